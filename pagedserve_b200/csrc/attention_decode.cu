@@ -122,7 +122,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                               float* __restrict__ part_acc, float* __restrict__ part_ml,
                               int* __restrict__ counters, int* __restrict__ status,
                               const int* __restrict__ q_start, const int* __restrict__ kv_len, int cluster,
-                              const int* __restrict__ token_row, SoftmaxExtras extras) {
+                              const int* __restrict__ token_row, SoftmaxExtras extras, int all_values) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     // page_size, chunk_keys and the unit are powers of two: shifts and masks instead of divisions
     const int unit = min(page_size, chunk_keys >> 3);                                // keys per copy
@@ -157,7 +157,9 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     };
 
     // ---- before the wait: only what no kernel of this step writes (positions, tables, older keys)
-    const int t = blockIdx.x, h = blockIdx.y, split = blockIdx.z;
+    // all_values: every query head meets the values of every key/value head, one (token, head, value head) per CTA column
+    const int t = blockIdx.x, column = blockIdx.y, columns = gridDim.y, split = blockIdx.z;
+    const int h = all_values ? column / n_kv_heads : column;
     const int lane = tid & 31, warp = tid >> 5;
     const int gq = lane >> 2, tq = lane & 3;
     const int p = positions[t];
@@ -181,6 +183,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     const int chunk_hi = active ? min(last_chunk, (split + 1) * split_chunks - 1) : 0;
 
     const int g = h / (n_heads / n_kv_heads);
+    const long long to_value = all_values ? (long long)(column % n_kv_heads - g) * page_size * head_dim : 0;
     // the token's block-table row: token_row[t] where the table is kept by request slot, else its item
     const int* bt = block_table + (size_t)(token_row ? token_row[t] : item) * bt_stride;
     const uint32_t unit_bytes = (uint32_t)unit * head_dim * 2;
@@ -205,7 +208,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                 const long long src = (long long)page * page_stride +
                                       ((long long)g * page_size + (key & (page_size - 1))) * head_dim;
                 bulk_copy_g2s(k_s + (size_t)tid * unit_elems, k_pool + src, unit_bytes, &bar);
-                bulk_copy_g2s(v_s + (size_t)tid * unit_elems, v_pool + src, unit_bytes, &bar);
+                bulk_copy_g2s(v_s + (size_t)tid * unit_elems, v_pool + src + to_value, unit_bytes, &bar);
             }
         }
     };
@@ -381,7 +384,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     if (n_splits == 1 || n_active == 1) {
         const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
         for (int d = tid_all; d < head_dim; d += THREADS)
-            out[(size_t)t * out_stride + h * head_dim + d] = __float2bfloat16_rn(o_s[d] * inv);
+            out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o_s[d] * inv);
         return;
     }
     if (by_cluster) {
@@ -421,9 +424,9 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             }
             // the others' shared memory has been read: they may leave while the result is written
             asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-            if (tid_all < head_dim) out[(size_t)t * out_stride + h * head_dim + tid_all] = __float2bfloat16_rn(o * inv);
+            if (tid_all < head_dim) out[(size_t)t * out_stride + column * head_dim + tid_all] = __float2bfloat16_rn(o * inv);
             if (tid_all + THREADS < head_dim)
-                out[(size_t)t * out_stride + h * head_dim + tid_all + THREADS] = __float2bfloat16_rn(more * inv);
+                out[(size_t)t * out_stride + column * head_dim + tid_all + THREADS] = __float2bfloat16_rn(more * inv);
             asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
             return;
         }
@@ -431,21 +434,21 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         return;
     }
     // several splits hold keys of this token: publish the partial state
-    const size_t slot = ((size_t)t * n_heads + h) * n_splits + split;
+    const size_t slot = ((size_t)t * columns + column) * n_splits + split;
     for (int d = tid_all; d < head_dim; d += THREADS) part_acc[slot * head_dim + d] = o_s[d];
     if (tid_all == 0) { part_ml[slot * 2] = m_run; part_ml[slot * 2 + 1] = l_run; }
     __threadfence();
     __syncthreads();
     if (tid_all == 0) {
-        int prev = atomicAdd(&counters[t * n_heads + h], 1);
+        int prev = atomicAdd(&counters[t * columns + column], 1);
         last_flag = (prev == n_active - 1);
-        if (last_flag) counters[t * n_heads + h] = 0;
+        if (last_flag) counters[t * columns + column] = 0;
     }
     __syncthreads();
     if (!last_flag) return;
     // (no fence on this side: the partial states below are read with ld.global.cg, from L2, where the other
     // CTAs' stores were performed before their fences let their counter increments through)
-    const size_t base = ((size_t)t * n_heads + h) * n_splits + first_split;
+    const size_t base = ((size_t)t * columns + column) * n_splits + first_split;
     // the partial accumulators are asked for first (they do not depend on the maxima), then the (max, sum)
     // pairs; the weight of each split is computed once and shared
     constexpr int HOLD = 8;                                   // splits whose values a thread keeps in flight
@@ -484,7 +487,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                 if (i < n_active)
                     o += (round == 0 ? held[i] : ldcg_f32(part_acc + (base + i) * head_dim + d)) * mh[i];
             }
-            out[(size_t)t * out_stride + h * head_dim + d] = __float2bfloat16_rn(o * inv);
+            out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o * inv);
         }
         return;
     }
@@ -519,7 +522,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             } else {
                 for (int i = 0; i < n_active; ++i) o += ldcg_f32(part_acc + (base + i) * head_dim + d) * w_s[i];
             }
-            out[(size_t)t * out_stride + h * head_dim + d] = __float2bfloat16_rn(o * inv);
+            out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o * inv);
         }
         return;
     }
@@ -533,7 +536,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         float o = 0.f;
         for (int i = 0; i < n_active; ++i)
             o += ldcg_f32(part_acc + (base + i) * head_dim + d) * exp2f(ldcg_f32(part_ml + (base + i) * 2) - M);
-        out[(size_t)t * out_stride + h * head_dim + d] = __float2bfloat16_rn(o * inv);
+        out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o * inv);
     }
 }
 
@@ -556,7 +559,7 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
                                    int split_tiles, int n_splits, float* part_acc, float* part_ml, int* counters,
                                    int* status, void* stream, const int* q_start = nullptr,
                                    const int* kv_len = nullptr, int cluster = 1, const int* token_row = nullptr,
-                                   float softcap = 0.f, const float* sink = nullptr) {
+                                   float softcap = 0.f, const float* sink = nullptr, int all_values = 0) {
     const ps::SoftmaxExtras extras = ps::softmax_extras(scale, softcap, sink);
     if (T <= 0) return PS_OK;
     if ((q_start == nullptr) != (kv_len == nullptr)) return PS_ERR_BAD_ARGUMENT;
@@ -564,7 +567,8 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return PS_ERR_BAD_ARGUMENT;
     if (head_dim <= 0 || head_dim % 16 != 0 || head_dim > 256) return PS_ERR_UNSUPPORTED;
     if (page_size <= 0 || page_size > 64 || (page_size & (page_size - 1))) return PS_ERR_UNSUPPORTED;
-    if (n_heads > 65535 || n_splits > 65535 || n_splits < 1 || split_tiles < 1) return PS_ERR_UNSUPPORTED;
+    const int columns = all_values ? n_heads * n_kv_heads : n_heads;
+    if (columns > 65535 || n_splits > 65535 || n_splits < 1 || split_tiles < 1) return PS_ERR_UNSUPPORTED;
     if (n_splits > 1 && cluster <= 1 && (!part_acc || !part_ml || !counters)) return PS_ERR_BAD_ARGUMENT;
     if (q_stride % 8 != 0 || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15) || page_stride % 8 != 0)
         return PS_ERR_UNSUPPORTED;
@@ -587,7 +591,7 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
     }
     // (a pair's chunks are walked in rounds of TEAMS: beyond two rounds, i.e. contexts of more than 12 chunks, the
     // split form's parallelism over more SMs is worth its merge again)
-    const bool teams = head_dim <= 64 && cluster <= 1 && n_splits > 1 && (long long)T * n_heads <= sm_count &&
+    const bool teams = head_dim <= 64 && cluster <= 1 && n_splits > 1 && (long long)T * columns <= sm_count &&
                        (long long)n_splits * split_chunks <= 2 * TEAMS;
     int groups = 1;
     if (teams) {
@@ -595,7 +599,7 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
         split_chunks *= n_splits;
         n_splits = 1;
     }
-    dim3 grid(T, n_heads, n_splits);
+    dim3 grid(T, columns, n_splits);
     size_t smem = (size_t)groups * (team_bytes + (size_t)head_dim * 4);
     cudaStream_t s = (cudaStream_t)stream;
     if (teams) {
@@ -607,7 +611,7 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
                                       (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, page_stride,
                                       token_item, positions, block_table, bt_stride, n_heads, n_kv_heads, head_dim,
                                       page_size, window, scale * 1.4426950408889634f, chunk_keys, split_chunks,
-                                      n_splits, part_acc, part_ml, counters, status, q_start, kv_len, 1, token_row, extras);
+                                      n_splits, part_acc, part_ml, counters, status, q_start, kv_len, 1, token_row, extras, all_values);
     }
 #define PS_DECODE_LAUNCH(KS)                                                                                          \
     {                                                                                                                \
@@ -620,7 +624,7 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
                                       token_item, positions, block_table, bt_stride, n_heads, n_kv_heads, head_dim,   \
                                       page_size, window, scale * 1.4426950408889634f, chunk_keys, split_chunks,       \
                                       n_splits, part_acc, part_ml, counters, status, q_start, kv_len, cluster,        \
-                                      token_row, extras);                                                             \
+                                      token_row, extras, all_values);                                                             \
     }
     if (head_dim <= 64) PS_DECODE_LAUNCH(4)
     if (head_dim <= 128) PS_DECODE_LAUNCH(8)
@@ -658,7 +662,9 @@ PS_EXPORT int ps_paged_attention_decode_checked(const void* q, int q_stride, voi
 // this step, so that a first chunk of such keys is fetched before the wait on the kernel before.
 // token_row (may be null): the block-table row of each token, where the table is kept by request slot
 // instead of by item. softcap > 0: scores become softcap * tanh(score / softcap); sink (may be null): one
-// float per query head whose exponential joins the softmax's denominator.
+// float per query head whose exponential joins the softmax's denominator.  all_values: every query head meets the
+// values of every key/value head; result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out, and the
+// scratch arrays are sized for n_heads * n_kv_heads heads.
 PS_EXPORT int ps_paged_attention_decode_ex(const void* q, int q_stride, void* out, int out_stride,
                                            const void* k_pool, const void* v_pool, long long page_stride,
                                            const int* token_item, const int* token_row, const int* positions,
@@ -667,11 +673,11 @@ PS_EXPORT int ps_paged_attention_decode_ex(const void* q, int q_stride, void* ou
                                            int n_heads, int n_kv_heads, int head_dim, int page_size, int window,
                                            float scale, int split_tiles, int n_splits, int cluster,
                                            float* part_acc, float* part_ml, int* counters, int* status,
-                                           float softcap, const float* sink, void* stream) {
+                                           float softcap, const float* sink, int all_values, void* stream) {
     return launch_attention_decode(q, q_stride, out, out_stride, k_pool, v_pool, page_stride, token_item, positions,
                                    block_table, bt_stride, T, n_heads, n_kv_heads, head_dim, page_size, window, scale,
                                    split_tiles, n_splits, part_acc, part_ml, counters, status, stream, q_start, kv_len,
-                                   cluster < 1 ? 1 : cluster, token_row, softcap, sink);
+                                   cluster < 1 ? 1 : cluster, token_row, softcap, sink, all_values);
 }
 
 // ------------------------------------------------------------------------------------------------

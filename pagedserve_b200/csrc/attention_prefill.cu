@@ -61,7 +61,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                          const int* __restrict__ block_table, int bt_stride, const int* __restrict__ item_row,
                          int first_item, int n_items, int n_heads, int n_kv_heads, int page_size, int window,
                          float scale_log2, SoftmaxExtras extras, const int* __restrict__ row_positions,
-                         int rows_per_item, float* __restrict__ partial, int key_splits) {
+                         int rows_per_item, float* __restrict__ partial, int key_splits, int all_values) {
     constexpr int RS = HD + 8;                         // padded row, in elements
     constexpr int CH = HD / 8;                         // 16-byte pieces of a row
     constexpr int KS = HD / 16;                        // k steps over the head dim
@@ -71,7 +71,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
     __nv_bfloat16* k_s = q_s + BQ * RS + wg * (4 * BKEY * RS);                 // this group's [2][BKEY][RS]
     // (a cache of one plane hands in the same pointer for keys and values: the rows are fetched once and read
     // from the key buffer for both products)
-    const bool one_plane = k_pool == v_pool;
+    const bool one_plane = k_pool == v_pool && !all_values;
     __nv_bfloat16* v_s = one_plane ? k_s : k_s + 2 * BKEY * RS;                // this group's [2][BKEY][RS]
 
     pdl_prologue();
@@ -95,7 +95,9 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
         }
     }
     if (item < 0) return;
-    const int h = blockIdx.y, g = h / (n_heads / n_kv_heads);
+    // all_values: every query head meets the values of every key/value head, one pair per CTA column
+    const int column = blockIdx.y, h = all_values ? column / n_kv_heads : column, g = h / (n_heads / n_kv_heads);
+    const long long to_value = all_values ? (long long)(column % n_kv_heads - g) * page_size * HD : 0;
     const int tid = threadIdx.x & (GROUP - 1), lane = tid & 31, warp = tid >> 5;   // within the group
     const int qs = one_position ? item * rows_per_item : q_start[item];
     const int q_len = one_position ? rows_per_item : q_start[item + 1] - qs;
@@ -137,7 +139,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                 off = (long long)page * page_stride + ((long long)g * page_size + (key % page_size)) * HD + piece * 8;
             }
             cp_async16(k_s + (buf * BKEY + r) * RS + piece * 8, k_pool + off, ok);
-            if (!one_plane) cp_async16(v_s + (buf * BKEY + r) * RS + piece * 8, v_pool + off, ok);
+            if (!one_plane) cp_async16(v_s + (buf * BKEY + r) * RS + piece * 8, v_pool + (ok ? off + to_value : 0), ok);
         }
     };
     if (kb_first + wg <= kb_last) load_kv(kb_first + wg, 0);
@@ -315,10 +317,10 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
     for (int dn = 0; dn < HD / 8; ++dn) {
         const int d = dn * 8 + tq * 2;
         if (row0 < rows)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + row0) * out_stride + h * HD + d) =
+            *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + row0) * out_stride + column * HD + d) =
                 pack_bf16(o[dn][0] * inv0, o[dn][1] * inv0);
         if (row1 < rows)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + row1) * out_stride + h * HD + d) =
+            *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + row1) * out_stride + column * HD + d) =
                 pack_bf16(o[dn][2] * inv1, o[dn][3] * inv1);
     }
 }
@@ -352,7 +354,8 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
            long long page_stride, const int* q_start, const int* kv_len, const int* block_table, int bt_stride,
            const int* item_row, int first_item, int n_items, int max_blocks, int n_heads, int n_kv_heads,
            int page_size, int window, float scale, float softcap, const float* sink, cudaStream_t stream,
-           const int* row_positions = nullptr, int rows_per_item = 0, float* partial = nullptr, int key_splits = 1) {
+           const int* row_positions = nullptr, int rows_per_item = 0, float* partial = nullptr, int key_splits = 1,
+           int all_values = 0) {
     constexpr int RS = HD + 8;
     size_t smem = (size_t)(BQ + 8 * BKEY) * RS * 2;
     auto kernel = prefill_attention_kernel<HD>;
@@ -365,16 +368,16 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
                                       kv_len, block_table, bt_stride, item_row, first_item, n_items, n_heads,
                                       n_kv_heads, page_size, window, scale * 1.4426950408889634f,
                                       softmax_extras(scale, softcap, sink), row_positions, rows_per_item, partial,
-                                      key_splits);
+                                      key_splits, 0);
         if (status != PS_OK) return status;
         return launch_pdl(merge_key_splits_kernel, dim3(n_items * rows_per_item), dim3(HD >= 64 ? 64 : 32), 0, stream,
                           (const float*)partial, key_splits, rows_per_item, HD, (__nv_bfloat16*)out, out_stride);
     }
-    return launch_pdl(kernel, dim3(max_blocks, n_heads), dim3(THREADS), smem, stream, (const __nv_bfloat16*)q, q_stride,
+    return launch_pdl(kernel, dim3(max_blocks, all_values ? n_heads * n_kv_heads : n_heads), dim3(THREADS), smem, stream, (const __nv_bfloat16*)q, q_stride,
                       (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool,
                       page_stride, q_start, kv_len, block_table, bt_stride, item_row, first_item, n_items, n_heads,
                       n_kv_heads, page_size, window, scale * 1.4426950408889634f, softmax_extras(scale, softcap, sink),
-                      row_positions, rows_per_item, (float*)nullptr, 1);
+                      row_positions, rows_per_item, (float*)nullptr, 1, all_values);
 }
 
 }  // namespace pf
@@ -385,15 +388,18 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
 // q and out point at row 0 of the step's flat token arrays. Head sizes: multiples of 16 up to 128.
 // item_row (may be null): the block-table row of each item, where the table is kept by request slot.
 // softcap > 0: scores become softcap * tanh(score / softcap); sink (may be null): one float per query head whose
-// exponential joins the softmax's denominator.
+// exponential joins the softmax's denominator.  all_values: every query head meets the values of every key/value head;
+// result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out.
 PS_EXPORT int ps_prefill_attention(const void* q, int q_stride, void* out, int out_stride, const void* k_pool,
                                    const void* v_pool, long long page_stride, const int* q_start, const int* kv_len,
                                    const int* block_table, int bt_stride, const int* item_row, int first_item,
                                    int n_items,
                                    int max_blocks, int n_heads, int n_kv_heads, int head_dim, int page_size,
-                                   int window, float scale, float softcap, const float* sink, void* stream) {
+                                   int window, float scale, float softcap, const float* sink, int all_values,
+                                   void* stream) {
     if (n_items <= 0 || max_blocks <= 0) return PS_OK;
-    if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0 || n_heads > 65535) return PS_ERR_BAD_ARGUMENT;
+    if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0 ||
+        (long long)n_heads * (all_values ? n_kv_heads : 1) > 65535) return PS_ERR_BAD_ARGUMENT;
     if (head_dim <= 0 || head_dim % 16 != 0 || head_dim > 128) return PS_ERR_UNSUPPORTED;
     if (page_size <= 0 || page_size > 64 || (page_size & (page_size - 1))) return PS_ERR_UNSUPPORTED;
     if (q_stride % 8 != 0 || out_stride % 2 != 0 || page_stride % 8 != 0) return PS_ERR_UNSUPPORTED;
@@ -404,7 +410,7 @@ PS_EXPORT int ps_prefill_attention(const void* q, int q_stride, void* out, int o
     case D:                                                                                                        \
         return ps::pf::launch<D>(q, q_stride, out, out_stride, k_pool, v_pool, page_stride, q_start, kv_len,       \
                                  block_table, bt_stride, item_row, first_item, n_items, max_blocks, n_heads,       \
-                                 n_kv_heads, page_size, window, scale, softcap, sink, s);
+                                 n_kv_heads, page_size, window, scale, softcap, sink, s, nullptr, 0, nullptr, 1, all_values);
     switch (head_dim) {
         PS_PF_CASE(16) PS_PF_CASE(32) PS_PF_CASE(48) PS_PF_CASE(64)
         PS_PF_CASE(80) PS_PF_CASE(96) PS_PF_CASE(112) PS_PF_CASE(128)

@@ -193,7 +193,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ item_row, int first_item, int n_items, int n_heads,
                             int n_kv_heads, int page_size, int window,
                             float scale_log2, long long k_row_base, long long v_row_base, long long page_rows,
-                            int* __restrict__ status, SoftmaxExtras extras) {
+                            int* __restrict__ status, SoftmaxExtras extras, int all_values) {
     using L = Layout<HD, SPLIT>;
     constexpr int ROW_THREADS = L::ROW_THREADS, THREADS = L::THREADS, COLS = L::COLS;
     extern __shared__ unsigned char smem_raw[];
@@ -221,7 +221,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         block -= blocks;
     }
     if (item < 0) return;
-    const int h = blockIdx.x, g = h / (n_heads / n_kv_heads);
+    // all_values: every query head meets the values of every key/value head, one pair per CTA column
+    const int column = blockIdx.x, h = all_values ? column / n_kv_heads : column, g = h / (n_heads / n_kv_heads);
+    const int to_value = all_values ? (column % n_kv_heads - g) * page_size : 0;       // rows from a key to its value
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int qs = q_start[item], q_len = q_start[item + 1] - qs;
     const int pos0 = kv_len[item] - q_len + qb * BQ;              // position of the block's first query
@@ -283,7 +285,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                 for (int c = 0; c < L::KCH; ++c) {
                     tma_load_2d(k_dst + c * (BKEY * 128) + lane * page_bytes, &map_kv, 64 * c, (int)(k_row_base + row), &kv_full[s]);
-                    tma_load_2d(v_dst + c * (BKEY * 128) + lane * page_bytes, &map_kv, 64 * c, (int)(v_row_base + row), &kv_full[s]);
+                    tma_load_2d(v_dst + c * (BKEY * 128) + lane * page_bytes, &map_kv, 64 * c, (int)(v_row_base + row) + to_value, &kv_full[s]);
                 }
             }
         }
@@ -473,7 +475,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (ok) {
             // the whole warp reads its O rows from TMEM (the load is warp-wide); rows of the portion store
             const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-            __nv_bfloat16* orow = out + (size_t)(tok0 + r) * out_stride + h * HD + half * OCOLS;
+            __nv_bfloat16* orow = out + (size_t)(tok0 + r) * out_stride + column * HD + half * OCOLS;
 #pragma unroll
             for (int c = 0; c < OCOLS; c += 32) {
                 uint32_t orr[32];
@@ -538,7 +540,7 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
            long long k_row_base, long long v_row_base, long long page_rows, const int* q_start, const int* kv_len,
            const int* block_table, int bt_stride, const int* item_row, int first_item, int n_items, int max_blocks,
            int n_heads, int n_kv_heads, int page_size, int window, float scale, int* status, float softcap,
-           const float* sink, cudaStream_t stream) {
+           const float* sink, int all_values, cudaStream_t stream) {
     CUtensorMap map_q, map_kv;
     if (!make_map(&map_q, q, T, n_heads * HD, q_stride, BQ)) return PS_ERR_LAUNCH;
     if (!make_map(&map_kv, pool, pool_rows, HD, HD, page_size)) return PS_ERR_LAUNCH;
@@ -547,10 +549,10 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
     static size_t raised[MAX_DEVICES] = {0};
     if (!ensure_dynamic_smem((const void*)kernel, (size_t)L::SMEM, raised)) return PS_ERR_LAUNCH;
     // heads vary fastest: the heaviest query blocks of all heads are scheduled first
-    return launch_pdl(kernel, dim3(n_heads, max_blocks), dim3(L::THREADS), L::SMEM, stream, map_q, map_kv,
+    return launch_pdl(kernel, dim3(all_values ? n_heads * n_kv_heads : n_heads, max_blocks), dim3(L::THREADS), L::SMEM, stream, map_q, map_kv,
                       (__nv_bfloat16*)out, out_stride, q_start, kv_len, block_table, bt_stride, item_row, first_item,
                       n_items, n_heads, n_kv_heads, page_size, window, scale * 1.4426950408889634f, k_row_base,
-                      v_row_base, page_rows, status, softmax_extras(scale, softcap, sink));
+                      v_row_base, page_rows, status, softmax_extras(scale, softcap, sink), all_values);
 }
 
 }  // namespace pftc
@@ -563,7 +565,8 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
 // row_threads: threads per query row, 1 or 2 (0: chosen here).
 // item_row (may be null): the block-table row of each item, where the table is kept by request slot.
 // softcap > 0: scores become softcap * tanh(score / softcap); sink (may be null): one float per query head whose
-// exponential joins the softmax's denominator.
+// exponential joins the softmax's denominator.  all_values: every query head meets the values of every key/value head;
+// result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out.
 PS_EXPORT int ps_prefill_attention_tc(const void* q, int q_stride, int T, void* out, int out_stride, const void* pool,
                                       long long pool_rows, long long k_row_base, long long v_row_base,
                                       long long page_rows, const int* q_start, const int* kv_len,
@@ -571,7 +574,7 @@ PS_EXPORT int ps_prefill_attention_tc(const void* q, int q_stride, int T, void* 
                                       int n_items,
                                       int max_blocks, int n_heads, int n_kv_heads, int head_dim, int page_size,
                                       int window, float scale, int row_threads, int* status, float softcap,
-                                      const float* sink, void* stream) {
+                                      const float* sink, int all_values, void* stream) {
     if (n_items <= 0 || max_blocks <= 0) return PS_OK;
     if (row_threads < 0 || row_threads > 2) return PS_ERR_BAD_ARGUMENT;
     if (!status) return PS_ERR_BAD_ARGUMENT;
@@ -591,7 +594,7 @@ PS_EXPORT int ps_prefill_attention_tc(const void* q, int q_stride, int T, void* 
     return ps::pftc::launch<HD, SPLIT>(q, q_stride, T, out, out_stride, pool, pool_rows, k_row_base, v_row_base,     \
                                        page_rows, q_start, kv_len, block_table, bt_stride, item_row, first_item,      \
                                        n_items, max_blocks, n_heads, n_kv_heads, page_size, window, scale, status,    \
-                                       softcap, sink, s)
+                                       softcap, sink, all_values, s)
     if (head_dim == 64) {
         if (two) PS_PFTC_LAUNCH(64, 2);
         PS_PFTC_LAUNCH(64, 1);

@@ -14,6 +14,8 @@
 //   s = (q.k) * scale, softmax in float32, o = p.v
 //   softcap > 0: s <- softcap * tanh(s / softcap) before the softmax;
 //   sink (one float per head, or null): exp(sink[h]) joins the softmax's denominator and nothing else.
+//   all_values: every query head meets the values of every key/value head (one CTA per pair), for a layer that mixes
+//   its heads' weights: result (h, g') = sum_j p_h(j) v_g'(j) stands at column (h * n_kv_heads + g') * head_dim.
 //   (reference: src/model/paged_attention.py:262-295; src/kernels/triton_paged_attention.py:219-331)
 // Keys are visited in tiles of 32 aligned to absolute positions; warp w takes tiles with
 // tile % 4 == w; the four partial (max, sum, acc) states are merged in warp order. The
@@ -106,7 +108,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
                             const int* __restrict__ token_item, const int* __restrict__ positions,
                             const int* __restrict__ block_table, int bt_stride,
                             int n_heads, int n_kv_heads, int head_dim, int page_size, int window, float scale,
-                            float softcap, const float* __restrict__ sink) {
+                            float softcap, const float* __restrict__ sink, int all_values) {
     extern __shared__ float smem[];
     float* q_s = smem;                                   // [head_dim]
     float* acc_s = smem + head_dim;                      // [ATT_WARPS][head_dim]
@@ -116,8 +118,11 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
     q = pdl_fresh(q);
     k_pool = pdl_fresh(k_pool);
     v_pool = pdl_fresh(v_pool);
-    int t = blockIdx.x, h = blockIdx.y;
+    int t = blockIdx.x, column = blockIdx.y;                // the head of the result
+    int h = all_values ? column / n_kv_heads : column;
     int g = h / (n_heads / n_kv_heads);
+    // from a key's row to the row of the value that it weighs
+    const long long to_value = all_values ? (long long)(column % n_kv_heads - g) * page_size * head_dim : 0;
     int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     int item = token_item[t];
     int p = positions[t];
@@ -159,7 +164,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
             if (!((mask >> j) & 1u)) continue;
             float pj = __shfl_sync(0xffffffffu, pr, j);
             long long rj = __shfl_sync(0xffffffffu, row, j);
-            const T* vr = v_pool + rj;
+            const T* vr = v_pool + rj + to_value;
 #pragma unroll
             for (int i = 0; i < NACC; ++i) {
                 int d = lane + 32 * i;
@@ -191,7 +196,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < ATT_WARPS; ++w) o += acc_s[w * head_dim + d] * wgt[w];
-        out[(size_t)t * out_stride + h * head_dim + d] = from_float<T>(o * inv);
+        out[(size_t)t * out_stride + column * head_dim + d] = from_float<T>(o * inv);
     }
 }
 
@@ -227,13 +232,14 @@ PS_EXPORT int ps_paged_attention_simt(const void* q, int q_stride, void* out, in
                                       const int* token_item, const int* positions, const int* block_table,
                                       int bt_stride, int T, int n_heads, int n_kv_heads, int head_dim,
                                       int page_size, int window, float scale, float softcap, const float* sink,
-                                      int dtype, void* stream) {
+                                      int all_values, int dtype, void* stream) {
     if (T <= 0) return PS_OK;
     int rc = check_attention_sizes(n_heads, n_kv_heads, head_dim, page_size);
     if (rc) return rc;
-    if (n_heads > 65535) return PS_ERR_UNSUPPORTED;
+    const int columns = all_values ? n_heads * n_kv_heads : n_heads;
+    if (columns > 65535) return PS_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(T, n_heads);
+    dim3 grid(T, columns);
     size_t smem = (size_t)(1 + ps::ATT_WARPS) * head_dim * sizeof(float);
     const bool wide = head_dim > ps::ATT_USUAL_HD;
     if (dtype == PS_F32) {
@@ -242,7 +248,7 @@ PS_EXPORT int ps_paged_attention_simt(const void* q, int q_stride, void* out, in
         return ps::launch_pdl(kernel, grid, dim3(ps::ATT_WARPS * 32), smem, s,
                               (const float*)q, q_stride, (float*)out, out_stride, (const float*)k_pool,
                               (const float*)v_pool, page_stride, token_item, positions, block_table, bt_stride,
-                              n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap, sink);
+                              n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap, sink, all_values);
     }
     if (dtype == PS_BF16) {
         auto kernel = wide ? ps::paged_attention_simt_kernel<__nv_bfloat16, ps::ATT_MAX_HD / 32>
@@ -251,7 +257,7 @@ PS_EXPORT int ps_paged_attention_simt(const void* q, int q_stride, void* out, in
                               (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride,
                               (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, page_stride, token_item,
                               positions, block_table, bt_stride, n_heads, n_kv_heads, head_dim, page_size, window,
-                              scale, softcap, sink);
+                              scale, softcap, sink, all_values);
     }
     return PS_ERR_UNSUPPORTED;
 }

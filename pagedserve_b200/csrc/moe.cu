@@ -15,6 +15,7 @@
 // The inner activation of a gated expert from its gate and up pre-activations g, u and the token's weight w
 // (GateForm):
 //     kind 0:  silu(g) * u * w                                   (the weight scales the expert's output)
+//     kind 2:  gelu_tanh(g) * u * w
 //     kind 1:  g' = min(w g, limit), u' = clamp(w u, -limit, limit);  g' * sigmoid(alpha g') * (u' + 1)
 //              (the weight scales the expert's input: without biases W (w h) = w (W h), so it is applied to the
 //              pre-activations in float32; the shared expert's columns have a limit of their own)
@@ -61,7 +62,7 @@ __device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
 }
 
 struct GateForm {
-    int kind;                 // 0: silu(g) u w; 1: clamped, weight on the input (see the top of the file)
+    int kind;                 // 0: silu(g) u w; 2: gelu_tanh(g) u w; 1: clamped, weight on the input (see the top of the file)
     float limit;              // kind 1: the routed experts' limit
     float shared_limit;       // kind 1: the shared expert's
     float alpha;              // kind 1: the sigmoid's slope
@@ -69,6 +70,7 @@ struct GateForm {
 
 __device__ __forceinline__ float gated_inner(float g, float u, float w, int kind, float limit, float alpha) {
     if (kind == 0) return silu(g) * u * w;
+    if (kind == 2) return gelu_tanh(g) * u * w;
     g = fminf(g * w, limit);
     u = fminf(fmaxf(u * w, -limit), limit);
     return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
@@ -540,7 +542,7 @@ PS_EXPORT int ps_moe_gate_mul(const void* gate_up, int gu_stride, const float* d
                               int kind, float limit, float shared_limit, float alpha, void* stream) {
     if (T <= 0 || columns <= 0) return PS_OK;
     if (!gate_up || !inner || E < 0 || (E > 0 && !dense) || F <= 0 || columns < E * F) return PS_ERR_BAD_ARGUMENT;
-    if (kind < 0 || kind > 1 || (kind == 1 && !(limit > 0.f && shared_limit > 0.f))) return PS_ERR_BAD_ARGUMENT;
+    if (kind < 0 || kind > 2 || (kind == 1 && !(limit > 0.f && shared_limit > 0.f))) return PS_ERR_BAD_ARGUMENT;
     const ps::GateForm form{kind, limit, shared_limit, alpha};
     cudaStream_t s = (cudaStream_t)stream;
     const int by8 = F % 8 == 0 && columns % 8 == 0 && gu_stride % 8 == 0 && inner_stride % 8 == 0 &&
@@ -594,7 +596,7 @@ PS_EXPORT int ps_moe_gate_mul_rows(const void* gate_up, int gu_stride, const flo
                                    void* stream) {
     if (R <= 0 || F <= 0) return PS_OK;
     if (!gate_up || !row_weight || !inner) return PS_ERR_BAD_ARGUMENT;
-    if (kind < 0 || kind > 1 || (kind == 1 && !(limit > 0.f))) return PS_ERR_BAD_ARGUMENT;
+    if (kind < 0 || kind > 2 || (kind == 1 && !(limit > 0.f))) return PS_ERR_BAD_ARGUMENT;
     const ps::GateForm form{kind, limit, limit, alpha};
     cudaStream_t s = (cudaStream_t)stream;
     const int by8 = F % 8 == 0 && gu_stride % 8 == 0 && inner_stride % 8 == 0 && !((uintptr_t)gate_up & 31) &&

@@ -14,6 +14,13 @@
 // x is also left in the compute type (`x_cast`, null where that is float32 itself) for the next product.
 //
 // depth_begin: history[0] <- x (if given), x_cast <- x, y <- 0.
+//
+// sandwich_close, one CTA per token, all float32: between two sublayers of a layer that norms what a sublayer reads and
+// what it returns.  A sublayer has left its result, up to a common factor y_scale, in the zeroed row y;
+//     x <- x + gain * norm(y_scale * y);   y <- 0          (norm(a) = a / sqrt(mean(a^2) + eps); gain null: only y <- 0)
+//     inverse = 1 / sqrt(mean(x^2) + eps)
+// and what the next sublayer wants of the new row: out <- x * inverse * next_gain (compute type), or the factor alone
+// (row_scale[t] <- inverse) where the next kernel reads x itself.
 #include "common.cuh"
 
 namespace ps {
@@ -144,6 +151,80 @@ depth_begin_kernel(const float* __restrict__ x, float* __restrict__ first, TC* _
     }
 }
 
+// the sum over the CTA's threads, in every thread, in a fixed order (`slots`: one float per warp)
+__device__ __forceinline__ float cta_sum(float v, float* slots) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) slots[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int w = 0; w < GROUP_NORM_THREADS / 32; ++w) total += slots[w];
+    return total;
+}
+
+template <typename TC, int V>
+__global__ void __launch_bounds__(GROUP_NORM_THREADS)
+sandwich_close_kernel(float* __restrict__ y, float* __restrict__ x, int H, const float* __restrict__ gain, float y_scale,
+                      float eps, const float* __restrict__ next_gain, TC* __restrict__ out, float* __restrict__ row_scale) {
+    using Pack = PackOf<V>;
+    extern __shared__ __align__(16) float staged[];          // the sublayer's row, the residual row
+    __shared__ float slots[2][GROUP_NORM_THREADS / 32];
+    float* row = staged;
+    float* kept = staged + H;
+    pdl_prologue();
+    y = pdl_fresh(y);
+    x = pdl_fresh(x);
+    const size_t base = (size_t)blockIdx.x * H;
+    Pack zero;
+#pragma unroll
+    for (int i = 0; i < V; ++i) zero.v[i] = 0.f;
+    float sq = 0.f, sq_x = 0.f;
+    for (int j = V * threadIdx.x; j < H; j += V * GROUP_NORM_THREADS) {
+        const Pack b = *reinterpret_cast<const Pack*>(x + base + j);
+        *reinterpret_cast<Pack*>(kept + j) = b;
+        if (gain) {
+            Pack a = *reinterpret_cast<const Pack*>(y + base + j);
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                a.v[i] *= y_scale;
+                sq = fmaf(a.v[i], a.v[i], sq);
+            }
+            *reinterpret_cast<Pack*>(row + j) = a;
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; ++i) sq_x = fmaf(b.v[i], b.v[i], sq_x);
+        }
+        *reinterpret_cast<Pack*>(y + base + j) = zero;
+    }
+    // (a thread reads back only what it has written itself: the two rows need no barrier of their own)
+    if (gain) {
+        const float inverse = 1.0f / sqrtf(cta_sum(sq, slots[0]) / (float)H + eps);
+        for (int j = V * threadIdx.x; j < H; j += V * GROUP_NORM_THREADS) {
+            const Pack g = *reinterpret_cast<const Pack*>(gain + j);
+            const Pack a = *reinterpret_cast<const Pack*>(row + j);
+            Pack b = *reinterpret_cast<const Pack*>(kept + j);
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                b.v[i] = fmaf(a.v[i] * inverse, g.v[i], b.v[i]);
+                sq_x = fmaf(b.v[i], b.v[i], sq_x);
+            }
+            *reinterpret_cast<Pack*>(kept + j) = b;
+            *reinterpret_cast<Pack*>(x + base + j) = b;
+        }
+    }
+    if (!out && !row_scale) return;
+    const float inverse = 1.0f / sqrtf(cta_sum(sq_x, slots[1]) / (float)H + eps);
+    if (row_scale && threadIdx.x == 0) row_scale[blockIdx.x] = inverse;
+    if (!out) return;
+    for (int j = V * threadIdx.x; j < H; j += V * GROUP_NORM_THREADS) {
+        const Pack g = *reinterpret_cast<const Pack*>(next_gain + j);
+        Pack b = *reinterpret_cast<const Pack*>(kept + j);
+#pragma unroll
+        for (int i = 0; i < V; ++i) b.v[i] = b.v[i] * inverse * g.v[i];
+        store_cast<V>(out + base + j, b);
+    }
+}
+
 template <typename TIn, typename TOut>
 inline int launch_group_norm(const void* x, long long x_stride, const int* rows, int n_rows, int H, int groups,
                              const float* gain, float eps, void* out, long long out_stride, cudaStream_t s) {
@@ -219,4 +300,33 @@ PS_EXPORT int ps_depth_begin(const float* x, float* first, void* x_cast, int cas
         return ps::launch_pdl(ps::depth_begin_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, x, first, (__nv_bfloat16*)x_cast,
                               y, count);
     return PS_ERR_UNSUPPORTED;
+}
+
+// y, x float32 [T, H] contiguous; gain, next_gain float32 [H] (gain null: nothing is added); out [T, H] of `out_dtype` or
+// null (then next_gain may be null); row_scale float32 [T] or null.
+PS_EXPORT int ps_sandwich_close(float* y, float* x, int T, int H, const float* gain, float y_scale, float eps,
+                                const float* next_gain, void* out, int out_dtype, float* row_scale, void* stream) {
+    if (T <= 0) return PS_OK;
+    if (!y || !x || H <= 0 || (out && !next_gain)) return PS_ERR_BAD_ARGUMENT;
+    const size_t smem = (size_t)2 * H * sizeof(float);
+    if (smem > 200 * 1024 || (out && out_dtype != PS_F32 && out_dtype != PS_BF16)) return PS_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool bf16 = out && out_dtype == PS_BF16;
+    const bool by4 = H % 4 == 0 && !(((uintptr_t)y | (uintptr_t)x | (uintptr_t)gain | (uintptr_t)next_gain) & 15) &&
+                     !((uintptr_t)out & (bf16 ? 7 : 15));
+#define PS_SANDWICH(TYPE, V)                                                                                         \
+    do {                                                                                                             \
+        static size_t raised[ps::MAX_DEVICES] = {0};                                                                 \
+        auto kernel = ps::sandwich_close_kernel<TYPE, V>;                                                            \
+        if (!ps::ensure_dynamic_smem((const void*)kernel, smem, raised)) return PS_ERR_LAUNCH;                       \
+        return ps::launch_pdl(kernel, dim3(T), dim3(ps::GROUP_NORM_THREADS), smem, s, y, x, H, gain, y_scale, eps,   \
+                              next_gain, (TYPE*)out, row_scale);                                                     \
+    } while (0)
+    if (bf16) {
+        if (by4) PS_SANDWICH(__nv_bfloat16, 4);
+        PS_SANDWICH(__nv_bfloat16, 1);
+    }
+    if (by4) PS_SANDWICH(float, 4);
+    PS_SANDWICH(float, 1);
+#undef PS_SANDWICH
 }

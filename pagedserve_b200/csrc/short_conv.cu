@@ -11,7 +11,11 @@
 // `head_slot` numbers of which the first `head_values` count.  mode 1: the convolved values are also stored, float32,
 // in `shared_values` [T, mix_heads * head_values]; mode 2: y <- (1 - m) y + m * shared_values[t], m = *mix.
 //
-// short_conv_keep, after it: the slot receives the last taps - 1 projected rows of the sequence (rows of this step,
+// row_scale (may be null): one float per token that multiplies its row of u wherever it is read (a row to be divided by
+// its root mean square, say, whose factor an earlier kernel has formed); kept rows are stored already multiplied.
+//
+// Entries of one token (decode) replace their slot's rows themselves: the thread of a channel has read them all.
+// short_conv_keep, after it, for the others: the slot receives the last taps - 1 projected rows of the sequence (rows of this step,
 // and older kept rows moved up where the entry brought fewer than taps - 1 tokens).  Two launches, because every
 // token of an entry may still read the old rows.
 #include "common.cuh"
@@ -23,12 +27,13 @@ constexpr int SHORT_CONV_MAX_TAPS = 16;
 template <typename TC>
 __global__ void __launch_bounds__(256)
 short_conv_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ weight, int taps,
-                  int conv_channels, int channels, const float* __restrict__ kept, long long kept_stride,
+                  int conv_channels, int channels, const float* __restrict__ row_scale, float* kept, long long kept_stride,
                   const int* __restrict__ token_item, const int* __restrict__ q_start, const int* __restrict__ item_slot,
                   TC* __restrict__ out, long long out_stride, int mode, int mix_lo, int mix_heads, int head_slot,
                   int head_values, float* __restrict__ shared_values, const float* __restrict__ mix, int tokens) {
     pdl_prologue();
     u = pdl_fresh(u);
+    row_scale = pdl_fresh(row_scale);
     shared_values = pdl_fresh(shared_values);
     const long long total = (long long)tokens * channels;
     const float blend = mode == 2 ? *mix : 0.f;
@@ -37,18 +42,24 @@ short_conv_kernel(const float* __restrict__ u, long long u_stride, const float* 
         const int t = (int)(i / channels), c = (int)(i - (long long)t * channels);
         float y;
         if (c >= conv_channels) {
-            y = u[(size_t)t * u_stride + c];
+            y = u[(size_t)t * u_stride + c] * (row_scale ? row_scale[t] : 1.f);
         } else {
             const int item = token_item[t];
             const int first = q_start[item];
-            const float* old = kept + (size_t)item_slot[item] * kept_stride;
+            float* old = kept + (size_t)item_slot[item] * kept_stride;
+            float now = 0.f;
             y = 0.f;
             for (int j = 0; j < taps; ++j) {
                 const int source = t - (taps - 1) + j;
                 // kept row k holds the projection of the token (taps - 1 - k) places before the entry's first
-                const float v = source >= first ? u[(size_t)source * u_stride + c]
+                const float v = source >= first ? u[(size_t)source * u_stride + c] * (row_scale ? row_scale[source] : 1.f)
                                                 : old[(size_t)(taps - 1 - (first - source)) * conv_channels + c];
                 y = fmaf(weight[(size_t)c * taps + j], v, y);
+                now = v;
+            }
+            if (taps > 1 && q_start[item + 1] - first == 1) {         // the entry's only token: its rows move up by one
+                for (int k = 0; k < taps - 2; ++k) old[(size_t)k * conv_channels + c] = old[(size_t)(k + 1) * conv_channels + c];
+                old[(size_t)(taps - 2) * conv_channels + c] = now;
             }
             if (mode) {
                 const int local = c - mix_lo;
@@ -88,8 +99,8 @@ constexpr int SHORT_CONV_THREADS = 128;
 template <typename TC, int TAPS>
 __global__ void __launch_bounds__(SHORT_CONV_THREADS)
 short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ weight,
-                       int conv_channels, int channels, const float* __restrict__ kept, long long kept_stride,
-                       const int* __restrict__ token_item, const int* __restrict__ q_start,
+                       int conv_channels, int channels, const float* __restrict__ row_scale, float* kept,
+                       long long kept_stride, const int* __restrict__ token_item, const int* __restrict__ q_start,
                        const int* __restrict__ item_slot, TC* __restrict__ out, long long out_stride, int mode, int mix_lo,
                        int mix_heads, int head_slot, int head_values, float* __restrict__ shared_values,
                        const float* __restrict__ mix, int tokens, int run) {
@@ -107,11 +118,20 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
     const float blend = mode == 2 ? *mix : 0.f;
     pdl_prologue();
     u = pdl_fresh(u);
+    row_scale = pdl_fresh(row_scale);
     shared_values = pdl_fresh(shared_values);
+    auto scaled = [&](int t) {
+        float4 v = *reinterpret_cast<const float4*>(u + (size_t)t * u_stride + c);
+        if (row_scale) {
+            const float f = row_scale[t];
+            v.x *= f; v.y *= f; v.z *= f; v.w *= f;
+        }
+        return v;
+    };
     if (c >= channels) return;
     if (!convolved) {
         for (int t = t0; t < t1; ++t) {
-            const float4 v = *reinterpret_cast<const float4*>(u + (size_t)t * u_stride + c);
+            const float4 v = scaled(t);
             const float y[4] = {v.x, v.y, v.z, v.w};
             store4<TC>(out + (size_t)t * out_stride + c, y);
         }
@@ -127,7 +147,6 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
         }
     }
     float4 held[TAPS > 1 ? TAPS - 1 : 1];                         // held[k]: the row k + 1 tokens back
-    int first = -1;
     for (int t = t0; t < t1; ++t) {
         const int item = token_item[t];
         const int start = q_start[item];
@@ -136,12 +155,11 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
 #pragma unroll
             for (int k = 0; k < TAPS - 1; ++k) {
                 const int source = t - 1 - k;
-                held[k] = source >= start ? *reinterpret_cast<const float4*>(u + (size_t)source * u_stride + c)
+                held[k] = source >= start ? scaled(source)
                                           : *reinterpret_cast<const float4*>(old + (size_t)(TAPS - 1 - (start - source)) * conv_channels + c);
             }
-            first = start;
         }
-        const float4 now = *reinterpret_cast<const float4*>(u + (size_t)t * u_stride + c);
+        const float4 now = scaled(t);
         float y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) {                      // tap j reads the row TAPS - 1 - j tokens back
@@ -154,6 +172,12 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
 #pragma unroll
         for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
         if (TAPS > 1) held[0] = now;
+        if (TAPS > 1 && q_start[item + 1] - start == 1) {              // the entry's only token: its rows move up by one
+            float* rows = kept + (size_t)item_slot[item] * kept_stride;
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k)
+                *reinterpret_cast<float4*>(rows + (size_t)(TAPS - 2 - k) * conv_channels + c) = held[k];
+        }
         if (common >= 0) {
             float* place = shared_values + (size_t)t * mix_heads * head_values + common;
             if (mode == 1) {
@@ -166,25 +190,26 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
         }
         store4<TC>(out + (size_t)t * out_stride + c, y);
     }
-    (void)first;
 }
 
 __global__ void __launch_bounds__(256)
-short_conv_keep_kernel(const float* __restrict__ u, long long u_stride, int taps, int conv_channels,
-                       float* __restrict__ kept, long long kept_stride, const int* __restrict__ q_start,
+short_conv_keep_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ row_scale, int taps,
+                       int conv_channels, float* __restrict__ kept, long long kept_stride, const int* __restrict__ q_start,
                        const int* __restrict__ item_slot) {
     const int item = blockIdx.y;
     const int first = q_start[item], count = q_start[item + 1] - first;
     pdl_prologue();
     u = pdl_fresh(u);
-    if (count <= 0) return;
+    row_scale = pdl_fresh(row_scale);
+    if (count <= 1) return;                                           // (one token: done by the convolution itself)
     float* rows = kept + (size_t)item_slot[item] * kept_stride;
     for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < conv_channels; c += gridDim.x * blockDim.x) {
         // new row k is the token at place count - (taps - 1) + k of the entry; before the entry's first token that
         // is the old row k + count, which lies above every row written so far
         for (int k = 0; k < taps - 1; ++k) {
             const int place = count - (taps - 1) + k;
-            rows[(size_t)k * conv_channels + c] = place >= 0 ? u[(size_t)(first + place) * u_stride + c]
+            rows[(size_t)k * conv_channels + c] = place >= 0 ? u[(size_t)(first + place) * u_stride + c] *
+                                                                   (row_scale ? row_scale[first + place] : 1.f)
                                                              : rows[(size_t)(k + count) * conv_channels + c];
         }
     }
@@ -192,11 +217,11 @@ short_conv_keep_kernel(const float* __restrict__ u, long long u_stride, int taps
 
 }  // namespace ps
 
-// u float32 [T, channels] rows (u_stride apart); weight float32 [conv_channels, taps]; kept float32
+// u float32 [T, channels] rows (u_stride apart); row_scale float32 [T] or null; weight float32 [conv_channels, taps]; kept float32
 // [slots, (taps - 1) * conv_channels] rows (kept_stride apart; may be null when taps = 1); out [T, channels] rows of
 // `dtype`.  mode 0: no blending; 1: store the convolved values; 2: blend with the stored ones by *mix.
 PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* weight, int taps, int conv_channels,
-                            int channels, const float* kept, long long kept_stride, const int* token_item,
+                            int channels, const float* row_scale, float* kept, long long kept_stride, const int* token_item,
                             const int* q_start, const int* item_slot, void* out, long long out_stride, int mode,
                             int mix_lo, int mix_heads, int head_slot, int head_values, float* shared_values,
                             const float* mix, int T, int dtype, void* stream) {
@@ -224,7 +249,7 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
         const dim3 grid(columns, (T + run - 1) / run), block(ps::SHORT_CONV_THREADS);
 #define PS_CONV_RUNS(TYPE, TAPS)                                                                                      \
     return ps::launch_pdl(ps::short_conv_runs_kernel<TYPE, TAPS>, grid, block, 0, s, u, u_stride, weight, conv_channels, \
-                          channels, kept, kept_stride, token_item, q_start, item_slot, (TYPE*)out, out_stride, mode,     \
+                          channels, row_scale, kept, kept_stride, token_item, q_start, item_slot, (TYPE*)out, out_stride, mode,     \
                           mix_lo, mix_heads, head_slot, head_values, shared_values, mix, T, run)
 #define PS_CONV_TAPS(TYPE)                                                                                            \
     switch (taps) {                                                                                                   \
@@ -243,17 +268,17 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
     const dim3 grid((unsigned)(blocks < 4736 ? blocks : 4736));
     if (dtype == PS_F32)
         return ps::launch_pdl(ps::short_conv_kernel<float>, grid, dim3(256), 0, s, u, u_stride, weight, taps,
-                              conv_channels, channels, kept, kept_stride, token_item, q_start, item_slot, (float*)out,
+                              conv_channels, channels, row_scale, kept, kept_stride, token_item, q_start, item_slot, (float*)out,
                               out_stride, mode, mix_lo, mix_heads, head_slot, head_values, shared_values, mix, T);
     if (dtype == PS_BF16)
         return ps::launch_pdl(ps::short_conv_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, u, u_stride, weight, taps,
-                              conv_channels, channels, kept, kept_stride, token_item, q_start, item_slot,
+                              conv_channels, channels, row_scale, kept, kept_stride, token_item, q_start, item_slot,
                               (__nv_bfloat16*)out, out_stride, mode, mix_lo, mix_heads, head_slot, head_values,
                               shared_values, mix, T);
     return PS_ERR_UNSUPPORTED;
 }
 
-PS_EXPORT int ps_short_conv_keep(const float* u, long long u_stride, int taps, int conv_channels, float* kept,
+PS_EXPORT int ps_short_conv_keep(const float* u, long long u_stride, const float* row_scale, int taps, int conv_channels, float* kept,
                                  long long kept_stride, const int* q_start, const int* item_slot, int items,
                                  void* stream) {
     if (items <= 0 || taps <= 1 || conv_channels <= 0) return PS_OK;
@@ -262,6 +287,6 @@ PS_EXPORT int ps_short_conv_keep(const float* u, long long u_stride, int taps, i
     cudaStream_t s = (cudaStream_t)stream;
     int blocks = (conv_channels + 255) / 256;
     if (blocks > 64) blocks = 64;
-    return ps::launch_pdl(ps::short_conv_keep_kernel, dim3(blocks, items), dim3(256), 0, s, u, u_stride, taps,
-                          conv_channels, kept, kept_stride, q_start, item_slot);
+    return ps::launch_pdl(ps::short_conv_keep_kernel, dim3(blocks, items), dim3(256), 0, s, u, u_stride, row_scale,
+                          taps, conv_channels, kept, kept_stride, q_start, item_slot);
 }

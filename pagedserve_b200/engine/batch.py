@@ -279,6 +279,7 @@ class StepContext:
         self.step_counter = views.step_counter
         self.block_tables = cache.slots.table_views
         self.decode_only = (layout.num_tokens == layout.num_items)
+        self.single_tokens = False   # every entry is known to bring exactly one token (set by the runner)
 
     @property
     def host(self) -> HostBatch:

@@ -217,6 +217,7 @@ class ModelRunner:
         ctx = StepContext(layout, self._device_buffer, host_batch, cache, self._status, max_q_len, max_kv_len,
                           num_short_items, num_short_tokens, num_long_blocks, views=views)
         ctx.real_logit_rows = real_rows
+        ctx.single_tokens = not pad and int(counts.max()) == 1
         return ctx
 
     def _fill(self, layout: BatchLayout, host: np.ndarray, item_slot, q_start, logit_rows, token_ids, fed: int):
@@ -344,6 +345,7 @@ class ModelRunner:
                                kv_len.astype(np.int32), ramp[:P], list(requests))
         ctx = StepContext(layout, self._device_buffer, host_batch, cache, self._status, 1,
                           int(kv_len.max()), P, P, 0, views=views)
+        ctx.single_tokens = True
         ctx.slots = slots
         ctx.real_items = I
         ctx.drained = self._drained                        # corrections staged but not yet uploaded

@@ -76,7 +76,7 @@ _SIGNATURES = {
         "ps_gemm_simt": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "ps_kv_append": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I, _P],
         "ps_paged_attention_simt": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P,
-                                    _I, _P],
+                                    _I, _I, _P],
         "ps_rotary_cache_write": [_P, _I, _P, _I, _P, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I,
                                   _I, _P],
         "ps_token_shift_mix": [_P, _I, _P, _I, _P, _L, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P],
@@ -99,8 +99,12 @@ _SIGNATURES = {
         "ps_post_norm_add": [_P, _P, _I, _I, _I, _P, _F, _P, _I, _P, _L, _I, _P, _P],
         "ps_depth_begin": [_P, _P, _P, _I, _P, _L, _P],
         "ps_mingru_scan": [_P, _L, _I, _P, _L, _P, _P, _I, _P, _L, _I, _I, _P],
-        "ps_short_conv": [_P, _L, _P, _I, _I, _I, _P, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P],
-        "ps_short_conv_keep": [_P, _L, _I, _I, _P, _L, _P, _P, _I, _P],
+        "ps_short_conv": [_P, _L, _P, _I, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P],
+        "ps_short_conv_keep": [_P, _L, _P, _I, _I, _P, _L, _P, _P, _I, _P],
+        "ps_sandwich_close": [_P, _P, _I, _I, _P, _F, _F, _P, _P, _I, _P, _P],
+        "ps_gla_recurrence": [_P, _L, _P, _P, _P, _I, _F, _F, _P, _F, _F, _P, _L, _P, _P, _I, _I, _I, _P, _P, _P, _L,
+                              _I, _I, _I, _I, _P],
+        "ps_head_mix": [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P],
         "ps_moe_plan": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P],
         "ps_moe_gather": [_P, _I, _P, _P, _I, _I, _I, _I, _P],
         "ps_moe_gate_mul_rows": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
@@ -122,10 +126,10 @@ _SIGNATURES = {
         "ps_paged_attention_decode_checked": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
                                               _F, _I, _I, _P, _P, _P, _P, _P],
         "ps_paged_attention_decode_ex": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I,
-                                         _I, _I, _F, _I, _I, _I, _P, _P, _P, _P, _F, _P, _P],
+                                         _I, _I, _F, _I, _I, _I, _P, _P, _P, _P, _F, _P, _I, _P],
         "ps_shared_position_attention": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P],
         "ps_prefill_attention": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F,
-                                 _F, _P, _P],
+                                 _F, _P, _I, _P],
     },
     "tc": {
         "ps_gemm_tc": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
@@ -135,7 +139,7 @@ _SIGNATURES = {
         "ps_gemm_tc_experts": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P],
         "ps_gemm_tc_qkv": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "ps_prefill_attention_tc": [_P, _I, _I, _P, _I, _P, _L, _L, _L, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I,
-                                    _I, _I, _F, _I, _P, _F, _P, _P],
+                                    _I, _I, _F, _I, _P, _F, _P, _I, _P],
     },
 }
 
@@ -612,10 +616,11 @@ class Ops:
                                       self.code, _stream()), "kv_append")
 
     def paged_attention_simt(self, q, out, k_pool, v_pool, page_stride, token_item, positions, block_table,
-                             n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap=None, sink=None):
+                             n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap=None, sink=None, all_values=False):
         """out[t, h] = softmax(q[t,h] . K[<=pos]) V over the request's pages; CUDA cores.  ``softcap``:
         scores become softcap * tanh(score / softcap); ``sink``: float32 [n_heads], exp(sink[h]) joins the
-        softmax's denominator."""
+        softmax's denominator; ``all_values``: every query head meets the values of every key/value head, ``out`` [T,
+        n_heads * n_kv_heads * head_dim] (see :meth:`head_mix`)."""
         if sink is not None:
             _require(sink, "sink", torch.float32)
             if sink.numel() != n_heads:
@@ -630,7 +635,7 @@ class Ops:
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_pool), _ptr(v_pool),
             page_stride, _ptr(token_item), _ptr(positions), _ptr(block_table),
             block_table.stride(0), T, n_heads, n_kv_heads, head_dim,
-            page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), self.code, _stream()),
+            page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), 1 if all_values else 0, self.code, _stream()),
             "paged_attention_simt")
         return out
 
@@ -671,7 +676,7 @@ class Ops:
     def paged_attention_decode(self, q, out, k_pool, v_pool, page_stride, token_item, positions, block_table,
                                n_heads, n_kv_heads, head_dim, page_size, window, scale, max_kv_len,
                                target_ctas=1184, status=None, q_start=None, kv_len=None, merge="global",
-                               largest_cluster=8, token_row=None, softcap=None, sink=None):
+                               largest_cluster=8, token_row=None, softcap=None, sink=None, all_values=False):
         """Split-key attention for few query tokens (bfloat16).  ``max_kv_len`` bounds the context of
         every token in the call; it fixes the grid, so a CUDA graph passes the model's maximum.
         ``q_start`` / ``kv_len`` (the step's per-item arrays) let the kernel fetch keys older than this step
@@ -679,13 +684,15 @@ class Ops:
         merge through scratch in global memory) or "cluster" (they are a thread-block cluster and merge
         through shared memory; falls back to "global" where more than ``largest_cluster`` splits pay).
         ``block_table`` rows are indexed by ``token_row[t]`` (a table kept by request slot) or, without it, by
-        ``token_item[t]``.  ``softcap`` / ``sink`` as in :meth:`paged_attention_simt`."""
+        ``token_item[t]``.  ``softcap`` / ``sink`` / ``all_values`` as in
+        :meth:`paged_attention_simt`."""
         T = q.shape[0]
         _require(q, "q", torch.bfloat16)
         _require(out, "out", torch.bfloat16)
+        columns = n_heads * n_kv_heads if all_values else n_heads          # results per token
         plan = None
         if merge == "cluster":
-            plan = self.attention_cluster_plan(T, n_heads, head_dim, page_size, max_kv_len, target_ctas,
+            plan = self.attention_cluster_plan(T, columns, head_dim, page_size, max_kv_len, target_ctas,
                                                largest_cluster)
         part_acc = part_ml = counters = None
         if plan is not None:
@@ -693,14 +700,14 @@ class Ops:
             n_splits = cluster
         else:
             cluster = 1
-            split_tiles, n_splits = self.attention_split_plan(T, n_heads, head_dim, page_size, max_kv_len,
+            split_tiles, n_splits = self.attention_split_plan(T, columns, head_dim, page_size, max_kv_len,
                                                               target_ctas)
             if n_splits > 1:
-                if self._counters is None or self._counters.numel() < T * n_heads:
-                    self._counters = torch.zeros(max(1024, T * n_heads), dtype=torch.int32, device=q.device)
+                if self._counters is None or self._counters.numel() < T * columns:
+                    self._counters = torch.zeros(max(1024, T * columns), dtype=torch.int32, device=q.device)
                 counters = self._counters
-                part_acc = self.empty((T * n_heads * n_splits, head_dim), torch.float32, q.device)
-                part_ml = self.empty((T * n_heads * n_splits, 2), torch.float32, q.device)
+                part_acc = self.empty((T * columns * n_splits, head_dim), torch.float32, q.device)
+                part_ml = self.empty((T * columns * n_splits, 2), torch.float32, q.device)
         self.launches += 1
         _check(self.fast.ps_paged_attention_decode_ex(
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_pool), _ptr(v_pool),
@@ -708,12 +715,12 @@ class Ops:
             block_table.stride(0), _ptr(q_start), _ptr(kv_len), T, n_heads, n_kv_heads, head_dim,
             page_size, window or 0, scale, split_tiles, n_splits, cluster,
             _ptr(part_acc), _ptr(part_ml), _ptr(counters), _ptr(status), float(softcap or 0.0), _ptr(sink),
-            _stream()), "paged_attention_decode")
+            1 if all_values else 0, _stream()), "paged_attention_decode")
         return out
 
     def prefill_attention(self, q, out, k_pool, v_pool, page_stride, q_start, kv_len, block_table, first_item,
                           n_items, max_blocks, n_heads, n_kv_heads, head_dim, page_size, window, scale,
-                          item_row=None, softcap=None, sink=None):
+                          item_row=None, softcap=None, sink=None, all_values=False):
         """Tensor-core causal attention of prompt portions (bfloat16): items ``first_item ..`` of the step,
         ``max_blocks`` >= the number of 64-query blocks they make up.  ``q`` / ``out`` are the step's flat
         token arrays (row 0 = token 0).  ``item_row``: the block-table row of each item (a table kept by request
@@ -727,8 +734,8 @@ class Ops:
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_pool), _ptr(v_pool),
             page_stride, _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), _ptr(item_row),
             first_item, n_items, max_blocks, n_heads, n_kv_heads,
-            head_dim, page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), _stream()),
-            "prefill_attention")
+            head_dim, page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), 1 if all_values else 0,
+            _stream()), "prefill_attention")
         return out
 
     def shared_position_attention(self, q, out, k_pool, v_pool, page_stride, positions, block_table, token_row,
@@ -764,7 +771,7 @@ class Ops:
 
     def prefill_attention_tc(self, q, out, pool, cache_layer_local, q_start, kv_len, block_table, first_item,
                              n_items, max_blocks, n_heads, n_kv_heads, head_dim, page_size, window, scale,
-                             status=None, row_threads=0, item_row=None, softcap=None, sink=None):
+                             status=None, row_threads=0, item_row=None, softcap=None, sink=None, all_values=False):
         """tcgen05 causal attention of prompt portions (bfloat16, head size 64 or 128).  ``pool`` is the cache
         group's whole pool ``[pages, layers, planes, kv heads, page size, head dim]`` (one plane: the values are the keys); ``cache_layer_local`` the
         layer's index inside it; ``max_blocks`` >= the number of 128-query blocks of the items.
@@ -785,14 +792,14 @@ class Ops:
             (cache_layer_local * planes + planes - 1) * rows_per_tensor, page_rows,
             _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), _ptr(item_row), first_item,
             n_items, max_blocks, n_heads, n_kv_heads, head_dim, page_size, window or 0, scale, row_threads,
-            _ptr(status), float(softcap or 0.0), _ptr(sink), _stream()),
+            _ptr(status), float(softcap or 0.0), _ptr(sink), 1 if all_values else 0, _stream()),
             "prefill_attention_tc")
         return out
 
     def attention(self, q, k, v, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale,
-                  write_cache=True, softcap=None, sink=None, chunk=None):
-        """Write the step's keys and values into the pages, then attend from the pages.  ``softcap`` and
-        ``sink`` as in :meth:`paged_attention_simt`.  Besides "no later key", a query sees the last ``window``
+                  write_cache=True, softcap=None, sink=None, chunk=None, all_values=False):
+        """Write the step's keys and values into the pages, then attend from the pages.  ``softcap``, ``sink`` and
+        ``all_values`` as in :meth:`paged_attention_simt`.  Besides "no later key", a query sees the last ``window``
         keys, or (``chunk`` C instead of a window) the keys j of its own run of C positions,
         ``j // C == i // C``, runs counted from position 0 of the sequence; neither: every earlier key.  Below
         this method the two travel as one integer: the window, or minus the chunk."""
@@ -810,9 +817,10 @@ class Ops:
             # up to 256
             return self.paged_attention_simt(q, out, layer.k_pool, layer.v_pool, layer.page_stride,
                                              ctx.token_slot, ctx.positions, layer.block_table, n_heads,
-                                             n_kv_heads, head_dim, layer.page_size, window, scale, softcap, sink)
+                                             n_kv_heads, head_dim, layer.page_size, window, scale, softcap, sink,
+                                             all_values)
         return tensorcore.attention(self, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale,
-                                    softcap=softcap, sink=sink)
+                                    softcap=softcap, sink=sink, all_values=all_values)
 
     # ------------------------------------------------------------------ rotary positions + cache write
     def rotary_cache_write(self, q, k, v, inv_freq, rot_dims, interleaved, ctx, layer, n_heads, n_kv_heads,
@@ -1132,6 +1140,95 @@ class Ops:
                                         dtype_code(x_cast.dtype) if x_cast is not None else PS_F32, _ptr(y), x.numel(),
                                         _stream()), "depth_begin")
 
+    def sandwich_close(self, y, x, gain, y_scale, eps, next_gain=None, out=None, row_scale=None):
+        """x += gain * rms_norm(y_scale * y), y = 0 (float32 [T, H]; ``gain`` None: only y = 0), then what comes next reads
+        of the new x: ``out`` = rms_norm(x) * next_gain (compute type or float32), and / or ``row_scale`` float32 [T] =
+        1 / sqrt(mean(x^2) + eps); csrc/post_norm.cu."""
+        for name, tensor in (("y", y), ("x", x)):
+            _require(tensor, name, torch.float32)
+        T, H = x.shape
+        if y.shape != x.shape or not (x.is_contiguous() and y.is_contiguous()):
+            raise KernelError("sandwich_close: shapes do not match")
+        for name, vector, count in (("gain", gain, H), ("next_gain", next_gain, H), ("row_scale", row_scale, T)):
+            if vector is not None:
+                _require(vector, name, torch.float32)
+                if vector.numel() != count or not vector.is_contiguous():
+                    raise KernelError(f"sandwich_close: {name} does not fit")
+        if out is not None and (next_gain is None or out.shape != x.shape or not out.is_contiguous()):
+            raise KernelError("sandwich_close: the normed rows need a gain and the rows' shape")
+        self.launches += 1
+        _check(self.core.ps_sandwich_close(_ptr(y), _ptr(x), T, H, _ptr(gain), float(y_scale), float(eps), _ptr(next_gain),
+                                           _ptr(out), dtype_code(out.dtype) if out is not None else PS_F32,
+                                           _ptr(row_scale), _stream()), "sandwich_close")
+
+    # ------------------------------------------------------------------ heads mixed across heads
+    def head_mix(self, every, mix, out, n_heads, n_kv_heads, head_dim):
+        """out[t, h] = sum_g mix[h, g] * every[t, g, G(h)], G(h) = h // (n_heads / n_kv_heads): the results of a layer
+        whose heads' weights are mixed by ``mix`` (float32 [H, H]) before they meet the values, from what attention
+        leaves with ``all_values`` (``every`` [T, H * n_kv_heads * head_dim]); csrc/head_mix.cu."""
+        _require(every, "every", self.dtype)
+        _require(out, "out", self.dtype)
+        _require(mix, "mix", torch.float32)
+        T = every.shape[0]
+        if (every.shape[1] != n_heads * n_kv_heads * head_dim or out.shape != (T, n_heads * head_dim)
+                or mix.shape != (n_heads, n_heads) or not mix.is_contiguous() or every.stride(1) != 1 or out.stride(1) != 1):
+            raise KernelError("head_mix: shapes do not match")
+        self.launches += 1
+        _check(self.core.ps_head_mix(_ptr(every), every.stride(0), _ptr(mix), _ptr(out), out.stride(0), T, n_heads,
+                                     n_kv_heads, head_dim, self.code, _stream()), "head_mix")
+        return out
+
+    # ------------------------------------------------------------------ gated linear attention
+    GLA_CTAS = 592                # CTAs that the recurrence of prompt portions is cut into at most, about
+    GLA_RUN = 64                  # and tokens of a run at least
+    GLA_SCRATCH_BYTES = 256 << 20
+
+    def gla_segments(self, ctx, heads, dk, dv):
+        """Runs that a prompt portion is cut into: enough CTAs to fill the GPU, no run shorter than GLA_RUN tokens."""
+        long_items = ctx.num_items - ctx.num_short_items
+        longest = int(ctx.max_q_len)
+        if long_items <= 0 or longest < 2 * self.GLA_RUN or max(dk, dv) > 128:
+            return 1
+        wanted = min(self.GLA_CTAS // max(1, long_items * heads), longest // self.GLA_RUN,
+                     self.GLA_SCRATCH_BYTES // (4 * long_items * heads * dk * (dv + 1)))
+        return max(1, min(64, wanted))
+
+    def gla_recurrence(self, rows, offsets, a2, bias, tau, q_scale, gain, eps, out_scale, state, ctx, out, heads, dk, dv,
+                       segments=None):
+        """The gated linear recurrence of every entry of the step, tokens in order, from and into the slots' state
+        (csrc/gla.cu).  ``rows`` [T, *] (compute dtype): the stacked projections, in which q, k [heads * dk], v, g
+        [heads * dv] and the decay's inner numbers [rank] begin at the five ``offsets``; ``a2`` float32 [heads * dk,
+        rank] and ``bias`` float32 [heads * dk] make the decay's argument of them; ``gain`` float32 [dv]; ``state``
+        float32 [slots, >= heads * dk * dv]; ``out`` [T, heads * dv] in the compute dtype, multiplied by ``out_scale``."""
+        _require(rows, "rows", self.dtype)
+        _require(out, "out", self.dtype)
+        for name, tensor in (("a2", a2), ("bias", bias), ("gain", gain), ("state", state)):
+            _require(tensor, name, torch.float32)
+        T, rank = rows.shape[0], a2.shape[1]
+        ends = [offsets[0] + heads * dk, offsets[1] + heads * dk, offsets[2] + heads * dv, offsets[3] + heads * dv,
+                offsets[4] + rank]
+        if (min(offsets) < 0 or max(ends) > rows.shape[1] or rows.stride(1) != 1 or a2.shape[0] != heads * dk
+                or not a2.is_contiguous() or bias.numel() != heads * dk or gain.numel() != dv
+                or state.shape[1] < heads * dk * dv or state.stride(1) != 1 or out.shape != (T, heads * dv)
+                or out.stride(1) != 1):
+            raise KernelError("gla_recurrence: shapes do not match")
+        if segments is None:
+            segments = self.gla_segments(ctx, heads, dk, dv)
+        first_cut = ctx.num_short_items
+        run_state = run_decay = None
+        if segments > 1:
+            runs = (ctx.num_items - first_cut) * heads * segments
+            run_state = self.empty((runs, dk * dv), torch.float32, rows.device)
+            run_decay = self.empty((runs, dk), torch.float32, rows.device)
+        places = (ctypes.c_int * 5)(*[int(o) for o in offsets])
+        self.launches += 2 if segments > 1 else 1
+        _check(self.core.ps_gla_recurrence(_ptr(rows), rows.stride(0), ctypes.addressof(places), _ptr(a2), _ptr(bias), rank,
+                                           1.0 / float(tau), float(q_scale), _ptr(gain), float(eps), float(out_scale),
+                                           _ptr(state), state.stride(0), _ptr(ctx.q_start), _ptr(ctx.item_slot),
+                                           ctx.num_items, first_cut, segments, _ptr(run_state), _ptr(run_decay), _ptr(out),
+                                           out.stride(0), heads, dk, dv, self.code, _stream()), "gla_recurrence")
+        return out
+
     # ------------------------------------------------------------------ minGRU
     def mingru_scan(self, zug, width, state, ctx, out):
         """The gated recurrence of every entry of the step from and into the slots' state (csrc/mingru.cu).  ``zug``
@@ -1156,14 +1253,15 @@ class Ops:
         return out
 
     # ------------------------------------------------------------------ short convolution over time
-    def short_conv(self, u, weight, taps, conv_channels, state, ctx, out, blend=None):
+    def short_conv(self, u, weight, taps, conv_channels, state, ctx, out, blend=None, row_scale=None):
         """out[t, c] = sum_j weight[c, j] * u[t - taps + 1 + j, c] for the first ``conv_channels`` channels, the rest
         passed through; what lies before an entry's first token comes from ``state`` (float32
         [slots, (taps - 1) * conv_channels]: a request's last projected rows), which is then brought up to date
         (csrc/short_conv.cu).  ``u`` float32 [T, channels], ``out`` the same shape in the compute type.
         ``blend`` = (mode, first channel, heads, head slot, head values, shared float32 [T, heads * head values],
         mix float32 scalar): mode "store" leaves the convolved values of those heads in ``shared``, "mix" blends
-        them, v <- (1 - mix) v + mix * shared."""
+        them, v <- (1 - mix) v + mix * shared.  ``row_scale`` float32 [T]: row t of ``u`` is multiplied by row_scale[t]
+        wherever it is read (and kept)."""
         _require(u, "u", torch.float32)
         _require(out, "out", self.dtype)
         T, channels = u.shape
@@ -1179,6 +1277,10 @@ class Ops:
                 raise KernelError("short_conv: the state holds taps - 1 rows of the convolved channels")
         else:
             state = None
+        if row_scale is not None:
+            _require(row_scale, "row_scale", torch.float32)
+            if row_scale.numel() != T or not row_scale.is_contiguous():
+                raise KernelError("short_conv: one scale per row")
         mode, lo, heads, slot, values, shared, mix = 0, 0, 0, 1, 1, None, None
         if blend is not None:
             kind, lo, heads, slot, values, shared, mix = blend
@@ -1189,14 +1291,15 @@ class Ops:
             if mode == 2:
                 _require(mix, "mix", torch.float32)
         self.launches += 1
-        _check(self.core.ps_short_conv(_ptr(u), u.stride(0), _ptr(weight), taps, conv_channels, channels, _ptr(state),
+        _check(self.core.ps_short_conv(_ptr(u), u.stride(0), _ptr(weight), taps, conv_channels, channels,
+                                       _ptr(row_scale), _ptr(state),
                                        state.stride(0) if state is not None else 0, _ptr(ctx.token_item),
                                        _ptr(ctx.q_start), _ptr(ctx.item_slot), _ptr(out), out.stride(0), mode, lo, heads,
                                        slot, values, _ptr(shared), _ptr(mix) if mode == 2 else None, T, self.code,
                                        _stream()), "short_conv")
-        if state is not None:
+        if state is not None and not getattr(ctx, "single_tokens", False):     # (entries of one token have kept theirs)
             self.launches += 1
-            _check(self.core.ps_short_conv_keep(_ptr(u), u.stride(0), taps, conv_channels, _ptr(state), state.stride(0),
+            _check(self.core.ps_short_conv_keep(_ptr(u), u.stride(0), _ptr(row_scale), taps, conv_channels, _ptr(state), state.stride(0),
                                                 _ptr(ctx.q_start), _ptr(ctx.item_slot), ctx.num_items, _stream()),
                    "short_conv_keep")
         return out
@@ -1253,11 +1356,13 @@ class Ops:
 
     @staticmethod
     def _gate_form(form):
-        """(kind, limit, shared limit, alpha) of the inner activation: None / "silu" = silu(g) * u * weight;
+        """(kind, limit, shared limit, alpha) of the inner activation: None / "silu" = silu(g) * u * weight; "gelu_tanh" likewise;
         ("clamped_swish", limit, shared_limit, alpha): g' = min(weight * g, limit), u' = clamp(weight * u, +-limit),
         g' * sigmoid(alpha * g') * (u' + 1): the weight scales the expert's input."""
         if form is None or form == "silu":
             return 0, 0.0, 0.0, 0.0
+        if form == "gelu_tanh":
+            return 2, 0.0, 0.0, 0.0
         kind, limit, shared_limit, alpha = form
         if kind != "clamped_swish":
             raise KernelError(f"unknown gated form {kind!r}")

@@ -54,11 +54,15 @@ def linear(ops, a, w, bias, out, act=None, accumulate=False, status=None):
 SHARED_POSITION_FROM = 8       # short tokens of a step from which heads that share a key head run as query rows
 
 
-def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale, softcap=None, sink=None):
+def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale, softcap=None, sink=None,
+              all_values=False):
     """Short entries (fewer than ``ctx.LONG_ENTRY`` tokens: decode tokens, short portions) come first in the
     step's flat batch and go token by token through the split-key kernel; long portions go through the
     tensor-core prefill kernel in blocks of 64 queries.  ``softcap``: scores become softcap * tanh(score /
-    softcap); ``sink``: float32 [n_heads], exp(sink[h]) joins the softmax's denominator of head h."""
+    softcap); ``sink``: float32 [n_heads], exp(sink[h]) joins the softmax's denominator of head h.
+    ``all_values``: every query head meets the values of every key/value head (``Ops.head_mix`` reads the results)."""
+    all_values = all_values and n_kv_heads > 1
+    columns = n_heads * n_kv_heads if all_values else n_heads
     short_tokens = ctx.num_short_tokens
     long_items = ctx.num_items - ctx.num_short_items
     if long_items and head_dim > 128:
@@ -86,21 +90,22 @@ def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, sc
                                    layer.page_stride, ctx.token_item[:short_tokens], ctx.positions[:short_tokens],
                                    layer.block_table, n_heads, n_kv_heads, head_dim, layer.page_size, window, scale,
                                    ctx.max_kv_len, status=ctx.status, q_start=ctx.q_start, kv_len=ctx.kv_len, merge=merge,
-                                   token_row=ctx.token_slot[:short_tokens], softcap=softcap, sink=sink)
+                                   token_row=ctx.token_slot[:short_tokens], softcap=softcap, sink=sink, all_values=all_values)
     if long_items:
         if ops.prefill_tc_ok(head_dim, layer.page_size, q, out, getattr(layer, "pool", None)):
             # blocks of 128 queries: never more than the count of 64-query blocks
             # Two threads per query row halve the chain of each 128-key tile but leave one CTA per SM: worth it
             # when all blocks are resident at once, or nearly so while some block runs over many tiles.
-            blocks = -(-ctx.num_long_blocks // 2) * n_heads          # an upper bound of the 128-query blocks
+            blocks = -(-ctx.num_long_blocks // 2) * columns          # an upper bound of the 128-query blocks
             two = blocks <= 148 or (blocks <= 296 and ctx.max_kv_len >= 768)
             ops.prefill_attention_tc(q, out, layer.pool, layer.pool_layer, ctx.q_start, ctx.kv_len, layer.block_table,
                                      ctx.num_short_items, long_items, ctx.num_long_blocks, n_heads, n_kv_heads,
                                      head_dim, layer.page_size, window, scale, status=ctx.status,
-                                     row_threads=2 if two else 1, item_row=ctx.item_slot, softcap=softcap, sink=sink)
+                                     row_threads=2 if two else 1, item_row=ctx.item_slot, softcap=softcap, sink=sink,
+                                     all_values=all_values)
         else:
             ops.prefill_attention(q, out, layer.k_pool, layer.v_pool, layer.page_stride, ctx.q_start, ctx.kv_len,
                                   layer.block_table, ctx.num_short_items, long_items, ctx.num_long_blocks, n_heads,
                                   n_kv_heads, head_dim, layer.page_size, window, scale, item_row=ctx.item_slot,
-                                  softcap=softcap, sink=sink)
+                                  softcap=softcap, sink=sink, all_values=all_values)
     return out

@@ -87,11 +87,11 @@ class Model:
 
     # ------------------------------------------------------------------ cache needs
     def _needs(self, which: str) -> list:
-        """Per cache layer, what the mixer of the run(s) that use it asks for."""
+        """Per cache layer, what the block (its mixer, mostly) of the run(s) that use it asks for."""
         needs = [None] * self.spec.num_cache_layers
         seen = [False] * self.spec.num_cache_layers
         for entry in self.spec.schedule:
-            need = getattr(self.blocks[entry.layer].mixer, which)()
+            need = getattr(self.blocks[entry.layer], which)()
             if seen[entry.cache_layer] and needs[entry.cache_layer] != need:
                 # runs that read the same rows through different masks: the rows stay for the longer look back
                 both = needs[entry.cache_layer]

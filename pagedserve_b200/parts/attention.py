@@ -132,10 +132,18 @@ class RotaryAttention(Mixer):
     ``slot_dim`` numbers, the larger of the two rounded up: the projections' matrices get zero rows there (zero keys add nothing to a score, zero values
     give zeros that the output projection's zero columns ignore), and every attention kernel runs unchanged.
 
+    ``head_norm`` without names divides by the root mean square alone; a turn keeps a head's length, so it makes no
+    difference whether that happens before the turn or behind it.  ``unit_sink``: a one in every head's denominator (a
+    sink of score 0 without a tensor).  ``talk_name``: the heads' weights (softmax, sinks in the denominators) are mixed
+    across heads before they meet the values, w'_h = sum_g M[h, g] w_g, M the tensor ``talk_name`` [H, H]; head h applies
+    w'_h to the values of its own key/value head.  This is linear in the weights: attention runs with every query head
+    meeting the values of every key/value head, and ``ops.head_mix`` adds the results up.
+
     params: hidden_size, n_heads, n_kv_heads, head_dim, v_dim (head_dim), scale, window, chunk, softcap,
     rotary (dict or None), q_name, k_name, v_name (None: values are the unturned keys), out_name, sink_name (None: no
-    sinks), bias (False; tensors ``<name>.b``), head_norm (None, or dict(q_name, k_name, eps)), kv_source (True),
-    conv (None), value_mix (None), gate_name (None), init_std, out_init_std.
+    sinks), unit_sink (False), bias (False; tensors ``<name>.b``), out_bias (False; likewise), head_norm (None, or
+    dict(q_name, k_name, eps), the names None for norms without gains), kv_source (True), conv (None), value_mix (None),
+    gate_name (None), talk_name (None), init_std, out_init_std.
     """
 
     graph_safe = True
@@ -153,9 +161,12 @@ class RotaryAttention(Mixer):
         self.head_norm = p.get("head_norm")
         if not self.has_v and self.v_dim != self.dim:
             raise ValueError("values that are the unturned keys have the keys' size")
+        rotary = p.get("rotary") or dict(dims=0, base=10000.0)
+        # heads that are normed, a stretched or slowed rotation: the kernel that turns heads as they are does not do it
+        prepared = self.head_norm is not None or bool(rotary.get("scaling"))
         # what a head takes in the cache and in the attention kernels
         slot = max(self.dim, self.v_dim)
-        if env.dtype == torch.bfloat16 and self.has_v:
+        if env.dtype == torch.bfloat16 and (self.has_v or prepared):
             slot = -(-slot // 16) * 16                 # the tensor-core attention kernels take multiples of 16
         self.slot_dim = slot
         if not (0 < self.slot_dim <= 256):
@@ -164,13 +175,12 @@ class RotaryAttention(Mixer):
             raise ValueError("window must be positive")
         if p.get("chunk") is not None and (p["chunk"] <= 0 or p.get("window") is not None):
             raise ValueError("chunk must be positive, and excludes a window")
-        rotary = p.get("rotary") or dict(dims=0, base=10000.0)
         # the plain kernel turns heads as they are; norms, padded heads, borrowed keys and stretched rotations take
         # the other one
-        self.plain = (self.head_norm is None and self.slot_dim == self.dim == self.v_dim and self.kv_source
-                      and not rotary.get("scaling"))
-        if not self.plain and not self.has_v:
-            raise ValueError("rotary_attention: head norms, padded heads and borrowed keys need a value projection")
+        self.plain = not prepared and self.slot_dim == self.dim == self.v_dim and self.kv_source
+        if p.get("sink_name") and p.get("unit_sink"):
+            raise ValueError("rotary_attention: learned sinks or a sink of one, not both")
+        self.talk_name = p.get("talk_name")
         self.q_width = p["n_heads"] * self.slot_dim
         self.kv_width = p["n_kv_heads"] * self.slot_dim
         from pagedserve_b200.parts.positions import RotaryPositions
@@ -230,13 +240,17 @@ class RotaryAttention(Mixer):
             specs.append((ParamSpec(self._n(self.value_mix["name"]), (), "vector"), ("normal", 0.3)))
         if self.gate_name:
             specs.append((ParamSpec(self._n(self.gate_name), (H * self.v_dim, W), "matmul"), ("normal", std)))
-        if self.head_norm:
+        if self.head_norm and self.head_norm.get("q_name"):
             specs.append((ParamSpec(self._n(self.head_norm["q_name"]), (self.dim,), "vector"), ("ones_plus_normal", 0.1)))
             if self.kv_source:
                 specs.append((ParamSpec(self._n(self.head_norm["k_name"]), (self.dim,), "vector"),
                               ("ones_plus_normal", 0.1)))
         specs.append((ParamSpec(self._n(p["out_name"]), (W, H * self.v_dim), "matmul"),
                       ("normal", p.get("out_init_std", std))))
+        if p.get("out_bias"):
+            specs.append((ParamSpec(self._n(p["out_name"] + ".b"), (W,), "vector"), ("normal", 0.3)))
+        if self.talk_name:
+            specs.append((ParamSpec(self._n(self.talk_name), (H, H), "vector"), ("eye_plus_normal", 0.3)))
         if p.get("sink_name"):
             specs.append((ParamSpec(self._n(p["sink_name"]), (H,), "vector"), ("normal", 1.0)))
         return specs
@@ -278,18 +292,60 @@ class RotaryAttention(Mixer):
         if self.v_dim != self.slot_dim:                             # zero columns where the heads are padded
             w_out = self._padded_rows(w_out.t().contiguous(), H, self.v_dim).t().contiguous()
         self.w_out = w_out
+        self.b_out = tensors[self._n(p["out_name"] + ".b")].contiguous() if p.get("out_bias") else None
         self.sink = tensors[self._n(p["sink_name"])].contiguous() if p.get("sink_name") else None
+        if p.get("unit_sink"):
+            self.sink = torch.zeros(H, dtype=torch.float32, device=self.w_in.device)
+        self.talk = tensors[self._n(self.talk_name)].contiguous() if self.talk_name else None
         self.q_gain = self.k_gain = None
-        if self.head_norm:
+        if self.head_norm and not self.head_norm.get("q_name"):
+            self.q_gain = self.k_gain = torch.ones(self.dim, dtype=torch.float32, device=self.w_in.device)
+        elif self.head_norm:
             self.q_gain = tensors[self._n(self.head_norm["q_name"])].contiguous()
             if self.kv_source:
                 self.k_gain = tensors[self._n(self.head_norm["k_name"])].contiguous()
+
+    def joint_in(self):
+        if self.staged:
+            raise ValueError("rotary_attention: a convolution, mixed values or a gate need a product of their own")
+        return self.w_in, self.b_in
+
+    def joint_out(self):
+        return self.w_out, self.b_out
+
+    def joint_mix(self, projected, context, ctx, layer, factor=1.0):
+        if factor != 1.0:
+            raise ValueError("rotary_attention: attention's result is not scaled")
+        p = self.params
+        ops = self.env.ops
+        H, G, D = p["n_heads"], p["n_kv_heads"], self.slot_dim
+        q = projected[:, :self.q_width]
+        k = v = None
+        if self.kv_source:
+            k = projected[:, self.q_width:self.q_width + self.kv_width]
+            v = projected[:, self.q_width + self.kv_width:self.q_width + 2 * self.kv_width] if self.has_v else None
+        write_cache = p.get("write_cache", True) and self.kv_source
+        if self.plain:
+            self.rotary.turn_and_store(q, k, v, ctx, layer, H, G, write_cache=write_cache)
+        else:
+            rotary = self.rotary.params
+            ops.head_norm_rotary_cache_write(
+                q, k, k if v is None else v, self.q_gain, self.k_gain,
+                float(self.head_norm["eps"]) if self.head_norm else 0.0,
+                self.rotary.inv_freq_split(), rotary["dims"], rotary.get("interleaved", True), self.dim, ctx, layer,
+                H, G, D, write_cache=write_cache, amplitude=self.rotary.amplitude)
+        mixes = self.talk is not None
+        result = ops.empty((projected.shape[0], H * G * D), self.env.dtype, projected.device) if mixes else context
+        ops.attention(q, k, v, result, ctx, layer, H, G, D, p.get("window"), float(p["scale"]), write_cache=False,
+                      softcap=p.get("softcap"), sink=self.sink, chunk=p.get("chunk"), all_values=mixes)
+        if mixes:
+            ops.head_mix(result, self.talk, context, H, G, D)
 
     def forward(self, x, residual, ctx, layer):
         p = self.params
         ops = self.env.ops
         tokens = x.shape[0]
-        H, G, D = p["n_heads"], p["n_kv_heads"], self.slot_dim
+        G, D = p["n_kv_heads"], self.slot_dim
         gate = None
         if self.staged:
             # float32 rows out of the product; one kernel convolves q, k and v over time from the request's kept
@@ -317,26 +373,11 @@ class RotaryAttention(Mixer):
         else:
             projected = ops.empty((tokens, self.w_in.shape[0]), self.env.dtype, residual.device)
             ops.linear(x, self.w_in, self.b_in, projected)
-        q = projected[:, :self.q_width]
-        k = v = None
-        if self.kv_source:
-            k = projected[:, self.q_width:self.q_width + self.kv_width]
-            v = projected[:, self.q_width + self.kv_width:self.q_width + 2 * self.kv_width] if self.has_v else None
-        write_cache = p.get("write_cache", True) and self.kv_source
-        if self.plain:
-            self.rotary.turn_and_store(q, k, v, ctx, layer, H, G, write_cache=write_cache)
-        else:
-            rotary = self.rotary.params
-            ops.head_norm_rotary_cache_write(
-                q, k, v, self.q_gain, self.k_gain, float(self.head_norm["eps"]) if self.head_norm else 0.0,
-                self.rotary.inv_freq_split(), rotary["dims"], rotary.get("interleaved", True), self.dim, ctx, layer,
-                H, G, D, write_cache=write_cache, amplitude=self.rotary.amplitude)
         context = ops.empty((tokens, self.q_width), self.env.dtype, residual.device)
-        ops.attention(q, k, v, context, ctx, layer, H, G, D, p.get("window"), float(p["scale"]), write_cache=False,
-                      softcap=p.get("softcap"), sink=self.sink, chunk=p.get("chunk"))
+        self.joint_mix(projected, context, ctx, layer)
         if gate is not None:
             ops.sigmoid_gate(context, gate)
-        ops.linear(context, self.w_out, None, residual, accumulate=True)
+        ops.linear(context, self.w_out, self.b_out, residual, accumulate=True)
 
 
 @register_part("mixer", "latent_attention")

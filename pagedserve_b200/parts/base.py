@@ -147,7 +147,28 @@ class Mixer(Part):
     def state_need(self) -> Optional[StateNeed]:
         return None
 
+    # What ``forward`` adds is the mixer's result divided by this common factor (1 for nearly all of them): a block that
+    # norms the result multiplies by it first (``Block.takes_output_scale``), other blocks refuse such a mixer.
+    output_scale = 1.0
+
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, layer: LayerContext) -> None:
+        raise NotImplementedError
+
+    # A mixer that can stand beside others, behind one product that makes all their inputs and in front of one that
+    # takes all their results (``parts/parallel.py``), cuts its ``forward`` into these.
+    def joint_in(self):
+        """(matrix [rows, hidden], bias [rows] or None) of its projections, stacked; after ``bind``."""
+        raise NotImplementedError
+
+    def joint_out(self):
+        """(matrix [hidden, columns], bias [hidden] or None) of its output projection."""
+        raise NotImplementedError
+
+    scales_joint = False        # whether ``joint_mix`` can multiply its result by a factor in float32
+
+    def joint_mix(self, projected: torch.Tensor, context: torch.Tensor, ctx, layer: LayerContext, factor: float = 1.0) -> None:
+        """From its columns of the projections' rows (compute dtype) to its columns of the rows that the output
+        projection reads."""
         raise NotImplementedError
 
 
@@ -166,8 +187,19 @@ class Block(Part):
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.norms = norms
+        if mixer.output_scale != 1.0 and not self.takes_output_scale:
+            raise ValueError("this arrangement cannot multiply a mixer's result by a factor")
 
     required_norms: Tuple[str, ...] = ()
+    takes_output_scale = False
+
+    # What a run of the layer needs of the cache: the mixer's needs, unless the arrangement keeps state of its own
+    # (``state_need``: it then hands the mixer its share of ``layer.state``).
+    def cache_need(self) -> Optional[KVNeed]:
+        return self.mixer.cache_need()
+
+    def state_need(self) -> Optional[StateNeed]:
+        return self.mixer.state_need()
 
     def forward(self, hidden: torch.Tensor, ctx, layer: LayerContext) -> None:
         raise NotImplementedError

@@ -4,7 +4,9 @@ from __future__ import annotations
 
 import torch
 
+from pagedserve_b200.cache.manager import StateNeed
 from pagedserve_b200.parts.base import Block, register_part
+from pagedserve_b200.parts.parallel import padded, state_share
 from pagedserve_b200.weights.loader import ParamSpec
 
 
@@ -211,6 +213,137 @@ class PostNormBlock(Block):
         if not alone:
             self.feed_forward.forward(carrier.x_cast, carrier.y, ctx)
             self._close(carrier, self.norms["post_feed_forward"], True)
+
+    def end(self, carrier, ctx):
+        return carrier.x
+
+
+class SandwichCarrier:
+    """What runs through the layers of a model that norms what its sublayers read and what they return: the float32 rows
+    ``x``, the zeroed float32 rows ``y`` a sublayer adds its result into, and ``inverse`` [T]: one over the root mean
+    square of every row of ``x``, which the next layer's first norm needs of it."""
+
+    def __init__(self, x, y, inverse):
+        self.x = x
+        self.y = y
+        self.inverse = inverse
+
+
+@register_part("block", "sandwich_norm")
+class SandwichNormBlock(Block):
+    """x <- x + s1 * post(mixer(c(pre(x)))); x <- x + s2 * post(feed_forward(pre(x))): norms before and after each
+    sublayer (four RMS norms without a mean; gains of one number or of the row's width), ``s1`` and ``s2`` a factor per
+    coordinate (``scales``: the tensors' names), and, with ``conv`` = dict(taps, name), c(h) = h + conv(h): a causal
+    convolution over time on each channel, conv(h)_t = sum_j w[:, j] h_(t - taps + 1 + j) with zeros before the
+    sequence's start; w [W, taps].  A layer whose feed-forward is the ``none`` part has the first sublayer only.  The
+    residual rows, norms, sums and the convolution are float32; a sublayer reads rows of the compute type.
+
+    A request keeps, in every layer, the last taps - 1 rows that the convolution read (float32, divided by their root
+    mean square, without the gain, which is folded into the taps) in front of the mixer's own state.
+
+    A sublayer adds its result into a zeroed row exactly as it would into the residual row of a pre-norm layer, so every
+    mixer and feed-forward works here unchanged.  One kernel (``ops.sandwich_close``) then norms that row, adds it, clears
+    it, and prepares what comes next: the feed-forward's normed rows, or the root mean square that the next layer's
+    convolution kernel (or the model's last norm) applies when it reads the rows.
+
+    params: scales = dict(mixer, feed_forward), conv (None), init_std."""
+
+    graph_safe = True
+    takes_output_scale = True
+
+    @property
+    def required_norms(self):
+        if getattr(self.feed_forward, "is_empty", False):
+            return ("pre_mixer", "post_mixer")
+        return ("pre_mixer", "post_mixer", "pre_feed_forward", "post_feed_forward")
+
+    def __init__(self, params, prefix, env, mixer, feed_forward, norms):
+        super().__init__(params, prefix, env, mixer, feed_forward, norms)
+        conv = self.params.get("conv")
+        if conv is not None and not (isinstance(conv["taps"], int) and 1 <= conv["taps"] <= 16):
+            raise ValueError("sandwich_norm: a convolution has 1 to 16 taps")
+        for norm in norms.values():
+            if norm.params.get("has_mean", True) or norm.params.get("has_bias", True):
+                raise ValueError("sandwich_norm: the norms are RMS norms without a bias")
+        self.width = norms["pre_mixer"].params["width"]
+        self.taps = conv["taps"] if conv is not None else 1
+        self.kept = (self.taps - 1) * self.width
+
+    def state_need(self):
+        own, need = self.kept, self.mixer.state_need()
+        if need is None:
+            return StateNeed((own,), "float32") if own else None
+        if not own:
+            return need
+        if need.dtype != "float32" or len(need.shape) != 1:
+            raise ValueError("sandwich_norm: a mixer's state is rows of float32 numbers")
+        return StateNeed((padded(own) + need.shape[0],), "float32")
+
+    def param_specs(self):
+        p, std = self.params, self.params.get("init_std", 0.1)
+        names = [p["scales"]["mixer"]]
+        if not getattr(self.feed_forward, "is_empty", False):
+            names.append(p["scales"]["feed_forward"])
+        specs = [(ParamSpec(self._n(name), (self.width,), "vector"), ("ones_plus_normal", std)) for name in names]
+        if p.get("conv"):
+            specs.append((ParamSpec(self._n(p["conv"]["name"]), (self.width, self.taps), "vector"),
+                          ("normal", 0.5 * self.taps ** -0.5)))
+        return specs
+
+    def bind(self, tensors):
+        # (the blocks are bound before their norms: the products with the norms' gains are formed when first needed)
+        p = self.params
+        self._tensors = {role: tensors[self._n(name)] for role, name in p["scales"].items()
+                         if self._n(name) in tensors}
+        self._taps = tensors[self._n(p["conv"]["name"])] if p.get("conv") else None
+        self._gains = None
+
+    def _folded(self):
+        """(gain behind the mixer, gain behind the feed-forward, taps of the rows divided by their root mean square)."""
+        if self._gains is None:
+            norms, scales = self.norms, self._tensors
+            after_mixer = (norms["post_mixer"].weight * scales["mixer"]).contiguous()
+            after_ff = None
+            if "post_feed_forward" in norms:
+                after_ff = (norms["post_feed_forward"].weight * scales["feed_forward"]).contiguous()
+            taps = torch.zeros((self.width, self.taps), dtype=torch.float32, device=after_mixer.device)
+            if self._taps is not None:
+                taps += self._taps
+            taps[:, -1] += 1.0                                        # h itself
+            self._gains = (after_mixer, after_ff, (taps * norms["pre_mixer"].weight[:, None]).contiguous())
+        return self._gains
+
+    def begin(self, hidden, ctx):
+        ops = self.env.ops
+        y = ops.empty(hidden.shape, torch.float32, hidden.device)
+        inverse = ops.empty((hidden.shape[0],), torch.float32, hidden.device)
+        ops.sandwich_close(y, hidden, None, 1.0, self.norms["pre_mixer"].params["eps"], row_scale=inverse)
+        return SandwichCarrier(hidden, y, inverse)
+
+    def forward(self, hidden, ctx, layer):
+        carrier, ops = hidden, self.env.ops
+        after_mixer, after_ff, taps = self._folded()
+        own = layer
+        kept = None
+        if layer.state is not None:
+            if self.kept:
+                kept = layer.state[:, :self.kept]
+                at = padded(self.kept)
+                own = state_share(layer, at, layer.state.shape[1] - at) if layer.state.shape[1] > at else layer
+        x = carrier.x
+        h = ops.empty(x.shape, self.env.dtype, x.device)
+        ops.short_conv(x, taps, self.taps, self.width, kept, ctx, h, row_scale=carrier.inverse)
+        self.mixer.forward(h, carrier.y, ctx, own)
+        alone = getattr(self.feed_forward, "is_empty", False)
+        eps = self.norms["post_mixer"].params["eps"]
+        if alone:
+            ops.sandwich_close(carrier.y, x, after_mixer, self.mixer.output_scale, eps, row_scale=carrier.inverse)
+            return
+        h = ops.empty(x.shape, self.env.dtype, x.device)
+        ops.sandwich_close(carrier.y, x, after_mixer, self.mixer.output_scale, eps,
+                           next_gain=self.norms["pre_feed_forward"].weight, out=h)
+        self.feed_forward.forward(h, carrier.y, ctx)
+        ops.sandwich_close(carrier.y, x, after_ff, 1.0, eps, row_scale=carrier.inverse)
 
     def end(self, carrier, ctx):
         return carrier.x

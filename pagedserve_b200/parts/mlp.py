@@ -14,8 +14,8 @@ ACTIVATIONS = ("gelu_tanh", "gelu_erf", "relu_squared", "silu")
 class DenseMLP(FeedForward):
     """residual += act(x W_up + b_up) W_down + b_down
     (reference: src/model/paged_decoder.py:178-179, 224-228, 273-280),
-    or, with ``gate_name``, the gated form residual += (act(x W_gate) * (x W_up)) W_down (activation 'silu', no
-    biases): gate and up run as one product over the stacked matrices, one elementwise kernel forms the inner row.
+    or, with ``gate_name``, the gated form residual += (act(x W_gate) * (x W_up)) W_down (activation 'silu' or
+    'gelu_tanh', no biases): gate and up run as one product over the stacked matrices, one elementwise kernel forms the inner row.
     params: hidden_size, inner_size, activation ('gelu_tanh' | 'gelu_erf' | 'relu_squared' = max(z, 0)^2 | 'silu'),
     has_bias,
     stored_in_out, up_name, down_name, gate_name (None), init_std, out_init_std."""
@@ -27,8 +27,9 @@ class DenseMLP(FeedForward):
         super().__init__(params, prefix, env)
         if self.params["activation"] not in ACTIVATIONS:
             raise ValueError(f"unsupported activation {self.params['activation']!r}; one of {ACTIVATIONS}")
-        if self.params.get("gate_name") and (self.params["activation"] != "silu" or self.params.get("has_bias", True)):
-            raise ValueError("dense_mlp: the gated form is silu(gate) * up without biases")
+        if self.params.get("gate_name") and (self.params["activation"] not in ("silu", "gelu_tanh")
+                                             or self.params.get("has_bias", True)):
+            raise ValueError("dense_mlp: the gated form is silu(gate) * up or gelu_tanh(gate) * up without biases")
 
     def _matrix(self, name, n_out, n_in, std):
         flip = self.params.get("stored_in_out", False)
@@ -66,7 +67,7 @@ class DenseMLP(FeedForward):
         if self.w_gate_up is not None:
             gate_up = ops.empty((x.shape[0], 2 * p["inner_size"]), self.env.dtype, x.device)
             ops.linear(x, self.w_gate_up, None, gate_up)
-            ops.moe_gate_mul(gate_up, None, None, inner, 0, p["inner_size"])
+            ops.moe_gate_mul(gate_up, None, None, inner, 0, p["inner_size"], form=p["activation"])
         else:
             ops.linear(x, self.w_up, self.b_up, inner, act=p["activation"])
         ops.linear(inner, self.w_down, self.b_down, residual, accumulate=True)

@@ -32,7 +32,9 @@ class LayerNorm(Norm):
     fused kernel src/kernels/triton_residual_layernorm.py:25-40.
     params: width, eps, name, has_mean (False gives the RMS form), has_bias, init_std,
     weight_offset (a constant added to the stored weight once, in float32, when it is bound: 1.0 for
-    gains that are stored as their distance from one; random weights are then drawn around zero).
+    gains that are stored as their distance from one; random weights are then drawn around zero),
+    scalar (the stored weight is one number for the whole row), weight_factor (a constant that multiplies the weight
+    once, in float32, when it is bound: a factor that the design puts on what the norm's one consumer makes of it).
     """
 
     graph_safe = True
@@ -40,7 +42,8 @@ class LayerNorm(Norm):
     def param_specs(self):
         p = self.params
         centred = bool(p.get("weight_offset"))
-        specs = [(ParamSpec(self._n(p["name"] + ".weight"), (p["width"],), "vector"),
+        shape = () if p.get("scalar") else (p["width"],)
+        specs = [(ParamSpec(self._n(p["name"] + ".weight"), shape, "vector"),
                   ("normal" if centred else "ones_plus_normal", p.get("init_std", 0.0)))]
         if p.get("has_bias", True):
             specs.append((ParamSpec(self._n(p["name"] + ".bias"), (p["width"],), "vector"),
@@ -52,6 +55,10 @@ class LayerNorm(Norm):
         self.weight = tensors[self._n(p["name"] + ".weight")]
         if p.get("weight_offset"):
             self.weight = self.weight + float(p["weight_offset"])        # float32: the "vector" role
+        if p.get("scalar"):
+            self.weight = self.weight.reshape(1).expand(p["width"]).contiguous()
+        if p.get("weight_factor", 1.0) != 1.0:
+            self.weight = self.weight * float(p["weight_factor"])
         self.bias = tensors[self._n(p["name"] + ".bias")] if p.get("has_bias", True) else None
 
     def defer(self, x, rows=None):

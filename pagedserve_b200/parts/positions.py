@@ -52,6 +52,10 @@ class RotaryPositions(PositionEncoding):
     hi = min(ceil(index(slow)), dims - 1), pair i keeps its frequency f_i below lo, turns at f_i / factor above hi and
     at the blend f_i / factor * r + f_i * (1 - r), r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), between; every
     sine and cosine is multiplied by ``amplitude`` = 0.1 ln(factor) + 1.
+    ``scaling`` = dict(factor) alone slows every pair down: f_i / factor, amplitude 1.
+    ``scaling`` = dict(factor, low, high, original), amplitude 1, goes by the turns a pair makes in ``original``
+    positions, n_i = original * f_i / (2 pi): above ``high`` the pair keeps f_i, below ``low`` it turns at f_i / factor,
+    and between, with s = (n_i - low) / (high - low), at (1 - s) f_i / factor + s f_i.
     params: dims, base, interleaved, head_dim, scaling (None)."""
 
     graph_safe = True
@@ -65,17 +69,21 @@ class RotaryPositions(PositionEncoding):
             raise ValueError("rotary: base must be positive")
         self._inv_freq = None
         scaling = p.get("scaling")
-        if scaling is not None and not (scaling["factor"] > 0 and scaling["original"] > 0 and scaling["fast"] > 0
-                                        and scaling["slow"] > 0):
-            raise ValueError("rotary: scaling needs positive factor, original, fast and slow")
+        if scaling is not None:
+            if set(scaling) not in ({"factor", "original", "fast", "slow"}, {"factor", "original", "low", "high"}, {"factor"}):
+                raise ValueError("rotary: scaling is (factor), (factor, original, fast, slow) or (factor, original, low, high)")
+            if not all(value > 0 for value in scaling.values()):
+                raise ValueError("rotary: scaling needs positive numbers")
+            if "low" in scaling and not scaling["low"] < scaling["high"]:
+                raise ValueError("rotary: scaling.low must lie below scaling.high")
 
     @property
     def amplitude(self) -> float:
-        """What every sine and cosine is multiplied by (1 without ``scaling``)."""
+        """What every sine and cosine is multiplied by (1 unless ``scaling`` is of the stretching kind)."""
         import math
 
         scaling = self.params.get("scaling")
-        return 0.1 * math.log(scaling["factor"]) + 1.0 if scaling else 1.0
+        return 0.1 * math.log(scaling["factor"]) + 1.0 if scaling and "fast" in scaling else 1.0
 
     def _frequencies(self):
         """The frequencies of the pairs in float64."""
@@ -87,7 +95,13 @@ class RotaryPositions(PositionEncoding):
         index = torch.arange(dims // 2, dtype=torch.float64)
         table = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * index / max(dims, 1))
         scaling = self.params.get("scaling")
-        if scaling and dims:
+        if scaling and dims and set(scaling) == {"factor"}:
+            table = table / float(scaling["factor"])
+        elif scaling and dims and "low" in scaling:
+            turns = float(scaling["original"]) * table / (2.0 * math.pi)
+            share = torch.clamp((turns - float(scaling["low"])) / float(scaling["high"] - scaling["low"]), 0.0, 1.0)
+            table = (1.0 - share) * table / float(scaling["factor"]) + share * table
+        elif scaling and dims:
             place = lambda turns: dims * math.log(scaling["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
             lo = max(math.floor(place(scaling["fast"])), 0)
             hi = min(math.ceil(place(scaling["slow"])), dims - 1)
