@@ -1215,6 +1215,8 @@ class Ops:
         if segments is None:
             segments = self.gla_segments(ctx, heads, dk, dv)
         first_cut = ctx.num_short_items
+        if first_cut >= ctx.num_items:
+            segments = 1
         run_state = run_decay = None
         if segments > 1:
             runs = (ctx.num_items - first_cut) * heads * segments
