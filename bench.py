@@ -307,7 +307,9 @@ def _run_reference(args, ref):
 # Zositar (chunked attention with normed heads and borrowed caches, routed experts with clamped activations and a
 # gated dense feed-forward) beside a Tefopel of attention layers only; Pagatar (layers that norm their sublayers'
 # results and end with an average over depth, a gated recurrence, latent attention without a window, attention with
-# short convolutions, routed experts) beside a Gozunex of equal width, depth, heads, latent and experts.
+# short convolutions, routed experts) beside a Gozunex of equal width, depth, heads, latent and experts; Suvunex (norms
+# before and after each sublayer, attention beside gated linear attention, attention with mixed heads) beside a Tefopel in
+# which every other layer is recurrent.
 DESIGN_SIZES = {"w1024": "w1024", "w2048": "w2048"}      # named sizes of config/tefopel.py and config/gozunex.py
 DESIGN_CONTEXT = 2048
 
@@ -332,8 +334,16 @@ def design_arm(args):
     steps, warmup = min(args.steps, 64), max(args.warmup, 3)
 
     def configs(name):
-        from pagedserve_b200.config import gozunex, pagatar, tefopel, zositar
+        from pagedserve_b200.config import gozunex, pagatar, suvunex, tefopel, zositar
 
+        if args.design == "suvunex":
+            # Tefopel of equal size: same width, depth, heads and head size, a recurrent layer wherever the design has a
+            # recurrence beside attention, windows that see every key, and a dense feed-forward that makes the weights equal
+            size = suvunex.NAMED_CONFIGS["suvunex-" + name]
+            like = tefopel.repeating_config(width=size["width"], heads=size["heads"], head_dim=size["head_dim"],
+                                            ff=size["width"] * 35 // 8, layers=size["layers"],
+                                            wkv_heads=size["width"] // 64, window=DESIGN_CONTEXT, vocab=size["vocab"], every=2)
+            return size, {"suvunex": suvunex.named_config("suvunex-" + name), "tefopel": like}
         if args.design == "pagatar":
             # Gozunex of equal size: same width, depth, heads, flat and turning sizes, latent, experts and vocabulary;
             # its windows as long as the chunks, its recurrent layers where the gated recurrence stands, two residual
@@ -465,6 +475,49 @@ def design_arm(args):
             run = microbench.time_experts(2048, width, size["experts"], size["top"], size["ff"])
             kernels[f"experts_2048_tokens_{name}"] = {**run, "frac_tensor": run["tflops"] / tensor,
                                                       "dense_frac_tensor": run["dense_tflops"] / tensor}
+    elif args.dtype == "bfloat16" and not args.skip_points and args.design == "suvunex":
+        from pagedserve_b200.config import suvunex
+
+        hbm, tensor = peaks["hbm_gbs"], peaks["bf16_tflops"]
+        kernels = report["kernels"]
+
+        def of_hbm(run):
+            return {**run, "frac_hbm": run["gbs"] / hbm}
+
+        def of_tensor(run):
+            return {**run, "frac_tensor": run["tflops"] / tensor}
+
+        for name in (args.design_sizes.split(",") if args.design_sizes else DESIGN_SIZES):
+            size = suvunex.NAMED_CONFIGS["suvunex-" + name]
+            H, d, width, G = size["heads"], size["head_dim"], size["width"], suvunex.repeating_config(**size).layers[0][
+                "mixer"]["left"]["kv_heads"]
+            # the two recurrences, each with the heads it has at this width
+            for label, items, each in (("prefill_2x1024", 2, 1024), ("decode_b64", 64, 1), ("decode_b8", 8, 1)):
+                kernels[f"recurrence_{label}_{name}"] = {
+                    "tefopel": of_hbm(microbench.time_wkv(items, each, width // 64, 64, width)),
+                    "suvunex": of_hbm(microbench.time_gla(items, each, H, d, d))}
+            # attention whose heads are mixed, with the mixing kernel, and plain attention of equal heads
+            for batch in (8, 64):
+                kernels[f"decode_attention_b{batch}_{name}"] = {
+                    "tefopel": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, softcap=50.0, sink=True)),
+                    "suvunex_left": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, sink=True)),
+                    "suvunex_mixed": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, sink=True, mixed=True))}
+            kernels[f"prefill_attention_{name}"] = {
+                "tefopel": of_tensor(microbench.time_prefill_attention(2, 1024, H, G, d, softcap=50.0, sink=True)),
+                "suvunex_left": of_tensor(microbench.time_prefill_attention(2, 1024, H, G, d, sink=True)),
+                "suvunex_mixed": of_tensor(microbench.time_prefill_attention(2, 1024, H, G, d, sink=True, mixed=True))}
+            for label, tokens in (("prefill_2048", 2048), ("decode_b64", 64), ("decode_b8", 8)):
+                like = microbench.time_cache_write(tokens, H, G, d, rot_dims=(d // 4) * 2)
+                kernels[f"cache_write_{label}_{name}"] = {
+                    "tefopel": {"us": like["us"], "gbs": like["gbs"], "frac_hbm": like["gbs"] / hbm},
+                    "suvunex": of_hbm(microbench.time_head_norm_cache_write(tokens, H, G, d, rot_dims=d))}
+                # what stands between two sublayers: a norm there, the close of one and the opening of the next here
+                kernels[f"between_sublayers_{label}_{name}"] = {
+                    "tefopel_norm": of_hbm(microbench.time_layernorm(tokens, width)),
+                    "pagatar_close": of_hbm(microbench.time_post_norm_add(tokens, width, 2, size["layers"] // 2 + 1)),
+                    "suvunex_close": of_hbm(microbench.time_sandwich_close(tokens, width)),
+                    "suvunex_convolution": of_hbm(microbench.time_row_conv(tokens, 2 if tokens > 64 else tokens, width, 4)),
+                    "pagatar_convolution": of_hbm(microbench.time_short_conv(tokens, 2 if tokens > 64 else tokens, H, H, d, 3))}
     elif args.dtype == "bfloat16" and not args.skip_points and args.design == "pagatar":
         from pagedserve_b200.config import pagatar
 
@@ -579,7 +632,7 @@ def main():
     parser.add_argument("--serving", type=int, default=0, metavar="REQUESTS",
                         help="instead of the decode measurement: this many requests (prompts U[64,1024), outputs "
                              "U[32,256]) through the scheduler, chunked prefill under a 2,048-token budget")
-    parser.add_argument("--design", default=None, choices=("tefopel", "gozunex", "zositar", "pagatar"),
+    parser.add_argument("--design", default=None, choices=("tefopel", "gozunex", "zositar", "pagatar", "suvunex"),
                         help="instead of the default workload: prefill and decode throughput of this design at a few "
                              "sizes beside GPT-2 of equal size, and its kernels alone against the measured peaks")
     parser.add_argument("--design-sizes", default=None, help="comma-separated names out of: " + ", ".join(DESIGN_SIZES))

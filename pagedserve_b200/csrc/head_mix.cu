@@ -75,6 +75,104 @@ head_mix_kernel(const T* __restrict__ all, long long all_stride, const float* __
     }
 }
 
+// The same by pieces of 16 bytes, for sizes, strides and addresses that allow it: a thread owns a piece of one head slot of
+// one token for all of its group's result heads.  M lies in shared memory by columns, every group's heads padded to
+// blocks of HEAD_MIX_BLOCK with zeros, so that a block's weights are two accesses for all threads of the group.
+template <typename T> struct HeadMixPiece;
+template <> struct HeadMixPiece<float> { static constexpr int V = 4; };
+template <> struct HeadMixPiece<__nv_bfloat16> { static constexpr int V = 8; };
+__device__ __forceinline__ void head_mix_unpack(const uint4& p, float (&x)[4]) {
+    x[0] = __uint_as_float(p.x); x[1] = __uint_as_float(p.y); x[2] = __uint_as_float(p.z); x[3] = __uint_as_float(p.w);
+}
+__device__ __forceinline__ void head_mix_unpack(const uint4& p, float (&x)[8]) {
+    const __nv_bfloat162* pair = reinterpret_cast<const __nv_bfloat162*>(&p);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(pair[i]);
+        x[2 * i] = f.x;
+        x[2 * i + 1] = f.y;
+    }
+}
+__device__ __forceinline__ uint4 head_mix_piece(const float (&x)[4]) {
+    return make_uint4(__float_as_uint(x[0]), __float_as_uint(x[1]), __float_as_uint(x[2]), __float_as_uint(x[3]));
+}
+__device__ __forceinline__ uint4 head_mix_piece(const float (&x)[8]) {
+    uint4 p;
+    uint32_t* word = reinterpret_cast<uint32_t*>(&p);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __nv_bfloat162 pair = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+        word[i] = *reinterpret_cast<const uint32_t*>(&pair);
+    }
+    return p;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(HEAD_MIX_THREADS)
+head_mix_pieces_kernel(const T* __restrict__ all, long long all_stride, const float* __restrict__ mix, T* __restrict__ out,
+                       long long out_stride, int tokens, int heads, int kv_heads, int dim) {
+    constexpr int V = HeadMixPiece<T>::V, AHEAD = 4;
+    extern __shared__ __align__(16) float head_mix_smem[];          // [g][group][padded heads of the group]
+    const int per = heads / kv_heads, padded = (per + HEAD_MIX_BLOCK - 1) / HEAD_MIX_BLOCK * HEAD_MIX_BLOCK;
+    for (int e = threadIdx.x; e < heads * kv_heads * padded; e += HEAD_MIX_THREADS) {
+        const int g = e / (kv_heads * padded), rest = e - g * kv_heads * padded, group = rest / padded, b = rest - group * padded;
+        head_mix_smem[e] = b < per ? mix[(size_t)(group * per + b) * heads + g] : 0.f;
+    }
+    const int pieces = dim / V, units = kv_heads * pieces;
+    const long long index = (long long)blockIdx.x * HEAD_MIX_THREADS + threadIdx.x;
+    const int t = (int)(index / units), unit = (int)(index - (long long)t * units);
+    const int group = unit / pieces, d = (unit - group * pieces) * V;
+    pdl_prologue();
+    all = pdl_fresh(all);
+    __syncthreads();
+    if (t >= tokens) return;
+    const T* source = all + (size_t)t * all_stride + group * dim + d;
+    T* target = out + (size_t)t * out_stride + (size_t)group * per * dim + d;
+    const size_t step = (size_t)kv_heads * dim;
+    for (int h0 = 0; h0 < padded; h0 += HEAD_MIX_BLOCK) {
+        float sum[HEAD_MIX_BLOCK][V];
+#pragma unroll
+        for (int b = 0; b < HEAD_MIX_BLOCK; ++b)
+#pragma unroll
+            for (int e = 0; e < V; ++e) sum[b][e] = 0.f;
+        const float* weights = head_mix_smem + group * padded + h0;
+        for (int g0 = 0; g0 < heads; g0 += AHEAD) {
+            uint4 raw[AHEAD];
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a)
+                if (g0 + a < heads) raw[a] = *reinterpret_cast<const uint4*>(source + (g0 + a) * step);
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a) {
+                if (g0 + a < heads) {
+                    float x[V];
+                    head_mix_unpack(raw[a], x);
+                    const float* w = weights + (size_t)(g0 + a) * kv_heads * padded;
+                    const float4 lo = *reinterpret_cast<const float4*>(w), hi = *reinterpret_cast<const float4*>(w + 4);
+                    const float m[HEAD_MIX_BLOCK] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+                    for (int b = 0; b < HEAD_MIX_BLOCK; ++b)
+#pragma unroll
+                        for (int e = 0; e < V; ++e) sum[b][e] = fmaf(m[b], x[e], sum[b][e]);
+                }
+            }
+        }
+#pragma unroll
+        for (int b = 0; b < HEAD_MIX_BLOCK; ++b)
+            if (h0 + b < per) *reinterpret_cast<uint4*>(target + (size_t)(h0 + b) * dim) = head_mix_piece(sum[b]);
+    }
+}
+
+template <typename T>
+inline int launch_head_mix_pieces(const void* all, long long all_stride, const float* mix, void* out, long long out_stride,
+                                  int T_tokens, int heads, int kv_heads, int dim, size_t smem, cudaStream_t s) {
+    auto kernel = head_mix_pieces_kernel<T>;
+    static size_t raised[MAX_DEVICES] = {0};
+    if (!ensure_dynamic_smem((const void*)kernel, smem, raised)) return PS_ERR_LAUNCH;
+    const long long threads = (long long)T_tokens * kv_heads * (dim / HeadMixPiece<T>::V);
+    return launch_pdl(kernel, dim3((unsigned)((threads + HEAD_MIX_THREADS - 1) / HEAD_MIX_THREADS)), dim3(HEAD_MIX_THREADS),
+                      smem, s, (const T*)all, all_stride, mix, (T*)out, out_stride, T_tokens, heads, kv_heads, dim);
+}
+
 }  // namespace ps
 
 PS_EXPORT int ps_head_mix(const void* all, long long all_stride, const float* mix, void* out, long long out_stride, int T,
@@ -83,6 +181,17 @@ PS_EXPORT int ps_head_mix(const void* all, long long all_stride, const float* mi
     if (!all || !mix || !out || heads <= 0 || kv_heads <= 0 || heads % kv_heads || dim <= 0) return PS_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const int elem = dtype == PS_F32 ? 4 : 2;
+    const int per = heads / kv_heads, padded = (per + ps::HEAD_MIX_BLOCK - 1) / ps::HEAD_MIX_BLOCK * ps::HEAD_MIX_BLOCK;
+    const size_t smem = (size_t)heads * kv_heads * padded * sizeof(float);
+    const int piece = 16 / elem;
+    if (dim % piece == 0 && all_stride % piece == 0 && out_stride % piece == 0 && !(((uintptr_t)all | (uintptr_t)out) & 15) &&
+        smem <= 48 * 1024) {
+        if (dtype == PS_F32)
+            return ps::launch_head_mix_pieces<float>(all, all_stride, mix, out, out_stride, T, heads, kv_heads, dim, smem, s);
+        if (dtype == PS_BF16)
+            return ps::launch_head_mix_pieces<__nv_bfloat16>(all, all_stride, mix, out, out_stride, T, heads, kv_heads, dim,
+                                                             smem, s);
+    }
     const bool pairs = dim % 2 == 0 && all_stride % 2 == 0 && out_stride % 2 == 0 &&
                        !(((uintptr_t)all | (uintptr_t)out) & (uintptr_t)(2 * elem - 1));
     const int units = kv_heads * (pairs ? dim / 2 : dim);

@@ -14,10 +14,9 @@
 // row_scale (may be null): one float per token that multiplies its row of u wherever it is read (a row to be divided by
 // its root mean square, say, whose factor an earlier kernel has formed); kept rows are stored already multiplied.
 //
-// Entries of one token (decode) replace their slot's rows themselves: the thread of a channel has read them all.
-// short_conv_keep, after it, for the others: the slot receives the last taps - 1 projected rows of the sequence (rows of this step,
-// and older kept rows moved up where the entry brought fewer than taps - 1 tokens).  Two launches, because every
-// token of an entry may still read the old rows.
+// The slot then receives the last taps - 1 rows of the sequence (rows of this step, and older kept rows moved up where the
+// entry brought fewer than taps - 1 tokens).  The old rows are read by the entry's first taps - 1 tokens only, and one
+// thread per channel works on all of those: it has read what it needs when it replaces them.
 #include "common.cuh"
 
 namespace ps {
@@ -40,40 +39,47 @@ short_conv_kernel(const float* __restrict__ u, long long u_stride, const float* 
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total;
          i += (long long)gridDim.x * blockDim.x) {
         const int t = (int)(i / channels), c = (int)(i - (long long)t * channels);
-        float y;
         if (c >= conv_channels) {
-            y = u[(size_t)t * u_stride + c] * (row_scale ? row_scale[t] : 1.f);
-        } else {
-            const int item = token_item[t];
-            const int first = q_start[item];
-            float* old = kept + (size_t)item_slot[item] * kept_stride;
-            float now = 0.f;
-            y = 0.f;
+            out[(size_t)t * out_stride + c] = from_float<TC>(u[(size_t)t * u_stride + c] * (row_scale ? row_scale[t] : 1.f));
+            continue;
+        }
+        const int item = token_item[t];
+        const int first = q_start[item], end = q_start[item + 1];
+        if (t != first && t - first < taps - 1) continue;             // (the thread of the first token does these)
+        float* old = kept + (size_t)item_slot[item] * kept_stride;
+        auto row = [&](int source) { return u[(size_t)source * u_stride + c] * (row_scale ? row_scale[source] : 1.f); };
+        const int last = t == first ? min(first + max(taps - 1, 1), end) : t + 1;
+        for (int now = t; now < last; ++now) {
+            float y = 0.f;
             for (int j = 0; j < taps; ++j) {
-                const int source = t - (taps - 1) + j;
+                const int source = now - (taps - 1) + j;
                 // kept row k holds the projection of the token (taps - 1 - k) places before the entry's first
-                const float v = source >= first ? u[(size_t)source * u_stride + c] * (row_scale ? row_scale[source] : 1.f)
+                const float v = source >= first ? row(source)
                                                 : old[(size_t)(taps - 1 - (first - source)) * conv_channels + c];
                 y = fmaf(weight[(size_t)c * taps + j], v, y);
-                now = v;
-            }
-            if (taps > 1 && q_start[item + 1] - first == 1) {         // the entry's only token: its rows move up by one
-                for (int k = 0; k < taps - 2; ++k) old[(size_t)k * conv_channels + c] = old[(size_t)(k + 1) * conv_channels + c];
-                old[(size_t)(taps - 2) * conv_channels + c] = now;
             }
             if (mode) {
                 const int local = c - mix_lo;
                 if (local >= 0 && local < mix_heads * head_slot) {
                     const int head = local / head_slot, place = local - head * head_slot;
                     if (place < head_values) {
-                        float* common = shared_values + (size_t)t * mix_heads * head_values + head * head_values + place;
+                        float* common = shared_values + (size_t)now * mix_heads * head_values + head * head_values + place;
                         if (mode == 1) *common = y;
                         else y = (1.0f - blend) * y + blend * *common;
                     }
                 }
             }
+            out[(size_t)now * out_stride + c] = from_float<TC>(y);
         }
-        out[(size_t)t * out_stride + c] = from_float<TC>(y);
+        if (t == first) {
+            // new row k is the token at place count - (taps - 1) + k of the entry; before the entry's first token that
+            // is the old row k + count, which lies above every row written so far
+            const int count = end - first;
+            for (int k = 0; k < taps - 1; ++k) {
+                const int place = count - (taps - 1) + k;
+                old[(size_t)k * conv_channels + c] = place >= 0 ? row(first + place) : old[(size_t)(k + count) * conv_channels + c];
+            }
+        }
     }
 }
 
@@ -147,70 +153,77 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
         }
     }
     float4 held[TAPS > 1 ? TAPS - 1 : 1];                         // held[k]: the row k + 1 tokens back
-    for (int t = t0; t < t1; ++t) {
-        const int item = token_item[t];
-        const int start = q_start[item];
-        if (t == t0 || t == start) {
-            const float* old = kept + (size_t)item_slot[item] * kept_stride;
+    bool fresh = true;
+    // a token among its entry's first TAPS - 1 belongs to the run that holds the entry's first token (see the top): the
+    // run before this one may have taken this one's first tokens, and this one may take some behind its end
+    const int limit = min(t1 + (TAPS > 1 ? TAPS - 2 : 0), tokens);
+    constexpr int AHEAD = 4;                                      // tokens whose rows are fetched together
+    for (int base = t0; base < limit; base += AHEAD) {
+        float4 rows[AHEAD];
+        int items[AHEAD], starts[AHEAD];
 #pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k) {
-                const int source = t - 1 - k;
-                held[k] = source >= start ? scaled(source)
-                                          : *reinterpret_cast<const float4*>(old + (size_t)(TAPS - 1 - (start - source)) * conv_channels + c);
+        for (int a = 0; a < AHEAD; ++a) {
+            if (base + a < limit) {
+                rows[a] = scaled(base + a);
+                items[a] = token_item[base + a];
             }
         }
-        const float4 now = scaled(t);
-        float y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) {                      // tap j reads the row TAPS - 1 - j tokens back
-            const float4 v = held[TAPS - 2 - j];
-            y[0] = fmaf(w[0][j], v.x, y[0]); y[1] = fmaf(w[1][j], v.y, y[1]);
-            y[2] = fmaf(w[2][j], v.z, y[2]); y[3] = fmaf(w[3][j], v.w, y[3]);
-        }
-        y[0] = fmaf(w[0][TAPS - 1], now.x, y[0]); y[1] = fmaf(w[1][TAPS - 1], now.y, y[1]);
-        y[2] = fmaf(w[2][TAPS - 1], now.z, y[2]); y[3] = fmaf(w[3][TAPS - 1], now.w, y[3]);
+        for (int a = 0; a < AHEAD; ++a)
+            if (base + a < limit) starts[a] = q_start[items[a]];
 #pragma unroll
-        for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
-        if (TAPS > 1) held[0] = now;
-        if (TAPS > 1 && q_start[item + 1] - start == 1) {              // the entry's only token: its rows move up by one
-            float* rows = kept + (size_t)item_slot[item] * kept_stride;
+        for (int a = 0; a < AHEAD; ++a) {
+            const int t = base + a;
+            if (t >= limit) break;
+            const int start = starts[a];
+            const int anchor = t - start < TAPS - 1 ? start : t;
+            if (anchor < t0 || anchor >= t1) continue;
+            const float4 now = rows[a];
+            if (TAPS > 1 && t == start) {
+                float* old = kept + (size_t)item_slot[items[a]] * kept_stride + c;
 #pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k)
-                *reinterpret_cast<float4*>(rows + (size_t)(TAPS - 2 - k) * conv_channels + c) = held[k];
-        }
-        if (common >= 0) {
-            float* place = shared_values + (size_t)t * mix_heads * head_values + common;
-            if (mode == 1) {
-                *reinterpret_cast<float4*>(place) = make_float4(y[0], y[1], y[2], y[3]);
-            } else {
-                const float4 other = *reinterpret_cast<const float4*>(place);
-                y[0] = (1.0f - blend) * y[0] + blend * other.x; y[1] = (1.0f - blend) * y[1] + blend * other.y;
-                y[2] = (1.0f - blend) * y[2] + blend * other.z; y[3] = (1.0f - blend) * y[3] + blend * other.w;
+                for (int k = 0; k < TAPS - 1; ++k)
+                    held[k] = *reinterpret_cast<const float4*>(old + (size_t)(TAPS - 2 - k) * conv_channels);
+                // new row k is the token at place count - (TAPS - 1) + k of the entry, or the old row k + count
+                const int count = q_start[items[a] + 1] - start;
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) {
+                    const int place = count - (TAPS - 1) + k;
+                    float4 v = now;
+                    if (place > 0) v = scaled(start + place);
+#pragma unroll
+                    for (int j = 0; j < TAPS - 1; ++j)
+                        if (TAPS - 2 - j == k + count) v = held[j];
+                    *reinterpret_cast<float4*>(old + (size_t)k * conv_channels) = v;
+                }
+            } else if (TAPS > 1 && fresh) {                       // all of these lie in the entry
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) held[k] = scaled(t - 1 - k);
             }
-        }
-        store4<TC>(out + (size_t)t * out_stride + c, y);
-    }
-}
-
-__global__ void __launch_bounds__(256)
-short_conv_keep_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ row_scale, int taps,
-                       int conv_channels, float* __restrict__ kept, long long kept_stride, const int* __restrict__ q_start,
-                       const int* __restrict__ item_slot) {
-    const int item = blockIdx.y;
-    const int first = q_start[item], count = q_start[item + 1] - first;
-    pdl_prologue();
-    u = pdl_fresh(u);
-    row_scale = pdl_fresh(row_scale);
-    if (count <= 1) return;                                           // (one token: done by the convolution itself)
-    float* rows = kept + (size_t)item_slot[item] * kept_stride;
-    for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < conv_channels; c += gridDim.x * blockDim.x) {
-        // new row k is the token at place count - (taps - 1) + k of the entry; before the entry's first token that
-        // is the old row k + count, which lies above every row written so far
-        for (int k = 0; k < taps - 1; ++k) {
-            const int place = count - (taps - 1) + k;
-            rows[(size_t)k * conv_channels + c] = place >= 0 ? u[(size_t)(first + place) * u_stride + c] *
-                                                                   (row_scale ? row_scale[first + place] : 1.f)
-                                                             : rows[(size_t)(k + count) * conv_channels + c];
+            fresh = false;
+            float y[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) {                  // tap j reads the row TAPS - 1 - j tokens back
+                const float4 v = held[TAPS - 2 - j];
+                y[0] = fmaf(w[0][j], v.x, y[0]); y[1] = fmaf(w[1][j], v.y, y[1]);
+                y[2] = fmaf(w[2][j], v.z, y[2]); y[3] = fmaf(w[3][j], v.w, y[3]);
+            }
+            y[0] = fmaf(w[0][TAPS - 1], now.x, y[0]); y[1] = fmaf(w[1][TAPS - 1], now.y, y[1]);
+            y[2] = fmaf(w[2][TAPS - 1], now.z, y[2]); y[3] = fmaf(w[3][TAPS - 1], now.w, y[3]);
+#pragma unroll
+            for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
+            if (TAPS > 1) held[0] = now;
+            if (common >= 0) {
+                float* place = shared_values + (size_t)t * mix_heads * head_values + common;
+                if (mode == 1) {
+                    *reinterpret_cast<float4*>(place) = make_float4(y[0], y[1], y[2], y[3]);
+                } else {
+                    const float4 other = *reinterpret_cast<const float4*>(place);
+                    y[0] = (1.0f - blend) * y[0] + blend * other.x; y[1] = (1.0f - blend) * y[1] + blend * other.y;
+                    y[2] = (1.0f - blend) * y[2] + blend * other.z; y[3] = (1.0f - blend) * y[3] + blend * other.w;
+                }
+            }
+            store4<TC>(out + (size_t)t * out_stride + c, y);
         }
     }
 }
@@ -242,10 +255,10 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
                        (!mode || (mix_lo % 4 == 0 && head_slot % 4 == 0 && head_values % 4 == 0 &&
                                   !((uintptr_t)shared_values & 15)));
     if (quads && (dtype == PS_F32 || dtype == PS_BF16)) {
-        // runs of 16 tokens re-read (taps - 1) / 16 of the rows; shorter runs where the step has few tokens
+        // runs of 16 tokens re-read (taps - 1) / 16 of the rows; shorter runs where the step has too few for the SMs
         const int columns = (channels / 4 + ps::SHORT_CONV_THREADS - 1) / ps::SHORT_CONV_THREADS;
         int run = 16;
-        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 296) run >>= 1;
+        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 1184) run >>= 1;
         const dim3 grid(columns, (T + run - 1) / run), block(ps::SHORT_CONV_THREADS);
 #define PS_CONV_RUNS(TYPE, TAPS)                                                                                      \
     return ps::launch_pdl(ps::short_conv_runs_kernel<TYPE, TAPS>, grid, block, 0, s, u, u_stride, weight, conv_channels, \
@@ -276,17 +289,4 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
                               (__nv_bfloat16*)out, out_stride, mode, mix_lo, mix_heads, head_slot, head_values,
                               shared_values, mix, T);
     return PS_ERR_UNSUPPORTED;
-}
-
-PS_EXPORT int ps_short_conv_keep(const float* u, long long u_stride, const float* row_scale, int taps, int conv_channels, float* kept,
-                                 long long kept_stride, const int* q_start, const int* item_slot, int items,
-                                 void* stream) {
-    if (items <= 0 || taps <= 1 || conv_channels <= 0) return PS_OK;
-    if (!u || !kept || !q_start || !item_slot) return PS_ERR_BAD_ARGUMENT;
-    if (taps > ps::SHORT_CONV_MAX_TAPS) return PS_ERR_UNSUPPORTED;
-    cudaStream_t s = (cudaStream_t)stream;
-    int blocks = (conv_channels + 255) / 256;
-    if (blocks > 64) blocks = 64;
-    return ps::launch_pdl(ps::short_conv_keep_kernel, dim3(blocks, items), dim3(256), 0, s, u, u_stride, row_scale,
-                          taps, conv_channels, kept, kept_stride, q_start, item_slot);
 }

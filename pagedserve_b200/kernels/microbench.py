@@ -132,9 +132,10 @@ def _paged_inputs(items, context, kv_heads, head_dim, page, rotate_mb=200, plane
 
 
 def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, window=None, softcap=None,
-                          sink=False, iters=20, planes=2, chunk=None):
+                          sink=False, iters=20, planes=2, chunk=None, mixed=False):
     """One decode token per request over ``context`` keys (bfloat16 split-key kernel); GB/s over the K and V
-    bytes a token may see (with one plane: over the rows once)."""
+    bytes a token may see (with one plane: over the rows once).  ``mixed``: a layer whose heads' weights are mixed
+    across heads (every query head meets all values, then the mixing kernel)."""
     from pagedserve_b200.kernels.ops import Ops
 
     ops = Ops(torch.bfloat16)
@@ -145,14 +146,18 @@ def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, wi
     positions = torch.full((batch,), context - 1, dtype=torch.int32, device="cuda")
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
     sinks = torch.randn(heads, device="cuda") if sink else None
+    every = torch.empty(batch, heads * kv_heads * head_dim, dtype=torch.bfloat16, device="cuda") if mixed else out
+    mix = torch.eye(heads, device="cuda")
     if chunk:                                           # a chunked mask travels as a negative window
         window = -chunk
 
     def run(i):
         layer = i % layers
-        ops.paged_attention_decode(q, out, pool[:, layer, 0], pool[:, layer, planes - 1], stride, token_item, positions,
+        ops.paged_attention_decode(q, every, pool[:, layer, 0], pool[:, layer, planes - 1], stride, token_item, positions,
                                    table, heads, kv_heads, head_dim, page, window, head_dim ** -0.5, context,
-                                   status=status, softcap=softcap, sink=sinks)
+                                   status=status, softcap=softcap, sink=sinks, all_values=mixed)
+        if mixed:
+            ops.head_mix(every, mix, out, heads, kv_heads, head_dim)
 
     seconds = _time(run, iters, graph=True)
     seen = min(context, window) if window and window > 0 else context
@@ -163,9 +168,9 @@ def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, wi
 
 
 def time_prefill_attention(prompts, prompt_len, heads, kv_heads, head_dim, page=16, window=None, softcap=None,
-                           sink=False, iters=10, planes=2, chunk=None):
+                           sink=False, iters=10, planes=2, chunk=None, mixed=False):
     """Whole prompts through the tcgen05 prompt kernel (bfloat16, head size 64 or 128); TFLOP/s over the
-    products of the keys a query may see."""
+    products of the keys a query may see.  ``mixed`` as in :func:`time_decode_attention` (the same products counted)."""
     from pagedserve_b200.kernels.ops import Ops
 
     ops = Ops(torch.bfloat16)
@@ -178,12 +183,17 @@ def time_prefill_attention(prompts, prompt_len, heads, kv_heads, head_dim, page=
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
     sinks = torch.randn(heads, device="cuda") if sink else None
     blocks = prompts * -(-prompt_len // 128)
+    every = torch.empty(total, heads * kv_heads * head_dim, dtype=torch.bfloat16, device="cuda") if mixed else out
+    mix = torch.eye(heads, device="cuda")
     if chunk:
         window = -chunk
 
     def run(i):
-        ops.prefill_attention_tc(q, out, pool, 0, q_start, kv_len, table, 0, prompts, blocks, heads, kv_heads,
-                                 head_dim, page, window, head_dim ** -0.5, status=status, softcap=softcap, sink=sinks)
+        ops.prefill_attention_tc(q, every, pool, 0, q_start, kv_len, table, 0, prompts, blocks, heads, kv_heads,
+                                 head_dim, page, window, head_dim ** -0.5, status=status, softcap=softcap, sink=sinks,
+                                 all_values=mixed)
+        if mixed:
+            ops.head_mix(every, mix, out, heads, kv_heads, head_dim)
 
     seconds = _time(run, iters, graph=True)
     if chunk:
@@ -411,6 +421,94 @@ def time_short_conv(tokens, items, heads, kv_heads, head_dim, taps, iters=20):
                     graph=True)
     moved = tokens * channels * 6 + tokens * kv_heads * head_dim * 4
     return {"us": seconds * 1e6, "gbs": moved / seconds / 1e9}
+
+
+def time_gla(items, tokens_each, heads, dk, dv, rank=16, dtype=torch.bfloat16, iters=10):
+    """The gated linear recurrence alone (the kernels of both launches where entries are cut into runs) on ``items``
+    entries of ``tokens_each`` tokens; GB/s over what it must move: the stacked projections in, one row out, and every
+    entry's state in and out."""
+    from types import SimpleNamespace
+
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    total, k, v = items * tokens_each, heads * dk, heads * dv
+    columns = 2 * k + 2 * v + rank
+    copies = max(1, int(200e6 // (total * columns * 2)) + 1)                       # rotate past the L2
+    copies = min(copies, 64)
+    rows = torch.randn(copies, total, columns + (-columns % 8), device="cuda").to(dtype)
+    a2, bias = torch.randn(k, rank, device="cuda") * rank ** -0.5, torch.randn(k, device="cuda")
+    gain = torch.ones(dv, device="cuda")
+    states = max(1, min(16, int(200e6 // (items * heads * dk * dv * 4)) + 1))
+    state = torch.zeros(states, items, heads * dk * dv, device="cuda")
+    out = torch.empty(total, v, dtype=dtype, device="cuda")
+    ctx = SimpleNamespace(q_start=torch.arange(0, total + 1, tokens_each, dtype=torch.int32, device="cuda"),
+                          item_slot=torch.arange(items, dtype=torch.int32, device="cuda"), num_items=items,
+                          num_short_items=items if tokens_each < 16 else 0, max_q_len=tokens_each,
+                          single_tokens=tokens_each == 1)
+    offsets = (0, k, 2 * k, 2 * k + v, 2 * k + 2 * v)
+
+    def run(i):
+        ops.gla_recurrence(rows[i % copies], offsets, a2, bias, 16.0, dk ** -0.5, gain, 1e-5, 1.0, state[i % states], ctx,
+                           out, heads, dk, dv)
+
+    seconds = _time(run, iters, graph=True)
+    nbytes = total * (columns + v) * out.element_size() + items * heads * dk * dv * 4 * 2
+    return {"us": seconds * 1e6, "gbs": nbytes / seconds / 1e9, "tokens_per_s": total / seconds}
+
+
+def time_sandwich_close(tokens, width, rows_out=True, iters=20):
+    """The kernel that closes a sublayer of a layer with norms before and after its sublayers; GB/s over the sublayer's
+    row read and zeroed, the residual row read and written and (``rows_out``) the next sublayer's row written."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = max(1, int(200e6 // (2 * tokens * width * 4)) + 1)                     # rotate past the L2
+    copies = min(copies, 256)
+    x, y = torch.randn(copies, tokens, width, device="cuda"), torch.randn(copies, tokens, width, device="cuda")
+    gain = torch.ones(width, device="cuda")
+    out = torch.empty(tokens, width, dtype=torch.bfloat16, device="cuda")
+    scale = torch.empty(tokens, device="cuda")
+    extra = dict(next_gain=gain, out=out) if rows_out else dict(row_scale=scale)
+    seconds = _time(lambda i: ops.sandwich_close(y[i % copies], x[i % copies], gain, 0.8, 1e-6, **extra), iters, graph=True)
+    moved = tokens * width * (16 + (2 if rows_out else 0))
+    return {"us": seconds * 1e6, "gbs": moved / seconds / 1e9}
+
+
+def time_layernorm(tokens, width, has_mean=False, iters=20):
+    """The norm kernel of a pre-norm layer; GB/s over float32 rows read and rounded rows written."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = min(256, max(1, int(200e6 // (tokens * width * 4)) + 1))               # rotate past the L2
+    x = torch.randn(copies, tokens, width, device="cuda")
+    gain = torch.ones(width, device="cuda")
+    out = torch.empty(tokens, width, dtype=torch.bfloat16, device="cuda")
+    seconds = _time(lambda i: ops.layernorm(x[i % copies], gain, None, 1e-6, out, has_mean=has_mean), iters, graph=True)
+    return {"us": seconds * 1e6, "gbs": tokens * width * 6 / seconds / 1e9}
+
+
+def time_row_conv(tokens, items, width, taps, iters=20):
+    """The short convolution on residual rows (with a factor per row) and the kernel that keeps the entries' last rows;
+    GB/s over the float32 rows read once and the rounded rows written."""
+    from types import SimpleNamespace
+
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = min(256, max(1, int(200e6 // (tokens * width * 6)) + 1))               # rotate past the L2
+    u = torch.randn(copies, tokens, width, device="cuda")
+    out = torch.empty(tokens, width, dtype=torch.bfloat16, device="cuda")
+    weight, scale = torch.randn(width, taps, device="cuda"), torch.ones(tokens, device="cuda")
+    state = torch.zeros(items + 1, (taps - 1) * width, device="cuda")
+    each = tokens // items
+    ctx = SimpleNamespace(q_start=torch.arange(0, tokens + 1, each, dtype=torch.int32, device="cuda"),
+                          item_slot=torch.arange(items, dtype=torch.int32, device="cuda"), num_items=items,
+                          token_item=(torch.arange(tokens, device="cuda") // each).to(torch.int32), single_tokens=each == 1)
+    seconds = _time(lambda i: ops.short_conv(u[i % copies], weight, taps, width, state, ctx, out, row_scale=scale), iters,
+                    graph=True)
+    kept = items * (taps - 1) * width * 4
+    return {"us": seconds * 1e6, "gbs": (tokens * width * 6 + 2 * kept) / seconds / 1e9}
 
 
 def time_experts(tokens, width, experts, top, ff, iters=10, score="softmax", normalize=True, form=None):

@@ -100,10 +100,9 @@ _SIGNATURES = {
         "ps_depth_begin": [_P, _P, _P, _I, _P, _L, _P],
         "ps_mingru_scan": [_P, _L, _I, _P, _L, _P, _P, _I, _P, _L, _I, _I, _P],
         "ps_short_conv": [_P, _L, _P, _I, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P],
-        "ps_short_conv_keep": [_P, _L, _P, _I, _I, _P, _L, _P, _P, _I, _P],
         "ps_sandwich_close": [_P, _P, _I, _I, _P, _F, _F, _P, _P, _I, _P, _P],
-        "ps_gla_recurrence": [_P, _L, _P, _P, _P, _I, _F, _F, _P, _F, _F, _P, _L, _P, _P, _I, _I, _I, _P, _P, _P, _L,
-                              _I, _I, _I, _I, _P],
+        "ps_gla_recurrence": [_P, _L, _P, _P, _P, _I, _F, _F, _P, _F, _F, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P,
+                              _L, _I, _I, _I, _I, _P],
         "ps_head_mix": [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P],
         "ps_moe_plan": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P],
         "ps_moe_gather": [_P, _I, _P, _P, _I, _I, _I, _I, _P],
@@ -1217,17 +1216,21 @@ class Ops:
         first_cut = ctx.num_short_items
         if first_cut >= ctx.num_items:
             segments = 1
-        run_state = run_decay = None
-        if segments > 1:
+        alpha = run_state = run_decay = None
+        if segments > 1 and max(dk, dv) <= 128 and rank <= 256:
+            alpha = self.empty((T, heads * dk), torch.float32, rows.device)
             runs = (ctx.num_items - first_cut) * heads * segments
             run_state = self.empty((runs, dk * dv), torch.float32, rows.device)
             run_decay = self.empty((runs, dk), torch.float32, rows.device)
+        else:
+            segments = 1
         places = (ctypes.c_int * 5)(*[int(o) for o in offsets])
-        self.launches += 2 if segments > 1 else 1
+        self.launches += 4 if segments > 1 else 1
         _check(self.core.ps_gla_recurrence(_ptr(rows), rows.stride(0), ctypes.addressof(places), _ptr(a2), _ptr(bias), rank,
                                            1.0 / float(tau), float(q_scale), _ptr(gain), float(eps), float(out_scale),
                                            _ptr(state), state.stride(0), _ptr(ctx.q_start), _ptr(ctx.item_slot),
-                                           ctx.num_items, first_cut, segments, _ptr(run_state), _ptr(run_decay), _ptr(out),
+                                           ctx.num_items, T, 1 if getattr(ctx, "single_tokens", False) else 0, first_cut,
+                                           segments, _ptr(alpha), _ptr(run_state), _ptr(run_decay), _ptr(out),
                                            out.stride(0), heads, dk, dv, self.code, _stream()), "gla_recurrence")
         return out
 
@@ -1299,11 +1302,6 @@ class Ops:
                                        _ptr(ctx.q_start), _ptr(ctx.item_slot), _ptr(out), out.stride(0), mode, lo, heads,
                                        slot, values, _ptr(shared), _ptr(mix) if mode == 2 else None, T, self.code,
                                        _stream()), "short_conv")
-        if state is not None and not getattr(ctx, "single_tokens", False):     # (entries of one token have kept theirs)
-            self.launches += 1
-            _check(self.core.ps_short_conv_keep(_ptr(u), u.stride(0), _ptr(row_scale), taps, conv_channels, _ptr(state), state.stride(0),
-                                                _ptr(ctx.q_start), _ptr(ctx.item_slot), ctx.num_items, _stream()),
-                   "short_conv_keep")
         return out
 
     # ------------------------------------------------------------------ routed experts

@@ -459,7 +459,7 @@ def recurrence_case(heads, dk, dv, rank, lengths, seed, dtype, tau=4.0):
     want = plain.rms_norm(want, gain.double(), eps) * gate * torch.sigmoid(gate) * out_scale
     short = sum(1 for n in lengths if n < 16)
     ctx = SimpleNamespace(max_q_len=max(lengths), q_start=torch.from_numpy(starts).to(DEV), item_slot=slots.to(DEV),
-                          num_items=items, num_short_items=short)
+                          num_items=items, num_short_items=short, single_tokens=max(lengths) == 1)
 
     def run(ops, segments=None):
         kept = state.to(DEV)
@@ -476,7 +476,8 @@ def recurrence_case(heads, dk, dv, rank, lengths, seed, dtype, tau=4.0):
 @pytest.mark.parametrize("heads,dk,dv,rank,lengths", [
     (3, 16, 24, 5, [1, 1, 1]), (2, 64, 64, 16, [1, 2, 15, 40, 200]), (1, 128, 128, 33, [3, 130]), (4, 20, 36, 1, [7, 17, 333]),
     (2, 40, 100, 70, [100]), (1, 96, 32, 8, [1, 64, 65]), (2, 8, 128, 12, [50, 31]), (2, 144, 160, 16, [1, 20]),
-    (5, 10, 14, 16, [16, 16, 150])])
+    (5, 10, 14, 16, [16, 16, 150]), (2, 64, 128, 16, [1] * 5), (3, 128, 64, 70, [1, 1]), (4, 10, 14, 3, [1] * 4),
+    (2, 32, 96, 9, [1] * 3)])
 def test_the_recurrence_alone(heads, dk, dv, rank, lengths, dtype):
     """Entries of unequal length (short ones first) from states that are not zero, in one piece and cut into runs that
     are worked on side by side (also into more runs than the entry has chunks), equal the plain loop; the state that is
