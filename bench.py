@@ -495,13 +495,18 @@ def design_arm(args):
             for label, items, each in (("prefill_2x1024", 2, 1024), ("decode_b64", 64, 1), ("decode_b8", 8, 1)):
                 kernels[f"recurrence_{label}_{name}"] = {
                     "tefopel": of_hbm(microbench.time_wkv(items, each, width // 64, 64, width)),
-                    "suvunex": of_hbm(microbench.time_gla(items, each, H, d, d))}
+                    "suvunex": of_hbm(microbench.time_gla(items, each, size.get("right_heads", H), size.get("right_dim", d),
+                                                          size.get("right_dim", d)))}
+            if d > 64:                                       # larger heads than the other recurrence has
+                for label, items, each in (("prefill_2x1024", 2, 1024), ("decode_b64", 64, 1)):
+                    kernels[f"recurrence_{label}_{name}"]["suvunex_large_heads"] = of_hbm(microbench.time_gla(items, each, H, d, d))
             # attention whose heads are mixed, with the mixing kernel, and plain attention of equal heads
             for batch in (8, 64):
                 kernels[f"decode_attention_b{batch}_{name}"] = {
                     "tefopel": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, softcap=50.0, sink=True)),
-                    "suvunex_left": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, sink=True)),
-                    "suvunex_mixed": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, sink=True, mixed=True))}
+                    "suvunex_left": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, sink=True, as_rows=True)),
+                    "suvunex_mixed": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, d, sink=True, mixed=True,
+                                                                            as_rows=True))}
             kernels[f"prefill_attention_{name}"] = {
                 "tefopel": of_tensor(microbench.time_prefill_attention(2, 1024, H, G, d, softcap=50.0, sink=True)),
                 "suvunex_left": of_tensor(microbench.time_prefill_attention(2, 1024, H, G, d, sink=True)),

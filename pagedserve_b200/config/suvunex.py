@@ -211,13 +211,14 @@ def attention_layer(heads: int, kv_heads: int, dim: int, ff: Optional[int], base
 
 
 def repeating_config(width: int, heads: int, head_dim: int, layers: int, vocab: int, ff: int, kv_heads: int = 2,
-                     right_heads: Optional[int] = None, taps: int = 4, eps: float = 1e-6,
+                     right_heads: Optional[int] = None, right_dim: Optional[int] = None, taps: int = 4, eps: float = 1e-6,
                      pattern=("parallel", "attention")) -> SuvunexConfig:
     """A model for random weights: the layer kinds of ``pattern`` in turn, all with a feed-forward."""
     entries = []
     for index in range(layers):
         if pattern[index % len(pattern)] == "parallel":
-            entries.append(parallel_layer(heads, kv_heads, head_dim, right_heads or heads, head_dim, head_dim, ff,
+            entries.append(parallel_layer(heads, kv_heads, head_dim, right_heads or heads, right_dim or head_dim,
+                                          right_dim or head_dim, ff,
                                           scaling={"factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}))
         else:
             entries.append(attention_layer(heads, kv_heads, head_dim, ff, factor=4.0))
@@ -229,7 +230,8 @@ def repeating_config(width: int, heads: int, head_dim: int, layers: int, vocab: 
 NAMED_CONFIGS = {
     "suvunex-tiny": dict(width=64, heads=4, head_dim=16, layers=3, vocab=512, ff=96),
     "suvunex-w1024": dict(width=1024, heads=16, head_dim=64, layers=8, vocab=32000, ff=2816),
-    "suvunex-w2048": dict(width=2048, heads=16, head_dim=128, layers=8, vocab=32000, ff=5632),
+    "suvunex-w2048": dict(width=2048, heads=16, head_dim=128, layers=8, vocab=32000, ff=5632,
+                          right_heads=32, right_dim=64),
 }
 
 

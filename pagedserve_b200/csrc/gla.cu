@@ -40,6 +40,8 @@ struct GlaInputs {
     int heads, dk, dv;
 };
 
+// x / (1 + exp(-x)), for the gate on the result (nothing of it is carried on)
+__device__ __forceinline__ float gla_silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 // log(sigmoid(z)) without overflow at either end
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
@@ -92,8 +94,8 @@ struct GlaLayout {
     static constexpr int up(int a, int b) { return (a + b - 1) / b; }
     static constexpr int K_PIECES = up(CH * DK / VEC, THREADS), V_PIECES = up(CH * DV / VEC, THREADS),
                          A_PIECES = up(CH * DK / 4, THREADS);
-    // floats: q, k, alpha in padded rows, v, g, sums, gain; then low [CH][rank], and A2 of the head [rank][DK] if it fits
-    static constexpr int Q = 0, K = CH * ROW, A = 2 * CH * ROW, V = 3 * CH * ROW, G = V + CH * DV, Y = G + CH * DV,
+    // floats: q, k, alpha in padded rows, v, g (two chunks of it), sums, gain; then low [CH][rank], and A2 of the head [rank][DK] if it fits
+    static constexpr int Q = 0, K = CH * ROW, A = 2 * CH * ROW, V = 3 * CH * ROW, G = V + CH * DV, Y = G + 2 * CH * DV,
                          GAIN = Y + CH * DV, LOW = GAIN + DV;
     static_assert(PARTS >= 4 && PARTS <= 16 && THREADS % 32 == 0 && THREADS % DK == 0 && VALUES >= 1, "layout");
     __host__ __device__ static bool a2_staged(int rank) { return rank <= 64; }
@@ -125,8 +127,7 @@ gla_decay_kernel(const T* __restrict__ rows, const GlaInputs in, float* __restri
     float z[GLA_DECAY_TOKENS];
 #pragma unroll
     for (int t = 0; t < GLA_DECAY_TOKENS; ++t) z[t] = 0.f;
-    for (int r = 0; r < rank; ++r) {
-        const float wr = w[r];
+    auto take = [&](int r, float wr) {
 #pragma unroll
         for (int t = 0; t < GLA_DECAY_TOKENS; t += 4) {
             const float4 low = *reinterpret_cast<const float4*>(gla_smem + r * GLA_DECAY_TOKENS + t);
@@ -135,6 +136,15 @@ gla_decay_kernel(const T* __restrict__ rows, const GlaInputs in, float* __restri
             z[t + 2] = fmaf(wr, low.z, z[t + 2]);
             z[t + 3] = fmaf(wr, low.w, z[t + 3]);
         }
+    };
+    if ((rank & 3) == 0 && !((uintptr_t)in.a2 & 15)) {
+#pragma unroll 4
+        for (int r = 0; r < rank; r += 4) {
+            const float4 four = *reinterpret_cast<const float4*>(w + r);
+            take(r, four.x); take(r + 1, four.y); take(r + 2, four.z); take(r + 3, four.w);
+        }
+    } else {
+        for (int r = 0; r < rank; ++r) take(r, w[r]);
     }
 #pragma unroll
     for (int t = 0; t < GLA_DECAY_TOKENS; ++t)
@@ -156,7 +166,7 @@ gla_recurrence_kernel(const T* __restrict__ rows, const GlaInputs in, int wide, 
     float* const s_k = gla_smem + L::K;
     float* const s_a = gla_smem + L::A;
     float* const s_v = gla_smem + L::V;
-    float* const s_g = gla_smem + L::G;
+    float* s_g = gla_smem + L::G;                                // the chunk's; the other buffer is the chunk's before
     float* const s_y = gla_smem + L::Y;
     float* const s_gain = gla_smem + L::GAIN;
     float* const s_low = gla_smem + L::LOW;
@@ -344,7 +354,9 @@ gla_recurrence_kernel(const T* __restrict__ rows, const GlaInputs in, int wide, 
 
     for (int t0 = lo; t0 < hi; t0 += CH) {
         const int n = min(CH, hi - t0);
-        settle(t0);                                              // (nobody reads these buffers any more: see below)
+        // q, k, v and the alphas of the chunk before were last read ahead of its second barrier; its gates, which the head
+        // norm may still be reading, lie in the other buffer; its sums are overwritten behind the next barrier only
+        settle(t0);
         __syncthreads();
         if (wide && t0 + CH < hi) fetch(t0 + CH);
         // ---- the decays: a thread's channel is fixed, its tokens are THREADS / DK apart
@@ -452,7 +464,7 @@ gla_recurrence_kernel(const T* __restrict__ rows, const GlaInputs in, int wide, 
                 const int j = (lane & 15) + 16 * m;
                 const bool here = valid && j < dv;
                 o[m] = here ? s_y[tt * DV + j] : 0.f;
-                factor[m] = here ? s_gain[j] * silu(s_g[tt * DV + j]) : 0.f;
+                factor[m] = here ? s_gain[j] * gla_silu(s_g[tt * DV + j]) : 0.f;
                 sq = fmaf(o[m], o[m], sq);
             }
 #pragma unroll
@@ -467,7 +479,7 @@ gla_recurrence_kernel(const T* __restrict__ rows, const GlaInputs in, int wide, 
                 }
             }
         }
-        __syncthreads();                                         // before the next chunk's rows (and sums) arrive
+        s_g = gla_smem + L::G + (s_g == gla_smem + L::G ? CH * DV : 0);
     }
     float end[8][4];
 #pragma unroll

@@ -225,6 +225,154 @@ sandwich_close_kernel(float* __restrict__ y, float* __restrict__ x, int H, const
     }
 }
 
+// The same with a row in registers, QUADS quads a thread whose loads are all in flight together: for widths that are
+// multiples of four on aligned rows.  With many rows a CTA has as few threads as the row allows, so that many rows are
+// resident; with few rows a thread has one quad.
+// TAPS > 0 (steps in which every entry brings one token, token t being entry t): what comes next is a short causal
+// convolution over time on the rows x / rms(x) (csrc/short_conv.cu), and an entry's one row meets its slot's kept rows here:
+// out <- sum_(j < TAPS - 1) taps[c][j] kept[j][c] + taps[c][TAPS - 1] x[c] / rms(x), and the kept rows move up by one.
+constexpr int CLOSE_QUADS = 4, CLOSE_MAX_THREADS = 1024;
+
+__device__ __forceinline__ float few_warps_sum(float v, float* slots) {
+    v = warp_sum(v);
+    const int warps = blockDim.x >> 5;
+    if (warps == 1) return v;
+    if ((threadIdx.x & 31) == 0) slots[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+    for (int w = 0; w < warps; ++w) total += slots[w];
+    return total;
+}
+
+template <typename TC, int QUADS, int TAPS>
+__global__ void __launch_bounds__(QUADS == 1 ? CLOSE_MAX_THREADS : CLOSE_MAX_THREADS / 2)
+sandwich_close_rows_kernel(float* __restrict__ y, float* __restrict__ x, int H, const float* __restrict__ gain, float y_scale,
+                           float eps, const float* __restrict__ next_gain, TC* __restrict__ out,
+                           float* __restrict__ row_scale, const float* __restrict__ taps, float* kept, long long kept_stride,
+                           const int* __restrict__ item_slot) {
+    using Pack = PackOf<4>;
+    __shared__ float slots[2][CLOSE_MAX_THREADS / 32];
+    const size_t base = (size_t)blockIdx.x * H;
+    Pack g[QUADS], a[QUADS], b[QUADS], zero;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) zero.v[i] = 0.f;
+    // before the wait: the gain, the taps, and the kept rows, which only this layer's kernels of an earlier step wrote
+    if (gain) {
+#pragma unroll
+        for (int k = 0; k < QUADS; ++k) {
+            const int j = 4 * (threadIdx.x + k * blockDim.x);
+            g[k] = j < H ? *reinterpret_cast<const Pack*>(gain + j) : zero;
+        }
+    }
+    constexpr int OLD = TAPS > 1 ? TAPS - 1 : 1;
+    Pack old[OLD];
+    float w[TAPS > 0 ? 4 * TAPS : 1];
+    float* slot = nullptr;
+    if constexpr (TAPS > 0) {
+        static_assert(QUADS == 1, "the convolution is for one quad a thread");
+        const int j = 4 * threadIdx.x;
+        if (j < H) {
+#pragma unroll
+            for (int p = 0; p < TAPS; ++p) {
+                const Pack v = *reinterpret_cast<const Pack*>(taps + (size_t)j * TAPS + 4 * p);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) w[4 * p + i] = v.v[i];
+            }
+            if constexpr (TAPS > 1) {
+                slot = kept + (size_t)item_slot[blockIdx.x] * kept_stride + j;
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) old[k] = *reinterpret_cast<const Pack*>(slot + (size_t)k * H);
+            }
+        }
+    }
+    pdl_prologue();
+    y = pdl_fresh(y);
+    x = pdl_fresh(x);
+#pragma unroll
+    for (int k = 0; k < QUADS; ++k) {
+        const int j = 4 * (threadIdx.x + k * blockDim.x);
+        const bool here = j < H;
+        b[k] = here ? *reinterpret_cast<const Pack*>(x + base + j) : zero;
+        if (gain) a[k] = here ? *reinterpret_cast<const Pack*>(y + base + j) : zero;
+    }
+    float sq = 0.f, sq_x = 0.f;
+    if (gain) {
+#pragma unroll
+        for (int k = 0; k < QUADS; ++k)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                a[k].v[i] *= y_scale;
+                sq = fmaf(a[k].v[i], a[k].v[i], sq);
+            }
+        const float inverse = 1.0f / sqrtf(few_warps_sum(sq, slots[0]) / (float)H + eps);
+#pragma unroll
+        for (int k = 0; k < QUADS; ++k)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) b[k].v[i] = fmaf(a[k].v[i] * inverse, g[k].v[i], b[k].v[i]);
+    }
+#pragma unroll
+    for (int k = 0; k < QUADS; ++k) {
+        const int j = 4 * (threadIdx.x + k * blockDim.x);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) sq_x = fmaf(b[k].v[i], b[k].v[i], sq_x);
+        if (j < H) {
+            if (gain) *reinterpret_cast<Pack*>(x + base + j) = b[k];
+            *reinterpret_cast<Pack*>(y + base + j) = zero;
+        }
+    }
+    if (!out && !row_scale) return;
+    const float inverse = 1.0f / sqrtf(few_warps_sum(sq_x, slots[1]) / (float)H + eps);
+    if (row_scale && threadIdx.x == 0) row_scale[blockIdx.x] = inverse;
+    if (!out) return;
+#pragma unroll
+    for (int k = 0; k < QUADS; ++k) {
+        const int j = 4 * (threadIdx.x + k * blockDim.x);
+        if (j >= H) continue;
+        if constexpr (TAPS > 0) {
+            Pack unit, sum = zero;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) unit.v[i] = b[k].v[i] * inverse;
+            if constexpr (TAPS > 1) {
+#pragma unroll
+                for (int p = 0; p < TAPS - 1; ++p) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) sum.v[i] = fmaf(w[i * TAPS + p], old[p].v[i], sum.v[i]);
+                    *reinterpret_cast<Pack*>(slot + (size_t)p * H) = p + 1 < TAPS - 1 ? old[p + 1 < OLD ? p + 1 : p] : unit;
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) sum.v[i] = fmaf(w[i * TAPS + TAPS - 1], unit.v[i], sum.v[i]);
+            store_cast<4>(out + base + j, sum);
+        } else {
+            const Pack n = *reinterpret_cast<const Pack*>(next_gain + j);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) b[k].v[i] = b[k].v[i] * inverse * n.v[i];
+            store_cast<4>(out + base + j, b[k]);
+        }
+    }
+}
+
+template <typename TC>
+int launch_sandwich_rows(float* y, float* x, int T, int H, const float* gain, float y_scale, float eps, const float* next_gain,
+                         void* out, float* row_scale, int n_taps, const float* taps, float* kept, long long kept_stride,
+                         const int* item_slot, cudaStream_t s) {
+    const bool few = n_taps > 0 || (T < 592 && H <= 4 * CLOSE_MAX_THREADS);
+    const int per_thread = few ? 4 : 4 * CLOSE_QUADS;
+    const dim3 block(((H + per_thread - 1) / per_thread + 31) / 32 * 32);
+#define PS_CLOSE_ROWS(QUADS, TAPS)                                                                                     \
+    return launch_pdl(sandwich_close_rows_kernel<TC, QUADS, TAPS>, dim3(T), block, 0, s, y, x, H, gain, y_scale, eps,    \
+                      next_gain, (TC*)out, row_scale, taps, kept, kept_stride, item_slot)
+    switch (n_taps) {
+        case 1: PS_CLOSE_ROWS(1, 1);
+        case 2: PS_CLOSE_ROWS(1, 2);
+        case 3: PS_CLOSE_ROWS(1, 3);
+        case 4: PS_CLOSE_ROWS(1, 4);
+    }
+    if (few) PS_CLOSE_ROWS(1, 0);
+    PS_CLOSE_ROWS(CLOSE_QUADS, 0);
+#undef PS_CLOSE_ROWS
+}
+
 template <typename TIn, typename TOut>
 inline int launch_group_norm(const void* x, long long x_stride, const int* rows, int n_rows, int H, int groups,
                              const float* gain, float eps, void* out, long long out_stride, cudaStream_t s) {
@@ -314,6 +462,13 @@ PS_EXPORT int ps_sandwich_close(float* y, float* x, int T, int H, const float* g
     const bool bf16 = out && out_dtype == PS_BF16;
     const bool by4 = H % 4 == 0 && !(((uintptr_t)y | (uintptr_t)x | (uintptr_t)gain | (uintptr_t)next_gain) & 15) &&
                      !((uintptr_t)out & (bf16 ? 7 : 15));
+    if (by4 && H <= 2 * ps::CLOSE_QUADS * ps::CLOSE_MAX_THREADS) {
+        if (bf16)
+            return ps::launch_sandwich_rows<__nv_bfloat16>(y, x, T, H, gain, y_scale, eps, next_gain, out, row_scale, 0, nullptr,
+                                                           nullptr, 0, nullptr, s);
+        return ps::launch_sandwich_rows<float>(y, x, T, H, gain, y_scale, eps, next_gain, out, row_scale, 0, nullptr, nullptr, 0,
+                                               nullptr, s);
+    }
 #define PS_SANDWICH(TYPE, V)                                                                                         \
     do {                                                                                                             \
         static size_t raised[ps::MAX_DEVICES] = {0};                                                                 \
@@ -329,4 +484,26 @@ PS_EXPORT int ps_sandwich_close(float* y, float* x, int T, int H, const float* g
     if (by4) PS_SANDWICH(float, 4);
     PS_SANDWICH(float, 1);
 #undef PS_SANDWICH
+}
+
+// The close of a sublayer and, for entries of one token each, the convolution in front of the next mixer: taps float32
+// [H, n_taps] (n_taps 1 to 4), kept float32 rows of kept_stride whose first (n_taps - 1) * H numbers are a slot's kept rows,
+// item_slot int32 [T].  H a multiple of 4 up to 4096, everything on 16-byte boundaries (out in the compute type: 8).
+PS_EXPORT int ps_sandwich_close_conv(float* y, float* x, int T, int H, const float* gain, float y_scale, float eps,
+                                     const float* taps, int n_taps, float* kept, long long kept_stride, const int* item_slot,
+                                     void* out, int out_dtype, void* stream) {
+    if (T <= 0) return PS_OK;
+    if (!y || !x || !out || !taps || H <= 0 || n_taps < 1 || (n_taps > 1 && (!kept || !item_slot))) return PS_ERR_BAD_ARGUMENT;
+    if (n_taps > 4 || H % 4 != 0 || H > 4 * ps::CLOSE_MAX_THREADS || kept_stride % 4 != 0 ||
+        (((uintptr_t)y | (uintptr_t)x | (uintptr_t)gain | (uintptr_t)taps | (uintptr_t)kept) & 15) ||
+        ((uintptr_t)out & (out_dtype == PS_BF16 ? 7 : 15)))
+        return PS_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (out_dtype == PS_BF16)
+        return ps::launch_sandwich_rows<__nv_bfloat16>(y, x, T, H, gain, y_scale, eps, nullptr, out, nullptr, n_taps, taps, kept,
+                                                       kept_stride, item_slot, s);
+    if (out_dtype == PS_F32)
+        return ps::launch_sandwich_rows<float>(y, x, T, H, gain, y_scale, eps, nullptr, out, nullptr, n_taps, taps, kept,
+                                               kept_stride, item_slot, s);
+    return PS_ERR_UNSUPPORTED;
 }

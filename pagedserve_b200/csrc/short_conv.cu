@@ -116,12 +116,22 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
     // the taps of the thread's four channels: static for the step, fetched before the wait
     float w[4][TAPS];
     if (convolved && c < channels) {
+        // (4 * TAPS neighbouring numbers)
+        float flat[4 * TAPS];
+#pragma unroll
+        for (int p = 0; p < TAPS; ++p) {
+            const float4 v = *reinterpret_cast<const float4*>(weight + (size_t)c * TAPS + 4 * p);
+            flat[4 * p] = v.x; flat[4 * p + 1] = v.y; flat[4 * p + 2] = v.z; flat[4 * p + 3] = v.w;
+        }
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) w[i][j] = weight[(size_t)(c + i) * TAPS + j];
+            for (int j = 0; j < TAPS; ++j) w[i][j] = flat[i * TAPS + j];
     }
     const float blend = mode == 2 ? *mix : 0.f;
+    // which entry the run lies in is static for the step too
+    const int item0 = convolved ? token_item[t0] : 0, item1 = convolved ? token_item[t1 - 1] : 0;
+    const int start0 = convolved ? q_start[item0] : 0;
     pdl_prologue();
     u = pdl_fresh(u);
     row_scale = pdl_fresh(row_scale);
@@ -135,11 +145,20 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
         return v;
     };
     if (c >= channels) return;
+    constexpr int AHEAD = 4;                                      // tokens whose rows are fetched together
     if (!convolved) {
-        for (int t = t0; t < t1; ++t) {
-            const float4 v = scaled(t);
-            const float y[4] = {v.x, v.y, v.z, v.w};
-            store4<TC>(out + (size_t)t * out_stride + c, y);
+        for (int t = t0; t < t1; t += AHEAD) {
+            float4 rows[AHEAD];
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a)
+                if (t + a < t1) rows[a] = scaled(t + a);
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a) {
+                if (t + a < t1) {
+                    const float y[4] = {rows[a].x, rows[a].y, rows[a].z, rows[a].w};
+                    store4<TC>(out + (size_t)(t + a) * out_stride + c, y);
+                }
+            }
         }
         return;
     }
@@ -152,79 +171,82 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
             if (place < head_values) common = head * head_values + place;
         }
     }
-    float4 held[TAPS > 1 ? TAPS - 1 : 1];                         // held[k]: the row k + 1 tokens back
+    constexpr int OLD = TAPS > 1 ? TAPS - 1 : 1;
+    float4 held[OLD];                                             // held[k]: the row k + 1 tokens back
+    // one token: its output, and its row becomes the newest of the held ones
+    auto emit = [&](int t, const float4& now) {
+        float y[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {                      // tap j reads the row TAPS - 1 - j tokens back
+            const float4 v = held[TAPS - 2 - j];
+            y[0] = fmaf(w[0][j], v.x, y[0]); y[1] = fmaf(w[1][j], v.y, y[1]);
+            y[2] = fmaf(w[2][j], v.z, y[2]); y[3] = fmaf(w[3][j], v.w, y[3]);
+        }
+        y[0] = fmaf(w[0][TAPS - 1], now.x, y[0]); y[1] = fmaf(w[1][TAPS - 1], now.y, y[1]);
+        y[2] = fmaf(w[2][TAPS - 1], now.z, y[2]); y[3] = fmaf(w[3][TAPS - 1], now.w, y[3]);
+#pragma unroll
+        for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
+        if (TAPS > 1) held[0] = now;
+        if (common >= 0) {
+            float* place = shared_values + (size_t)t * mix_heads * head_values + common;
+            if (mode == 1) {
+                *reinterpret_cast<float4*>(place) = make_float4(y[0], y[1], y[2], y[3]);
+            } else {
+                const float4 other = *reinterpret_cast<const float4*>(place);
+                y[0] = (1.0f - blend) * y[0] + blend * other.x; y[1] = (1.0f - blend) * y[1] + blend * other.y;
+                y[2] = (1.0f - blend) * y[2] + blend * other.z; y[3] = (1.0f - blend) * y[3] + blend * other.w;
+            }
+        }
+        store4<TC>(out + (size_t)t * out_stride + c, y);
+    };
+    if (item0 == item1 && t0 - start0 >= TAPS - 1) {
+        // the run lies inside one entry, behind its first TAPS - 1 tokens: no kept rows
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k) held[k] = scaled(t0 - 1 - k);
+        for (int t = t0; t < t1; t += AHEAD) {
+            float4 rows[AHEAD];
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a)
+                if (t + a < t1) rows[a] = scaled(t + a);
+#pragma unroll
+            for (int a = 0; a < AHEAD; ++a)
+                if (t + a < t1) emit(t + a, rows[a]);
+        }
+        return;
+    }
     bool fresh = true;
     // a token among its entry's first TAPS - 1 belongs to the run that holds the entry's first token (see the top): the
     // run before this one may have taken this one's first tokens, and this one may take some behind its end
     const int limit = min(t1 + (TAPS > 1 ? TAPS - 2 : 0), tokens);
-    constexpr int AHEAD = 4;                                      // tokens whose rows are fetched together
-    for (int base = t0; base < limit; base += AHEAD) {
-        float4 rows[AHEAD];
-        int items[AHEAD], starts[AHEAD];
+#pragma unroll 1
+    for (int t = t0; t < limit; ++t) {
+        const int item = token_item[t], start = q_start[item];
+        const int anchor = t - start < TAPS - 1 ? start : t;
+        if (anchor < t0 || anchor >= t1) continue;
+        const float4 now = scaled(t);
+        if (TAPS > 1 && t == start) {
+            float* old = kept + (size_t)item_slot[item] * kept_stride + c;
 #pragma unroll
-        for (int a = 0; a < AHEAD; ++a) {
-            if (base + a < limit) {
-                rows[a] = scaled(base + a);
-                items[a] = token_item[base + a];
+            for (int k = 0; k < TAPS - 1; ++k)
+                held[k] = *reinterpret_cast<const float4*>(old + (size_t)(TAPS - 2 - k) * conv_channels);
+            // new row k is the token at place count - (TAPS - 1) + k of the entry, or the old row k + count
+            const int count = q_start[item + 1] - start;
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k) {
+                const int place = count - (TAPS - 1) + k;
+                float4 v = now;
+                if (place > 0) v = scaled(start + place);
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j)
+                    if (TAPS - 2 - j == k + count) v = held[j];
+                *reinterpret_cast<float4*>(old + (size_t)k * conv_channels) = v;
             }
+        } else if (TAPS > 1 && fresh) {                           // all of these lie in the entry
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k) held[k] = scaled(t - 1 - k);
         }
-#pragma unroll
-        for (int a = 0; a < AHEAD; ++a)
-            if (base + a < limit) starts[a] = q_start[items[a]];
-#pragma unroll
-        for (int a = 0; a < AHEAD; ++a) {
-            const int t = base + a;
-            if (t >= limit) break;
-            const int start = starts[a];
-            const int anchor = t - start < TAPS - 1 ? start : t;
-            if (anchor < t0 || anchor >= t1) continue;
-            const float4 now = rows[a];
-            if (TAPS > 1 && t == start) {
-                float* old = kept + (size_t)item_slot[items[a]] * kept_stride + c;
-#pragma unroll
-                for (int k = 0; k < TAPS - 1; ++k)
-                    held[k] = *reinterpret_cast<const float4*>(old + (size_t)(TAPS - 2 - k) * conv_channels);
-                // new row k is the token at place count - (TAPS - 1) + k of the entry, or the old row k + count
-                const int count = q_start[items[a] + 1] - start;
-#pragma unroll
-                for (int k = 0; k < TAPS - 1; ++k) {
-                    const int place = count - (TAPS - 1) + k;
-                    float4 v = now;
-                    if (place > 0) v = scaled(start + place);
-#pragma unroll
-                    for (int j = 0; j < TAPS - 1; ++j)
-                        if (TAPS - 2 - j == k + count) v = held[j];
-                    *reinterpret_cast<float4*>(old + (size_t)k * conv_channels) = v;
-                }
-            } else if (TAPS > 1 && fresh) {                       // all of these lie in the entry
-#pragma unroll
-                for (int k = 0; k < TAPS - 1; ++k) held[k] = scaled(t - 1 - k);
-            }
-            fresh = false;
-            float y[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int j = 0; j < TAPS - 1; ++j) {                  // tap j reads the row TAPS - 1 - j tokens back
-                const float4 v = held[TAPS - 2 - j];
-                y[0] = fmaf(w[0][j], v.x, y[0]); y[1] = fmaf(w[1][j], v.y, y[1]);
-                y[2] = fmaf(w[2][j], v.z, y[2]); y[3] = fmaf(w[3][j], v.w, y[3]);
-            }
-            y[0] = fmaf(w[0][TAPS - 1], now.x, y[0]); y[1] = fmaf(w[1][TAPS - 1], now.y, y[1]);
-            y[2] = fmaf(w[2][TAPS - 1], now.z, y[2]); y[3] = fmaf(w[3][TAPS - 1], now.w, y[3]);
-#pragma unroll
-            for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
-            if (TAPS > 1) held[0] = now;
-            if (common >= 0) {
-                float* place = shared_values + (size_t)t * mix_heads * head_values + common;
-                if (mode == 1) {
-                    *reinterpret_cast<float4*>(place) = make_float4(y[0], y[1], y[2], y[3]);
-                } else {
-                    const float4 other = *reinterpret_cast<const float4*>(place);
-                    y[0] = (1.0f - blend) * y[0] + blend * other.x; y[1] = (1.0f - blend) * y[1] + blend * other.y;
-                    y[2] = (1.0f - blend) * y[2] + blend * other.z; y[3] = (1.0f - blend) * y[3] + blend * other.w;
-                }
-            }
-            store4<TC>(out + (size_t)t * out_stride + c, y);
-        }
+        fresh = false;
+        emit(t, now);
     }
 }
 
@@ -250,7 +272,7 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
     // quads of channels over runs of tokens, where every boundary between kinds of channels falls between quads
     const int elem = dtype == PS_F32 ? 4 : 2;
     const bool quads = taps <= 4 && conv_channels > 0 && channels % 4 == 0 && conv_channels % 4 == 0 && u_stride % 4 == 0 &&
-                       out_stride % 4 == 0 && kept_stride % 4 == 0 && !((uintptr_t)u & 15) && !((uintptr_t)kept & 15) &&
+                       out_stride % 4 == 0 && kept_stride % 4 == 0 && !((uintptr_t)u & 15) && !((uintptr_t)kept & 15) && !((uintptr_t)weight & 15) &&
                        !((uintptr_t)out & (uintptr_t)(4 * elem - 1)) &&
                        (!mode || (mix_lo % 4 == 0 && head_slot % 4 == 0 && head_values % 4 == 0 &&
                                   !((uintptr_t)shared_values & 15)));
@@ -258,7 +280,7 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
         // runs of 16 tokens re-read (taps - 1) / 16 of the rows; shorter runs where the step has too few for the SMs
         const int columns = (channels / 4 + ps::SHORT_CONV_THREADS - 1) / ps::SHORT_CONV_THREADS;
         int run = 16;
-        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 1184) run >>= 1;
+        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 592) run >>= 1;
         const dim3 grid(columns, (T + run - 1) / run), block(ps::SHORT_CONV_THREADS);
 #define PS_CONV_RUNS(TYPE, TAPS)                                                                                      \
     return ps::launch_pdl(ps::short_conv_runs_kernel<TYPE, TAPS>, grid, block, 0, s, u, u_stride, weight, conv_channels, \

@@ -35,7 +35,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "core": ["embed_norm.cu", "gemm_simt.cu", "attention_simt.cu", "sampling.cu", "host_io.cu", "step_state.cu", "step_build.cu",
              "rotary.cu", "wkv.cu", "embed_pair.cu", "hyper.cu", "latent.cu", "moe.cu", "post_norm.cu", "mingru.cu",
              "short_conv.cu", "gla.cu", "head_mix.cu"],
-    "bf16": ["gemm_skinny.cu", "attention_decode.cu", "attention_prefill.cu"],
+    "bf16": ["gemm_skinny.cu", "attention_decode.cu", "attention_prefill.cu", "attention_rows.cu"],
     "tc": ["gemm_tc.cu", "gemm_rows_tc.cu", "attention_prefill_tc.cu"],
 }
 

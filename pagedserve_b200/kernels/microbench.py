@@ -132,10 +132,11 @@ def _paged_inputs(items, context, kv_heads, head_dim, page, rotate_mb=200, plane
 
 
 def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, window=None, softcap=None,
-                          sink=False, iters=20, planes=2, chunk=None, mixed=False):
+                          sink=False, iters=20, planes=2, chunk=None, mixed=False, as_rows=False, splits=None):
     """One decode token per request over ``context`` keys (bfloat16 split-key kernel); GB/s over the K and V
     bytes a token may see (with one plane: over the rows once).  ``mixed``: a layer whose heads' weights are mixed
-    across heads (every query head meets all values, then the mixing kernel)."""
+    across heads (every query head meets all values, then the mixing kernel).  ``as_rows``: the kernel with the heads of a
+    group (mixed: all heads) as the rows of a tile, a token's keys shared out over ``splits`` CTAs (None: its own rule)."""
     from pagedserve_b200.kernels.ops import Ops
 
     ops = Ops(torch.bfloat16)
@@ -158,6 +159,13 @@ def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, wi
                                    status=status, softcap=softcap, sink=sinks, all_values=mixed)
         if mixed:
             ops.head_mix(every, mix, out, heads, kv_heads, head_dim)
+
+    if as_rows:
+        def run(i):
+            layer = i % layers
+            ops.attention_rows(q, out, pool[:, layer, 0], pool[:, layer, planes - 1], stride, token_item, positions, table,
+                               heads, kv_heads, head_dim, page, window, head_dim ** -0.5, context, softcap=softcap,
+                               sink=sinks, mix=mix if mixed else None, splits=splits)
 
     seconds = _time(run, iters, graph=True)
     seen = min(context, window) if window and window > 0 else context

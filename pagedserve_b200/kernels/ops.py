@@ -101,6 +101,7 @@ _SIGNATURES = {
         "ps_mingru_scan": [_P, _L, _I, _P, _L, _P, _P, _I, _P, _L, _I, _I, _P],
         "ps_short_conv": [_P, _L, _P, _I, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P],
         "ps_sandwich_close": [_P, _P, _I, _I, _P, _F, _F, _P, _P, _I, _P, _P],
+        "ps_sandwich_close_conv": [_P, _P, _I, _I, _P, _F, _F, _P, _I, _P, _L, _P, _P, _I, _P],
         "ps_gla_recurrence": [_P, _L, _P, _P, _P, _I, _F, _F, _P, _F, _F, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P,
                               _L, _I, _I, _I, _I, _P],
         "ps_head_mix": [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P],
@@ -127,6 +128,8 @@ _SIGNATURES = {
         "ps_paged_attention_decode_ex": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I,
                                          _I, _I, _F, _I, _I, _I, _P, _P, _P, _P, _F, _P, _I, _P],
         "ps_shared_position_attention": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P],
+        "ps_attention_rows": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P,
+                              _P, _P],
         "ps_prefill_attention": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F,
                                  _F, _P, _I, _P],
     },
@@ -763,6 +766,63 @@ class Ops:
             scale, _ptr(partial), splits, _stream()), "shared_position_attention")
         return out
 
+    ROWS_KERNEL_WARPS = 4
+    ROWS_KERNEL_HEADS = 16        # rows of the tile
+
+    @staticmethod
+    def _rows_groups(n_kv_heads, mixed):
+        """Key/value heads that a CTA of the heads-as-rows kernel is compiled for."""
+        groups = 1
+        while mixed and groups < n_kv_heads:
+            groups *= 2
+        return groups
+
+    def attention_rows_ok(self, q, out, n_heads, n_kv_heads, head_dim, mixed=False):
+        """Whether :meth:`attention_rows` takes these heads."""
+        rows = n_heads if mixed else n_heads // n_kv_heads
+        return (self.dtype == torch.bfloat16 and rows <= self.ROWS_KERNEL_HEADS and head_dim % 16 == 0 and head_dim <= 128
+                and self._rows_groups(n_kv_heads, mixed) * head_dim <= 256
+                and self._rows_groups(n_kv_heads, mixed) <= (8 if head_dim <= 32 else 4 if head_dim <= 64 else 2)
+                and q.stride(0) % 8 == 0 and out.stride(0) % 4 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 8 == 0)
+
+    def attention_rows_splits(self, T, n_heads, n_kv_heads, head_dim, max_kv_len, mixed=False):
+        """CTAs that share a token's keys: as many as are resident at once, none without a key tile for every warp."""
+        wide = self._rows_groups(n_kv_heads, mixed) * head_dim
+        nbytes = 16 * (head_dim + 8) * 2 + max(self.ROWS_KERNEL_WARPS * 2 * 2 * 16 * (wide + 8) * 2,
+                                               (self.ROWS_KERNEL_WARPS + 1) * 16 * wide * 4)
+        resident = 148 * max(1, min(6, 225_000 // (nbytes + 1024)))
+        ctas, tiles = T * (1 if mixed else n_kv_heads), -(-int(max_kv_len) // 16)
+        splits = 1
+        while splits < 8 and ctas * splits * 2 <= resident and splits * 2 * self.ROWS_KERNEL_WARPS <= tiles:
+            splits *= 2
+        return splits
+
+    def attention_rows(self, q, out, k_pool, v_pool, page_stride, token_item, positions, block_table, n_heads, n_kv_heads,
+                       head_dim, page_size, window, scale, max_kv_len, q_start=None, kv_len=None, token_row=None,
+                       softcap=None, sink=None, mix=None, splits=None):
+        """Attention of single tokens (bfloat16) with the query heads of a group (or, with ``mix``, all query heads) as the
+        rows of one tile: a group's keys are fetched once (csrc/attention_rows.cu).  ``mix`` float32 [n_heads, n_heads]: the
+        heads' weights are mixed by it before they meet the values.  Otherwise as :meth:`paged_attention_decode`."""
+        T = q.shape[0]
+        _require(q, "q", torch.bfloat16)
+        _require(out, "out", torch.bfloat16)
+        if q.shape[1] != n_heads * head_dim or out.shape != q.shape or q.stride(1) != 1 or out.stride(1) != 1:
+            raise KernelError("attention_rows: q and out must be rows of n_heads * head_dim")
+        for name, vector, count in (("sink", sink, n_heads), ("mix", mix, n_heads * n_heads)):
+            if vector is not None:
+                _require(vector, name, torch.float32)
+                if vector.numel() != count or not vector.is_contiguous():
+                    raise KernelError(f"attention_rows: {name} does not fit")
+        if splits is None:
+            splits = self.attention_rows_splits(T, n_heads, n_kv_heads, head_dim, max_kv_len, mix is not None)
+        self.launches += 1
+        _check(self.fast.ps_attention_rows(
+            _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_pool), _ptr(v_pool), page_stride, _ptr(token_item),
+            _ptr(token_row), _ptr(positions), _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), T, n_heads,
+            n_kv_heads, head_dim, page_size, window or 0, scale, splits, float(softcap or 0.0), _ptr(sink), _ptr(mix),
+            _stream()), "attention_rows")
+        return out
+
     @staticmethod
     def prefill_tc_ok(head_dim, page_size, q, out, pool):
         return (head_dim in (64, 128) and 8 <= page_size <= 64 and pool is not None and q.stride(0) % 8 == 0
@@ -796,9 +856,10 @@ class Ops:
         return out
 
     def attention(self, q, k, v, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale,
-                  write_cache=True, softcap=None, sink=None, chunk=None, all_values=False):
-        """Write the step's keys and values into the pages, then attend from the pages.  ``softcap``, ``sink`` and
-        ``all_values`` as in :meth:`paged_attention_simt`.  Besides "no later key", a query sees the last ``window``
+                  write_cache=True, softcap=None, sink=None, chunk=None, mix=None):
+        """Write the step's keys and values into the pages, then attend from the pages.  ``softcap`` and ``sink`` as in
+        :meth:`paged_attention_simt`; ``mix`` float32 [n_heads, n_heads]: the heads' weights are mixed by it before they
+        meet the values (:meth:`head_mix`).  Besides "no later key", a query sees the last ``window``
         keys, or (``chunk`` C instead of a window) the keys j of its own run of C positions,
         ``j // C == i // C``, runs counted from position 0 of the sequence; neither: every earlier key.  Below
         this method the two travel as one integer: the window, or minus the chunk."""
@@ -814,12 +875,13 @@ class Ops:
         if self.dtype == torch.float32 or head_dim % 16 != 0 or head_dim > 256:
             # the CUDA-core kernel takes every head size (up to 1,024); the tensor-core kernels want multiples of 16
             # up to 256
-            return self.paged_attention_simt(q, out, layer.k_pool, layer.v_pool, layer.page_stride,
-                                             ctx.token_slot, ctx.positions, layer.block_table, n_heads,
-                                             n_kv_heads, head_dim, layer.page_size, window, scale, softcap, sink,
-                                             all_values)
+            every = out if mix is None else self.empty((q.shape[0], n_heads * n_kv_heads * head_dim), self.dtype, q.device)
+            self.paged_attention_simt(q, every, layer.k_pool, layer.v_pool, layer.page_stride, ctx.token_slot,
+                                      ctx.positions, layer.block_table, n_heads, n_kv_heads, head_dim, layer.page_size,
+                                      window, scale, softcap, sink, all_values=mix is not None)
+            return out if mix is None else self.head_mix(every, mix, out, n_heads, n_kv_heads, head_dim)
         return tensorcore.attention(self, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale,
-                                    softcap=softcap, sink=sink, all_values=all_values)
+                                    softcap=softcap, sink=sink, mix=mix)
 
     # ------------------------------------------------------------------ rotary positions + cache write
     def rotary_cache_write(self, q, k, v, inv_freq, rot_dims, interleaved, ctx, layer, n_heads, n_kv_heads,
@@ -1159,6 +1221,36 @@ class Ops:
         _check(self.core.ps_sandwich_close(_ptr(y), _ptr(x), T, H, _ptr(gain), float(y_scale), float(eps), _ptr(next_gain),
                                            _ptr(out), dtype_code(out.dtype) if out is not None else PS_F32,
                                            _ptr(row_scale), _stream()), "sandwich_close")
+
+    @staticmethod
+    def close_conv_ok(y, taps, n_taps, state):
+        """Whether :meth:`sandwich_close_conv` takes these sizes."""
+        H = y.shape[1]
+        return (n_taps <= 4 and H % 4 == 0 and H <= 4096 and taps.data_ptr() % 16 == 0
+                and (state is None or (state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0)))
+
+    def sandwich_close_conv(self, y, x, gain, y_scale, eps, taps, n_taps, state, ctx, out):
+        """``sandwich_close`` and, for a step in which every entry brings one token, the :meth:`short_conv` of the new
+        rows divided by their root mean square, in one kernel (csrc/post_norm.cu)."""
+        for name, tensor in (("y", y), ("x", x), ("taps", taps)):
+            _require(tensor, name, torch.float32)
+        T, H = x.shape
+        if (y.shape != x.shape or not (x.is_contiguous() and y.is_contiguous()) or taps.shape != (H, n_taps)
+                or not taps.is_contiguous() or out.shape != x.shape or not out.is_contiguous()
+                or (gain is not None and (gain.numel() != H or not gain.is_contiguous()))):
+            raise KernelError("sandwich_close_conv: shapes do not match")
+        if ctx.num_items != T:
+            raise KernelError("sandwich_close_conv: one token per entry")
+        if n_taps > 1:
+            _require(state, "state", torch.float32)
+            if state.shape[1] != (n_taps - 1) * H or state.stride(1) != 1:
+                raise KernelError("sandwich_close_conv: the state holds taps - 1 rows")
+        self.launches += 1
+        _check(self.core.ps_sandwich_close_conv(
+            _ptr(y), _ptr(x), T, H, _ptr(gain), float(y_scale), float(eps), _ptr(taps), n_taps,
+            _ptr(state) if n_taps > 1 else None, state.stride(0) if n_taps > 1 else 0, _ptr(ctx.item_slot), _ptr(out),
+            dtype_code(out.dtype), _stream()), "sandwich_close_conv")
+        return out
 
     # ------------------------------------------------------------------ heads mixed across heads
     def head_mix(self, every, mix, out, n_heads, n_kv_heads, head_dim):

@@ -51,24 +51,31 @@ def linear(ops, a, w, bias, out, act=None, accumulate=False, status=None):
     return ops.linear_simt(a, w, bias, out, act, accumulate)
 
 
+ROWS_FROM_HEADS = 4            # query heads per key head from which single tokens run with the heads as rows
 SHARED_POSITION_FROM = 8       # short tokens of a step from which heads that share a key head run as query rows
 
 
-def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale, softcap=None, sink=None,
-              all_values=False):
+def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale, softcap=None, sink=None, mix=None):
     """Short entries (fewer than ``ctx.LONG_ENTRY`` tokens: decode tokens, short portions) come first in the
-    step's flat batch and go token by token through the split-key kernel; long portions go through the
+    step's flat batch and go token by token through a kernel for single tokens; long portions go through the
     tensor-core prefill kernel in blocks of 64 queries.  ``softcap``: scores become softcap * tanh(score /
-    softcap); ``sink``: float32 [n_heads], exp(sink[h]) joins the softmax's denominator of head h.
-    ``all_values``: every query head meets the values of every key/value head (``Ops.head_mix`` reads the results)."""
-    all_values = all_values and n_kv_heads > 1
-    columns = n_heads * n_kv_heads if all_values else n_heads
+    softcap); ``sink``: float32 [n_heads], exp(sink[h]) joins the softmax's denominator of head h; ``mix``: float32
+    [n_heads, n_heads], the heads' weights are mixed by it before they meet the values."""
     short_tokens = ctx.num_short_tokens
     long_items = ctx.num_items - ctx.num_short_items
     if long_items and head_dim > 128:
         short_tokens, long_items = ctx.num_tokens, 0
+    # Mixed heads: where a kernel does not mix itself, every query head meets the values of every key/value head and the
+    # mixing kernel adds the results up.
+    every, columns = out, n_heads
+    rows = short_tokens and ops.attention_rows_ok(q, out, n_heads, n_kv_heads, head_dim, mixed=mix is not None)
+    if mix is not None:
+        columns = n_heads * n_kv_heads
+        if long_items or not rows:
+            every = ops.empty((ctx.num_tokens, columns * head_dim), out.dtype, out.device)
+    all_values = mix is not None
     if short_tokens >= SHARED_POSITION_FROM and n_kv_heads == 1 and n_heads >= 4 and head_dim <= 128 \
-            and softcap is None and sink is None and q.is_contiguous() and out.is_contiguous():
+            and softcap is None and sink is None and mix is None and q.is_contiguous() and out.is_contiguous():
         # Every query head reads the one key/value head: the heads of a token become the query rows of one
         # tile of the prompt kernel, all at the token's position, and the token's keys are fetched once instead
         # of once per head; with few tokens the key tiles of a token are shared out over up to 8 CTAs and merged
@@ -79,6 +86,12 @@ def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, sc
                                       layer.page_stride, ctx.positions[:short_tokens], layer.block_table,
                                       ctx.token_slot[:short_tokens], n_heads, head_dim, layer.page_size, window, scale,
                                       max_kv_len=ctx.max_kv_len)
+    elif rows and (mix is not None or n_heads >= ROWS_FROM_HEADS * n_kv_heads):
+        # Groups of several heads (or heads that are mixed): the heads of a token as the rows of one tile.
+        ops.attention_rows(q[:short_tokens], out[:short_tokens], layer.k_pool, layer.v_pool, layer.page_stride,
+                           ctx.token_item[:short_tokens], ctx.positions[:short_tokens], layer.block_table, n_heads,
+                           n_kv_heads, head_dim, layer.page_size, window, scale, ctx.max_kv_len, q_start=ctx.q_start,
+                           kv_len=ctx.kv_len, token_row=ctx.token_slot[:short_tokens], softcap=softcap, sink=sink, mix=mix)
     elif short_tokens:
         # The splits of a (token, head) pair merge through global memory. (With at most one pair per SM the
         # kernel makes one CTA of six teams per pair instead and merges in shared memory: batch 8, 278 -> 259 us
@@ -86,26 +99,29 @@ def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, sc
         # whole clusters costs more than the trip through memory it saves, 354 vs 317 us at batch 8 when measured,
         # and 4,636 vs 4,734 tokens/s at batch 1 against the teams.)
         merge = "global"
-        ops.paged_attention_decode(q[:short_tokens], out[:short_tokens], layer.k_pool, layer.v_pool,
+        ops.paged_attention_decode(q[:short_tokens], every[:short_tokens], layer.k_pool, layer.v_pool,
                                    layer.page_stride, ctx.token_item[:short_tokens], ctx.positions[:short_tokens],
                                    layer.block_table, n_heads, n_kv_heads, head_dim, layer.page_size, window, scale,
                                    ctx.max_kv_len, status=ctx.status, q_start=ctx.q_start, kv_len=ctx.kv_len, merge=merge,
                                    token_row=ctx.token_slot[:short_tokens], softcap=softcap, sink=sink, all_values=all_values)
     if long_items:
-        if ops.prefill_tc_ok(head_dim, layer.page_size, q, out, getattr(layer, "pool", None)):
+        if ops.prefill_tc_ok(head_dim, layer.page_size, q, every, getattr(layer, "pool", None)):
             # blocks of 128 queries: never more than the count of 64-query blocks
             # Two threads per query row halve the chain of each 128-key tile but leave one CTA per SM: worth it
             # when all blocks are resident at once, or nearly so while some block runs over many tiles.
             blocks = -(-ctx.num_long_blocks // 2) * columns          # an upper bound of the 128-query blocks
             two = blocks <= 148 or (blocks <= 296 and ctx.max_kv_len >= 768)
-            ops.prefill_attention_tc(q, out, layer.pool, layer.pool_layer, ctx.q_start, ctx.kv_len, layer.block_table,
+            ops.prefill_attention_tc(q, every, layer.pool, layer.pool_layer, ctx.q_start, ctx.kv_len, layer.block_table,
                                      ctx.num_short_items, long_items, ctx.num_long_blocks, n_heads, n_kv_heads,
                                      head_dim, layer.page_size, window, scale, status=ctx.status,
                                      row_threads=2 if two else 1, item_row=ctx.item_slot, softcap=softcap, sink=sink,
                                      all_values=all_values)
         else:
-            ops.prefill_attention(q, out, layer.k_pool, layer.v_pool, layer.page_stride, ctx.q_start, ctx.kv_len,
+            ops.prefill_attention(q, every, layer.k_pool, layer.v_pool, layer.page_stride, ctx.q_start, ctx.kv_len,
                                   layer.block_table, ctx.num_short_items, long_items, ctx.num_long_blocks, n_heads,
                                   n_kv_heads, head_dim, layer.page_size, window, scale, item_row=ctx.item_slot,
                                   softcap=softcap, sink=sink, all_values=all_values)
+    if mix is not None and every is not out:
+        first = short_tokens if rows else 0
+        ops.head_mix(every[first:], mix, out[first:], n_heads, n_kv_heads, head_dim)
     return out

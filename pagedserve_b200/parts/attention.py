@@ -136,8 +136,8 @@ class RotaryAttention(Mixer):
     difference whether that happens before the turn or behind it.  ``unit_sink``: a one in every head's denominator (a
     sink of score 0 without a tensor).  ``talk_name``: the heads' weights (softmax, sinks in the denominators) are mixed
     across heads before they meet the values, w'_h = sum_g M[h, g] w_g, M the tensor ``talk_name`` [H, H]; head h applies
-    w'_h to the values of its own key/value head.  This is linear in the weights: attention runs with every query head
-    meeting the values of every key/value head, and ``ops.head_mix`` adds the results up.
+    w'_h to the values of its own key/value head.  This is linear in the weights: every query head meets the values of every
+    key/value head, and the results are added up with M's numbers (``ops.attention``: ``mix``).
 
     params: hidden_size, n_heads, n_kv_heads, head_dim, v_dim (head_dim), scale, window, chunk, softcap,
     rotary (dict or None), q_name, k_name, v_name (None: values are the unturned keys), out_name, sink_name (None: no
@@ -334,12 +334,8 @@ class RotaryAttention(Mixer):
                 float(self.head_norm["eps"]) if self.head_norm else 0.0,
                 self.rotary.inv_freq_split(), rotary["dims"], rotary.get("interleaved", True), self.dim, ctx, layer,
                 H, G, D, write_cache=write_cache, amplitude=self.rotary.amplitude)
-        mixes = self.talk is not None
-        result = ops.empty((projected.shape[0], H * G * D), self.env.dtype, projected.device) if mixes else context
-        ops.attention(q, k, v, result, ctx, layer, H, G, D, p.get("window"), float(p["scale"]), write_cache=False,
-                      softcap=p.get("softcap"), sink=self.sink, chunk=p.get("chunk"), all_values=mixes)
-        if mixes:
-            ops.head_mix(result, self.talk, context, H, G, D)
+        ops.attention(q, k, v, context, ctx, layer, H, G, D, p.get("window"), float(p["scale"]), write_cache=False,
+                      softcap=p.get("softcap"), sink=self.sink, chunk=p.get("chunk"), mix=self.talk)
 
     def forward(self, x, residual, ctx, layer):
         p = self.params

@@ -220,13 +220,15 @@ class PostNormBlock(Block):
 
 class SandwichCarrier:
     """What runs through the layers of a model that norms what its sublayers read and what they return: the float32 rows
-    ``x``, the zeroed float32 rows ``y`` a sublayer adds its result into, and ``inverse`` [T]: one over the root mean
-    square of every row of ``x``, which the next layer's first norm needs of it."""
+    ``x``, the float32 rows ``y`` a sublayer adds its result into, ``inverse`` [T] (room for one over the root mean
+    square of every row of ``x``, which a layer's first norm needs), and what the last sublayer has left to do:
+    ``pending`` = (gain of its norm or None, factor on its result, eps)."""
 
-    def __init__(self, x, y, inverse):
+    def __init__(self, x, y, inverse, pending):
         self.x = x
         self.y = y
         self.inverse = inverse
+        self.pending = pending
 
 
 @register_part("block", "sandwich_norm")
@@ -243,8 +245,9 @@ class SandwichNormBlock(Block):
 
     A sublayer adds its result into a zeroed row exactly as it would into the residual row of a pre-norm layer, so every
     mixer and feed-forward works here unchanged.  One kernel (``ops.sandwich_close``) then norms that row, adds it, clears
-    it, and prepares what comes next: the feed-forward's normed rows, or the root mean square that the next layer's
-    convolution kernel (or the model's last norm) applies when it reads the rows.
+    it, and prepares what comes next.  Behind the mixer that is the feed-forward's normed rows.  Behind a layer it is left
+    pending for the next one: in a step of single tokens the same kernel goes on with that layer's convolution, else it
+    forms the root mean square that the convolution's kernel applies when it reads the rows.
 
     params: scales = dict(mixer, feed_forward), conv (None), init_std."""
 
@@ -317,8 +320,7 @@ class SandwichNormBlock(Block):
         ops = self.env.ops
         y = ops.empty(hidden.shape, torch.float32, hidden.device)
         inverse = ops.empty((hidden.shape[0],), torch.float32, hidden.device)
-        ops.sandwich_close(y, hidden, None, 1.0, self.norms["pre_mixer"].params["eps"], row_scale=inverse)
-        return SandwichCarrier(hidden, y, inverse)
+        return SandwichCarrier(hidden, y, inverse, (None, 1.0, self.norms["pre_mixer"].params["eps"]))
 
     def forward(self, hidden, ctx, layer):
         carrier, ops = hidden, self.env.ops
@@ -332,18 +334,24 @@ class SandwichNormBlock(Block):
                 own = state_share(layer, at, layer.state.shape[1] - at) if layer.state.shape[1] > at else layer
         x = carrier.x
         h = ops.empty(x.shape, self.env.dtype, x.device)
-        ops.short_conv(x, taps, self.taps, self.width, kept, ctx, h, row_scale=carrier.inverse)
+        gain, factor, eps = carrier.pending
+        if getattr(ctx, "single_tokens", False) and ops.close_conv_ok(carrier.y, taps, self.taps, kept):
+            ops.sandwich_close_conv(carrier.y, x, gain, factor, eps, taps, self.taps, kept, ctx, h)
+        else:
+            ops.sandwich_close(carrier.y, x, gain, factor, eps, row_scale=carrier.inverse)
+            ops.short_conv(x, taps, self.taps, self.width, kept, ctx, h, row_scale=carrier.inverse)
         self.mixer.forward(h, carrier.y, ctx, own)
         alone = getattr(self.feed_forward, "is_empty", False)
         eps = self.norms["post_mixer"].params["eps"]
         if alone:
-            ops.sandwich_close(carrier.y, x, after_mixer, self.mixer.output_scale, eps, row_scale=carrier.inverse)
+            carrier.pending = (after_mixer, self.mixer.output_scale, eps)
             return
         h = ops.empty(x.shape, self.env.dtype, x.device)
         ops.sandwich_close(carrier.y, x, after_mixer, self.mixer.output_scale, eps,
                            next_gain=self.norms["pre_feed_forward"].weight, out=h)
         self.feed_forward.forward(h, carrier.y, ctx)
-        ops.sandwich_close(carrier.y, x, after_ff, 1.0, eps, row_scale=carrier.inverse)
+        carrier.pending = (after_ff, 1.0, eps)
 
     def end(self, carrier, ctx):
+        self.env.ops.sandwich_close(carrier.y, carrier.x, *carrier.pending)
         return carrier.x

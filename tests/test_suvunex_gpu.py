@@ -361,8 +361,9 @@ def run_layer(block, layer, rows, ctx):
     """The whole layer on residual rows."""
     carrier = block.begin(rows.float().clone(), ctx)
     block.forward(carrier, ctx, layer)
+    rows = block.end(carrier, ctx)
     assert float(carrier.y.abs().max()) == 0.0                       # ready for the next sublayer
-    return block.end(carrier, ctx)
+    return rows
 
 
 def plain_mixer(which, index, fed):
@@ -558,7 +559,7 @@ def test_the_convolution_on_scaled_rows(taps, lengths, width):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("rows,width", [(1, 64), (37, 50), (9, 1024), (5, 2056)])
+@pytest.mark.parametrize("rows,width", [(1, 64), (37, 50), (9, 1024), (5, 2056), (3, 9000), (6, 36)])
 def test_the_close_of_a_sublayer(rows, width, dtype):
     from pagedserve_b200.kernels.ops import Ops
 
@@ -581,6 +582,36 @@ def test_the_close_of_a_sublayer(rows, width, dtype):
     assert float(ys.abs().max()) == 0.0 and rel_err(xs, summed) < 2e-6
 
 
+@pytest.mark.parametrize("taps", [1, 2, 3, 4])
+@pytest.mark.parametrize("rows,width", [(1, 64), (6, 1024), (3, 2052)])
+def test_the_close_and_the_next_convolution_in_one_kernel(rows, width, taps):
+    """Single tokens: the fused kernel leaves what the close and the convolution one after the other leave, the kept rows
+    included, twice in a row."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    g = torch.Generator().manual_seed(width + taps)
+    gain, weight = torch.randn(width, generator=g).to(DEV), torch.randn(width, taps, generator=g).to(DEV)
+    slots = torch.randperm(rows, generator=g).to(torch.int32).to(DEV)
+    state = torch.randn(rows + 1, (taps - 1) * width + 4, generator=g).to(DEV)
+    ctx = SimpleNamespace(token_item=torch.arange(rows, dtype=torch.int32, device=DEV), item_slot=slots, num_items=rows,
+                          q_start=torch.arange(rows + 1, dtype=torch.int32, device=DEV), single_tokens=True)
+    kept_a, kept_b = state.clone(), state.clone()
+    share = lambda kept: kept[:, :(taps - 1) * width] if taps > 1 else None
+    for factor in (0.7, None):
+        x, y = torch.randn(rows, width, generator=g).to(DEV), torch.randn(rows, width, generator=g).to(DEV)
+        xa, ya, xb, yb = x.clone(), y.clone(), x.clone(), y.clone()
+        own = gain if factor is not None else None
+        scale = torch.empty(rows, device=DEV)
+        a, b = (torch.empty(rows, width, dtype=torch.bfloat16, device=DEV) for _ in range(2))
+        ops.sandwich_close(ya, xa, own, factor or 1.0, 1e-5, row_scale=scale)
+        ops.short_conv(xa, weight, taps, width, share(kept_a), ctx, a, row_scale=scale)
+        assert ops.close_conv_ok(yb, weight, taps, share(kept_b))
+        ops.sandwich_close_conv(yb, xb, own, factor or 1.0, 1e-5, weight, taps, share(kept_b), ctx, b)
+        assert rel_err(xb, xa.cpu()) < 1e-6 and float(yb.abs().max()) == 0.0
+        assert rel_err(b.float(), a.float().cpu()) < 5e-3 and rel_err(kept_b, kept_a.cpu()) < 1e-6
+
+
 def paged_case(tokens, positions, kv_heads, dim, page, seed, dtype):
     """A pool of keys and values in shuffled pages and one block-table row per token's request."""
     g = torch.Generator().manual_seed(seed)
@@ -594,7 +625,8 @@ def paged_case(tokens, positions, kv_heads, dim, page, seed, dtype):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("heads,kv_heads,dim,page", [(4, 2, 16, 16), (6, 3, 48, 8), (8, 8, 64, 16), (4, 2, 128, 32), (5, 1, 64, 16),
-                                                     (6, 2, 20, 16), (12, 4, 96, 16)])
+                                                     (6, 2, 20, 16), (12, 4, 96, 16), (20, 4, 32, 16), (16, 4, 64, 16),
+                                                     (16, 8, 32, 8), (12, 3, 64, 16)])
 @pytest.mark.parametrize("form", ["single", "portion"])
 def test_every_query_head_meets_every_value_head(heads, kv_heads, dim, page, form, dtype):
     """Attention with all values and the mixing kernel against the equations: single tokens at many positions, and a
@@ -637,15 +669,49 @@ def test_every_query_head_meets_every_value_head(heads, kv_heads, dim, page, for
                           kv_len=place + 1 if single else torch.tensor([positions[-1] + 1], dtype=torch.int32, device=DEV),
                           item_slot=torch.zeros(items, dtype=torch.int32, device=DEV))
     q = q.to(DEV)
-    every = torch.full((count, heads * kv_heads * dim), 9.0, dtype=dtype, device=DEV)
-    ops.attention(q, None, None, every, ctx, layer, heads, kv_heads, dim, None, scale, write_cache=False, sink=sink.to(DEV),
-                  all_values=True)
     tol = 5e-6 if dtype == torch.float32 else 1.2e-2
+    wide = torch.full((count, heads * dim + 8), 9.0, dtype=dtype, device=DEV)
+    ops.attention(q, None, None, wide[:, :heads * dim], ctx, layer, heads, kv_heads, dim, None, scale, write_cache=False,
+                  sink=sink.to(DEV), mix=talk.to(DEV).contiguous())
+    assert rel_err(wide[:, :heads * dim], want) < tol and bool((wide[:, heads * dim:] == 9.0).all())
+    # the two steps alone, on the kernel that takes every head size
+    every = torch.full((count, heads * kv_heads * dim), 9.0, dtype=dtype, device=DEV)
+    ops.paged_attention_simt(q, every, layer.k_pool, layer.v_pool, layer.page_stride, zeros, place, table, heads, kv_heads, dim,
+                             page, None, scale, sink=sink.to(DEV), all_values=True)
     assert rel_err(every, want_all.reshape(count, -1)) < tol
     out = torch.empty(count, heads * dim, dtype=dtype, device=DEV)
     ops.head_mix(every, talk.to(DEV).contiguous(), out, heads, kv_heads, dim)
     assert rel_err(out, want) < tol
     assert int(ops.status_flag(DEV).item()) == 0
+
+
+@pytest.mark.parametrize("heads,kv_heads,dim,page,window,softcap,with_sink", [
+    (8, 2, 64, 16, None, None, True), (16, 1, 128, 16, None, None, False), (12, 3, 48, 8, 100, None, True),
+    (20, 4, 96, 32, None, 20.0, True), (4, 1, 16, 16, -70, None, False), (32, 2, 32, 16, 33, None, True),
+    (7, 7, 112, 16, None, None, True), (10, 2, 80, 64, None, None, False)])
+@pytest.mark.parametrize("splits", [1, 2, 8, None])
+def test_heads_of_a_group_as_rows(heads, kv_heads, dim, page, window, softcap, with_sink, splits):
+    """Single tokens with the heads of a group as the rows of a tile against the CUDA-core kernel: positions at tile and
+    page borders, windows and chunked masks, capped scores, sinks, and more CTAs than some tokens have key tiles."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    positions = [0, 1, 15, 16, 31, 63, 64, 130, 255, 256, 299, 700]
+    count = len(positions)
+    pool, table, _, _ = paged_case(count, positions, kv_heads, dim, page, seed=dim + heads, dtype=torch.bfloat16)
+    g = torch.Generator().manual_seed(heads)
+    q = (torch.randn(count, heads * dim + 16, generator=g)).to(torch.bfloat16).to(DEV)[:, :heads * dim]
+    sink = torch.randn(heads, generator=g).to(DEV) if with_sink else None
+    zeros, place = torch.zeros(count, dtype=torch.int32, device=DEV), torch.tensor(positions, dtype=torch.int32, device=DEV)
+    own = torch.arange(count, dtype=torch.int32, device=DEV)
+    want, got = torch.empty(count, heads * dim, dtype=torch.bfloat16, device=DEV), torch.empty(count, heads * dim,
+                                                                                           dtype=torch.bfloat16, device=DEV)
+    args = (pool[:, 0, 0], pool[:, 0, 1], pool.stride(0))
+    ops.paged_attention_simt(q, want, *args, zeros, place, table, heads, kv_heads, dim, page, window, dim ** -0.5, softcap, sink)
+    ops.attention_rows(q, got, *args, own, place, table, heads, kv_heads, dim, page, window, dim ** -0.5, max(positions) + 1,
+                       q_start=torch.arange(count + 1, dtype=torch.int32, device=DEV), kv_len=place + 1, token_row=zeros,
+                       softcap=softcap, sink=sink, splits=splits)
+    assert rel_err(got, want.float().cpu()) < 1.2e-2
 
 
 # ------------------------------------------------------------------ a key that stands out, at page borders and far back
