@@ -68,9 +68,15 @@ struct GateForm {
     float alpha;              // kind 1: the sigmoid's slope
 };
 
+// the tanh form of gelu, written 0.5 z (1 + tanh(a)) = z / (1 + exp(-2 a)): no difference of nearly equal numbers where z is
+// negative, and one exponential and one division on the special function units instead of tanhf
+__device__ __forceinline__ float gelu_tanh_sigmoid(float z) {
+    const float a = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return __fdividef(z, 1.0f + __expf(-2.0f * a));
+}
 __device__ __forceinline__ float gated_inner(float g, float u, float w, int kind, float limit, float alpha) {
     if (kind == 0) return silu(g) * u * w;
-    if (kind == 2) return gelu_tanh(g) * u * w;
+    if (kind == 2) return gelu_tanh_sigmoid(g) * u * w;
     g = fminf(g * w, limit);
     u = fminf(fmaxf(u * w, -limit), limit);
     return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);

@@ -102,7 +102,7 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16*
 
 constexpr int SHORT_CONV_THREADS = 128;
 
-template <typename TC, int TAPS>
+template <typename TC, int TAPS, bool SCALED>
 __global__ void __launch_bounds__(SHORT_CONV_THREADS)
 short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ weight,
                        int conv_channels, int channels, const float* __restrict__ row_scale, float* kept,
@@ -138,7 +138,7 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
     shared_values = pdl_fresh(shared_values);
     auto scaled = [&](int t) {
         float4 v = *reinterpret_cast<const float4*>(u + (size_t)t * u_stride + c);
-        if (row_scale) {
+        if constexpr (SCALED) {
             const float f = row_scale[t];
             v.x *= f; v.y *= f; v.z *= f; v.w *= f;
         }
@@ -280,12 +280,14 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
         // runs of 16 tokens re-read (taps - 1) / 16 of the rows; shorter runs where the step has too few for the SMs
         const int columns = (channels / 4 + ps::SHORT_CONV_THREADS - 1) / ps::SHORT_CONV_THREADS;
         int run = 16;
-        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 592) run >>= 1;
+        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 1200) run >>= 1;
         const dim3 grid(columns, (T + run - 1) / run), block(ps::SHORT_CONV_THREADS);
 #define PS_CONV_RUNS(TYPE, TAPS)                                                                                      \
-    return ps::launch_pdl(ps::short_conv_runs_kernel<TYPE, TAPS>, grid, block, 0, s, u, u_stride, weight, conv_channels, \
-                          channels, row_scale, kept, kept_stride, token_item, q_start, item_slot, (TYPE*)out, out_stride, mode,     \
-                          mix_lo, mix_heads, head_slot, head_values, shared_values, mix, T, run)
+    return ps::launch_pdl(row_scale ? ps::short_conv_runs_kernel<TYPE, TAPS, true>                                     \
+                                    : ps::short_conv_runs_kernel<TYPE, TAPS, false>,                                    \
+                          grid, block, 0, s, u, u_stride, weight, conv_channels, channels, row_scale, kept, kept_stride, \
+                          token_item, q_start, item_slot, (TYPE*)out, out_stride, mode, mix_lo, mix_heads, head_slot,   \
+                          head_values, shared_values, mix, T, run)
 #define PS_CONV_TAPS(TYPE)                                                                                            \
     switch (taps) {                                                                                                   \
         case 1: PS_CONV_RUNS(TYPE, 1);                                                                                \

@@ -1270,17 +1270,21 @@ class Ops:
         return out
 
     # ------------------------------------------------------------------ gated linear attention
-    GLA_CTAS = 592                # CTAs that the recurrence of prompt portions is cut into at most, about
-    GLA_RUN = 64                  # and tokens of a run at least
+    GLA_RUN = 32                  # tokens of a run at least
     GLA_SCRATCH_BYTES = 256 << 20
 
     def gla_segments(self, ctx, heads, dk, dv):
-        """Runs that a prompt portion is cut into: enough CTAs to fill the GPU, no run shorter than GLA_RUN tokens."""
+        """Runs that a prompt portion is cut into: as many CTAs as are resident at once (512 threads an SM, which is what
+        the registers allow), no run shorter than GLA_RUN tokens.  us for 2 x 1,024 tokens: 16 heads of 64: 1 / 4 / 8 / 16 /
+        32 runs 411 / 198 / 111 / 70 / 70; 16 heads of 128 (a CTA fills an SM): 674 / 216 / 221 / 240 / 252."""
         long_items = ctx.num_items - ctx.num_short_items
         longest = int(ctx.max_q_len)
         if long_items <= 0 or longest < 2 * self.GLA_RUN or max(dk, dv) > 128:
             return 1
-        wanted = min(self.GLA_CTAS // max(1, long_items * heads), longest // self.GLA_RUN,
+        padded = lambda size: 32 if size <= 32 else 64 if size <= 64 else 128
+        threads = padded(dk) // 8 * (padded(dv) // 4)
+        resident = 148 * max(1, 512 // threads)
+        wanted = min(resident // (long_items * heads), longest // self.GLA_RUN,
                      self.GLA_SCRATCH_BYTES // (4 * long_items * heads * dk * (dv + 1)))
         return max(1, min(64, wanted))
 
