@@ -135,8 +135,8 @@ class RotaryAttention(Mixer):
     ``head_norm`` without names divides by the root mean square alone; a turn keeps a head's length, so it makes no
     difference whether that happens before the turn or behind it.  ``unit_sink``: a one in every head's denominator (a
     sink of score 0 without a tensor).  ``talk_name``: the heads' weights (softmax, sinks in the denominators) are mixed
-    across heads before they meet the values, w'_h = sum_g M[h, g] w_g, M the tensor ``talk_name`` [H, H]; head h applies
-    w'_h to the values of its own key/value head.  This is linear in the weights: every query head meets the values of every
+    across heads before they meet the values, w'_h = sum_g M[h, g] w_g, M the tensor ``talk_name`` [H, H]; which values
+    head h weighs stays a matter of its group.  This is linear in the weights: every query head meets the values of every
     key/value head, and the results are added up with M's numbers (``ops.attention``: ``mix``).
 
     params: hidden_size, n_heads, n_kv_heads, head_dim, v_dim (head_dim), scale, window, chunk, softcap,

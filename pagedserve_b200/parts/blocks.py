@@ -235,10 +235,10 @@ class SandwichCarrier:
 class SandwichNormBlock(Block):
     """x <- x + s1 * post(mixer(c(pre(x)))); x <- x + s2 * post(feed_forward(pre(x))): norms before and after each
     sublayer (four RMS norms without a mean; gains of one number or of the row's width), ``s1`` and ``s2`` a factor per
-    coordinate (``scales``: the tensors' names), and, with ``conv`` = dict(taps, name), c(h) = h + conv(h): a causal
-    convolution over time on each channel, conv(h)_t = sum_j w[:, j] h_(t - taps + 1 + j) with zeros before the
-    sequence's start; w [W, taps].  A layer whose feed-forward is the ``none`` part has the first sublayer only.  The
-    residual rows, norms, sums and the convolution are float32; a sublayer reads rows of the compute type.
+    coordinate (``scales``: the tensors' names), and, with ``conv`` = dict(taps, name), c(h)_t = h_t + sum over d < taps of
+    w[:, taps - 1 - d] h_(t-d), channel by channel, rows before position 0 taken as zero; w [W, taps].  A layer whose
+    feed-forward is the ``none`` part has the first sublayer only.  The residual rows, norms, sums and the convolution are
+    float32; a sublayer reads rows of the compute type.
 
     A request keeps, in every layer, the last taps - 1 rows that the convolution read (float32, divided by their root
     mean square, without the gain, which is folded into the taps) in front of the mixer's own state.

@@ -15,13 +15,13 @@ class GatedLinearAttention(Mixer):
     is alpha = sigmoid(z)^(1 / tau), z = W_a2 (W_a1 x) + b, a number in (0, 1).  Per head, with S a dim x v_dim matrix that
     starts at zero:
 
-        S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,        o_t = S_t^T q_t
+        S[i, j] <- alpha[i] S[i, j] + k[i] v[j],        o[j] = sum_i q[i] S[i, j]
 
     Each head's o is divided by its root mean square and multiplied by a gain of v_dim numbers (one for all heads), the
     heads are joined, multiplied by silu(W_g x), and W_o adds the result into the residual row.
 
-    A request keeps S (float32) in its slot, so a step runs only the tokens it brings: a prompt portion runs its tokens in
-    order from the stored state, a decode step is a portion of one token.  The projections (W_a1's too) are one product in
+    A request keeps S (float32) in its slot: a prompt portion runs its tokens in order from the stored state and leaves the
+    new one there, a decode step is a portion of one token.  The projections (W_a1's too) are one product in
     the compute type; everything behind it, from the decay's argument on, is float32 (csrc/gla.cu).
 
     params: hidden_size, n_heads, head_dim, v_dim, tau, eps, random_decay_rank (the inner size of W_a1 / W_a2, which only a

@@ -163,7 +163,7 @@ def gated_ff(tensors, prefix, h):
 
 
 def with_convolution(h, w):
-    """h + conv(h): conv(h)_t = sum_j w[:, j] h_(t - taps + 1 + j), zeros before the first token."""
+    """Every row plus the ``taps`` newest rows (itself included, none before the first token) weighed by w, newest last."""
     taps = w.shape[1]
     out = h.clone()
     for t in range(h.shape[0]):

@@ -195,7 +195,7 @@ def test_portions_of_every_size(which, dtype):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("which", ["a", "b", "c", "d"])
 def test_mixed_batches_reuse_pages_and_slots(which, dtype):
-    """Nine unequal requests through four slots: portions of some beside single tokens of others, requests left
+    """Nine unequal requests through four slots: prompts in portions next to decoded tokens, requests left
     out of steps, pages and state slots handed out again; every request must equal itself alone."""
     sequences = sequences_for(which, [90, 33, 200, 5, 61, 148, 17, 75, 2], seed=30)
     steps = helpers.trace_mixed(sequences, seed=3, live=4, decode_tail=20, max_portion=40)
