@@ -15,3 +15,4 @@ from pagedserve_b200.config.tefopel import TefopelConfig  # noqa: F401
 from pagedserve_b200.config.zositar import ZositarConfig  # noqa: F401
 from pagedserve_b200.config.pagatar import PagatarConfig  # noqa: F401
 from pagedserve_b200.config.suvunex import SuvunexConfig  # noqa: F401
+from pagedserve_b200.config.vozirax import VoziraxConfig  # noqa: F401

@@ -27,6 +27,11 @@
 #define PS_ACT_SILU 4
 #define PS_ACT_TANH 5
 
+// what a product does with its result, in its `accumulate` argument: add it to a float32 output instead of storing it; and
+// what its vector of one number per column (`bias`) is, a factor on the column instead of a summand
+#define PS_ACCUMULATE 1
+#define PS_COLUMN_FACTOR 2
+
 #define PS_EXPORT extern "C" __attribute__((visibility("default")))
 
 namespace ps {
@@ -105,6 +110,26 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
+}
+
+// two float32 numbers in one 64-bit register, multiplied and added as a pair
+__device__ __forceinline__ unsigned long long pair_of(float lo, float hi) {
+    unsigned long long p;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(lo), "f"(hi));
+    return p;
+}
+__device__ __forceinline__ void pair_split(unsigned long long p, float& lo, float& hi) {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(p));
+}
+__device__ __forceinline__ unsigned long long pair_mul(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ unsigned long long pair_fma(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
 }
 
 // Extras of the attention softmax, in the units the tensor-core kernels work in (scores times log2 e):

@@ -1,4 +1,4 @@
-// Embedding gather (token table + optional learned position table) and LayerNorm.
+// Embedding gather (token table + optional learned position table, or sines of the position) and LayerNorm.
 //
 // The residual stream is float32 in every mode: the sum of the two embeddings,
 // every residual add and all norm statistics are 32-bit.
@@ -32,6 +32,116 @@ __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict_
         if (q) v += to_float(q[c]);
         out[(size_t)t * H + c] = v;
     }
+}
+
+// h[t] = wte[id_t] + sinusoids of the position: number 2i is sin(p f_i), number 2i + 1 is cos(p f_i).  The angle is formed to
+// more than one float: f_i comes as (high, low) parts, the product's rounding error is recovered with an fma, and what the
+// float that sincosf takes cannot hold is applied to first order.
+template <typename T>
+__global__ void embed_sinusoid_kernel(const int* __restrict__ ids, const int* __restrict__ pos, const T* __restrict__ wte,
+                                      const float2* __restrict__ freq, float* __restrict__ out, int H, int V,
+                                      int* __restrict__ status) {
+    pdl_prologue();
+    ids = pdl_fresh(ids);
+    pos = pdl_fresh(pos);
+    const int t = blockIdx.x, id = ids[t];
+    const float p = (float)pos[t];
+    const bool bad = id < 0 || id >= V;
+    if (bad && threadIdx.x == 0 && blockIdx.y == 0 && status) atomicExch(status, 1);
+    const T* e = wte + (size_t)(bad ? 0 : id) * H;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; 2 * i < H; i += gridDim.y * blockDim.x) {
+        const int c = 2 * i;
+        const float a = to_float(e[c]), b = c + 1 < H ? to_float(e[c + 1]) : 0.f;
+        const float2 f = freq[i];
+        const float high = p * f.x, low = fmaf(p, f.x, -high) + p * f.y;
+        float sn, cs;
+        sincosf(high, &sn, &cs);
+        out[(size_t)t * H + c] = bad ? 0.f : a + fmaf(low, cs, sn);
+        if (c + 1 < H) out[(size_t)t * H + c + 1] = bad ? 0.f : b + fmaf(-low, sn, cs);
+    }
+}
+
+// Two RMS norms of the same row with gains of their own, out_a = n(x) gain_a and out_b = n(x) gain_b: one warp per row held in
+// registers (H <= 128 * WMAX, a multiple of four, 16-byte addresses), or one CTA per row of any width (WMAX 0).
+template <typename TOut, int WMAX>
+__global__ void __launch_bounds__(256)
+rms_norm_pair_kernel(const float* __restrict__ x, const float* __restrict__ gain_a, const float* __restrict__ gain_b, float eps,
+                     TOut* __restrict__ out_a, TOut* __restrict__ out_b, int n_rows, int H) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const float inv_h = 1.0f / (float)H;
+    if constexpr (WMAX > 0) {
+        const int quads = H >> 2;
+        pdl_prologue();
+        x = pdl_fresh(x);
+        const int r = blockIdx.x * (blockDim.x >> 5) + warp;
+        if (r >= n_rows) return;
+        const float4* xr = reinterpret_cast<const float4*>(x + (size_t)r * H);
+        float4 v[WMAX];
+        float sq = 0.f;
+#pragma unroll
+        for (int i = 0; i < WMAX; ++i) {
+            const int c = lane + 32 * i;
+            v[i] = c < quads ? xr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < WMAX; ++i) sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+        const float inverse = 1.0f / sqrtf(warp_sum(sq) * inv_h + eps);
+        auto put = [&](TOut* out, const float* gain) {
+#pragma unroll
+            for (int i = 0; i < WMAX; ++i) {
+                const int c = lane + 32 * i;
+                if (c < quads) {
+                    const float4 g = reinterpret_cast<const float4*>(gain)[c];
+                    const float y0 = v[i].x * inverse * g.x, y1 = v[i].y * inverse * g.y;
+                    const float y2 = v[i].z * inverse * g.z, y3 = v[i].w * inverse * g.w;
+                    if constexpr (sizeof(TOut) == 2) {
+                        __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
+                        *reinterpret_cast<uint2*>(out + (size_t)r * H + 4 * c) =
+                            make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+                    } else {
+                        *reinterpret_cast<float4*>(out + (size_t)r * H + 4 * c) = make_float4(y0, y1, y2, y3);
+                    }
+                }
+            }
+        };
+        put(out_a, gain_a);
+        put(out_b, gain_b);
+    } else {
+        __shared__ float red[8];
+        pdl_prologue();
+        x = pdl_fresh(x);
+        const size_t base = (size_t)blockIdx.x * H;
+        float sq = 0.f;
+        for (int c = threadIdx.x; c < H; c += blockDim.x) sq = fmaf(x[base + c], x[base + c], sq);
+        sq = warp_sum(sq);
+        if (lane == 0) red[warp] = sq;
+        __syncthreads();
+        float total = 0.f;
+        for (int w = 0; w < (int)(blockDim.x >> 5); ++w) total += red[w];
+        const float inverse = 1.0f / sqrtf(total * inv_h + eps);
+        for (int c = threadIdx.x; c < H; c += blockDim.x) {
+            const float n = x[base + c] * inverse;
+            out_a[base + c] = from_float<TOut>(n * gain_a[c]);
+            out_b[base + c] = from_float<TOut>(n * gain_b[c]);
+        }
+    }
+}
+
+template <typename TOut>
+int launch_rms_norm_pair(const float* x, const float* gain_a, const float* gain_b, float eps, TOut* out_a, TOut* out_b,
+                         int n_rows, int H, cudaStream_t s) {
+    // (which form runs depends on the width and the alignment alone)
+    const bool aligned = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)gain_a | (uintptr_t)gain_b | (uintptr_t)out_a |
+                                         (uintptr_t)out_b) & 15) == 0;
+    if (aligned && H <= 2048) {
+        const int warps = n_rows <= 256 ? 2 : 8;
+        const dim3 grid((n_rows + warps - 1) / warps), block(32 * warps);
+        if (H <= 1024)
+            return launch_pdl(rms_norm_pair_kernel<TOut, 8>, grid, block, 0, s, x, gain_a, gain_b, eps, out_a, out_b, n_rows, H);
+        return launch_pdl(rms_norm_pair_kernel<TOut, 16>, grid, block, 0, s, x, gain_a, gain_b, eps, out_a, out_b, n_rows, H);
+    }
+    return launch_pdl(rms_norm_pair_kernel<TOut, 0>, dim3(n_rows), dim3(256), 0, s, x, gain_a, gain_b, eps, out_a, out_b,
+                      n_rows, H);
 }
 
 // One CTA per row. Row kept in registers when H <= NT*MAXV, else re-read.
@@ -215,6 +325,38 @@ PS_EXPORT int ps_embed(const int* ids, const int* pos, const void* wte, const vo
     if (dtype == PS_BF16)
         return ps::launch_pdl(ps::embed_kernel<__nv_bfloat16>, dim3(T), dim3(nt), 0, s, ids, pos,
                               (const __nv_bfloat16*)wte, (const __nv_bfloat16*)wpe, out, H, V, P, status);
+    return PS_ERR_UNSUPPORTED;
+}
+
+// As ps_embed with sines and cosines of the position instead of a table; freq float32 [ceil(H / 2)][2] (high, low) parts.
+PS_EXPORT int ps_embed_sinusoid(const int* ids, const int* pos, const void* wte, const float* freq, float* out, int T, int H,
+                                int V, int dtype, int* status, void* stream) {
+    if (T <= 0) return PS_OK;
+    if (H <= 0 || V <= 0 || !ids || !pos || !wte || !freq || !out || ((uintptr_t)freq & 7)) return PS_ERR_BAD_ARGUMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int pairs = (H + 1) / 2, nt = 128;
+    // a few tokens: a token's numbers over several CTAs
+    const dim3 grid(T, T >= 512 ? 1 : (pairs + nt - 1) / nt);
+    if (dtype == PS_F32)
+        return ps::launch_pdl(ps::embed_sinusoid_kernel<float>, grid, dim3(nt), 0, s, ids, pos, (const float*)wte,
+                              (const float2*)freq, out, H, V, status);
+    if (dtype == PS_BF16)
+        return ps::launch_pdl(ps::embed_sinusoid_kernel<__nv_bfloat16>, grid, dim3(nt), 0, s, ids, pos,
+                              (const __nv_bfloat16*)wte, (const float2*)freq, out, H, V, status);
+    return PS_ERR_UNSUPPORTED;
+}
+
+// out_a = rms_norm(x) * gain_a, out_b = rms_norm(x) * gain_b; x float32 [n_rows, H], gains float32 [H]
+PS_EXPORT int ps_rms_norm_pair(const float* x, int n_rows, int H, const float* gain_a, const float* gain_b, float eps,
+                               void* out_a, void* out_b, int out_dtype, void* stream) {
+    if (n_rows <= 0) return PS_OK;
+    if (H <= 0 || !x || !gain_a || !gain_b || !out_a || !out_b) return PS_ERR_BAD_ARGUMENT;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (out_dtype == PS_F32)
+        return ps::launch_rms_norm_pair<float>(x, gain_a, gain_b, eps, (float*)out_a, (float*)out_b, n_rows, H, s);
+    if (out_dtype == PS_BF16)
+        return ps::launch_rms_norm_pair<__nv_bfloat16>(x, gain_a, gain_b, eps, (__nv_bfloat16*)out_a, (__nv_bfloat16*)out_b,
+                                                       n_rows, H, s);
     return PS_ERR_UNSUPPORTED;
 }
 

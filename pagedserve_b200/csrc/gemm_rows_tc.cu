@@ -292,7 +292,7 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             if (n >= N) continue;
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                v[j] += b[j];
+                v[j] = (accumulate & PS_COLUMN_FACTOR) ? v[j] * b[j] : v[j] + b[j];
                 if (act == PS_ACT_GELU_TANH) v[j] = sizeof(TOut) == 2 ? gelu_tanh_fast(v[j]) : gelu_tanh(v[j]);
                 else if (act != PS_ACT_NONE) v[j] = apply_act(v[j], act);
             }
@@ -326,7 +326,7 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             if (out_vector) {
                 if constexpr (sizeof(TOut) == 4) {
                     float4 o = make_float4(v[0], v[1], v[2], v[3]);
-                    if (accumulate) {
+                    if (accumulate & PS_ACCUMULATE) {
                         const float4 old = *reinterpret_cast<const float4*>(dst);
                         o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w;
                     }
@@ -341,7 +341,7 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             } else {
                 for (int j = 0; j < 4 && n + j < N; ++j) {
                     float x = v[j];
-                    if (accumulate) x += to_float(dst[j]);
+                    if (accumulate & PS_ACCUMULATE) x += to_float(dst[j]);
                     dst[j] = from_float<TOut>(x);
                 }
             }
@@ -443,7 +443,7 @@ PS_EXPORT int ps_gemm_rows_tc(const void* A, int lda, const void* W, int ldw, co
     if (K <= 0 || K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0 || lda < K || ldw < K || ldo < N)
         return PS_ERR_UNSUPPORTED;
     if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return PS_ERR_UNSUPPORTED;
-    if (accumulate && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
+    if ((accumulate & PS_ACCUMULATE) && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
     if (splits == 0) splits = ps::rows::pick_splits(N, K);
     if (splits != 1 && splits != 2 && splits != 4 && splits != 8) return PS_ERR_BAD_ARGUMENT;
     ps::KvScatter kv = {};

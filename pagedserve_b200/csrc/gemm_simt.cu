@@ -65,10 +65,10 @@ gemm_simt_kernel(const TIn* __restrict__ A, int lda, const TIn* __restrict__ W, 
             int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if (bias) v += bias[n];
+            if (bias) v = (accumulate & PS_COLUMN_FACTOR) ? v * bias[n] : v + bias[n];
             v = apply_act(v, act);
             size_t o = (size_t)m * ldo + n;
-            if (accumulate) v += to_float(out[o]);
+            if (accumulate & PS_ACCUMULATE) v += to_float(out[o]);
             out[o] = from_float<TOut>(v);
         }
     }
@@ -84,13 +84,14 @@ int launch_gemm_simt(const void* A, int lda, const void* W, int ldw, const float
 
 }  // namespace ps
 
-// in_dtype: dtype of A and W. out_dtype: dtype of out. accumulate: out += result (out must be f32).
+// in_dtype: dtype of A and W. out_dtype: dtype of out. accumulate: PS_ACCUMULATE: out += result (out must be f32);
+// PS_COLUMN_FACTOR: the numbers of `bias` multiply the columns.
 PS_EXPORT int ps_gemm_simt(const void* A, int lda, const void* W, int ldw, const float* bias, void* out,
                            int ldo, int M, int N, int K, int in_dtype, int out_dtype, int act,
                            int accumulate, void* stream) {
     if (M <= 0 || N <= 0) return PS_OK;
     if (K <= 0 || lda < K || ldw < K || ldo < N) return PS_ERR_BAD_ARGUMENT;
-    if (accumulate && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
+    if ((accumulate & PS_ACCUMULATE) && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     using bf = __nv_bfloat16;
     if (in_dtype == PS_F32 && out_dtype == PS_F32)

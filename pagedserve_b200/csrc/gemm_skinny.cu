@@ -130,7 +130,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bflo
         for (int j = 0; j < EPT; ++j) {
             const int e = threadIdx.x + j * WARPS * 32;
             const int n = n0 + (e & 15), m = e >> 4;
-            prev[j] = (accumulate && e < 16 * TOK && m < M && n < N) ? to_float(out[(size_t)m * ldo + n - n_shift]) : 0.f;
+            prev[j] = ((accumulate & PS_ACCUMULATE) && e < 16 * TOK && m < M && n < N) ? to_float(out[(size_t)m * ldo + n - n_shift]) : 0.f;
         }
     };
     // the bias of this thread's output column (the same in every epilogue round: the CTA's thread count is a
@@ -189,7 +189,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bflo
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) v += red[(size_t)w * 16 * TOK + r * TOK + m];
-        v += bias_mine;
+        v = (accumulate & PS_COLUMN_FACTOR) ? v * bias_mine : v + bias_mine;
         v = apply_act(v, act);
         if (kv.k_pool && n >= kv.q_width) {        // a key or value column: into the row's page
             const KvColumn col = kv_column(kv, n, N);
@@ -505,7 +505,7 @@ gemm_skinny_fused_kernel(NormInput in, const __nv_bfloat16* __restrict__ W, int 
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) v += red[(size_t)w * 16 * TOK + r * TOK + m];
-        v += bias_mine;
+        v = (accumulate & PS_COLUMN_FACTOR) ? v * bias_mine : v + bias_mine;
         v = apply_act(v, act);
         if (kv_col.which) {
             const long long base = dst_s[m];
@@ -513,7 +513,7 @@ gemm_skinny_fused_kernel(NormInput in, const __nv_bfloat16* __restrict__ W, int 
             continue;
         }
         size_t o = (size_t)m * ldo + n;
-        if (accumulate) v += to_float(out[o]);
+        if (accumulate & PS_ACCUMULATE) v += to_float(out[o]);
         out[o] = from_float<TOut>(v);
     }
 }
@@ -570,7 +570,7 @@ PS_EXPORT int ps_gemm_skinny(const void* A, int lda, const void* W, int ldw, con
     if (K <= 0 || K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0 || lda < K || ldw < K || ldo < N)
         return PS_ERR_UNSUPPORTED;
     if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return PS_ERR_UNSUPPORTED;
-    if (accumulate && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
+    if ((accumulate & PS_ACCUMULATE) && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
     if (k_pool && (q_width + 2 * kv_width != N || head_dim <= 0 || kv_width % head_dim != 0 || page_size <= 0))
         return PS_ERR_BAD_ARGUMENT;
     ps::KvScatter kv{(__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, page_stride, token_item, positions, block_table,
@@ -622,7 +622,7 @@ PS_EXPORT int ps_gemm_skinny_fused(const float* x, int ldx, const int* rows, con
     if (K <= 0 || K % 8 != 0 || ldx % 4 != 0 || ldw % 8 != 0 || ldx < K || ldw < K || ldo < N) return PS_ERR_UNSUPPORTED;
     if (((uintptr_t)x & 15) || ((uintptr_t)W & 15) || ((uintptr_t)gamma & 15) || ((uintptr_t)beta & 15))
         return PS_ERR_UNSUPPORTED;
-    if (accumulate && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
+    if ((accumulate & PS_ACCUMULATE) && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
     if (k_pool && (q_width + 2 * kv_width != N || head_dim <= 0 || kv_width % head_dim != 0 || page_size <= 0))
         return PS_ERR_BAD_ARGUMENT;
     ps::NormInput in{x, ldx, rows, gamma, beta, eps, has_mean};

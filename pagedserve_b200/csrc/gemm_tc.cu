@@ -353,8 +353,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(rr[j]);
                         if (bias) {
                             const float mine = bias_lane[group * (COLS / 32) + half];
+                            if (accumulate & PS_COLUMN_FACTOR) {
 #pragma unroll
-                            for (int j = 0; j < 32; ++j) v[j] += __shfl_sync(0xffffffffu, mine, j);
+                                for (int j = 0; j < 32; ++j) v[j] *= __shfl_sync(0xffffffffu, mine, j);
+                            } else {
+#pragma unroll
+                                for (int j = 0; j < 32; ++j) v[j] += __shfl_sync(0xffffffffu, mine, j);
+                            }
                         }
                         if (act == PS_ACT_GELU_TANH) {
 #pragma unroll
@@ -402,7 +407,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                         // (key and value columns of a scattering q|k|v product were written by the rows themselves;
                         // the query width is a multiple of the 64-column group, so a group is all one or the other)
                         if (n0 + c < N && !(sizeof(TOut) == 2 && kv.k_pool && n0 + c >= kv.q_width)) {
-                            if (accumulate) tma_reduce_add_2d(&map_out, stage_buf, n0 + c, m0);
+                            if (accumulate & PS_ACCUMULATE) tma_reduce_add_2d(&map_out, stage_buf, n0 + c, m0);
                             else tma_store_2d(&map_out, stage_buf, n0 + c, m0);
                         }
                         asm volatile("cp.async.bulk.commit_group;" ::: "memory");
@@ -430,7 +435,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                     float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
-                    if (bias) {
+                    if (bias && (accumulate & PS_COLUMN_FACTOR)) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j)
+                            if (n + j < N) v[j] *= bias[n + j];
+                    } else if (bias) {
                         if (full_chunk && ((((uintptr_t)(bias + n)) & 15) == 0)) {
 #pragma unroll
                             for (int j = 0; j < 32; j += 4) {
@@ -470,7 +479,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             for (int j = 0; j < 32; j += 4) {
                                 float4* dst = reinterpret_cast<float4*>(orow + n + j);
                                 float4 o = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
-                                if (accumulate) {
+                                if (accumulate & PS_ACCUMULATE) {
                                     float4 old = *dst;
                                     o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w;
                                 }
@@ -481,7 +490,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             for (int j = 0; j < 32; ++j) {
                                 if (n + j < N) {
                                     float x = v[j];
-                                    if (accumulate) x += to_float(orow[n + j]);
+                                    if (accumulate & PS_ACCUMULATE) x += to_float(orow[n + j]);
                                     orow[n + j] = from_float<TOut>(x);
                                 }
                             }
@@ -657,7 +666,7 @@ static int gemm_tc_entry(const void* A, int lda, const void* W, int ldw, const f
     if (K <= 0 || K % 8 != 0 || lda % 8 != 0 || ldw % 8 != 0 || lda < K || ldw < K || ldo < N)
         return PS_ERR_UNSUPPORTED;
     if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return PS_ERR_UNSUPPORTED;
-    if (accumulate && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
+    if ((accumulate & PS_ACCUMULATE) && out_dtype != PS_F32) return PS_ERR_BAD_ARGUMENT;
     if (ex.tile_expert && ex.k_per_expert % 8 != 0) return PS_ERR_UNSUPPORTED;      // TMA: x in units of 16 bytes
     if (cg.groups && (cg.a_cols % 8 != 0 || ex.tile_expert || kv.k_pool || bias || accumulate)) return PS_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;

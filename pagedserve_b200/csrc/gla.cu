@@ -45,26 +45,6 @@ __device__ __forceinline__ float gla_silu(float x) { return __fdividef(x, 1.0f +
 // log(sigmoid(z)) without overflow at either end
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
-// two float32 numbers in one 64-bit register, multiplied and added as a pair
-__device__ __forceinline__ unsigned long long pair_of(float lo, float hi) {
-    unsigned long long p;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(p) : "f"(lo), "f"(hi));
-    return p;
-}
-__device__ __forceinline__ void pair_split(unsigned long long p, float& lo, float& hi) {
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(p));
-}
-__device__ __forceinline__ unsigned long long pair_mul(unsigned long long a, unsigned long long b) {
-    unsigned long long d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-__device__ __forceinline__ unsigned long long pair_fma(unsigned long long a, unsigned long long b, unsigned long long c) {
-    unsigned long long d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-
 // elements of one 16-byte access, as floats
 __device__ __forceinline__ void gla_unpack(const uint4& raw, float (&x)[4]) {
     x[0] = __uint_as_float(raw.x); x[1] = __uint_as_float(raw.y); x[2] = __uint_as_float(raw.z); x[3] = __uint_as_float(raw.w);

@@ -3,11 +3,12 @@
 // moe_route, one CTA per token, float32 throughout:
 //     z = W_router h                    (E numbers; the operands may be bfloat16, sums are float32)
 //     s = softmax(z) over all E experts, or s = sigmoid(z) expert by expert (score_kind 1)
-//     with groups: the experts are `groups` runs of E / groups neighbours; a group's mark is its largest s; only
-//     experts of the `keep` groups with the largest marks stand for election
+//     with groups: the experts are `groups` runs of E / groups neighbours; a group's mark is its largest s, or
+//     (mark_kind 1) the sum of its two largest s + correction; only experts of the `keep` groups with the largest
+//     marks stand for election
 //     the `top` largest s among them are chosen (ties: the lower index), and their weights are s / (sum of the
-//     chosen s + 1e-20), or the chosen s themselves (normalize 0); the lanes of one warp hold the scores and run
-//     every round together
+//     chosen s + 1e-20), or the chosen s themselves (normalize 0), times a constant; the lanes of one warp hold the
+//     scores and run every round together
 //     shared gate: sigmoid(w_sg . h), one number per token (where the layer has a shared expert)
 // Results: dense weights [T, E] (0 where an expert is not chosen), the chosen experts and their weights
 // [T, top], and the shared gate [T].
@@ -19,6 +20,8 @@
 //     kind 1:  g' = min(w g, limit), u' = clamp(w u, -limit, limit);  g' * sigmoid(alpha g') * (u' + 1)
 //              (the weight scales the expert's input: without biases W (w h) = w (W h), so it is applied to the
 //              pre-activations in float32; the shared expert's columns have a limit of their own)
+// An expert without a gate (kind 3) has one block of F columns in the stacked product: inner = max(u, 0)^2 * w.  With
+// sorted rows its activation is the first product's own epilogue, and the weight joins in moe_combine.
 // moe_gate_mul: inner[t, c] = silu(gate) * up * weight[t, expert of column c] over one stacked product of all
 // experts: expert e's block of 2 F columns is its gate columns, then its up columns; the shared expert's block
 // follows the experts' (weight = the shared gate, or 1 without one; E = 0: a dense gated feed-forward).  inner's columns [e * F, (e + 1) * F) belong to expert e, those
@@ -89,7 +92,7 @@ moe_route_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ ro
                  float* __restrict__ chosen_w, float* __restrict__ shared_gate, int tokens, int W, int E, int top,
                  int groups, int keep, int by8, const float* __restrict__ raw, int raw_stride,
                  const float* __restrict__ gain, float eps, T* __restrict__ x_out, int score_kind, int normalize,
-                 const float* __restrict__ correction) {
+                 const float* __restrict__ correction, int mark_kind, float weight_scale) {
     pdl_prologue();
     x = pdl_fresh(x);
     raw = pdl_fresh(raw);
@@ -231,9 +234,14 @@ moe_route_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ ro
         const int per = E / groups;
         __shared__ float group_mark[MOE_MAX_EXPERTS];
         for (int g = lane; g < groups; g += 32) {
-            float m = -INFINITY;
-            for (int j = 0; j < per; ++j) m = fmaxf(m, score[g * per + j]);
-            group_mark[g] = m;
+            float m = -INFINITY, second = -INFINITY;
+            for (int j = 0; j < per; ++j) {
+                const int e = g * per + j;
+                const float s = score[e] + (mark_kind == 1 && correction ? correction[e] : 0.f);
+                second = fmaxf(second, fminf(m, s));
+                m = fmaxf(m, s);
+            }
+            group_mark[g] = mark_kind == 1 && per > 1 ? m + second : m;
         }
         __syncwarp();
         for (int drop = 0; drop < groups - keep; ++drop) {
@@ -291,7 +299,7 @@ moe_route_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ ro
         if (best_e >= 0) total += correction ? score[best_e] : best;
     }
     __syncwarp();
-    const float scale = normalize ? 1.0f / (total + 1e-20f) : 1.0f;
+    const float scale = normalize ? weight_scale / (total + 1e-20f) : weight_scale;
     for (int k = lane; k < top; k += 32) {
         const int e = winner[k];
         const float w = winner_score[k] * scale;
@@ -311,7 +319,7 @@ moe_gate_mul_kernel(const T* __restrict__ gate_up, int gu_stride, const float* _
     dense = pdl_fresh(dense);
     shared_gate = pdl_fresh(shared_gate);
     const long long total = (long long)tokens * columns;
-    const int shared_ff = columns - E * F;
+    const int shared_ff = columns - E * F, blocks = form.kind == 3 ? 1 : 2;       // blocks of F columns of an expert
     if (by8) {                                  // eight neighbouring columns (of one expert) per thread and turn
         const int groups = columns >> 3;
         for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < (long long)tokens * groups;
@@ -323,12 +331,17 @@ moe_gate_mul_kernel(const T* __restrict__ gate_up, int gu_stride, const float* _
             float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
             if (w != 0.f) {
                 const int j = c - e * F;
-                const T* block = gate_up + (size_t)t * gu_stride + 2 * (size_t)e * F;
+                const T* block = gate_up + (size_t)t * gu_stride + blocks * (size_t)e * F;
                 float g[8], u[8];
                 load8(block + j, g);
-                load8(block + (e < E ? F : shared_ff) + j, u);
+                if (form.kind == 3) {
 #pragma unroll
-                for (int k = 0; k < 8; ++k) v[k] = gated_inner(g[k], u[k], w, form.kind, limit, form.alpha);
+                    for (int k = 0; k < 8; ++k) v[k] = relu_squared(g[k]) * w;
+                } else {
+                    load8(block + (e < E ? F : shared_ff) + j, u);
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) v[k] = gated_inner(g[k], u[k], w, form.kind, limit, form.alpha);
+                }
             }
             store8(inner + (size_t)t * inner_stride + c, v);
         }
@@ -343,9 +356,10 @@ moe_gate_mul_kernel(const T* __restrict__ gate_up, int gu_stride, const float* _
         if (w != 0.f) {
             // an expert's block of the stacked product is its gate columns, then its up columns
             const int j = c - e * F;
-            const T* block = gate_up + (size_t)t * gu_stride + 2 * (size_t)e * F;
-            v = gated_inner(to_float(block[j]), to_float(block[(e < E ? F : shared_ff) + j]), w, form.kind,
-                            e < E ? form.limit : form.shared_limit, form.alpha);
+            const T* block = gate_up + (size_t)t * gu_stride + blocks * (size_t)e * F;
+            if (form.kind == 3) v = relu_squared(to_float(block[j])) * w;
+            else v = gated_inner(to_float(block[j]), to_float(block[(e < E ? F : shared_ff) + j]), w, form.kind,
+                                 e < E ? form.limit : form.shared_limit, form.alpha);
         }
         inner[(size_t)t * inner_stride + c] = from_float<T>(v);
     }
@@ -469,15 +483,48 @@ moe_gate_mul_rows_kernel(const T* __restrict__ gate_up, int gu_stride, const flo
     }
 }
 
-// y[t] += sum over k (in rising order) of down[row_of[t * top + k]]
+// y[t] += sum over k (in rising order) of down[row_of[t * top + k]]; with weights, factor * sum of weight[t * top + k] *
+// down[...] (factor: one number per column, null: 1)
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ down, int down_stride, const int* __restrict__ row_of, int top,
-                   float* __restrict__ y, int y_stride, int W, int by4) {
+                   const float* __restrict__ weights, const float* __restrict__ factor, float* __restrict__ y, int y_stride,
+                   int W, int by4) {
     pdl_prologue();
     down = pdl_fresh(down);
     row_of = pdl_fresh(row_of);
+    weights = pdl_fresh(weights);
     y = pdl_fresh(y);
     const int t = blockIdx.x;
+    if (weights) {
+        if (by4) {
+            for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
+                float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+                float4 old = *reinterpret_cast<const float4*>(y + (size_t)t * y_stride + c);
+                const float4 f = factor ? *reinterpret_cast<const float4*>(factor + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+                for (int k = 0; k < top; ++k) {
+                    const int r = row_of[t * top + k];
+                    if (r < 0) continue;
+                    const float w = weights[t * top + k];
+                    const float4 d = *reinterpret_cast<const float4*>(down + (size_t)r * down_stride + c);
+                    acc.x = fmaf(w, d.x, acc.x); acc.y = fmaf(w, d.y, acc.y);
+                    acc.z = fmaf(w, d.z, acc.z); acc.w = fmaf(w, d.w, acc.w);
+                }
+                old.x = fmaf(f.x, acc.x, old.x); old.y = fmaf(f.y, acc.y, old.y);
+                old.z = fmaf(f.z, acc.z, old.z); old.w = fmaf(f.w, acc.w, old.w);
+                *reinterpret_cast<float4*>(y + (size_t)t * y_stride + c) = old;
+            }
+            return;
+        }
+        for (int c = threadIdx.x; c < W; c += blockDim.x) {
+            float acc = 0.f;
+            for (int k = 0; k < top; ++k) {
+                const int r = row_of[t * top + k];
+                if (r >= 0) acc = fmaf(weights[t * top + k], down[(size_t)r * down_stride + c], acc);
+            }
+            y[(size_t)t * y_stride + c] = fmaf(factor ? factor[c] : 1.f, acc, y[(size_t)t * y_stride + c]);
+        }
+        return;
+    }
     if (by4) {
         for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
             float4 acc = *reinterpret_cast<const float4*>(y + (size_t)t * y_stride + c);
@@ -507,12 +554,12 @@ moe_combine_kernel(const float* __restrict__ down, int down_stride, const int* _
 // chosen int32 [T, top]; chosen_w float32 [T, top]; shared_gate float32 [T] (written only with shared_gate_w).
 // raw (may be null): float32 [T, W] rows whose RMS norm (gain float32 [W], eps) is what the router reads: the normed
 // rows are then written to x (which the experts' products read) instead of being read from it.  correction (may be
-// null): float32 [E] added to the scores for the election only.
+// null): float32 [E] added to the scores for the election only.  mark_kind: see the top of the file.
 PS_EXPORT int ps_moe_route(const void* x, int x_stride, const void* router, int router_stride,
                            const void* shared_gate_w, float* dense, int* chosen, float* chosen_w, float* shared_gate,
                            int T, int W, int E, int top, int groups, int keep, int dtype, const float* raw,
                            int raw_stride, const float* gain, float eps, int score_kind, int normalize,
-                           const float* correction, void* stream) {
+                           const float* correction, int mark_kind, float weight_scale, void* stream) {
     if (T <= 0) return PS_OK;
     if (raw && !gain) return PS_ERR_BAD_ARGUMENT;
     if (W <= 0 || E <= 0 || top <= 0 || top > E || !x || !router || !dense || !chosen || !chosen_w)
@@ -531,24 +578,24 @@ PS_EXPORT int ps_moe_route(const void* x, int x_stride, const void* router, int 
         return ps::launch_pdl(ps::moe_route_kernel<float>, grid, block, 0, s, (const float*)x, x_stride,
                               (const float*)router, router_stride, (const float*)shared_gate_w, dense, chosen,
                               chosen_w, shared_gate, T, W, E, top, groups, keep, by8, raw, raw_stride, gain, eps,
-                              (float*)const_cast<void*>(x), score_kind, normalize, correction);
+                              (float*)const_cast<void*>(x), score_kind, normalize, correction, mark_kind, weight_scale);
     if (dtype == PS_BF16)
         return ps::launch_pdl(ps::moe_route_kernel<__nv_bfloat16>, grid, block, 0, s, (const __nv_bfloat16*)x,
                               x_stride, (const __nv_bfloat16*)router, router_stride,
                               (const __nv_bfloat16*)shared_gate_w, dense, chosen, chosen_w, shared_gate, T, W, E, top,
                               groups, keep, by8, raw, raw_stride, gain, eps, (__nv_bfloat16*)const_cast<void*>(x),
-                              score_kind, normalize, correction);
+                              score_kind, normalize, correction, mark_kind, weight_scale);
     return PS_ERR_UNSUPPORTED;
 }
 
-// gate_up [T, 2 * columns] (per expert: gates, then ups); dense float32 [T, E]; shared_gate float32 [T] (read for
+// gate_up [T, 2 * columns] (per expert: gates, then ups; kind 3: [T, columns]); dense float32 [T, E]; shared_gate float32 [T] (read for
 // columns from E * F on); inner [T, columns].
 PS_EXPORT int ps_moe_gate_mul(const void* gate_up, int gu_stride, const float* dense, const float* shared_gate,
                               void* inner, int inner_stride, int T, int columns, int E, int F, int dtype,
                               int kind, float limit, float shared_limit, float alpha, void* stream) {
     if (T <= 0 || columns <= 0) return PS_OK;
     if (!gate_up || !inner || E < 0 || (E > 0 && !dense) || F <= 0 || columns < E * F) return PS_ERR_BAD_ARGUMENT;
-    if (kind < 0 || kind > 2 || (kind == 1 && !(limit > 0.f && shared_limit > 0.f))) return PS_ERR_BAD_ARGUMENT;
+    if (kind < 0 || kind > 3 || (kind == 1 && !(limit > 0.f && shared_limit > 0.f)) || (kind == 3 && columns != E * F)) return PS_ERR_BAD_ARGUMENT;
     const ps::GateForm form{kind, limit, shared_limit, alpha};
     cudaStream_t s = (cudaStream_t)stream;
     const int by8 = F % 8 == 0 && columns % 8 == 0 && gu_stride % 8 == 0 && inner_stride % 8 == 0 &&
@@ -619,13 +666,14 @@ PS_EXPORT int ps_moe_gate_mul_rows(const void* gate_up, int gu_stride, const flo
     return PS_ERR_UNSUPPORTED;
 }
 
-// down float32 [R, W]; row_of int32 [T * top]; y float32 [T, W]
-PS_EXPORT int ps_moe_combine(const float* down, int down_stride, const int* row_of, int top, float* y, int y_stride,
-                             int T, int W, void* stream) {
+// down float32 [R, W]; row_of int32 [T * top]; y float32 [T, W]; weights (may be null) float32 [T * top]; factor (null
+// without weights; may be null) float32 [W]
+PS_EXPORT int ps_moe_combine(const float* down, int down_stride, const int* row_of, int top, const float* weights,
+                             const float* factor, float* y, int y_stride, int T, int W, void* stream) {
     if (T <= 0 || W <= 0) return PS_OK;
-    if (!down || !row_of || !y || top <= 0) return PS_ERR_BAD_ARGUMENT;
+    if (!down || !row_of || !y || top <= 0 || (factor && !weights)) return PS_ERR_BAD_ARGUMENT;
     const int by4 = W % 4 == 0 && down_stride % 4 == 0 && y_stride % 4 == 0 && !((uintptr_t)down & 15) &&
-                    !((uintptr_t)y & 15);
+                    !((uintptr_t)y & 15) && !((uintptr_t)factor & 15);
     return ps::launch_pdl(ps::moe_combine_kernel, dim3(T), dim3(W >= 1024 ? 256 : 128), 0, (cudaStream_t)stream, down,
-                          down_stride, row_of, top, y, y_stride, W, by4);
+                          down_stride, row_of, top, weights, factor, y, y_stride, W, by4);
 }

@@ -11,6 +11,9 @@
 // `head_slot` numbers of which the first `head_values` count.  mode 1: the convolved values are also stored, float32,
 // in `shared_values` [T, mix_heads * head_values]; mode 2: y <- (1 - m) y + m * shared_values[t], m = *mix.
 //
+// bias and act (optional): y <- act(y + bias[c]) before the result is rounded (act: one of the activation codes); kept rows
+// are the projection's own.  u may be rows of the compute type too.
+//
 // row_scale (may be null): one float per token that multiplies its row of u wherever it is read (a row to be divided by
 // its root mean square, say, whose factor an earlier kernel has formed); kept rows are stored already multiplied.
 //
@@ -23,13 +26,14 @@ namespace ps {
 
 constexpr int SHORT_CONV_MAX_TAPS = 16;
 
-template <typename TC>
+template <typename TI, typename TC>
 __global__ void __launch_bounds__(256)
-short_conv_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ weight, int taps,
+short_conv_kernel(const TI* __restrict__ u, long long u_stride, const float* __restrict__ weight, int taps,
                   int conv_channels, int channels, const float* __restrict__ row_scale, float* kept, long long kept_stride,
                   const int* __restrict__ token_item, const int* __restrict__ q_start, const int* __restrict__ item_slot,
                   TC* __restrict__ out, long long out_stride, int mode, int mix_lo, int mix_heads, int head_slot,
-                  int head_values, float* __restrict__ shared_values, const float* __restrict__ mix, int tokens) {
+                  int head_values, float* __restrict__ shared_values, const float* __restrict__ mix,
+                  const float* __restrict__ bias, int act, int tokens) {
     pdl_prologue();
     u = pdl_fresh(u);
     row_scale = pdl_fresh(row_scale);
@@ -40,14 +44,14 @@ short_conv_kernel(const float* __restrict__ u, long long u_stride, const float* 
          i += (long long)gridDim.x * blockDim.x) {
         const int t = (int)(i / channels), c = (int)(i - (long long)t * channels);
         if (c >= conv_channels) {
-            out[(size_t)t * out_stride + c] = from_float<TC>(u[(size_t)t * u_stride + c] * (row_scale ? row_scale[t] : 1.f));
+            out[(size_t)t * out_stride + c] = from_float<TC>(to_float(u[(size_t)t * u_stride + c]) * (row_scale ? row_scale[t] : 1.f));
             continue;
         }
         const int item = token_item[t];
         const int first = q_start[item], end = q_start[item + 1];
         if (t != first && t - first < taps - 1) continue;             // (the thread of the first token does these)
         float* old = kept + (size_t)item_slot[item] * kept_stride;
-        auto row = [&](int source) { return u[(size_t)source * u_stride + c] * (row_scale ? row_scale[source] : 1.f); };
+        auto row = [&](int source) { return to_float(u[(size_t)source * u_stride + c]) * (row_scale ? row_scale[source] : 1.f); };
         const int last = t == first ? min(first + max(taps - 1, 1), end) : t + 1;
         for (int now = t; now < last; ++now) {
             float y = 0.f;
@@ -58,6 +62,8 @@ short_conv_kernel(const float* __restrict__ u, long long u_stride, const float* 
                                                 : old[(size_t)(taps - 1 - (first - source)) * conv_channels + c];
                 y = fmaf(weight[(size_t)c * taps + j], v, y);
             }
+            if (bias) y += bias[c];
+            y = apply_act(y, act);
             if (mode) {
                 const int local = c - mix_lo;
                 if (local >= 0 && local < mix_heads * head_slot) {
@@ -100,16 +106,25 @@ template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16*
     *reinterpret_cast<uint2*>(p) = packed;
 }
 
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
 constexpr int SHORT_CONV_THREADS = 128;
 
-template <typename TC, int TAPS, bool SCALED>
+// FORM: 0 plain, 1 rows multiplied by row_scale, 2 a bias and silu
+template <typename TI, typename TC, int TAPS, int FORM>
 __global__ void __launch_bounds__(SHORT_CONV_THREADS)
-short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const float* __restrict__ weight,
+short_conv_runs_kernel(const TI* __restrict__ u, long long u_stride, const float* __restrict__ weight,
                        int conv_channels, int channels, const float* __restrict__ row_scale, float* kept,
                        long long kept_stride, const int* __restrict__ token_item, const int* __restrict__ q_start,
                        const int* __restrict__ item_slot, TC* __restrict__ out, long long out_stride, int mode, int mix_lo,
                        int mix_heads, int head_slot, int head_values, float* __restrict__ shared_values,
-                       const float* __restrict__ mix, int tokens, int run) {
+                       const float* __restrict__ mix, const float* __restrict__ bias, int tokens, int run) {
     const int c = 4 * (blockIdx.x * SHORT_CONV_THREADS + threadIdx.x);
     const int t0 = blockIdx.y * run, t1 = min(t0 + run, tokens);
     const bool convolved = c < conv_channels;
@@ -128,6 +143,10 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) w[i][j] = flat[i * TAPS + j];
     }
+    float4 shift = make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (FORM == 2) {
+        if (convolved && c < channels) shift = *reinterpret_cast<const float4*>(bias + c);
+    }
     const float blend = mode == 2 ? *mix : 0.f;
     // which entry the run lies in is static for the step too
     const int item0 = convolved ? token_item[t0] : 0, item1 = convolved ? token_item[t1 - 1] : 0;
@@ -137,8 +156,8 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
     row_scale = pdl_fresh(row_scale);
     shared_values = pdl_fresh(shared_values);
     auto scaled = [&](int t) {
-        float4 v = *reinterpret_cast<const float4*>(u + (size_t)t * u_stride + c);
-        if constexpr (SCALED) {
+        float4 v = load4(u + (size_t)t * u_stride + c);
+        if constexpr (FORM == 1) {
             const float f = row_scale[t];
             v.x *= f; v.y *= f; v.z *= f; v.w *= f;
         }
@@ -187,6 +206,10 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
 #pragma unroll
         for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
         if (TAPS > 1) held[0] = now;
+        if constexpr (FORM == 2) {
+            y[0] = silu(y[0] + shift.x); y[1] = silu(y[1] + shift.y);
+            y[2] = silu(y[2] + shift.z); y[3] = silu(y[3] + shift.w);
+        }
         if (common >= 0) {
             float* place = shared_values + (size_t)t * mix_heads * head_values + common;
             if (mode == 1) {
@@ -252,14 +275,15 @@ short_conv_runs_kernel(const float* __restrict__ u, long long u_stride, const fl
 
 }  // namespace ps
 
-// u float32 [T, channels] rows (u_stride apart); row_scale float32 [T] or null; weight float32 [conv_channels, taps]; kept float32
-// [slots, (taps - 1) * conv_channels] rows (kept_stride apart; may be null when taps = 1); out [T, channels] rows of
-// `dtype`.  mode 0: no blending; 1: store the convolved values; 2: blend with the stored ones by *mix.
-PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* weight, int taps, int conv_channels,
+// u [T, channels] rows (u_stride apart), float32 or (u_dtype) of `dtype`; row_scale float32 [T] or null; weight float32
+// [conv_channels, taps]; kept float32 [slots, (taps - 1) * conv_channels] rows (kept_stride apart; may be null when taps = 1);
+// out [T, channels] rows of `dtype`.  mode 0: no blending; 1: store the convolved values; 2: blend with the stored ones by
+// *mix.  bias float32 [conv_channels] or null, act an activation code: behind the convolution.
+PS_EXPORT int ps_short_conv(const void* u, int u_dtype, long long u_stride, const float* weight, int taps, int conv_channels,
                             int channels, const float* row_scale, float* kept, long long kept_stride, const int* token_item,
                             const int* q_start, const int* item_slot, void* out, long long out_stride, int mode,
                             int mix_lo, int mix_heads, int head_slot, int head_values, float* shared_values,
-                            const float* mix, int T, int dtype, void* stream) {
+                            const float* mix, const float* bias, int act, int T, int dtype, void* stream) {
     if (T <= 0 || channels <= 0) return PS_OK;
     if (!u || !out || conv_channels < 0 || conv_channels > channels || taps < 1) return PS_ERR_BAD_ARGUMENT;
     if (conv_channels && (!weight || !token_item || !q_start || !item_slot || (taps > 1 && !kept)))
@@ -267,50 +291,63 @@ PS_EXPORT int ps_short_conv(const float* u, long long u_stride, const float* wei
     if (mode < 0 || mode > 2 || (mode && (!shared_values || head_slot <= 0 || head_values <= 0 || head_values > head_slot)))
         return PS_ERR_BAD_ARGUMENT;
     if (mode == 2 && !mix) return PS_ERR_BAD_ARGUMENT;
+    if ((dtype != PS_F32 && dtype != PS_BF16) || (u_dtype != PS_F32 && u_dtype != dtype)) return PS_ERR_UNSUPPORTED;
     if (taps > ps::SHORT_CONV_MAX_TAPS) return PS_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
+    using bf = __nv_bfloat16;
     // quads of channels over runs of tokens, where every boundary between kinds of channels falls between quads
-    const int elem = dtype == PS_F32 ? 4 : 2;
+    const int elem = dtype == PS_F32 ? 4 : 2, in_elem = u_dtype == PS_F32 ? 4 : 2;
+    const int form = row_scale ? 1 : (bias && act == PS_ACT_SILU) ? 2 : 0;
+    const bool plain = bias == nullptr && act == PS_ACT_NONE;
     const bool quads = taps <= 4 && conv_channels > 0 && channels % 4 == 0 && conv_channels % 4 == 0 && u_stride % 4 == 0 &&
-                       out_stride % 4 == 0 && kept_stride % 4 == 0 && !((uintptr_t)u & 15) && !((uintptr_t)kept & 15) && !((uintptr_t)weight & 15) &&
-                       !((uintptr_t)out & (uintptr_t)(4 * elem - 1)) &&
+                       out_stride % 4 == 0 && kept_stride % 4 == 0 && !((uintptr_t)u & (uintptr_t)(4 * in_elem - 1)) &&
+                       !((uintptr_t)kept & 15) && !((uintptr_t)weight & 15) && !((uintptr_t)bias & 15) &&
+                       !((uintptr_t)out & (uintptr_t)(4 * elem - 1)) && (plain || form == 2) &&
+                       (u_dtype == PS_F32 || form == 2) &&
                        (!mode || (mix_lo % 4 == 0 && head_slot % 4 == 0 && head_values % 4 == 0 &&
                                   !((uintptr_t)shared_values & 15)));
-    if (quads && (dtype == PS_F32 || dtype == PS_BF16)) {
+    if (quads) {
         // runs of 16 tokens re-read (taps - 1) / 16 of the rows; shorter runs where the step has too few for the SMs
         const int columns = (channels / 4 + ps::SHORT_CONV_THREADS - 1) / ps::SHORT_CONV_THREADS;
         int run = 16;
         while (run > 1 && (long long)columns * ((T + run - 1) / run) < 1200) run >>= 1;
         const dim3 grid(columns, (T + run - 1) / run), block(ps::SHORT_CONV_THREADS);
-#define PS_CONV_RUNS(TYPE, TAPS)                                                                                      \
-    return ps::launch_pdl(row_scale ? ps::short_conv_runs_kernel<TYPE, TAPS, true>                                     \
-                                    : ps::short_conv_runs_kernel<TYPE, TAPS, false>,                                    \
-                          grid, block, 0, s, u, u_stride, weight, conv_channels, channels, row_scale, kept, kept_stride, \
-                          token_item, q_start, item_slot, (TYPE*)out, out_stride, mode, mix_lo, mix_heads, head_slot,   \
-                          head_values, shared_values, mix, T, run)
-#define PS_CONV_TAPS(TYPE)                                                                                            \
+#define PS_CONV_RUNS(TI, TC, TAPS, FORM)                                                                              \
+    return ps::launch_pdl(ps::short_conv_runs_kernel<TI, TC, TAPS, FORM>, grid, block, 0, s, (const TI*)u, u_stride,    \
+                          weight, conv_channels, channels, row_scale, kept, kept_stride, token_item, q_start, item_slot, \
+                          (TC*)out, out_stride, mode, mix_lo, mix_heads, head_slot, head_values, shared_values, mix,     \
+                          bias, T, run)
+#define PS_CONV_TAPS(TI, TC, FORM)                                                                                    \
     switch (taps) {                                                                                                   \
-        case 1: PS_CONV_RUNS(TYPE, 1);                                                                                \
-        case 2: PS_CONV_RUNS(TYPE, 2);                                                                                \
-        case 3: PS_CONV_RUNS(TYPE, 3);                                                                                \
-        default: PS_CONV_RUNS(TYPE, 4);                                                                               \
+        case 1: PS_CONV_RUNS(TI, TC, 1, FORM);                                                                        \
+        case 2: PS_CONV_RUNS(TI, TC, 2, FORM);                                                                        \
+        case 3: PS_CONV_RUNS(TI, TC, 3, FORM);                                                                        \
+        default: PS_CONV_RUNS(TI, TC, 4, FORM);                                                                       \
     }
-        if (dtype == PS_F32) PS_CONV_TAPS(float)
-        PS_CONV_TAPS(__nv_bfloat16)
+        if (form == 2) {
+            if (dtype == PS_F32) PS_CONV_TAPS(float, float, 2)
+            if (u_dtype == PS_F32) PS_CONV_TAPS(float, bf, 2)
+            PS_CONV_TAPS(bf, bf, 2)
+        }
+        if (dtype == PS_F32) {
+            if (form == 1) PS_CONV_TAPS(float, float, 1)
+            PS_CONV_TAPS(float, float, 0)
+        }
+        if (form == 1) PS_CONV_TAPS(float, bf, 1)
+        PS_CONV_TAPS(float, bf, 0)
 #undef PS_CONV_TAPS
 #undef PS_CONV_RUNS
     }
     const long long total = (long long)T * channels;
     const long long blocks = (total + 255) / 256;
     const dim3 grid((unsigned)(blocks < 4736 ? blocks : 4736));
-    if (dtype == PS_F32)
-        return ps::launch_pdl(ps::short_conv_kernel<float>, grid, dim3(256), 0, s, u, u_stride, weight, taps,
-                              conv_channels, channels, row_scale, kept, kept_stride, token_item, q_start, item_slot, (float*)out,
-                              out_stride, mode, mix_lo, mix_heads, head_slot, head_values, shared_values, mix, T);
-    if (dtype == PS_BF16)
-        return ps::launch_pdl(ps::short_conv_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, u, u_stride, weight, taps,
-                              conv_channels, channels, row_scale, kept, kept_stride, token_item, q_start, item_slot,
-                              (__nv_bfloat16*)out, out_stride, mode, mix_lo, mix_heads, head_slot, head_values,
-                              shared_values, mix, T);
-    return PS_ERR_UNSUPPORTED;
+#define PS_CONV(TI, TC)                                                                                               \
+    return ps::launch_pdl(ps::short_conv_kernel<TI, TC>, grid, dim3(256), 0, s, (const TI*)u, u_stride, weight, taps,   \
+                          conv_channels, channels, row_scale, kept, kept_stride, token_item, q_start, item_slot,        \
+                          (TC*)out, out_stride, mode, mix_lo, mix_heads, head_slot, head_values, shared_values, mix,     \
+                          bias, act, T)
+    if (dtype == PS_F32) PS_CONV(float, float);
+    if (u_dtype == PS_F32) PS_CONV(float, bf);
+    PS_CONV(bf, bf);
+#undef PS_CONV
 }

@@ -34,7 +34,7 @@ NVCC_FLAGS = [
 LIBRARIES: Dict[str, List[str]] = {
     "core": ["embed_norm.cu", "gemm_simt.cu", "attention_simt.cu", "sampling.cu", "host_io.cu", "step_state.cu", "step_build.cu",
              "rotary.cu", "wkv.cu", "embed_pair.cu", "hyper.cu", "latent.cu", "moe.cu", "post_norm.cu", "mingru.cu",
-             "short_conv.cu", "gla.cu", "head_mix.cu"],
+             "short_conv.cu", "gla.cu", "head_mix.cu", "ssd.cu", "diff_attention.cu"],
     "bf16": ["gemm_skinny.cu", "attention_decode.cu", "attention_prefill.cu", "attention_rows.cu"],
     "tc": ["gemm_tc.cu", "gemm_rows_tc.cu", "attention_prefill_tc.cu"],
 }

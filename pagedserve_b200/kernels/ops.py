@@ -18,6 +18,7 @@ from pagedserve_b200.kernels.build import load as _load_library
 
 PS_F32, PS_BF16 = 0, 1
 _DTYPE_CODE = {torch.float32: PS_F32, torch.bfloat16: PS_BF16}
+COLUMN_FACTOR = 2             # in a product's ``accumulate``: its vector multiplies the columns instead of being added
 _ACT_CODE = {None: 0, "none": 0, "gelu_tanh": 1, "gelu_erf": 2, "relu_squared": 3, "silu": 4, "tanh": 5}
 _STATUS = {1: "bad argument", 2: "unsupported size or dtype", 3: "kernel launch failed"}
 
@@ -72,6 +73,8 @@ _P, _I, _F, _L = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlon
 _SIGNATURES = {
     "core": {
         "ps_embed": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
+        "ps_embed_sinusoid": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+        "ps_rms_norm_pair": [_P, _I, _I, _P, _P, _F, _P, _P, _I, _P],
         "ps_layernorm": [_P, _P, _I, _I, _P, _P, _F, _I, _P, _I, _P],
         "ps_gemm_simt": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "ps_kv_append": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I, _P],
@@ -91,7 +94,7 @@ _SIGNATURES = {
         "ps_latent_prepare": [_P, _I, _P, _I, _P, _F, _P, _I, _P, _P, _P, _I, _P, _L, _I, _P, _I, _I, _I, _I, _I, _I,
                               _I, _P],
         "ps_sigmoid_gate": [_P, _I, _P, _I, _I, _I, _I, _I, _P],
-        "ps_moe_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _F, _I, _I, _P, _P],
+        "ps_moe_route": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P, _F, _I, _I, _P, _I, _F, _P],
         "ps_moe_gate_mul": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _P],
         "ps_head_norm_rotary_cache_write": [_P, _I, _P, _I, _P, _I, _P, _P, _F, _P, _I, _I, _P, _P, _P, _I, _P, _P, _L,
                                             _I, _I, _I, _I, _I, _I, _I, _F, _P],
@@ -99,16 +102,21 @@ _SIGNATURES = {
         "ps_post_norm_add": [_P, _P, _I, _I, _I, _P, _F, _P, _I, _P, _L, _I, _P, _P],
         "ps_depth_begin": [_P, _P, _P, _I, _P, _L, _P],
         "ps_mingru_scan": [_P, _L, _I, _P, _L, _P, _P, _I, _P, _L, _I, _I, _P],
-        "ps_short_conv": [_P, _L, _P, _I, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P],
+        "ps_short_conv": [_P, _I, _L, _P, _I, _I, _I, _P, _P, _L, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P],
         "ps_sandwich_close": [_P, _P, _I, _I, _P, _F, _F, _P, _P, _I, _P, _P],
         "ps_sandwich_close_conv": [_P, _P, _I, _I, _P, _F, _F, _P, _I, _P, _L, _P, _P, _I, _P],
         "ps_gla_recurrence": [_P, _L, _P, _P, _P, _I, _F, _F, _P, _F, _F, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P,
                               _L, _I, _I, _I, _I, _P],
+        "ps_ssd": [_P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I,
+                   _P],
+        "ps_diff_prepare": [_P, _L, _I, _I, _P, _P, _F, _F, _I, _P, _P, _P, _I, _P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _I,
+                            _I, _I, _I, _P],
+        "ps_diff_combine": [_P, _L, _P, _L, _P, _L, _F, _F, _F, _I, _I, _I, _I, _I, _P],
         "ps_head_mix": [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P],
         "ps_moe_plan": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P],
         "ps_moe_gather": [_P, _I, _P, _P, _I, _I, _I, _I, _P],
         "ps_moe_gate_mul_rows": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
-        "ps_moe_combine": [_P, _I, _P, _I, _P, _I, _I, _I, _P],
+        "ps_moe_combine": [_P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P],
         "ps_step_shape": [_I, _P, _P, _P, _I, _I, _I, _I, _P],
         "ps_step_fill": [_I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _L, _P, _I, _I, _I, _I, _P],
         "ps_step_begin": [_P, _P, _P, _P, _P, _P],
@@ -283,7 +291,39 @@ class Ops:
                                   _ptr(status), _stream()), "embed")
         return out
 
+    def embed_sinusoid(self, ids, positions, wte, freq, out, status=None):
+        """out[t] = wte[ids[t]] + sines and cosines of the position, float32 [T, H]: number 2i gets sin(p * f_i), number
+        2i + 1 cos(p * f_i); ``freq`` float32 [ceil(H / 2), 2]: the f_i as (high, low) parts."""
+        T, H = out.shape
+        _require(out, "out", torch.float32)
+        _require(ids, "ids", torch.int32)
+        _require(positions, "positions", torch.int32)
+        _require(wte, "wte", self.dtype)
+        _require(freq, "freq", torch.float32)
+        if wte.shape[1] != H or ids.numel() != T or freq.shape != ((H + 1) // 2, 2) or not freq.is_contiguous():
+            raise KernelError("embed_sinusoid: shapes do not match")
+        self.launches += 1
+        _check(self.core.ps_embed_sinusoid(_ptr(ids), _ptr(positions), _ptr(wte), _ptr(freq), _ptr(out), T, H, wte.shape[0],
+                                           self.code, _ptr(status), _stream()), "embed_sinusoid")
+        return out
+
     # ------------------------------------------------------------------ norm
+    def rms_norm_pair(self, x, gain_a, gain_b, eps, out_a, out_b):
+        """out_a = rms_norm(x) * gain_a and out_b = rms_norm(x) * gain_b of the same float32 rows [T, H]."""
+        _require(x, "x", torch.float32)
+        T, H = x.shape
+        for name, gain in (("gain_a", gain_a), ("gain_b", gain_b)):
+            _require(gain, name, torch.float32)
+            if gain.numel() != H or not gain.is_contiguous():
+                raise KernelError("rms_norm_pair: one gain per number of the row")
+        if (out_a.shape != x.shape or out_b.shape != x.shape or out_a.dtype != out_b.dtype or not x.is_contiguous()
+                or not (out_a.is_contiguous() and out_b.is_contiguous())):
+            raise KernelError("rms_norm_pair: shapes do not match")
+        self.launches += 1
+        _check(self.core.ps_rms_norm_pair(_ptr(x), T, H, _ptr(gain_a), _ptr(gain_b), float(eps), _ptr(out_a), _ptr(out_b),
+                                          dtype_code(out_a.dtype), _stream()), "rms_norm_pair")
+        return out_a, out_b
+
     def layernorm(self, x, gamma, beta, eps, out, rows=None, has_mean=True):
         """out[r] = norm(x[rows[r]] or x[r]); x float32 [*, H]; out compute dtype or float32."""
         _require(x, "x", torch.float32)
@@ -322,13 +362,13 @@ class Ops:
                 raise KernelError("linear: bias length")
         if a.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1:
             raise KernelError("linear: innermost stride must be 1")
-        if accumulate and out.dtype != torch.float32:
+        if int(accumulate) & 1 and out.dtype != torch.float32:
             raise KernelError("linear: accumulate needs a float32 output")
         self.launches += 1
         _check(self.core.ps_gemm_simt(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(bias),
                                       _ptr(out), out.stride(0), M, N, K,
                                       dtype_code(a.dtype), dtype_code(out.dtype),
-                                      _ACT_CODE[act], 1 if accumulate else 0, _stream()),
+                                      _ACT_CODE[act], int(accumulate), _stream()),
                "gemm_simt")
         return out
 
@@ -351,7 +391,7 @@ class Ops:
         _check(self.fast.ps_gemm_skinny(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(bias),
                                         _ptr(out), out.stride(0), M, N, K,
                                         dtype_code(out.dtype), _ACT_CODE[act],
-                                        1 if accumulate else 0, *self._kv_arguments(kv, N), _stream()), "gemm_skinny")
+                                        int(accumulate), *self._kv_arguments(kv, N), _stream()), "gemm_skinny")
         return out
 
     GROUPED_ROWS = 32             # most rows for which equal products run as one grouped launch
@@ -434,7 +474,7 @@ class Ops:
         _check(self._tc.ps_gemm_tc(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(bias), _ptr(out),
                                    out.stride(0), M, N, K,
                                    dtype_code(out.dtype), _ACT_CODE[act],
-                                   1 if accumulate else 0, _ptr(status), bn, _stream()), "gemm_tc")
+                                   int(accumulate), _ptr(status), bn, _stream()), "gemm_tc")
         return out
 
     def linear_rows_tc(self, a, w, bias, out, act=None, accumulate=False, kv=None, status=None, splits=0):
@@ -459,7 +499,7 @@ class Ops:
         self.launches += 1
         _check(self._tc.ps_gemm_rows_tc(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(bias), _ptr(out),
                                         out.stride(0), M, N, K, dtype_code(out.dtype), _ACT_CODE[act],
-                                        1 if accumulate else 0, _ptr(status), splits,
+                                        int(accumulate), _ptr(status), splits,
                                         *self._kv_arguments(kv, N), _stream()), "gemm_rows_tc")
         return out
 
@@ -537,7 +577,7 @@ class Ops:
             _ptr(a.x), a.x.stride(0), _ptr(a.rows), _ptr(norm.weight), _ptr(norm.bias),
             float(norm.eps), 1 if norm.has_mean else 0,
             _ptr(w), w.stride(0), _ptr(bias), _ptr(out), out.stride(0), M, N,
-            K, dtype_code(out.dtype), _ACT_CODE[act], 1 if accumulate else 0,
+            K, dtype_code(out.dtype), _ACT_CODE[act], int(accumulate),
             *kv_args, _stream()), "gemm_skinny_fused")
         return out
 
@@ -587,9 +627,15 @@ class Ops:
             q_width, kv_width, head_dim, layer.page_size, _stream()), "gemm_tc_qkv")
         return out
 
-    def linear(self, a, w, bias, out, act=None, accumulate=False):
+    def linear(self, a, w, bias, out, act=None, accumulate=False, factor=None):
         """The matrix product of the model: float32 runs on FFMA, bfloat16 on tensor cores.
-        ``a`` may be a DeferredNorm: it is folded into the product where a kernel can, else evaluated."""
+        ``a`` may be a DeferredNorm: it is folded into the product where a kernel can, else evaluated.
+        ``factor`` (float32, one number per column, instead of a bias) multiplies the product before it is stored or
+        added: the product kernels take it as their vector of one number per column."""
+        if factor is not None:
+            if bias is not None or act is not None:
+                raise KernelError("linear: a factor per column goes with neither a bias nor an activation")
+            bias, accumulate = factor, int(accumulate) | COLUMN_FACTOR
         if hasattr(a, "materialize"):
             if self._fused_norm_ok(a, w):
                 return self.linear_skinny_fused(a, w, bias, out, act, accumulate)
@@ -1330,6 +1376,110 @@ class Ops:
                                            out.stride(0), heads, dk, dv, self.code, _stream()), "gla_recurrence")
         return out
 
+    # ------------------------------------------------------------------ state space
+    SSD_RUN = 64                  # no run of a prompt portion is shorter than this
+    SSD_SCRATCH_BYTES = 256 << 20
+
+    def ssd_segments(self, ctx, heads, N, P):
+        """Runs that a prompt portion is cut into: about as many CTAs as the device holds at once."""
+        long_items = ctx.num_items - ctx.num_short_items
+        longest = int(ctx.max_q_len)
+        if long_items <= 0 or longest < 2 * self.SSD_RUN:
+            return 1
+        tiles = -(-P // 32)
+        wanted = min(148 * 3 // (long_items * heads * tiles), longest // self.SSD_RUN,
+                     self.SSD_SCRATCH_BYTES // (4 * long_items * heads * N * P))
+        return max(1, min(64, wanted))
+
+    def ssd(self, conv, raw, offsets, a_log, dt_bias, d, state, ctx, out, heads, groups, N, P, segments=None):
+        """The state-space recurrence of every entry of the step, tokens in order, from and into the slots' state, with the
+        skip and the gate behind it (csrc/ssd.cu).  ``conv`` / ``raw`` [T, *] (compute dtype): convolved and projected rows in
+        which x [heads * P], B and C [groups * N] (``conv``), z [heads * P] and dt [heads] (``raw``) begin at the five
+        ``offsets``; ``a_log``, ``dt_bias``, ``d`` float32 [heads]; ``state`` float32 [slots, >= heads * N * P]; ``out``
+        [T, heads * P] in the compute dtype or float32."""
+        _require(conv, "conv", self.dtype)
+        _require(raw, "raw", self.dtype)
+        for name, tensor in (("a_log", a_log), ("dt_bias", dt_bias), ("d", d), ("state", state)):
+            _require(tensor, name, torch.float32)
+        _require(out, "out", out.dtype if out.dtype in (self.dtype, torch.float32) else self.dtype)
+        T = conv.shape[0]
+        ends = [offsets[0] + heads * P, offsets[1] + groups * N, offsets[2] + groups * N]
+        if (min(offsets) < 0 or max(ends) > conv.shape[1] or max(offsets[3] + heads * P, offsets[4] + heads) > raw.shape[1]
+                or raw.shape[0] != T or conv.stride(1) != 1 or raw.stride(1) != 1 or heads % groups
+                or any(t.numel() != heads or not t.is_contiguous() for t in (a_log, dt_bias, d))
+                or state.shape[1] < heads * N * P or state.stride(1) != 1 or out.shape != (T, heads * P)
+                or out.stride(1) != 1):
+            raise KernelError("ssd: shapes do not match")
+        single = bool(getattr(ctx, "single_tokens", False))
+        if segments is None:
+            segments = 1 if single else self.ssd_segments(ctx, heads, N, P)
+        first_cut = ctx.num_short_items
+        if single or first_cut >= ctx.num_items:
+            segments = 1
+        run_state = run_decay = None
+        if segments > 1:
+            runs = (ctx.num_items - first_cut) * heads * segments
+            run_state = self.empty((runs, N * P), torch.float32, conv.device)
+            run_decay = self.empty((runs,), torch.float32, conv.device)
+        places = (ctypes.c_int * 5)(*[int(o) for o in offsets])
+        self.launches += 3 if segments > 1 else 1
+        _check(self.core.ps_ssd(_ptr(conv), conv.stride(0), _ptr(raw), raw.stride(0), ctypes.addressof(places), _ptr(a_log),
+                                _ptr(dt_bias), _ptr(d), _ptr(state), state.stride(0), _ptr(ctx.q_start), _ptr(ctx.item_slot),
+                                ctx.num_items, T, 1 if single else 0, first_cut, segments, _ptr(run_state), _ptr(run_decay),
+                                _ptr(out), out.stride(0), heads, groups, N, P, self.code, dtype_code(out.dtype), _stream()),
+               "ssd")
+        return out
+
+    # ------------------------------------------------------------------ differential attention
+    def diff_prepare(self, row, k_offset, v_offset, q_gain, k_gain, eps, q_temp, ctx, layer, q_out, n_heads, n_kv_heads, dim,
+                     vdim, slot, has_kv=True):
+        """Queries and pages of attention with two maps per head (csrc/diff_attention.cu).  ``row`` [T, *] (compute dtype):
+        q [n_heads, 2, dim], then (``has_kv``) k [n_kv_heads, 2, dim] at ``k_offset`` and v [n_kv_heads, vdim] at
+        ``v_offset``; ``q_out`` [T, 2 * n_heads * slot]; gains float32 [dim]; ``q_temp`` (coef, every) or None."""
+        _require(row, "row", self.dtype)
+        _require(q_out, "q_out", self.dtype)
+        T = row.shape[0]
+        for name, gain in (("q_gain", q_gain), ("k_gain", k_gain)):
+            if gain is not None:
+                _require(gain, name, torch.float32)
+                if gain.numel() != dim or not gain.is_contiguous():
+                    raise KernelError("diff_prepare: one gain per number of a map's head")
+        width = max(v_offset + n_kv_heads * vdim, k_offset + 2 * n_kv_heads * dim) if has_kv else 0
+        if (row.stride(1) != 1 or row.shape[1] < max(width, 2 * n_heads * dim) or q_out.shape != (T, 2 * n_heads * slot)
+                or q_out.stride(1) != 1 or slot < max(2 * dim, vdim) or (has_kv and k_gain is None)):
+            raise KernelError("diff_prepare: shapes do not match")
+        if has_kv:
+            _require(layer.k_pool, "k_pool", self.dtype)
+        coef, every = q_temp if q_temp is not None else (0.0, 0)
+        self.launches += 1
+        _check(self.core.ps_diff_prepare(
+            _ptr(row), row.stride(0), k_offset, v_offset, _ptr(q_gain), _ptr(k_gain), float(eps), float(coef), int(every),
+            _ptr(ctx.token_slot) if has_kv else None, _ptr(ctx.positions), _ptr(layer.block_table) if has_kv else None,
+            layer.block_table.stride(0) if has_kv else 0, _ptr(layer.k_pool) if has_kv else None,
+            _ptr(layer.v_pool) if has_kv else None, layer.page_stride if has_kv else 0, layer.page_size if has_kv else 1,
+            _ptr(q_out), q_out.stride(0), T, n_heads, n_kv_heads, dim, vdim, slot, 1 if has_kv else 0, self.code, _stream()),
+            "diff_prepare")
+        return q_out
+
+    def diff_combine(self, maps, gate, out, share, eps, scale, n_heads, vdim, slot):
+        """Per head o = a1 - share * a2 of the two maps' results in ``maps`` [T, 2 * n_heads * slot]; ``out``
+        [T, n_heads * vdim] = o / sqrt(mean(o^2) + eps) * scale * sigmoid(gate), ``gate`` [T, n_heads] or None."""
+        T = maps.shape[0]
+        for name, tensor in (("maps", maps), ("out", out)):
+            _require(tensor, name, self.dtype)
+        if gate is not None:
+            _require(gate, "gate", self.dtype)
+            if gate.shape != (T, n_heads) or gate.stride(1) != 1:
+                raise KernelError("diff_combine: one gate per head")
+        if (maps.shape != (T, 2 * n_heads * slot) or maps.stride(1) != 1 or out.shape != (T, n_heads * vdim)
+                or out.stride(1) != 1 or slot < vdim):
+            raise KernelError("diff_combine: shapes do not match")
+        self.launches += 1
+        _check(self.core.ps_diff_combine(_ptr(maps), maps.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                         _ptr(out), out.stride(0), float(share), float(eps), float(scale), T, n_heads, vdim,
+                                         slot, self.code, _stream()), "diff_combine")
+        return out
+
     # ------------------------------------------------------------------ minGRU
     def mingru_scan(self, zug, width, state, ctx, out):
         """The gated recurrence of every entry of the step from and into the slots' state (csrc/mingru.cu).  ``zug``
@@ -1354,7 +1504,7 @@ class Ops:
         return out
 
     # ------------------------------------------------------------------ short convolution over time
-    def short_conv(self, u, weight, taps, conv_channels, state, ctx, out, blend=None, row_scale=None):
+    def short_conv(self, u, weight, taps, conv_channels, state, ctx, out, blend=None, row_scale=None, bias=None, act=None):
         """out[t, c] = sum_j weight[c, j] * u[t - taps + 1 + j, c] for the first ``conv_channels`` channels, the rest
         passed through; what lies before an entry's first token comes from ``state`` (float32
         [slots, (taps - 1) * conv_channels]: a request's last projected rows), which is then brought up to date
@@ -1362,8 +1512,15 @@ class Ops:
         ``blend`` = (mode, first channel, heads, head slot, head values, shared float32 [T, heads * head values],
         mix float32 scalar): mode "store" leaves the convolved values of those heads in ``shared``, "mix" blends
         them, v <- (1 - mix) v + mix * shared.  ``row_scale`` float32 [T]: row t of ``u`` is multiplied by row_scale[t]
-        wherever it is read (and kept)."""
-        _require(u, "u", torch.float32)
+        wherever it is read (and kept).  ``bias`` float32 [conv_channels] and ``act``: act(y + bias) behind the convolution;
+        ``u`` may then be of the compute dtype too."""
+        if u.dtype != torch.float32:
+            _require(u, "u", self.dtype)
+        if bias is not None:
+            _require(bias, "bias", torch.float32)
+            if bias.numel() != conv_channels or not bias.is_contiguous():
+                raise KernelError("short_conv: one bias per convolved channel")
+        _require(u, "u")
         _require(out, "out", self.dtype)
         T, channels = u.shape
         if out.shape != u.shape or u.stride(1) != 1 or out.stride(1) != 1 or not (0 <= conv_channels <= channels):
@@ -1392,17 +1549,17 @@ class Ops:
             if mode == 2:
                 _require(mix, "mix", torch.float32)
         self.launches += 1
-        _check(self.core.ps_short_conv(_ptr(u), u.stride(0), _ptr(weight), taps, conv_channels, channels,
+        _check(self.core.ps_short_conv(_ptr(u), dtype_code(u.dtype), u.stride(0), _ptr(weight), taps, conv_channels, channels,
                                        _ptr(row_scale), _ptr(state),
                                        state.stride(0) if state is not None else 0, _ptr(ctx.token_item),
                                        _ptr(ctx.q_start), _ptr(ctx.item_slot), _ptr(out), out.stride(0), mode, lo, heads,
-                                       slot, values, _ptr(shared), _ptr(mix) if mode == 2 else None, T, self.code,
-                                       _stream()), "short_conv")
+                                       slot, values, _ptr(shared), _ptr(mix) if mode == 2 else None, _ptr(bias),
+                                       _ACT_CODE[act], T, self.code, _stream()), "short_conv")
         return out
 
     # ------------------------------------------------------------------ routed experts
     def moe_route(self, x, router, shared_gate_w, dense, chosen, chosen_w, shared_gate, top, groups, keep, norm=None,
-                  score="softmax", normalize=True, correction=None):
+                  score="softmax", normalize=True, correction=None, group_mark="largest", scale=1.0):
         """The router of a layer of experts (csrc/moe.cu): softmax of ``x @ router.T`` in float32, the ``top``
         largest among the experts of the ``keep`` best of ``groups`` groups (0 or 1 groups: all experts stand),
         weights normalised to sum 1.  ``dense`` float32 [T, E] gets the weights (0 where not chosen), ``chosen``
@@ -1411,7 +1568,10 @@ class Ops:
         first writes the RMS norm of ``raw`` into ``x`` (the rows the experts' products then read) instead of
         reading ``x``.  ``score`` "sigmoid": the scores are sigmoid(z) expert by expert instead of the softmax;
         ``normalize`` False: the weights are the chosen scores themselves.  ``correction`` float32 [E]: added to the
-        scores for the election only (the weights stay the scores)."""
+        scores for the election only (the weights stay the scores).  ``group_mark`` "two_largest": a group's mark is the sum
+        of its two largest corrected scores instead of its largest score; ``scale`` multiplies the weights."""
+        if group_mark not in ("largest", "two_largest"):
+            raise KernelError(f"moe_route: unknown mark of a group {group_mark!r}")
         if correction is not None:
             _require(correction, "correction", torch.float32)
             if correction.numel() != router.shape[0] or not correction.is_contiguous():
@@ -1448,17 +1608,20 @@ class Ops:
                                       int(groups or 0), int(keep or 0), self.code, _ptr(raw),
                                       raw.stride(0) if raw is not None else 0, _ptr(gain), float(eps),
                                       1 if score == "sigmoid" else 0, 1 if normalize else 0, _ptr(correction),
-                                      _stream()), "moe_route")
+                                      1 if group_mark == "two_largest" else 0, float(scale), _stream()), "moe_route")
 
     @staticmethod
     def _gate_form(form):
         """(kind, limit, shared limit, alpha) of the inner activation: None / "silu" = silu(g) * u * weight; "gelu_tanh" likewise;
+        "relu_squared" = max(u, 0)^2 * weight, without a gate;
         ("clamped_swish", limit, shared_limit, alpha): g' = min(weight * g, limit), u' = clamp(weight * u, +-limit),
         g' * sigmoid(alpha * g') * (u' + 1): the weight scales the expert's input."""
         if form is None or form == "silu":
             return 0, 0.0, 0.0, 0.0
         if form == "gelu_tanh":
             return 2, 0.0, 0.0, 0.0
+        if form == "relu_squared":
+            return 3, 0.0, 0.0, 0.0
         kind, limit, shared_limit, alpha = form
         if kind != "clamped_swish":
             raise KernelError(f"unknown gated form {kind!r}")
@@ -1469,11 +1632,12 @@ class Ops:
         expert e's block of 2 * expert_ff columns is its gates, then its ups, and the shared expert's block follows;
         the weight of inner's column c is ``dense[t, c // expert_ff]`` for the experts' columns and
         ``shared_gate[t]`` (None: 1) from column ``n_experts * expert_ff`` on (csrc/moe.cu).  ``n_experts`` 0: the
-        product of a shared expert alone, or of a dense gated feed-forward.  ``form``: see :meth:`_gate_form`."""
+        product of a shared expert alone, or of a dense gated feed-forward.  ``form``: see :meth:`_gate_form`; without a
+        gate ``gate_up`` is [T, C], one block of expert_ff columns per expert."""
         T, C = inner.shape
         _require(gate_up, "gate_up", self.dtype)
         _require(inner, "inner", self.dtype)
-        if (gate_up.shape != (T, 2 * C) or gate_up.stride(1) != 1 or inner.stride(1) != 1
+        if (gate_up.shape != (T, C if form == "relu_squared" else 2 * C) or gate_up.stride(1) != 1 or inner.stride(1) != 1
                 or (n_experts and (dense.shape != (T, n_experts) or not dense.is_contiguous()))):
             raise KernelError("moe_gate_mul: shapes do not match")
         if n_experts:
@@ -1541,17 +1705,23 @@ class Ops:
                "moe_gate_mul_rows")
         return inner
 
-    def moe_combine(self, down, row_of, top, y):
-        """y[t] += sum_k down[row_of[t * top + k]] (float32; k in rising order, rows < 0 skipped)."""
+    def moe_combine(self, down, row_of, top, y, weights=None, factor=None):
+        """y[t] += sum_k down[row_of[t * top + k]] (float32; k in rising order, rows < 0 skipped); with ``weights`` float32
+        [T, top], y[t] += factor * sum_k weights[t, k] * down[...] (``factor`` float32, one number per column, or None)."""
         T, W = y.shape
         _require(down, "down", torch.float32)
         _require(y, "y", torch.float32)
         _require(row_of, "row_of", torch.int32)
         if down.shape[1] != W or row_of.numel() != T * top or down.stride(1) != 1 or y.stride(1) != 1:
             raise KernelError("moe_combine: shapes do not match")
+        for name, vector, count in (("weights", weights, T * top), ("factor", factor, W)):
+            if vector is not None:
+                _require(vector, name, torch.float32)
+                if vector.numel() != count or not vector.is_contiguous() or weights is None:
+                    raise KernelError(f"moe_combine: {name} do not fit")
         self.launches += 1
-        _check(self.core.ps_moe_combine(_ptr(down), down.stride(0), _ptr(row_of), top, _ptr(y), y.stride(0), T, W,
-                                        _stream()), "moe_combine")
+        _check(self.core.ps_moe_combine(_ptr(down), down.stride(0), _ptr(row_of), top, _ptr(weights), _ptr(factor), _ptr(y),
+                                        y.stride(0), T, W, _stream()), "moe_combine")
         return y
 
     def linear_experts(self, a, w, out, tile_expert, experts, along_k=False, act=None, status=None):

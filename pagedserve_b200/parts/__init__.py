@@ -16,4 +16,4 @@ from pagedserve_b200.parts.base import (  # noqa: F401
     register_part,
 )
 from pagedserve_b200.parts import (  # noqa: F401
-    attention, blocks, embedding, gla, mingru, mlp, moe, norms, parallel, positions, wkv)
+    attention, blocks, differential, embedding, gla, mingru, mlp, moe, norms, parallel, positions, ssd, wkv)

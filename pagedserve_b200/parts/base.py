@@ -67,6 +67,16 @@ class Part:
     # with such a part runs every step eagerly.
     graph_safe = False
 
+    # A factor per coordinate (float32 [H]) that an arrangement puts on what a mixer or a feed-forward adds to the residual
+    # rows (:meth:`set_result_factor`); parts that can apply it where their last product is stored say so.
+    result_factor = None
+    takes_result_factor = False
+
+    def set_result_factor(self, factor: torch.Tensor) -> None:
+        if not self.takes_result_factor:
+            raise ValueError(f"{type(self).__name__} cannot multiply its result by a factor per coordinate")
+        self.result_factor = factor
+
     def __init__(self, params: dict, prefix: str, env: PartEnv):
         self.params = dict(params)
         self.prefix = prefix
@@ -102,6 +112,11 @@ class PositionEncoding(Part):
 
     def embedding_table(self) -> Optional[torch.Tensor]:
         """A ``[positions, H]`` table to be added to the token embedding, if this encoding has one."""
+        return None
+
+    def sinusoids(self) -> Optional[torch.Tensor]:
+        """Frequencies ``[ceil(H / 2), 2]`` ((high, low) floats) of sines and cosines of the position that are added to the
+        token embedding, if this encoding is made of them."""
         return None
 
     def add_to_hidden(self, hidden: torch.Tensor, ctx) -> None:

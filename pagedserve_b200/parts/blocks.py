@@ -41,6 +41,62 @@ class PreNormBlock(Block):
                                   hidden, ctx)
 
 
+@register_part("block", "parallel_pre_norm")
+class ParallelPreNormBlock(Block):
+    """x <- x + s1 * mixer(norm1(x)) + s2 * feed_forward(norm2(x)), both of the same x: two RMS norms (``pre_mixer``,
+    ``pre_feed_forward``) with gains of their own, ``s1`` and ``s2`` a factor per coordinate (``scales``: the tensors'
+    names; absent: 1).  A layer whose feed-forward is the ``none`` part has the mixer only, and no second norm.
+
+    One kernel norms the row for both; after it x may change, so both results are added into x where they are made, times
+    their factors, by the epilogues of the mixer's and the feed-forward's last products (``Part.set_result_factor``).  The
+    residual rows, norms and sums are float32.
+
+    params: scales = dict(mixer, feed_forward) or None, init_std."""
+
+    graph_safe = True
+
+    def __init__(self, params, prefix, env, mixer, feed_forward, norms):
+        super().__init__(params, prefix, env, mixer, feed_forward, norms)
+        self.alone = getattr(feed_forward, "is_empty", False)
+        for norm in norms.values():
+            if norm.params.get("has_mean", True) or norm.params.get("has_bias", True):
+                raise ValueError("parallel_pre_norm: the norms are RMS norms without a bias")
+        if not self.alone and norms["pre_mixer"].params["eps"] != norms["pre_feed_forward"].params["eps"]:
+            raise ValueError("parallel_pre_norm: both norms have one eps")
+
+    @property
+    def required_norms(self):
+        return ("pre_mixer",) if self.alone else ("pre_mixer", "pre_feed_forward")
+
+    def _scaled(self):
+        scales = self.params.get("scales") or {}
+        return [(scales[role], part) for role, part in (("mixer", self.mixer), ("feed_forward", self.feed_forward))
+                if role in scales and not (role == "feed_forward" and self.alone)]
+
+    def param_specs(self):
+        width = self.norms["pre_mixer"].params["width"]
+        return [(ParamSpec(self._n(name), (width,), "vector"), ("ones_plus_normal", self.params.get("init_std", 0.1)))
+                for name, _ in self._scaled()]
+
+    def bind(self, tensors):
+        for name, part in self._scaled():
+            part.set_result_factor(tensors[self._n(name)].contiguous())
+
+    def forward(self, hidden, ctx, layer):
+        ops = self.env.ops
+        norm = self.norms["pre_mixer"]
+        if self.alone:
+            deferred = getattr(self.mixer, "accepts_deferred_norm", False)
+            self.mixer.forward(norm.defer(hidden) if deferred else norm.forward(hidden), hidden, ctx, layer)
+            return
+        second = self.norms["pre_feed_forward"]
+        h1 = ops.empty(hidden.shape, self.env.dtype, hidden.device)
+        h2 = ops.empty(hidden.shape, self.env.dtype, hidden.device)
+        ops.rms_norm_pair(hidden, norm.weight, second.weight, float(norm.params["eps"]), h1, h2)
+        self.mixer.forward(h1, hidden, ctx, layer)
+        self.feed_forward.forward(h2, hidden, ctx)
+
+
 class StreamCarrier:
     """What runs through the layers of a model with several residual streams: the streams ``[S, T, W]``, the
     row ``u`` that the open sublayer reads, the row ``y`` it adds its result into, and the (mix, out) weights of

@@ -10,7 +10,7 @@ from pagedserve_b200.weights.loader import ParamSpec
 
 @register_part("embedding", "token_embedding")
 class TokenEmbedding(Embedding):
-    """hidden[t] = table[id_t] (+ the position encoding's table row, fused into the same gather).
+    """hidden[t] = table[id_t] (+ the position encoding's table row, or its sines and cosines, in the same kernel).
 
     reference: src/model/paged_decoder.py:288, 306-314.  The result is float32:
     it starts the residual stream.  params: vocab_size, hidden_size, name, init_std."""
@@ -28,6 +28,9 @@ class TokenEmbedding(Embedding):
     def forward(self, ctx, positions):
         hidden = self.env.ops.empty((ctx.num_tokens, self.params["hidden_size"]), torch.float32, self.table.device)
         position_table = positions.embedding_table()
+        sinusoids = positions.sinusoids()
+        if sinusoids is not None:
+            return self.env.ops.embed_sinusoid(ctx.token_ids, ctx.positions, self.table, sinusoids, hidden, ctx.status)
         self.env.ops.embed(ctx.token_ids, ctx.positions, self.table, position_table, hidden, ctx.status)
         if position_table is None:
             positions.add_to_hidden(hidden, ctx)
@@ -103,6 +106,8 @@ class TokenPairEmbedding(TokenEmbedding):
     def forward(self, ctx, positions, state=None):
         p = self.params
         pair = p.get("pair") or {}
+        if positions.sinusoids() is not None:
+            raise ValueError("token_pair_embedding: positions made of sines are added by the plain token embedding only")
         hidden = self.env.ops.empty((ctx.num_tokens, p["hidden_size"]), torch.float32, self.table.device)
         if self.pair_table is not None and state is None:
             raise ValueError("token_pair_embedding: the cache holds no slot state for the token before")

@@ -23,6 +23,10 @@ class DenseMLP(FeedForward):
     graph_safe = True
     accepts_deferred_norm = True       # x goes straight into ops.linear
 
+    @property
+    def takes_result_factor(self):
+        return not self.params.get("has_bias", True)
+
     def __init__(self, params, prefix, env):
         super().__init__(params, prefix, env)
         if self.params["activation"] not in ACTIVATIONS:
@@ -70,7 +74,7 @@ class DenseMLP(FeedForward):
             ops.moe_gate_mul(gate_up, None, None, inner, 0, p["inner_size"], form=p["activation"])
         else:
             ops.linear(x, self.w_up, self.b_up, inner, act=p["activation"])
-        ops.linear(inner, self.w_down, self.b_down, residual, accumulate=True)
+        ops.linear(inner, self.w_down, self.b_down, residual, accumulate=True, factor=self.result_factor)
 
 
 @register_part("feed_forward", "none")
@@ -79,6 +83,7 @@ class NoFeedForward(FeedForward):
 
     graph_safe = True
     is_empty = True
+    takes_result_factor = True
 
     def forward(self, x, residual, ctx):
         return None

@@ -19,7 +19,9 @@ class RoutedExperts(FeedForward):
     chosen s (+ 1e-20).  A shared expert of the same form (its own inner size) runs for every token, multiplied by
     sigmoid(w_sg . x), one number per token (``shared_gate`` False: the shared expert is added as it is).
 
-    Other forms of the same part.  ``score`` "sigmoid": s = sigmoid(z), expert by expert, instead of the softmax;
+    Other forms of the same part.  ``expert_form`` dict(kind="relu_squared"): an expert is W_down max(W_up x, 0)^2, without a
+    gate matrix.  ``group_mark`` "two_largest": a group's mark is the sum of its two largest corrected scores (not its
+    largest score); ``weight_scale`` multiplies the weights.    ``score`` "sigmoid": s = sigmoid(z), expert by expert, instead of the softmax;
     ``normalize`` False: the weights are the chosen s themselves.  ``expert_form`` dict(kind="clamped_swish", limit,
     alpha): an expert is W_down (g sigmoid(alpha g) (u + 1)) with g = min(W_gate x', limit), u = clamp(W_up x',
     -limit, limit), and its weight multiplies its input, x' = w x, not its output; the shared expert has a limit of
@@ -41,7 +43,7 @@ class RoutedExperts(FeedForward):
     sums up to their order.
 
     params: hidden_size, n_experts, expert_ff, top, groups, group_keep, shared_ff (None: no shared expert),
-    score ("softmax"), normalize (True), expert_form (None: silu), shared_limit, shared_gate (True),
+    score ("softmax"), normalize (True), group_mark ("largest"), weight_scale (1), expert_form (None: silu), shared_limit, shared_gate (True),
     correction_name (None; a float32 tensor of one number per expert that is added to the scores for the election
     only: the chosen experts' weights stay their scores),
     init_std, out_init_std; tensors ``router``, ``e<i>.gate / up / down``, ``shared.gate / up / down / sg``.
@@ -49,6 +51,7 @@ class RoutedExperts(FeedForward):
 
     graph_safe = True
     accepts_deferred_norm = True       # an RMS norm in front is computed by the router's kernel
+    takes_result_factor = True
 
     def __init__(self, params, prefix, env):
         super().__init__(params, prefix, env)
@@ -64,7 +67,12 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: score is 'softmax' or 'sigmoid'")
         form = p.get("expert_form")
         self.form = None
-        if form is not None and form.get("kind", "silu") != "silu":
+        self.gated = form is None or form.get("kind", "silu") != "relu_squared"
+        if not self.gated:
+            self.form = "relu_squared"
+            if p.get("shared_ff"):
+                raise ValueError("routed_experts: a shared expert has a gate")
+        elif form is not None and form.get("kind", "silu") != "silu":
             if form["kind"] != "clamped_swish" or not form["limit"] > 0:
                 raise ValueError("routed_experts: expert_form is silu, or clamped_swish with a positive limit")
             self.form = ("clamped_swish", float(form["limit"]), float(p.get("shared_limit") or form["limit"]),
@@ -82,8 +90,9 @@ class RoutedExperts(FeedForward):
         specs = [(ParamSpec(self._n("router"), (p["n_experts"], W), "matmul"), ("normal", 4.0 * std))]
         for name in self._expert_names():
             F = p["shared_ff"] if name == "shared." else p["expert_ff"]
-            specs += [(ParamSpec(self._n(name + "gate"), (F, W), "matmul"), ("normal", std)),
-                      (ParamSpec(self._n(name + "up"), (F, W), "matmul"), ("normal", std)),
+            if self.gated:
+                specs.append((ParamSpec(self._n(name + "gate"), (F, W), "matmul"), ("normal", std)))
+            specs += [(ParamSpec(self._n(name + "up"), (F, W), "matmul"), ("normal", std)),
                       (ParamSpec(self._n(name + "down"), (W, F), "matmul"), ("normal", out_std))]
         if self.has_shared_gate:
             specs.append((ParamSpec(self._n("shared.sg"), (1, W), "matmul"), ("normal", std)))
@@ -95,7 +104,7 @@ class RoutedExperts(FeedForward):
         t = lambda name: tensors[self._n(name)]
         names = self._expert_names()
         self.router = t("router").contiguous()
-        self.w_gate_up = torch.cat([t(name + which) for name in names for which in ("gate", "up")],
+        self.w_gate_up = torch.cat([t(name + which) for name in names for which in (("gate", "up") if self.gated else ("up",))],
                                    dim=0).contiguous()           # [2 * columns, W]: per expert its gates, then its ups
         self.w_down = torch.cat([t(name + "down") for name in names], dim=1).contiguous()      # [W, columns]
         self.w_shared_gate = t("shared.sg").reshape(-1).contiguous() if self.has_shared_gate else None
@@ -122,16 +131,17 @@ class RoutedExperts(FeedForward):
         shared_gate = ops.empty((tokens,), torch.float32, device) if self.w_shared_gate is not None else None
         ops.moe_route(x, self.router, self.w_shared_gate, dense, chosen, chosen_w, shared_gate, p["top"],
                       p.get("groups") or 0, p.get("group_keep") or 0, norm=norm, score=p.get("score", "softmax"),
-                      normalize=p.get("normalize", True), correction=self.correction)
+                      normalize=p.get("normalize", True), correction=self.correction,
+                      group_mark=p.get("group_mark", "largest"), scale=float(p.get("weight_scale", 1.0)))
         F, width = p["expert_ff"], p["hidden_size"]
         if self._sorted_rows(tokens, x):
             self._forward_sorted(x, residual, dense, chosen, chosen_w, shared_gate)
             return
-        gate_up = ops.empty((tokens, 2 * self.columns), dtype, device)
+        gate_up = ops.empty((tokens, self.w_gate_up.shape[0]), dtype, device)
         ops.linear(x, self.w_gate_up, None, gate_up)
         inner = ops.empty((tokens, self.columns), dtype, device)
         ops.moe_gate_mul(gate_up, dense, shared_gate, inner, E, F, form=self.form)
-        ops.linear(inner, self.w_down, None, residual, accumulate=True)
+        ops.linear(inner, self.w_down, None, residual, accumulate=True, factor=self.result_factor)
 
     SORTED_FROM = 128             # tokens of a step from which the rows are sorted by expert
 
@@ -156,17 +166,33 @@ class RoutedExperts(FeedForward):
         ops.moe_plan(chosen, chosen_w, E, row_of, row_token, row_weight, tile_expert)
         rows = ops.empty((rows_cap, width), dtype, device)
         ops.moe_gather(x, row_token, rows)
+        inner = ops.empty((rows_cap, F), dtype, device)
+        down = ops.empty((rows_cap, width), torch.float32, device)
+        if not self.gated:
+            # the activation is the first product's epilogue, the weights join where the rows come together
+            ops.linear_experts(rows, self.w_gate_up, inner, tile_expert, E, act="relu_squared")
+            ops.linear_experts(inner, self.w_down, down, tile_expert, E, along_k=True)
+            ops.moe_combine(down, row_of, top, residual, weights=chosen_w, factor=self.result_factor)
+            return
         gate_up = ops.empty((rows_cap, 2 * F), dtype, device)
         ops.linear_experts(rows, self.w_gate_up[:E * 2 * F], gate_up, tile_expert, E)
-        inner = ops.empty((rows_cap, F), dtype, device)
         ops.moe_gate_mul_rows(gate_up, row_weight, inner, form=self.form)
-        down = ops.empty((rows_cap, width), torch.float32, device)
         ops.linear_experts(inner, self.w_down[:, :E * F], down, tile_expert, E, along_k=True)
-        ops.moe_combine(down, row_of, top, residual)
+        if self.result_factor is None:
+            ops.moe_combine(down, row_of, top, residual)
+        else:                                                   # (the weights are in the inner rows already)
+            ops.moe_combine(down, row_of, top, residual, weights=self._ones(chosen_w), factor=self.result_factor)
         shared_ff = p.get("shared_ff") or 0
         if shared_ff:
             gate_up_shared = ops.empty((tokens, 2 * shared_ff), dtype, device)
             ops.linear(x, self.w_gate_up[E * 2 * F:], None, gate_up_shared)
             inner_shared = ops.empty((tokens, shared_ff), dtype, device)
             ops.moe_gate_mul(gate_up_shared, dense, shared_gate, inner_shared, 0, shared_ff, form=self.form)
-            ops.linear(inner_shared, self.w_down[:, E * F:], None, residual, accumulate=True)
+            ops.linear(inner_shared, self.w_down[:, E * F:], None, residual, accumulate=True, factor=self.result_factor)
+
+    def _ones(self, like):
+        """Float32 ones of the shape of ``like``, kept for the life of the part."""
+        held = getattr(self, "_held_ones", None)
+        if held is None or held.numel() < like.numel():
+            self._held_ones = held = torch.ones(like.numel(), dtype=torch.float32, device=like.device)
+        return held[:like.numel()]

@@ -36,6 +36,34 @@ class NoPositions(PositionEncoding):
     graph_safe = True
 
 
+@register_part("positions", "sinusoidal")
+class SinusoidalPositions(PositionEncoding):
+    """h0[t] gets a vector of sines and cosines of the position p: number 2i is sin(p * base^(-2i / hidden_size)), number
+    2i + 1 the cosine of the same angle.  Nothing bounds the positions; the embedding's kernel forms the angles, float32
+    with frequencies of more than one float (``sinusoids``).
+    params: hidden_size, base."""
+
+    graph_safe = True
+
+    def __init__(self, params, prefix, env):
+        super().__init__(params, prefix, env)
+        if not self.params["base"] > 0:
+            raise ValueError("sinusoidal: base must be positive")
+        self._table = None
+
+    def sinusoids(self):
+        if self._table is None:
+            import torch
+
+            width = self.params["hidden_size"]
+            index = torch.arange((width + 1) // 2, dtype=torch.float64)
+            exact = torch.pow(torch.tensor(float(self.params["base"]), dtype=torch.float64), -2.0 * index / width)
+            high = exact.to(torch.float32)
+            low = (exact - high.to(torch.float64)).to(torch.float32)
+            self._table = torch.stack([high, low], dim=1).contiguous().to(self.env.device)
+        return self._table
+
+
 @register_part("positions", "rotary")
 class RotaryPositions(PositionEncoding):
     """Queries and keys turn by their position: of the first ``dims`` dimensions of every head, pair i turns by
