@@ -250,3 +250,109 @@ def read_folder(folder, dtype=torch.float64):
             raise ValueError(f"{name}: {entry['dtype']}")
         tensors[name] = array.reshape(entry["shape"]).to(dtype)
     return tensors, config
+
+
+# ------------------------------------------------------------------------------- random models for the tests
+def tensor_shapes(config):
+    """{checkpoint name: shape} of a model of ``config``."""
+    W, V = config["width"], config["vocab"]
+    shapes = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    for index, layer in enumerate(config["layers"]):
+        p, m = f"l{index}.", layer["mixer"]
+        shapes.update({p + "norm1": (W,), p + "ls1": (W,)})
+        mix = lambda name: p + "mix." + name
+        H, e = m["heads"], m["vdim"]
+        if layer["type"] == "mamba2":
+            inner, channels = H * e, H * e + 2 * m["groups"] * m["state"]
+            shapes.update({mix("in"): (inner + channels + H, W), mix("conv"): (channels, m["conv"]), mix("conv.b"): (channels,),
+                           mix("dt_bias"): (H,), mix("A_log"): (H,), mix("D"): (H,), mix("norm"): (inner,),
+                           mix("o"): (W, inner)})
+        else:
+            d, G = m["dim"], m["kv_heads"]
+            shapes.update({mix("q"): (2 * H * d, W), mix("q.norm"): (d,), mix("g"): (H, W), mix("o"): (W, H * e)})
+            shapes.update({mix(name): (d,) for name in ("lq1", "lk1", "lq2", "lk2")})
+            if m.get("kv_from") is None:
+                shapes.update({mix("k"): (2 * G * d, W), mix("k.norm"): (d,), mix("v"): (G * e, W)})
+        mlp = layer.get("mlp")
+        if mlp is None:
+            continue
+        shapes.update({p + "norm2": (W,), p + "ls2": (W,)})
+        ff = lambda name: p + "mlp." + name
+        if mlp["kind"] == "dense":
+            shapes.update({ff("gate"): (mlp["ff"], W), ff("up"): (mlp["ff"], W), ff("down"): (W, mlp["ff"])})
+        else:
+            E, F = mlp["router"]["experts"], mlp["expert"]["ff"]
+            shapes.update({ff("router"): (E, W), ff("correction"): (E,)})
+            for index_e in range(E):
+                shapes.update({ff(f"e{index_e}.up"): (F, W), ff(f"e{index_e}.down"): (W, F)})
+    return shapes
+
+
+def random_model(config, seed):
+    """Random tensors (rounded to bfloat16, stored as such) that keep activations of order one: states that remember from a
+    few to hundreds of tokens, second maps that take a good part off the first, corrections that turn elections and make
+    choice scores negative."""
+    g = torch.Generator().manual_seed(seed)
+    tensors = {}
+    for name, shape in tensor_shapes(config).items():
+        leaf = name.split(".")[-1]
+        if name == "embed":
+            value = torch.randn(shape, generator=g)
+        elif name.endswith(("q.norm", "k.norm")):
+            value = 1.3 + 0.2 * torch.randn(shape, generator=g)
+        elif name.endswith("mix.norm"):
+            value = 1.0 + 0.2 * torch.randn(shape, generator=g)
+        elif leaf in ("norm", "norm1", "norm2"):
+            value = 0.2 * torch.randn(shape, generator=g)
+        elif leaf in ("ls1", "ls2"):
+            value = 0.6 + 0.2 * torch.randn(shape, generator=g)
+        elif leaf == "conv":
+            value = torch.randn(shape, generator=g) / math.sqrt(shape[1])
+        elif leaf == "b":
+            value = 0.3 * torch.randn(shape, generator=g)
+        elif leaf == "dt_bias":
+            value = torch.randn(shape, generator=g) - 1.0
+        elif leaf == "A_log":
+            value = 5.0 * torch.rand(shape, generator=g) - 4.0
+        elif leaf == "D":
+            value = torch.randn(shape, generator=g)
+        elif leaf in ("lq1", "lk1", "lq2", "lk2"):
+            value = 0.6 * torch.randn(shape, generator=g) / math.sqrt(shape[0]) ** 0.5
+        elif leaf == "correction":
+            value = 0.5 * torch.randn(shape, generator=g) - 0.6
+        elif leaf == "router":
+            value = 2.0 * torch.randn(shape, generator=g) / math.sqrt(shape[1])
+        else:
+            value = torch.randn(shape, generator=g) / math.sqrt(shape[1])
+        tensors[name] = value.to(torch.bfloat16)
+    return tensors
+
+
+def dense_mlp(ff=48):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe_mlp(experts=6, top=2, ff=24, groups=(3, 2), scale=1.5):
+    router = {"experts": experts, "top": top, "scale": scale}
+    if groups is not None:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "expert": {"ff": ff}, "router": router}
+
+
+def mamba_layer(heads=4, vdim=16, state=24, groups=2, norm_groups=2, conv=3, mlp=None):
+    return {"type": "mamba2", "mlp": mlp, "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups,
+                                                    "norm_groups": norm_groups, "conv": conv}}
+
+
+def diff_layer(heads=4, kv_heads=2, dim=12, vdim=20, scale=0.3, diff=0.4, q_temp=(0.2, 16), kv_from=None, mlp=None):
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "diff": diff}
+    if q_temp is not None:
+        mixer["q_temp"] = {"coef": q_temp[0], "every": q_temp[1]}
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    return {"type": "attention", "mlp": mlp, "mixer": mixer}
+
+
+def make_config(layers, width=64, vocab=97, eps=1e-5, logit_scale=0.7):
+    return {"architecture": "Vozirax", "layers": layers, "logit_scale": logit_scale, "norm": {"eps": eps}, "vocab": vocab,
+            "width": width}

@@ -1,0 +1,879 @@
+"""Vozirax in the engine against the plain implementation (tests/plain_vozirax.py): every mechanism alone, then whole
+models through the step function, the trace replay and the scheduler, in float32 and bfloat16.
+
+The configurations are made here, with random weights; sizes differ from model to model so that nothing rests on a
+value that happens to be 1 or on two sizes that happen to be equal."""
+
+import io
+import json
+import os
+import tempfile
+from types import SimpleNamespace
+
+import numpy as np
+import pytest
+import torch
+
+import helpers
+import plain_vozirax as plain
+
+pytestmark = pytest.mark.gpu
+
+DEV = "cuda:0"
+CLOSE_CALL = 0.03                       # elections closer than this may turn under bfloat16 rounding
+
+M, D, X, E = plain.mamba_layer, plain.diff_layer, plain.dense_mlp, plain.moe_mlp
+# both mixers with both feed-forwards and none, three groups, two norm groups, two layers that borrow from one, values
+# larger than two keys and smaller
+CONFIG_A = plain.make_config(
+    [M(6, 16, 24, groups=3, norm_groups=2, conv=3, mlp=E(6, 2, 24)),
+     D(4, 2, 12, 20, q_temp=(0.3, 24), mlp=X(48)),
+     D(6, 2, 12, 20, diff=0.7, q_temp=(0.1, 7), kv_from=1, mlp=E(8, 3, 16, groups=(4, 2), scale=2.0)),
+     M(4, 24, 16, groups=1, norm_groups=3, conv=4),
+     D(2, 2, 12, 20, diff=-0.1, q_temp=None, kv_from=1, mlp=X(40)),
+     D(5, 1, 20, 56, scale=0.2, mlp=E(4, 2, 20, groups=None))],
+    width=64, vocab=97)
+# heads of 2 x 32 and 2 x 64 numbers (the tensor-core attention kernels), state sizes of the tensor-core recurrence
+CONFIG_B = plain.make_config(
+    [D(4, 2, 32, 64, scale=0.15, q_temp=(0.2, 100), mlp=E(8, 2, 64, groups=(2, 1), scale=2.5)),
+     M(8, 32, 64, groups=2, norm_groups=1, conv=4, mlp=X(160)),
+     D(4, 1, 64, 128, scale=0.1, mlp=X(96)),
+     M(4, 64, 128, groups=1, norm_groups=4, conv=2, mlp=E(16, 4, 32, groups=(4, 2), scale=1.3)),
+     D(8, 1, 64, 128, scale=0.12, diff=0.2, kv_from=2)],
+    width=128, vocab=211, eps=1e-6, logit_scale=0.5)
+# nothing a multiple of 8 or 16, single heads, an odd width
+CONFIG_C = plain.make_config(
+    [M(3, 14, 10, groups=1, norm_groups=1, conv=2, mlp=X(36)),
+     D(3, 3, 7, 9, scale=0.5, q_temp=(0.4, 5), mlp=E(5, 2, 14, groups=None, scale=0.7)),
+     M(1, 20, 36, groups=1, norm_groups=5, conv=1, mlp=E(6, 1, 10, groups=(2, 1))),
+     D(1, 1, 22, 6, scale=0.3, mlp=X(20)),
+     D(9, 3, 7, 9, kv_from=1)],
+    width=71, vocab=53, eps=1e-4, logit_scale=1.7)
+# wide states and heads, every expert chosen, many norm groups
+CONFIG_D = plain.make_config(
+    [M(2, 96, 40, groups=2, norm_groups=8, conv=5, mlp=E(4, 4, 24, groups=(2, 2))),
+     D(2, 1, 40, 64, mlp=E(3, 3, 16, groups=None)),
+     M(3, 130, 72, groups=1, norm_groups=6, conv=4, mlp=X(64)),
+     D(6, 2, 16, 112, scale=0.25, diff=0.5, mlp=None)],
+    width=96, vocab=131, eps=1e-3)
+# one layer of each kind alone
+CONFIG_E = plain.make_config([M(4, 20, 12, groups=4, norm_groups=4, conv=6, mlp=E(4, 1, 16, groups=(2, 1)))], width=48, vocab=61)
+CONFIG_F = plain.make_config([D(4, 4, 10, 12, mlp=X(8))], width=40, vocab=77)
+# states and cached heads beyond what the fast kernels take
+CONFIG_W = plain.make_config([M(2, 72, 300, groups=1, norm_groups=1, conv=3), D(2, 1, 136, 290, scale=0.1, mlp=X(16))], width=56,
+                             vocab=41)
+# layers for keys that stand out: large gains, second maps that hardly count or count fully
+CONFIG_S = plain.make_config(
+    [D(4, 2, 16, 24, scale=0.5, diff=0.3), D(4, 2, 32, 64, scale=0.3, diff=0.5, q_temp=(0.3, 50)),
+     D(2, 1, 64, 128, scale=0.2, diff=0.4), D(6, 3, 10, 14, scale=0.6, diff=-0.3)],
+    width=96, vocab=67)
+# layers as wide as a small model's (the tensor-core products, prompt attention and recurrence run at these sizes)
+CONFIG_M = plain.make_config(
+    [M(16, 64, 128, groups=2, norm_groups=1, conv=4, mlp=X(700)),
+     D(8, 4, 32, 64, scale=0.18, q_temp=(0.1, 256), mlp=E(8, 2, 192, groups=(2, 1), scale=2.5)),
+     M(24, 32, 64, groups=3, norm_groups=2, conv=4, mlp=E(8, 3, 160, groups=(4, 2), scale=1.5)),
+     D(12, 4, 32, 64, scale=0.15, kv_from=1, mlp=X(500)),
+     D(4, 2, 48, 80, scale=0.15, mlp=None)],
+    width=512, vocab=700, eps=1e-6)
+
+CONFIGS = {"a": (CONFIG_A, 1, 16), "b": (CONFIG_B, 2, 16), "c": (CONFIG_C, 3, 8), "d": (CONFIG_D, 4, 32),   # config, seed, page
+           "e": (CONFIG_E, 5, 16), "f": (CONFIG_F, 6, 8), "w": (CONFIG_W, 7, 16), "s": (CONFIG_S, 8, 16),
+           "m": (CONFIG_M, 9, 16)}
+
+_FOLDERS, _TENSORS, _LOGITS, _CLEAR = {}, {}, {}, {}
+
+
+def folder_of(which):
+    if which not in _FOLDERS:
+        from pagedserve_b200.weights.safetensors_io import write_safetensors
+
+        config, seed, _ = CONFIGS[which]
+        holder = tempfile.TemporaryDirectory(prefix=f"ps_vozirax_{which}_")
+        tensors = plain.random_model(config, seed)
+        if which == "s":                                             # large query gains: one key can stand out
+            for name in tensors:
+                if name.endswith("mix.q.norm"):
+                    tensors[name] = (tensors[name].float() * 3.0).to(torch.bfloat16)
+        _TENSORS[which] = tensors
+        with open(os.path.join(holder.name, "config.json"), "w") as handle:
+            json.dump(config, handle)
+        write_safetensors(os.path.join(holder.name, "model.safetensors"), tensors)
+        _FOLDERS[which] = holder
+    return _FOLDERS[which].name
+
+
+def plain_logits(which, sequences):
+    """Logits of every sequence; beside them which rows' elections were all clear."""
+    folder_of(which)
+    out, clear = {}, {}
+    for name, tokens in sequences.items():
+        key = (which, tuple(tokens))
+        if key not in _LOGITS:
+            margins = []
+            _LOGITS[key] = plain.forward(_TENSORS[which], CONFIGS[which][0], tokens, margins=margins).numpy()
+            _CLEAR[key] = np.array([margin > CLOSE_CALL for margin in margins])
+        out[name], clear[name] = _LOGITS[key], _CLEAR[key]
+    return out, clear
+
+
+def assert_rows_close(got, want, dtype, what, clear=None):
+    """float32: every logit within 3e-5 of the scale (sums differ in order only), the best token the same.
+    bfloat16: a row's error is the root mean square over the vocabulary against that of the logits; rounding alone
+    gives about 1 % in the mean over the rows and a few per cent at single rows, while a wrong key, a lost state or a
+    map that is not taken off moves a row by 30 % and more.  Rows in which an election was a close call are left out."""
+    assert got.shape == want.shape and np.isfinite(got).all(), what
+    if dtype == "float32":
+        scale = float(np.abs(want).max())
+        error = np.abs(got.astype(np.float64) - want).max(-1)
+        assert float(error.max()) <= 3e-5 * scale, \
+            f"{what}: row {int(error.argmax())} is off by {float(error.max()):.3e}, scale {scale:.3e}"
+        ordered = np.sort(want, axis=-1)
+        sure = (ordered[:, -1] - ordered[:, -2]) > 1e-4 * scale
+        assert (got.argmax(-1) == want.argmax(-1))[sure].all(), f"{what}: another best token"
+        return
+    error = np.sqrt(((got - want) ** 2).mean(-1)) / np.sqrt((want ** 2).mean())
+    if clear is not None:
+        error = error[clear]
+    if error.size:
+        assert float(error.max()) < 0.12, f"{what}: row {int(error.argmax())} of the clear ones is off by {float(error.max()):.3f}"
+        assert float(error.mean()) < 0.03, f"{what}: rows are off by {float(error.mean()):.4f} in the mean"
+
+
+def build_engine(which, dtype, **options):
+    from pagedserve_b200.config.engine_config import EngineConfig
+    from pagedserve_b200.engine.engine import Engine
+
+    defaults = dict(dtype=dtype, block_size=CONFIGS[which][2], num_blocks=96, max_num_seqs=4, max_model_len=512)
+    defaults.update(options)
+    return Engine.from_folder(folder_of(which), EngineConfig(**defaults))
+
+
+def sequences_for(which, lengths, seed=0):
+    vocab = CONFIGS[which][0]["vocab"]
+    return {f"s{i}": helpers.random_tokens(vocab, n, seed=seed + i) for i, n in enumerate(lengths)}
+
+
+def rel_err(got, want):
+    want = want.double()
+    return float((got.double().cpu() - want).abs().max() / want.abs().max().clamp_min(1e-30))
+
+
+# ------------------------------------------------------------------ the replay program on whole models
+def run_replay(which, dtype, steps, slots=4):
+    from pagedserve_b200.engine import replay as replay_module
+
+    with tempfile.TemporaryDirectory(prefix="ps_out_") as out:
+        args = SimpleNamespace(model=folder_of(which), dtype=dtype, out=out, max_tokens=helpers.peak_tokens(steps),
+                               block_size=CONFIGS[which][2], max_num_seqs=slots, disable_cuda_graphs=False)
+        stdin = io.StringIO("".join(json.dumps(step) + "\n" for step in steps))
+        assert replay_module.run(args, stdin=stdin, stdout=io.StringIO()) == 0
+        return helpers.collect(out, steps)
+
+
+def check_replay(which, dtype, steps, sequences, what, slots=4):
+    got = run_replay(which, dtype, steps, slots)
+    want, clear = plain_logits(which, sequences)
+    for name in sequences:
+        assert_rows_close(got[name], want[name], dtype, f"{what}/{which}/{name}", clear[name])
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which", ["a", "b", "c", "d"])
+def test_whole_prompts_and_decoded_tails(which, dtype):
+    """Each request alone: whole in one step, and most of it in one step with its tail token by token, so that
+    prefill and decoding through the cache and the kept state give the same logits.  Sequences of one and two tokens
+    (shorter than a convolution) included."""
+    sequences = sequences_for(which, [1, 2, 37, 150, 301], seed=10)
+    check_replay(which, dtype, helpers.trace_whole(sequences), sequences, "whole")
+    check_replay(which, dtype, helpers.trace_tail(sequences, tail=48), sequences, "tail")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which", ["a", "b", "c", "d"])
+def test_portions_of_every_size(which, dtype):
+    """Portions down to two tokens (fewer than the convolution's taps), cut inside pages, key tiles, chunks and runs of
+    the recurrence."""
+    sequences = sequences_for(which, [61, 143, 260], seed=20)
+    check_replay(which, dtype, helpers.trace_chunks(sequences, seed=1), sequences, "portions")
+    check_replay(which, dtype, helpers.trace_chunks(sequences, seed=2, sizes=(2, 2, 17, 64, 3, 130, 2, 31)), sequences,
+                 "portions-2")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which", ["a", "b", "c", "d"])
+def test_mixed_batches_reuse_pages_and_slots(which, dtype):
+    """Nine unequal requests through four slots: prompts in portions next to decoded tokens, requests left
+    out of steps, pages and state slots handed out again; every request must equal itself alone."""
+    sequences = sequences_for(which, [90, 33, 200, 5, 61, 148, 17, 75, 2], seed=30)
+    steps = helpers.trace_mixed(sequences, seed=3, live=4, decode_tail=20, max_portion=40)
+    assert helpers.peak_tokens(steps) < sum(len(t) for t in sequences.values())
+    check_replay(which, dtype, steps, sequences, "mixed")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_many_requests_decoded_together(dtype):
+    """Eleven requests live at once, most of them decoding: batches of single tokens that are padded to shared sizes."""
+    sequences = sequences_for("b", [40, 52, 33, 47, 60, 35, 44, 58, 39, 50, 41, 36, 55], seed=90)
+    steps = helpers.trace_mixed(sequences, seed=8, live=11, decode_tail=26, max_portion=40)
+    check_replay("b", dtype, steps, sequences, "many", slots=11)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which", ["e", "f", "w"])
+def test_models_of_few_layers(which, dtype):
+    sequences = sequences_for(which, [70, 3, 131, 29, 64, 1], seed=70)
+    check_replay(which, dtype, helpers.trace_whole(sequences), sequences, "whole")
+    steps = helpers.trace_mixed(sequences, seed=5, live=4, decode_tail=16, max_portion=30)
+    check_replay(which, dtype, steps, sequences, "mixed")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_model_of_middle_size(dtype):
+    """Hundreds of tokens whole, then unequal requests mixed, at layer sizes where the tensor-core kernels run."""
+    sequences = sequences_for("m", [700, 260, 97, 23, 1], seed=60)
+    check_replay("m", dtype, helpers.trace_whole(sequences), sequences, "whole")
+    steps = helpers.trace_mixed(sequences, seed=6, live=4, decode_tail=24, max_portion=170)
+    check_replay("m", dtype, steps, sequences, "mixed")
+
+
+@pytest.mark.parametrize("which,count,tail", [("a", 340, 330), ("c", 200, 190)])
+def test_long_decoding_float32(which, count, tail):
+    """A short prompt, then hundreds of tokens one by one: the recurrent state and the kept rows of the convolutions
+    are carried through every step."""
+    sequences = sequences_for(which, [count], seed=40)
+    check_replay(which, "float32", helpers.trace_tail(sequences, tail=tail), sequences, "long decode")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_long_prompt_in_one_step_and_in_portions(dtype):
+    """1,500 tokens: angles of more than a thousand radians, a recurrence cut into many runs, then the tail decoded."""
+    which = "b"
+    sequences = sequences_for(which, [1500], seed=80)
+    wanted = list(range(0, 1500, 97)) + list(range(1460, 1500))
+    whole = [{"step": 0, "entries": [{"id": "s0", "tokens": sequences["s0"], "want": wanted}], "end": ["s0"]}]
+    got = run_replay(which, dtype, whole)
+    logits, clear = plain_logits(which, sequences)
+    want, clear = logits["s0"][wanted], clear["s0"][wanted]
+    assert_rows_close(got["s0"], want, dtype, "long prompt in one step", clear)
+    steps, number, done = [], 0, 0
+    for size in [700, 500, 270] + [1] * 30:
+        places = [i for i in range(size) if done + i in wanted]
+        steps.append({"step": number, "entries": [{"id": "s0", "tokens": sequences["s0"][done:done + size],
+                                                   "want": places}], "end": []})
+        number, done = number + 1, done + size
+    steps[-1]["end"] = ["s0"]
+    got = run_replay(which, dtype, steps)
+    assert_rows_close(got["s0"], want, dtype, "long prompt in portions", clear)
+
+
+# ------------------------------------------------------------------ generation through the scheduler
+@pytest.mark.parametrize("strategy", ["orca", "sarathi"])
+@pytest.mark.parametrize("which", ["a", "c"])
+def test_greedy_generation_equals_the_plain_model(which, strategy):
+    from pagedserve_b200.engine.engine import generate
+
+    engine = build_engine(which, "float32", strategy=strategy, prefill_chunk_size=7, max_num_seqs=3)
+    prompts = list(sequences_for(which, [9, 30, 3, 55, 1], seed=60).values())
+    got = generate(engine, prompts, max_new_tokens=12)
+    config, tensors = CONFIGS[which][0], _TENSORS[which]
+    for prompt, tokens in zip(prompts, got):
+        sequence = list(prompt)
+        for _ in range(12):
+            logits = plain.forward(tensors, config, sequence)[-1]
+            top = torch.topk(logits, 2).values
+            if float(top[0] - top[1]) < 1e-3 * float(logits.abs().max()):
+                break                                        # a near tie: either token is a correct greedy choice
+            sequence.append(int(logits.argmax()))
+        made = len(sequence) - len(prompt)
+        assert tokens[:made] == sequence[len(prompt):]
+    engine.check_status()
+
+
+def test_command_line_runs_a_model_folder(capsys):
+    from pagedserve_b200.main import main
+
+    assert main(["--model", folder_of("c"), "--dtype", "bfloat16", "--max-new-tokens", "4", "--block-size", "8",
+                 "--num-blocks", "64", "--max-batch-size", "2", "--prompt-ids", "1 2 3 4 5"]) == 0
+    assert "request 0:" in capsys.readouterr().out
+    # a named size with random weights
+    assert main(["--model", "vozirax-tiny", "--seed", "3", "--dtype", "float32", "--max-new-tokens", "5",
+                 "--num-blocks", "32", "--max-batch-size", "2", "--prompt-ids", "7 8 9"]) == 0
+    assert "request 0:" in capsys.readouterr().out
+
+
+# ------------------------------------------------------------------ each part alone
+def make_ctx(engine, entries):
+    from pagedserve_b200.engine.batch import StepEntry
+
+    ctx = engine.runner.prepare([StepEntry(*entry) for entry in entries])
+    engine.runner.begin(ctx)
+    ctx.shared = {}
+    return ctx
+
+
+def layer_context(engine, index):
+    from pagedserve_b200.parts.base import LayerContext
+
+    entry = engine.spec.schedule[index]
+    layer = LayerContext(entry.layer, entry.cache_layer, engine.model.positions)
+    cache = engine.cache
+    group_index = cache.group_of_layer.get(entry.cache_layer)
+    if group_index is not None:
+        group = cache.groups[group_index]
+        layer.k_pool, layer.v_pool = group.layer_views(entry.cache_layer)
+        layer.page_stride, layer.page_size = group.page_stride, group.page_size
+        layer.pool, layer.pool_layer = group.pool, group.cache_layers.index(entry.cache_layer)
+        layer.block_table = cache.slots.table_views[group_index]
+    layer.state = cache.state.get(entry.cache_layer)
+    return engine.model.blocks[entry.layer], layer
+
+
+def run_in_portions(engine, index, fed, tokens, cuts, run, name="x", others=(), lender=None):
+    """``run(block, layer, rows, ctx) -> [T, W] results`` over ``fed`` in portions ``cuts`` (so that later ones start
+    from pages, state and kept rows).  ``others``: (name, token) of requests whose single tokens ride in the last
+    portion's step.  ``lender`` = (layer, rows): its mixer runs first in every portion and writes the keys and values that
+    layer ``index`` borrows."""
+    block, layer = layer_context(engine, index)
+    result = torch.zeros(fed.shape[0], fed.shape[1], dtype=torch.float32, device=DEV)
+    for number, (lo, hi) in enumerate(zip(cuts[:-1], cuts[1:])):
+        entries = [(name, tokens[lo:hi], [])]
+        rows = fed[lo:hi]
+        beside = others if number == len(cuts) - 2 else ()
+        if beside:
+            entries = [(other, [token], []) for other, token in beside] + entries
+            g = torch.Generator().manual_seed(number)
+            rows = torch.cat([torch.randn(len(beside), fed.shape[1], generator=g).to(fed.dtype), rows])
+        ctx = make_ctx(engine, entries)
+        if lender is not None:
+            other_block, other_layer = layer_context(engine, lender[0])
+            run_mixer(other_block, other_layer, lender[1][lo:hi].to(DEV).contiguous(), ctx)
+        result[lo:hi] = run(block, layer, rows.to(DEV).contiguous(), ctx)[len(beside):]
+        engine.cache.commit_many([entry[0] for entry in entries])
+    engine.cache.free(name)
+    return result
+
+
+def run_mixer(block, layer, rows, ctx):
+    """What the mixer adds, the factor of its layer included."""
+    out = torch.zeros(rows.shape, dtype=torch.float32, device=DEV)
+    block.mixer.forward(rows, out, ctx, layer)
+    return out
+
+
+def run_layer(block, layer, rows, ctx):
+    """The whole layer on residual rows."""
+    rows = rows.float().clone()
+    carrier = block.begin(rows, ctx)
+    block.forward(carrier, ctx, layer)
+    return block.end(carrier, ctx)
+
+
+def double_tensors(which):
+    folder_of(which)
+    return {name: t.double() for name, t in _TENSORS[which].items()}
+
+
+def plain_mixer(which, index, fed, lender_rows=None):
+    config, tensors = CONFIGS[which][0], double_tensors(which)
+    entry, p, eps = config["layers"][index], f"l{index}.", config["norm"]["eps"]
+    if entry["type"] == "mamba2":
+        return tensors[p + "ls1"] * plain.mamba(tensors, p + "mix.", entry["mixer"], fed, eps)
+    lender = entry["mixer"].get("kv_from")
+    source = index if lender is None else lender
+    kv = plain.keys_and_values(tensors, f"l{source}.mix.", config["layers"][source]["mixer"],
+                               fed if lender is None else lender_rows, eps)
+    return tensors[p + "ls1"] * plain.differential_attention(tensors, p + "mix.", entry["mixer"], fed,
+                                                             torch.arange(fed.shape[0]), eps, kv)
+
+
+def plain_feed_forward(which, index, fed, margins=None):
+    tensors, mlp, p = double_tensors(which), CONFIGS[which][0]["layers"][index]["mlp"], f"l{index}."
+    if mlp["kind"] == "dense":
+        return tensors[p + "ls2"] * plain.gated_ff(tensors, p + "mlp.", fed)
+    return tensors[p + "ls2"] * plain.routed_experts(tensors, p + "mlp.", mlp, fed, margins)
+
+
+@pytest.mark.parametrize("dtype,tol", [("float32", 1e-5), ("bfloat16", 2.5e-2)])
+@pytest.mark.parametrize("which", ["a", "b", "c", "d"])
+def test_each_part_alone(which, dtype, tol):
+    """Every mixer, every whole layer, the feed-forwards, the embedding and the head, each fed with the plain
+    implementation's own values.  Mixers and layers run a prompt in four portions (the last two of two tokens and one), so
+    the later ones start from pages, state and kept rows."""
+    engine = build_engine(which, dtype)
+    config, tensors = CONFIGS[which][0], _TENSORS[which]
+    eps, compute, width = config["norm"]["eps"], engine.dtype, config["width"]
+    count, cuts = 46, [0, 29, 43, 45, 46]
+    tokens = helpers.random_tokens(config["vocab"], count, seed=9)
+    g = torch.Generator().manual_seed(5)
+    stream = torch.randn(count, width, generator=g, dtype=torch.float64) * 2.0
+    t = lambda name: tensors[name].double()
+    for index, entry in enumerate(config["layers"]):
+        fed = (stream * 0.5).to(compute)
+        lender = entry["mixer"].get("kv_from")
+        lent = torch.randn(count, width, generator=g, dtype=torch.float64).to(compute) if lender is not None else None
+        lending = None if lender is None else (lender, lent)
+        got = run_in_portions(engine, index, fed, tokens, cuts, run_mixer, lender=lending)
+        want = plain_mixer(which, index, fed.double(), None if lent is None else lent.double())
+        assert rel_err(got, want) < tol, (which, index, entry["type"])
+        # the whole layer: mixer and feed-forward of the same rows
+        rows = stream.float()
+        got = run_in_portions(engine, index, rows, tokens, cuts, run_layer, lender=lending)
+        h = plain.centred_norm(rows.double(), t(f"l{index}.norm1"), eps)
+        want = rows.double() + plain_mixer(which, index, h, None if lent is None else lent.double())
+        clear = np.ones(count, dtype=bool)
+        if entry["mlp"] is not None:
+            margins = [float("inf")] * count
+            want = want + plain_feed_forward(which, index, plain.centred_norm(rows.double(), t(f"l{index}.norm2"), eps), margins)
+            clear = np.array(margins) > (1e-5 if dtype == "float32" else CLOSE_CALL)
+            assert clear.any()
+        assert rel_err(got.cpu()[clear], want[clear]) < tol, (which, index, "layer")
+        if entry["mlp"] is not None:
+            margins = [float("inf")] * count
+            want = plain_feed_forward(which, index, fed.double(), margins)
+            clear = np.array(margins) > 1e-3
+            residual = torch.zeros(count, width, dtype=torch.float32, device=DEV)
+            engine.model.blocks[index].feed_forward.forward(fed.to(DEV), residual, None)
+            assert rel_err(residual.cpu()[clear], want[clear]) < tol, (which, index, "feed-forward")
+    # the embedding with its sines, the model's norm on chosen rows, and the head times its constant
+    ctx = make_ctx(engine, [("z", tokens, [0, 7, 44])])
+    embedded = engine.model.embedding.forward(ctx, engine.model.positions)
+    assert rel_err(embedded, t("embed")[tokens] + plain.position_rows(torch.arange(count), width)) < 1e-6
+    picked = engine.model.final_norm.forward(stream.float().to(DEV), rows=ctx.logit_rows)
+    logits = engine.model.head.forward(picked, engine.model.embedding)
+    want = plain.centred_norm(stream, t("final.norm"), eps)[[0, 7, 44]] @ t("head").T * config["logit_scale"]
+    assert rel_err(logits, want) < tol
+    engine.cache.rollback("z")
+    engine.cache.free("z")
+    engine.check_status()
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("width", [64, 37, 1030])
+def test_sines_of_far_positions(width, dtype):
+    """Positions of tens of thousands: an angle rounded to one float would be off by thousandths of a radian."""
+    from pagedserve_b200.kernels.ops import Ops
+    from pagedserve_b200.parts.base import PartEnv
+    from pagedserve_b200.parts.positions import SinusoidalPositions
+
+    ops = Ops(dtype)
+    part = SinusoidalPositions(dict(hidden_size=width, base=10000.0), "", PartEnv(ops=ops, dtype=dtype, device=DEV))
+    g = torch.Generator().manual_seed(width)
+    table = torch.randn(11, width, generator=g).to(dtype)
+    positions = torch.tensor([0, 1, 2, 63, 1000, 4095, 32767, 65535, 99999], dtype=torch.int32)
+    ids = torch.randint(0, 11, (len(positions),), generator=g).to(torch.int32)
+    out = torch.empty(len(positions), width, device=DEV)
+    ops.embed_sinusoid(ids.to(DEV), positions.to(DEV), table.to(DEV), part.sinusoids(), out)
+    want = table.double()[ids.long()] + plain.position_rows(positions, width)
+    assert float((out.cpu().double() - want).abs().max()) < 2e-6
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
+    ids[3] = 11                                                      # not in the table: reported, the row is zeros
+    ops.embed_sinusoid(ids.to(DEV), positions.to(DEV), table.to(DEV), part.sinusoids(), out, status)
+    assert int(status.item()) == 1 and float(out[3].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows,width", [(1, 64), (37, 50), (300, 1024), (5, 2048), (3, 2052), (6, 37)])
+def test_two_norms_of_one_row(rows, width, dtype):
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    g = torch.Generator().manual_seed(width)
+    x = torch.randn(rows, width, generator=g) * 0.01                  # eps shows beside rows this small
+    gains = [1.0 + 0.3 * torch.randn(width, generator=g) for _ in range(2)]
+    outs = [torch.empty(rows, width, dtype=dtype, device=DEV) for _ in range(2)]
+    ops.rms_norm_pair(x.to(DEV), gains[0].to(DEV), gains[1].to(DEV), 1e-4, *outs)
+    for out, gain in zip(outs, gains):
+        assert rel_err(out, plain.unit_rms(x.double(), 1e-4) * gain.double()) < (2e-6 if dtype == torch.float32 else 5e-3)
+
+
+# ------------------------------------------------------------------ products with a factor per column
+@pytest.mark.parametrize("accumulate", [False, True])
+@pytest.mark.parametrize("rows,columns,depth", [(1, 64, 64), (8, 200, 136), (20, 4100, 64), (40, 3000, 1024), (64, 256, 320),
+                                                (130, 256, 512), (257, 100, 72), (70, 129, 40), (5, 37, 21)])
+def test_products_with_a_factor_per_column(rows, columns, depth, accumulate):
+    """Every product kernel (few rows, few rows of a large matrix, many rows, odd sizes) with a factor per column instead
+    of a bias, stored and added to float32 rows, in bfloat16 and float32."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    g = torch.Generator().manual_seed(rows + columns)
+    for dtype, tol in ((torch.float32, 3e-6), (torch.bfloat16, 3e-6)):
+        ops = Ops(dtype)
+        a = torch.randn(rows, depth, generator=g).to(dtype)
+        w = (torch.randn(columns, depth, generator=g) * depth ** -0.5).to(dtype)
+        factor, base = torch.randn(columns, generator=g), torch.randn(rows, columns, generator=g)
+        product = a.double() @ w.double().T * factor.double()
+        out = base.to(DEV)
+        ops.linear(a.to(DEV), w.to(DEV), None, out, accumulate=accumulate, factor=factor.to(DEV))
+        assert rel_err(out, product + base.double() if accumulate else product) < tol
+        if dtype == torch.bfloat16 and rows <= 64 and depth % 8 == 0:
+            for product_kernel in ("linear_skinny", "linear_rows_tc"):
+                out = base.to(DEV)
+                getattr(ops, product_kernel)(a.to(DEV), w.to(DEV), factor.to(DEV), out, accumulate=int(accumulate) | 2)
+                assert rel_err(out, product + base.double() if accumulate else product) < tol, product_kernel
+    assert int(ops.status_flag(DEV).item()) == 0
+
+
+@pytest.mark.parametrize("rows", [1, 7, 16, 30])
+def test_a_folded_norm_with_a_factor_per_column(rows):
+    from pagedserve_b200.kernels.ops import Ops
+    from pagedserve_b200.parts.norms import DeferredNorm, LayerNorm
+    from pagedserve_b200.parts.base import PartEnv
+
+    ops = Ops(torch.bfloat16)
+    g = torch.Generator().manual_seed(rows)
+    depth, columns = 264, 104
+    x, gain = torch.randn(rows, depth, generator=g), 1.0 + 0.2 * torch.randn(depth, generator=g)
+    w = (torch.randn(columns, depth, generator=g) * depth ** -0.5).to(torch.bfloat16)
+    factor, base = torch.randn(columns, generator=g), torch.randn(rows, columns, generator=g)
+    norm = LayerNorm(dict(width=depth, eps=1e-5, name="n", has_mean=False, has_bias=False), "", PartEnv(ops, torch.bfloat16, DEV))
+    norm.weight, norm.bias = gain.to(DEV), None
+    out = base.to(DEV)
+    deferred = DeferredNorm(norm, x.to(DEV))
+    assert ops._fused_norm_ok(deferred, w.to(DEV))
+    ops.linear(deferred, w.to(DEV), None, out, accumulate=True, factor=factor.to(DEV))
+    want = base.double() + (plain.unit_rms(x.double(), 1e-5) * gain.double()) @ w.double().T * factor.double()
+    assert rel_err(out, want) < 6e-3
+
+
+# ------------------------------------------------------------------ the recurrence alone
+def recurrence_case(heads, groups, N, P, lengths, seed, dtype, slow=False):
+    g = torch.Generator().manual_seed(seed)
+    total = sum(lengths)
+    gap = 3 if P % 8 else 0                                             # odd places in the rows
+    inner, shared = heads * P, groups * N
+    conv = torch.randn(total, gap + inner + 2 * shared + (-(inner + 2 * shared) % 8 if not gap else 2), generator=g).to(dtype)
+    raw = torch.randn(total, inner + heads + (-(inner + heads) % 8), generator=g).to(dtype)
+    offsets = (gap, gap + inner, gap + inner + shared, 0, inner)
+    a_log = (5.0 * torch.rand(heads, generator=g) - 4.0) - (4.0 if slow else 0.0)
+    dt_bias, d = torch.randn(heads, generator=g) - 1.0, torch.randn(heads, generator=g)
+    items = len(lengths)
+    state = torch.randn(items + 1, heads * N * P + 8, generator=g)
+    starts = np.concatenate([[0], np.cumsum(lengths)]).astype(np.int32)
+    slots = torch.randperm(items, generator=g).to(torch.int32)
+    x = conv[:, gap:gap + inner].double().reshape(total, heads, P)
+    b = conv[:, offsets[1]:offsets[1] + shared].double().reshape(total, groups, N).repeat_interleave(heads // groups, 1)
+    c = conv[:, offsets[2]:offsets[2] + shared].double().reshape(total, groups, N).repeat_interleave(heads // groups, 1)
+    z = raw[:, :inner].double().reshape(total, heads, P)
+    dt = plain.softplus(raw[:, inner:inner + heads].double() + dt_bias.double())
+    keep = torch.exp(-torch.exp(a_log.double()) * dt)
+    want = torch.empty(total, heads, P, dtype=torch.float64)
+    final = state.double().clone()
+    for item, (lo, hi) in enumerate(zip(starts[:-1], starts[1:])):
+        S = state[slots[item], :heads * N * P].double().reshape(heads, N, P)
+        for t in range(lo, hi):
+            S = keep[t][:, None, None] * S + (dt[t][:, None] * b[t])[:, :, None] * x[t][:, None, :]
+            want[t] = torch.einsum("hn,hnp->hp", c[t], S) + d.double()[:, None] * x[t]
+        final[slots[item], :heads * N * P] = S.reshape(-1)
+    want = (want * plain.silu(z)).reshape(total, inner)
+    short = sum(1 for n in lengths if n < 16)
+    ctx = SimpleNamespace(max_q_len=max(lengths), q_start=torch.from_numpy(starts).to(DEV), item_slot=slots.to(DEV),
+                          num_items=items, num_short_items=short, num_short_tokens=sum(n for n in lengths if n < 16),
+                          single_tokens=max(lengths) == 1)
+
+    def run(ops, segments=None, out_dtype=None):
+        kept = state.to(DEV)
+        out = torch.full((total, inner + 5), 7.0, dtype=out_dtype or dtype, device=DEV)
+        ops.ssd(conv.to(DEV), raw.to(DEV), offsets, a_log.to(DEV), dt_bias.to(DEV), d.to(DEV), kept, ctx, out[:, :inner], heads,
+                groups, N, P, segments=segments)
+        assert bool((out[:, inner:] == 7.0).all())
+        assert torch.equal(kept[:, heads * N * P:].cpu(), state[:, heads * N * P:])       # what lies behind S stays
+        return out[:, :inner], kept
+
+    return run, want, final
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("heads,groups,N,P,lengths", [
+    (3, 1, 16, 24, [1, 1, 1]), (4, 2, 64, 64, [1, 2, 15, 40, 200]), (2, 1, 128, 64, [3, 130, 64, 65]), (4, 4, 20, 36, [7, 17, 333]),
+    (2, 1, 40, 100, [100]), (1, 1, 96, 32, [1, 64, 65, 127]), (6, 3, 8, 128, [50, 31]), (2, 2, 144, 160, [1, 20]),
+    (5, 1, 10, 14, [16, 16, 150]), (2, 1, 128, 64, [1] * 5), (3, 3, 64, 128, [1, 1]), (4, 1, 10, 14, [1] * 4),
+    (2, 2, 32, 96, [1] * 3), (2, 1, 300, 72, [1, 1]), (1, 1, 500, 40, [3, 70]), (3, 1, 256, 256, [1, 1]), (2, 1, 16, 8, [16, 300]),
+    (2, 2, 128, 128, [18, 200]), (8, 2, 32, 32, [1, 500])])
+def test_the_recurrence_alone(heads, groups, N, P, lengths, dtype):
+    """Entries of unequal length (short ones first) from states that are not zero, in one piece and cut into runs that
+    are worked on side by side (also into more runs than the entry has chunks), equal the plain loop; the state that is
+    left is where a next step starts from."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    run, want, final = recurrence_case(heads, groups, N, P, lengths, seed=heads + N + P, dtype=dtype)
+    for segments in (1, 2, 5, 64, None):
+        out, kept = run(ops, segments)
+        assert rel_err(out, want) < (1e-5 if dtype == torch.float32 else 6e-3), segments
+        assert rel_err(kept, final) < 5e-6, segments
+    if dtype == torch.bfloat16:                                          # rows that go into a norm stay float32
+        out, _ = run(ops, None, torch.float32)
+        assert rel_err(out, want) < 2e-5
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_a_token_is_remembered_for_a_thousand(dtype):
+    """Decays near one: what a far token left in the state is still there, to float32, after a thousand others."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    run, want, final = recurrence_case(2, 1, 64, 64, [1100], seed=3, dtype=dtype, slow=True)
+    for segments in (1, 6):
+        out, kept = run(Ops(dtype), segments, torch.float32)
+        assert rel_err(out, want) < 2e-5 and rel_err(kept, final) < 1e-5
+
+
+def test_decays_at_both_ends():
+    """Step sizes of 1e-7 and 60 with rates that make decays of one and of zero: nothing overflows on the way."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    heads, N, P, total = 4, 16, 16, 150
+    g = torch.Generator().manual_seed(0)
+    a_log, dt_bias = torch.tensor([3.0, -3.0, 4.0, 0.0]), torch.tensor([60.0, -16.0, 2.0, -60.0])
+    for dtype in (torch.float32, torch.bfloat16):
+        conv, raw = torch.randn(total, heads * P + 2 * N, generator=g).to(dtype), torch.randn(total, heads * P + heads + 4, generator=g).to(dtype)
+        dt = plain.softplus(raw[:, heads * P:heads * P + heads].double() + dt_bias.double())
+        b, c = conv[:, heads * P:heads * P + N].double(), conv[:, heads * P + N:].double()
+        x = conv[:, :heads * P].double().reshape(total, heads, P)
+        want = plain.state_space(x, b[:, None], c[:, None], dt, a_log.double(), torch.ones(heads).double())
+        want = want.reshape(total, -1) * plain.silu(raw[:, :heads * P].double())
+        ctx = SimpleNamespace(max_q_len=total, q_start=torch.tensor([0, total], dtype=torch.int32, device=DEV),
+                              item_slot=torch.zeros(1, dtype=torch.int32, device=DEV), num_items=1, num_short_items=0,
+                              num_short_tokens=0)
+        for segments in (1, 2):
+            state = torch.zeros(1, heads * N * P, device=DEV)
+            out = torch.empty(total, heads * P, device=DEV)
+            Ops(dtype).ssd(conv.to(DEV), raw.to(DEV), (0, heads * P, heads * P + N, 0, heads * P), a_log.to(DEV), dt_bias.to(DEV),
+                           torch.ones(heads, device=DEV), state, ctx, out, heads, 1, N, P, segments=segments)
+            for h in range(heads):                                       # (heads differ in size by many orders)
+                cut = slice(h * P, (h + 1) * P)
+                assert rel_err(out[:, cut], want[:, cut]) < 3e-5, (h, dtype)
+
+
+# ------------------------------------------------------------------ the convolution with bias and silu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("channels", [40, 37])
+@pytest.mark.parametrize("taps,lengths", [(1, [5, 1]), (2, [1, 1, 9]), (3, [2, 1, 40, 1]), (4, [1, 2, 3, 200]), (4, [1, 1, 1]),
+                                          (7, [3, 3, 1])])
+def test_the_convolution_with_bias_and_silu(taps, lengths, channels, dtype):
+    """Rows of the compute type, entries shorter and longer than the convolution, four steps in a row: each starts from the
+    rows that the one before kept."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    g = torch.Generator().manual_seed(taps)
+    weight, bias = torch.randn(channels, taps, generator=g), torch.randn(channels, generator=g)
+    items = len(lengths)
+    slots = torch.randperm(items, generator=g).to(torch.int32)
+    state = torch.zeros(items + 1, (taps - 1) * channels + 12, device=DEV)
+    kept = state[:, :(taps - 1) * channels] if taps > 1 else None        # a share of a longer row
+    history = [torch.zeros(0, channels, dtype=torch.float64) for _ in lengths]
+    for step in range(4):
+        counts = [1] * items if step == 2 else lengths if step % 2 == 0 else lengths[::-1]
+        starts = np.concatenate([[0], np.cumsum(counts)]).astype(np.int32)
+        wide = torch.randn(int(starts[-1]), channels + 8, generator=g).to(dtype)      # rows inside wider rows
+        u = wide[:, 4:4 + channels]
+        token_item = torch.repeat_interleave(torch.arange(items), torch.tensor(counts)).to(torch.int32)
+        want = torch.empty(u.shape, dtype=torch.float64)
+        for item, (lo, hi) in enumerate(zip(starts[:-1], starts[1:])):
+            before = history[item].shape[0]
+            history[item] = torch.cat([history[item], u[lo:hi].double()])
+            want[lo:hi] = plain.silu(plain.causal_convolution(history[item], weight.double(), bias.double()))[before:]
+        ctx = SimpleNamespace(token_item=token_item.to(DEV), q_start=torch.from_numpy(starts).to(DEV),
+                              item_slot=slots.to(DEV), num_items=items, single_tokens=max(counts) == 1)
+        out = torch.empty(u.shape, dtype=dtype, device=DEV)
+        ops.short_conv(wide.to(DEV)[:, 4:4 + channels], weight.to(DEV), taps, channels, kept, ctx, out, bias=bias.to(DEV), act="silu")
+        assert rel_err(out, want) < (3e-6 if dtype == torch.float32 else 5e-3), (taps, step)
+    assert float(state[:, (taps - 1) * channels:].abs().max()) == 0.0
+
+
+# ------------------------------------------------------------------ experts
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("experts,top,groups", [(8, 2, (2, 1)), (6, 3, (3, 2)), (12, 4, (4, 4)), (5, 5, None), (64, 6, (8, 3)),
+                                                (3, 1, (3, 1)), (256, 8, (8, 4)), (4, 2, (1, 1))])
+def test_the_election_by_groups(experts, top, groups, dtype):
+    """Corrections that turn elections and make most choice scores negative: closed groups stay closed, groups are marked by
+    their two largest corrected scores, the weights are the plain scores over their sum, times the constant."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    compute = torch.float32 if dtype == "float32" else torch.bfloat16
+    ops = Ops(compute)
+    g = torch.Generator().manual_seed(experts * 10 + top)
+    tokens, width = 200, 48
+    x = torch.randn(tokens, width, generator=g).to(compute)
+    router = (2.0 * torch.randn(experts, width, generator=g) / width ** 0.5).to(compute)
+    correction = 0.5 * torch.randn(experts, generator=g) - 0.8
+    rule = {"experts": experts, "top": top, "scale": 2.5}
+    if groups:
+        rule["groups"] = {"count": groups[0], "keep": groups[1]}
+    dense = torch.empty(tokens, experts, dtype=torch.float32, device=DEV)
+    got = torch.empty(tokens, top, dtype=torch.int32, device=DEV)
+    got_w = torch.empty(tokens, top, dtype=torch.float32, device=DEV)
+    count, keep = groups or (0, 0)
+    ops.moe_route(x.to(DEV), router.to(DEV), None, dense, got, got_w, None, top, count, keep, score="sigmoid", normalize=True,
+                  correction=correction.to(DEV), group_mark="two_largest", scale=2.5)
+    scores = torch.sigmoid(x.double() @ router.double().T)
+    checked = other = 0
+    for t in range(tokens):
+        weights, margin = plain.election(scores[t], correction.double(), rule)
+        if margin < 1e-4:
+            continue
+        checked += 1
+        assert sorted(got[t].tolist()) == sorted(weights)
+        for e, w in zip(got[t].tolist(), got_w[t].tolist()):
+            assert abs(w - float(weights[e])) < 1e-5 * 2.5
+        other += set(torch.topk(scores[t], top).indices.tolist()) != set(weights)
+    assert checked > tokens * 0.8 and (other > 0 or top == experts)
+    picked = torch.zeros(tokens, experts).scatter_(1, got.cpu().long(), got_w.cpu())
+    assert torch.equal(picked, dense.cpu())
+
+
+@pytest.mark.parametrize("dtype,tol", [("float32", 1e-5), ("bfloat16", 2.5e-2)])
+@pytest.mark.parametrize("which,count", [("a", 300), ("b", 130), ("m", 200), ("d", 160)])
+def test_experts_with_many_tokens(which, count, dtype, tol):
+    """Steps of many tokens sort their rows by expert (bfloat16): the same sums as token by token.  Tokens whose election
+    is a close call are left out: the two sides may elect differently there."""
+    engine = build_engine(which, dtype, max_model_len=1024)
+    config = CONFIGS[which][0]
+    g = torch.Generator().manual_seed(count)
+    fed = torch.randn(count, config["width"], generator=g, dtype=torch.float64).to(engine.dtype)
+    for index, entry in enumerate(config["layers"]):
+        if entry["mlp"] is None or entry["mlp"]["kind"] != "moe":
+            continue
+        margins = [float("inf")] * count
+        want = plain_feed_forward(which, index, fed.double(), margins)
+        clear = np.array(margins) > 1e-3
+        residual = torch.zeros(count, config["width"], dtype=torch.float32, device=DEV)
+        engine.model.blocks[index].feed_forward.forward(fed.to(DEV), residual, None)
+        assert rel_err(residual.cpu()[clear], want[clear]) < tol, (which, index)
+    engine.check_status()
+
+
+# ------------------------------------------------------------------ what comes before and behind the attention kernels
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,slot", [(4, 2, 16, 32, 32), (6, 3, 12, 20, 32), (2, 1, 64, 128, 128), (3, 3, 7, 9, 16),
+                                                          (2, 2, 24, 80, 80), (5, 1, 40, 16, 80), (2, 1, 136, 290, 304)])
+def test_two_maps_before_and_behind_attention(heads, kv_heads, dim, vdim, slot, dtype):
+    """Queries, pages and the combined rows against the equations: maps in their halves with zeros beside them, the
+    temperature on both sides of its steps, a layer that brings queries only, gates and none."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    g = torch.Generator().manual_seed(heads * dim)
+    page, positions = 16, [0, 5, 6, 7, 13, 14, 31, 32, 100]
+    count = len(positions)
+    q_width, k_width, v_width = 2 * heads * dim, 2 * kv_heads * dim, kv_heads * vdim
+    pad = lambda n: n + (-n) % 8
+    k_offset, v_offset = pad(q_width), pad(q_width) + pad(k_width)
+    row = torch.randn(count, v_offset + pad(v_width), generator=g).to(dtype)
+    gains = [1.3 + 0.2 * torch.randn(dim, generator=g) for _ in range(2)]
+    pool = torch.full((10, 1, 2, kv_heads, page, slot), 5.0, dtype=dtype, device=DEV)
+    table = torch.randperm(10, generator=g).to(torch.int32)[None]
+    layer = SimpleNamespace(k_pool=pool[:, 0, 0], v_pool=pool[:, 0, 1], page_stride=pool.stride(0), page_size=page,
+                            block_table=table.to(DEV))
+    place = torch.tensor(positions, dtype=torch.int32, device=DEV)
+    ctx = SimpleNamespace(token_slot=torch.zeros(count, dtype=torch.int32, device=DEV), positions=place)
+    eps, temp = 1e-2, (0.3, 7)
+    q = plain.unit_rms(row[:, :q_width].double().reshape(count, heads, 2, dim), eps) * gains[0].double()
+    q = q * plain.temperature(torch.tensor(positions), {"coef": 0.3, "every": 7})[:, None, None, None]
+    k = plain.unit_rms(row[:, k_offset:k_offset + k_width].double().reshape(count, kv_heads, 2, dim), eps) * gains[1].double()
+    v = row[:, v_offset:v_offset + v_width].double().reshape(count, kv_heads, vdim)
+    want_q = torch.zeros(count, heads, 2, slot, dtype=torch.float64)
+    want_k, want_v = torch.zeros(count, kv_heads, slot).double(), torch.zeros(count, kv_heads, slot).double()
+    for i in (0, 1):
+        want_q[:, :, i, i * dim:(i + 1) * dim] = q[:, :, i]
+        want_k[:, :, i * dim:(i + 1) * dim] = k[:, :, i]
+    want_v[:, :, :vdim] = v
+    tol = 2e-6 if dtype == torch.float32 else 5e-3
+    for has_kv in (True, False):
+        out = torch.full((count, 2 * heads * slot), 9.0, dtype=dtype, device=DEV)
+        before = pool.clone()
+        ops.diff_prepare(row.to(DEV), k_offset, v_offset, gains[0].to(DEV), gains[1].to(DEV) if has_kv else None, eps, temp, ctx,
+                         layer, out, heads, kv_heads, dim, vdim, slot, has_kv=has_kv)
+        assert rel_err(out, want_q.reshape(count, -1)) < tol
+        if has_kv:
+            pages, inside = table[0, torch.tensor(positions) // page].long(), torch.tensor(positions) % page
+            assert rel_err(pool[pages, 0, 0, :, inside], want_k) < tol and rel_err(pool[pages, 0, 1, :, inside], want_v) < tol
+            assert int((pool == 5.0).sum()) == pool.numel() - count * 2 * kv_heads * slot     # nothing else was written
+        else:
+            assert torch.equal(before, pool)
+    maps = torch.randn(count, 2 * heads * slot, generator=g).to(dtype)
+    wide = torch.randn(count, heads + 3, generator=g).to(dtype)
+    a = maps.double().reshape(count, heads, 2, slot)[..., :vdim]
+    for gate in (wide[:, 2:2 + heads], None):
+        want = plain.unit_rms(a[:, :, 0] - 0.8 * a[:, :, 1], eps) * 0.6
+        if gate is not None:
+            want = want * torch.sigmoid(gate.double())[:, :, None]
+        out = torch.full((count, heads * vdim + 8), 9.0, dtype=dtype, device=DEV)
+        ops.diff_combine(maps.to(DEV), wide.to(DEV)[:, 2:2 + heads] if gate is not None else None, out[:, :heads * vdim], 0.8, eps, 0.6,
+                         heads, vdim, slot)
+        assert rel_err(out[:, :heads * vdim], want.reshape(count, -1)) < tol and bool((out[:, heads * vdim:] == 9.0).all())
+
+
+# ------------------------------------------------------------------ a key that stands out, at page borders and far back
+def standing_out(index, which_map, key_at, query_at, count, seed):
+    """Rows for the mixer of layer ``index`` such that one map of query head 0 at ``query_at`` points straight along that
+    map's key of key head 0 at ``key_at``.  The norms remove the query's size, so the rows are solved for its direction
+    only; steep scales and large query gains make the key decide."""
+    config, tensors = CONFIGS["s"][0], double_tensors("s")
+    m, eps, d = config["layers"][index]["mixer"], config["norm"]["eps"], config["layers"][index]["mixer"]["dim"]
+    g = torch.Generator().manual_seed(seed)
+    rows = torch.randn(count, config["width"], generator=g, dtype=torch.float64)
+    keys, _ = plain.keys_and_values(tensors, f"l{index}.mix.", m, rows, eps)
+    wanted = 4.0 * keys[key_at, 0, which_map] / tensors[f"l{index}.mix.q.norm"]
+    matrix = tensors[f"l{index}.mix.q"].reshape(m["heads"], 2, d, -1)[0, which_map]
+    rows[query_at] = torch.linalg.lstsq(matrix, wanted[:, None], driver="gelsd").solution[:, 0]
+    return rows
+
+
+@pytest.mark.parametrize("dtype,tol", [("float32", 2e-5), ("bfloat16", 3e-2)])
+@pytest.mark.parametrize("index", [0, 1, 2, 3])
+def test_a_key_that_stands_out_at_page_borders_and_far_back(index, dtype, tol):
+    """One map of one query made to point at one key: at the sequence's first token, at the token before, on both sides of
+    page and tile borders and hundreds of tokens back; in a prompt in one step, in two portions cut between the two tokens,
+    with the query decoded alone, and decoded among single tokens of other requests."""
+    from pagedserve_b200.engine.batch import StepEntry
+
+    engine = build_engine("s", dtype)
+    config = CONFIGS["s"][0]
+    count = 300
+    tokens = helpers.random_tokens(config["vocab"], count, seed=2)
+    for other in ("p", "q", "r"):                        # three other requests hold pages of their own
+        engine.step([StepEntry(other, helpers.random_tokens(config["vocab"], 20, seed=ord(other)), [])])
+    pairs = ((299, 0), (299, 3), (150, 1), (255, 16), (256, 255), (272, 271), (17, 15), (128, 127))
+    for number, (query_at, key_at) in enumerate(pairs):
+        fed = standing_out(index, number % 2, key_at, query_at, count, seed=query_at + key_at).to(engine.dtype)
+        want = plain_mixer("s", index, fed.double())
+        # the key decides the row: with another key in its place the plain result is another one altogether
+        changed = fed.double().clone()
+        changed[key_at] = torch.randn(config["width"], generator=torch.Generator().manual_seed(number)).double()
+        moved = plain_mixer("s", index, changed)[query_at]
+        assert float((moved - want[query_at]).abs().max()) > 0.05 * float(want[query_at].abs().max())
+        alone = [0, query_at, query_at + 1, count] if query_at + 1 < count else [0, query_at, count]
+        for cuts, others in (([0, count], ()), ([0, key_at + 1, count], ()), (alone, ()),
+                             (alone[:-1] if len(alone) == 4 else alone, (("p", 1), ("q", 2), ("r", 3)))):
+            got = run_in_portions(engine, index, fed[:cuts[-1]], tokens, cuts, run_mixer, others=others)
+            assert rel_err(got[query_at], want[query_at]) < tol, (index, query_at, key_at, cuts)
+            assert rel_err(got, want[:cuts[-1]]) < tol, (index, query_at, key_at, cuts)
+    engine.check_status()
+
+
+def test_each_mechanism_of_the_attention_shows():
+    """The second map, the temperature, the gate, the borrowed keys: the plain layer without one of them differs from the
+    engine's by far more than the tolerance."""
+    engine = build_engine("a", "float32")
+    config, eps = CONFIGS["a"][0], CONFIGS["a"][0]["norm"]["eps"]
+    g = torch.Generator().manual_seed(1)
+    count, index = 60, 2
+    fed, lent = (torch.randn(count, config["width"], generator=g) for _ in range(2))
+    tokens = helpers.random_tokens(config["vocab"], count, seed=3)
+    got = run_in_portions(engine, index, fed, tokens, [0, 40, count], run_mixer, lender=(1, lent))
+    assert rel_err(got, plain_mixer("a", index, fed.double(), lent.double())) < 1e-5
+    tensors, m = double_tensors("a"), dict(config["layers"][index]["mixer"])
+
+    def without(change=None, **values):
+        own, mine = dict(tensors), dict(m, **values)
+        if change:
+            change(own)
+        kv = plain.keys_and_values(own, "l1.mix.", config["layers"][1]["mixer"], lent.double(), eps)
+        return own["l2.ls1"] * plain.differential_attention(own, "l2.mix.", mine, fed.double(), torch.arange(count), eps, kv)
+
+    assert rel_err(got, without()) < 1e-5
+    assert rel_err(got, without(q_temp=None)) > 0.02
+    assert rel_err(got, without(lambda own: own.update({"l2.mix.g": torch.zeros_like(own["l2.mix.g"])}))) > 0.05
+    assert rel_err(got, without(lambda own: own.update({"l2.mix.lq1": torch.zeros_like(own["l2.mix.lq1"])}))) > 0.02
+    assert rel_err(got, plain_mixer("a", index, fed.double(), fed.double())) > 0.05
