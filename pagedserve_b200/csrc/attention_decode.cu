@@ -384,7 +384,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
     if (n_splits == 1 || n_active == 1) {
         const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
         for (int d = tid_all; d < head_dim; d += THREADS)
-            out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o_s[d] * inv);
+            store_result(out, (size_t)t * out_stride + column * head_dim + d, o_s[d] * inv, extras);
         return;
     }
     if (by_cluster) {
@@ -424,9 +424,9 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             }
             // the others' shared memory has been read: they may leave while the result is written
             asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-            if (tid_all < head_dim) out[(size_t)t * out_stride + column * head_dim + tid_all] = __float2bfloat16_rn(o * inv);
+            if (tid_all < head_dim) store_result(out, (size_t)t * out_stride + column * head_dim + tid_all, o * inv, extras);
             if (tid_all + THREADS < head_dim)
-                out[(size_t)t * out_stride + column * head_dim + tid_all + THREADS] = __float2bfloat16_rn(more * inv);
+                store_result(out, (size_t)t * out_stride + column * head_dim + tid_all + THREADS, more * inv, extras);
             asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
             return;
         }
@@ -487,7 +487,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
                 if (i < n_active)
                     o += (round == 0 ? held[i] : ldcg_f32(part_acc + (base + i) * head_dim + d)) * mh[i];
             }
-            out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o * inv);
+            store_result(out, (size_t)t * out_stride + column * head_dim + d, o * inv, extras);
         }
         return;
     }
@@ -522,7 +522,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
             } else {
                 for (int i = 0; i < n_active; ++i) o += ldcg_f32(part_acc + (base + i) * head_dim + d) * w_s[i];
             }
-            out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o * inv);
+            store_result(out, (size_t)t * out_stride + column * head_dim + d, o * inv, extras);
         }
         return;
     }
@@ -536,7 +536,7 @@ paged_attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride,
         float o = 0.f;
         for (int i = 0; i < n_active; ++i)
             o += ldcg_f32(part_acc + (base + i) * head_dim + d) * exp2f(ldcg_f32(part_ml + (base + i) * 2) - M);
-        out[(size_t)t * out_stride + column * head_dim + d] = __float2bfloat16_rn(o * inv);
+        store_result(out, (size_t)t * out_stride + column * head_dim + d, o * inv, extras);
     }
 }
 
@@ -559,8 +559,8 @@ static int launch_attention_decode(const void* q, int q_stride, void* out, int o
                                    int split_tiles, int n_splits, float* part_acc, float* part_ml, int* counters,
                                    int* status, void* stream, const int* q_start = nullptr,
                                    const int* kv_len = nullptr, int cluster = 1, const int* token_row = nullptr,
-                                   float softcap = 0.f, const float* sink = nullptr, int all_values = 0) {
-    const ps::SoftmaxExtras extras = ps::softmax_extras(scale, softcap, sink);
+                                   float softcap = 0.f, const float* sink = nullptr, int all_values = 0, int wide = 0) {
+    const ps::SoftmaxExtras extras = ps::softmax_extras(scale, softcap, sink, wide);
     if (T <= 0) return PS_OK;
     if ((q_start == nullptr) != (kv_len == nullptr)) return PS_ERR_BAD_ARGUMENT;
     if (cluster > 1 && (cluster != n_splits || cluster > 8 || (cluster & (cluster - 1)))) return PS_ERR_BAD_ARGUMENT;
@@ -664,7 +664,7 @@ PS_EXPORT int ps_paged_attention_decode_checked(const void* q, int q_stride, voi
 // instead of by item. softcap > 0: scores become softcap * tanh(score / softcap); sink (may be null): one
 // float per query head whose exponential joins the softmax's denominator.  all_values: every query head meets the
 // values of every key/value head; result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out, and the
-// scratch arrays are sized for n_heads * n_kv_heads heads.
+// scratch arrays are sized for n_heads * n_kv_heads heads.  wide: out is float32.
 PS_EXPORT int ps_paged_attention_decode_ex(const void* q, int q_stride, void* out, int out_stride,
                                            const void* k_pool, const void* v_pool, long long page_stride,
                                            const int* token_item, const int* token_row, const int* positions,
@@ -673,11 +673,11 @@ PS_EXPORT int ps_paged_attention_decode_ex(const void* q, int q_stride, void* ou
                                            int n_heads, int n_kv_heads, int head_dim, int page_size, int window,
                                            float scale, int split_tiles, int n_splits, int cluster,
                                            float* part_acc, float* part_ml, int* counters, int* status,
-                                           float softcap, const float* sink, int all_values, void* stream) {
+                                           float softcap, const float* sink, int all_values, int wide, void* stream) {
     return launch_attention_decode(q, q_stride, out, out_stride, k_pool, v_pool, page_stride, token_item, positions,
                                    block_table, bt_stride, T, n_heads, n_kv_heads, head_dim, page_size, window, scale,
                                    split_tiles, n_splits, part_acc, part_ml, counters, status, stream, q_start, kv_len,
-                                   cluster < 1 ? 1 : cluster, token_row, softcap, sink, all_values);
+                                   cluster < 1 ? 1 : cluster, token_row, softcap, sink, all_values, wide);
 }
 
 // ------------------------------------------------------------------------------------------------

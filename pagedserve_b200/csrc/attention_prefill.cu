@@ -317,11 +317,9 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
     for (int dn = 0; dn < HD / 8; ++dn) {
         const int d = dn * 8 + tq * 2;
         if (row0 < rows)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + row0) * out_stride + column * HD + d) =
-                pack_bf16(o[dn][0] * inv0, o[dn][1] * inv0);
+            store_result2(out, (size_t)(tok0 + row0) * out_stride + column * HD + d, o[dn][0] * inv0, o[dn][1] * inv0, extras);
         if (row1 < rows)
-            *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + row1) * out_stride + column * HD + d) =
-                pack_bf16(o[dn][2] * inv1, o[dn][3] * inv1);
+            store_result2(out, (size_t)(tok0 + row1) * out_stride + column * HD + d, o[dn][2] * inv1, o[dn][3] * inv1, extras);
     }
 }
 
@@ -355,7 +353,7 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
            const int* item_row, int first_item, int n_items, int max_blocks, int n_heads, int n_kv_heads,
            int page_size, int window, float scale, float softcap, const float* sink, cudaStream_t stream,
            const int* row_positions = nullptr, int rows_per_item = 0, float* partial = nullptr, int key_splits = 1,
-           int all_values = 0) {
+           int all_values = 0, int wide = 0) {
     constexpr int RS = HD + 8;
     size_t smem = (size_t)(BQ + 8 * BKEY) * RS * 2;
     auto kernel = prefill_attention_kernel<HD>;
@@ -376,7 +374,7 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
     return launch_pdl(kernel, dim3(max_blocks, all_values ? n_heads * n_kv_heads : n_heads), dim3(THREADS), smem, stream, (const __nv_bfloat16*)q, q_stride,
                       (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool,
                       page_stride, q_start, kv_len, block_table, bt_stride, item_row, first_item, n_items, n_heads,
-                      n_kv_heads, page_size, window, scale * 1.4426950408889634f, softmax_extras(scale, softcap, sink),
+                      n_kv_heads, page_size, window, scale * 1.4426950408889634f, softmax_extras(scale, softcap, sink, wide),
                       row_positions, rows_per_item, (float*)nullptr, 1, all_values);
 }
 
@@ -389,14 +387,14 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
 // item_row (may be null): the block-table row of each item, where the table is kept by request slot.
 // softcap > 0: scores become softcap * tanh(score / softcap); sink (may be null): one float per query head whose
 // exponential joins the softmax's denominator.  all_values: every query head meets the values of every key/value head;
-// result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out.
+// result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out.  wide: out is float32.
 PS_EXPORT int ps_prefill_attention(const void* q, int q_stride, void* out, int out_stride, const void* k_pool,
                                    const void* v_pool, long long page_stride, const int* q_start, const int* kv_len,
                                    const int* block_table, int bt_stride, const int* item_row, int first_item,
                                    int n_items,
                                    int max_blocks, int n_heads, int n_kv_heads, int head_dim, int page_size,
                                    int window, float scale, float softcap, const float* sink, int all_values,
-                                   void* stream) {
+                                   int wide, void* stream) {
     if (n_items <= 0 || max_blocks <= 0) return PS_OK;
     if (n_heads <= 0 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0 ||
         (long long)n_heads * (all_values ? n_kv_heads : 1) > 65535) return PS_ERR_BAD_ARGUMENT;
@@ -410,7 +408,8 @@ PS_EXPORT int ps_prefill_attention(const void* q, int q_stride, void* out, int o
     case D:                                                                                                        \
         return ps::pf::launch<D>(q, q_stride, out, out_stride, k_pool, v_pool, page_stride, q_start, kv_len,       \
                                  block_table, bt_stride, item_row, first_item, n_items, max_blocks, n_heads,       \
-                                 n_kv_heads, page_size, window, scale, softcap, sink, s, nullptr, 0, nullptr, 1, all_values);
+                                 n_kv_heads, page_size, window, scale, softcap, sink, s, nullptr, 0, nullptr, 1, all_values,  \
+                                 wide);
     switch (head_dim) {
         PS_PF_CASE(16) PS_PF_CASE(32) PS_PF_CASE(48) PS_PF_CASE(64)
         PS_PF_CASE(80) PS_PF_CASE(96) PS_PF_CASE(112) PS_PF_CASE(128)

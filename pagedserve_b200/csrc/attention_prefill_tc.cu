@@ -481,7 +481,14 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 uint32_t orr[32];
                 tmem_ld32(lane_base + L::O_COL + half * OCOLS + c, orr);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                if (r < rows) {
+                if (r < rows && extras.wide) {
+                    float* wide = reinterpret_cast<float*>(out) + (size_t)(tok0 + r) * out_stride + column * HD + half * OCOLS + c;
+#pragma unroll
+                    for (int d = 0; d < 32; d += 4)
+                        *reinterpret_cast<float4*>(wide + d) =
+                            make_float4(__uint_as_float(orr[d]) * inv, __uint_as_float(orr[d + 1]) * inv,
+                                        __uint_as_float(orr[d + 2]) * inv, __uint_as_float(orr[d + 3]) * inv);
+                } else if (r < rows) {
 #pragma unroll
                     for (int d = 0; d < 32; d += 8) {
                         uint4 pack;
@@ -540,7 +547,7 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
            long long k_row_base, long long v_row_base, long long page_rows, const int* q_start, const int* kv_len,
            const int* block_table, int bt_stride, const int* item_row, int first_item, int n_items, int max_blocks,
            int n_heads, int n_kv_heads, int page_size, int window, float scale, int* status, float softcap,
-           const float* sink, int all_values, cudaStream_t stream) {
+           const float* sink, int all_values, int wide, cudaStream_t stream) {
     CUtensorMap map_q, map_kv;
     if (!make_map(&map_q, q, T, n_heads * HD, q_stride, BQ)) return PS_ERR_LAUNCH;
     if (!make_map(&map_kv, pool, pool_rows, HD, HD, page_size)) return PS_ERR_LAUNCH;
@@ -552,7 +559,7 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
     return launch_pdl(kernel, dim3(all_values ? n_heads * n_kv_heads : n_heads, max_blocks), dim3(L::THREADS), L::SMEM, stream, map_q, map_kv,
                       (__nv_bfloat16*)out, out_stride, q_start, kv_len, block_table, bt_stride, item_row, first_item,
                       n_items, n_heads, n_kv_heads, page_size, window, scale * 1.4426950408889634f, k_row_base,
-                      v_row_base, page_rows, status, softmax_extras(scale, softcap, sink), all_values);
+                      v_row_base, page_rows, status, softmax_extras(scale, softcap, sink, wide), all_values);
 }
 
 }  // namespace pftc
@@ -566,7 +573,7 @@ int launch(const void* q, int q_stride, int T, void* out, int out_stride, const 
 // item_row (may be null): the block-table row of each item, where the table is kept by request slot.
 // softcap > 0: scores become softcap * tanh(score / softcap); sink (may be null): one float per query head whose
 // exponential joins the softmax's denominator.  all_values: every query head meets the values of every key/value head;
-// result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out.
+// result (h, g') stands at column (h * n_kv_heads + g') * head_dim of out.  wide: out is float32.
 PS_EXPORT int ps_prefill_attention_tc(const void* q, int q_stride, int T, void* out, int out_stride, const void* pool,
                                       long long pool_rows, long long k_row_base, long long v_row_base,
                                       long long page_rows, const int* q_start, const int* kv_len,
@@ -574,7 +581,7 @@ PS_EXPORT int ps_prefill_attention_tc(const void* q, int q_stride, int T, void* 
                                       int n_items,
                                       int max_blocks, int n_heads, int n_kv_heads, int head_dim, int page_size,
                                       int window, float scale, int row_threads, int* status, float softcap,
-                                      const float* sink, int all_values, void* stream) {
+                                      const float* sink, int all_values, int wide, void* stream) {
     if (n_items <= 0 || max_blocks <= 0) return PS_OK;
     if (row_threads < 0 || row_threads > 2) return PS_ERR_BAD_ARGUMENT;
     if (!status) return PS_ERR_BAD_ARGUMENT;
@@ -594,7 +601,7 @@ PS_EXPORT int ps_prefill_attention_tc(const void* q, int q_stride, int T, void* 
     return ps::pftc::launch<HD, SPLIT>(q, q_stride, T, out, out_stride, pool, pool_rows, k_row_base, v_row_base,     \
                                        page_rows, q_start, kv_len, block_table, bt_stride, item_row, first_item,      \
                                        n_items, max_blocks, n_heads, n_kv_heads, page_size, window, scale, status,    \
-                                       softcap, sink, all_values, s)
+                                       softcap, sink, all_values, wide, s)
     if (head_dim == 64) {
         if (two) PS_PFTC_LAUNCH(64, 2);
         PS_PFTC_LAUNCH(64, 1);

@@ -302,10 +302,7 @@ attention_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bf
         if (mixed) {
             *reinterpret_cast<float4*>(final_rows + r * WIDE + d) = total;
         } else {
-            uint2 packed;
-            packed.x = pack(total.x, total.y);
-            packed.y = pack(total.z, total.w);
-            *reinterpret_cast<uint2*>(out + (size_t)t * out_stride + (head0 + r) * D + d) = packed;
+            store_result4(out, (size_t)t * out_stride + (head0 + r) * D + d, total, extras);
         }
     }
     __syncthreads();
@@ -323,10 +320,7 @@ attention_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_bf
                 total.x = fmaf(weight, v.x, total.x); total.y = fmaf(weight, v.y, total.y);
                 total.z = fmaf(weight, v.z, total.z); total.w = fmaf(weight, v.w, total.w);
             }
-            uint2 packed;
-            packed.x = pack(total.x, total.y);
-            packed.y = pack(total.z, total.w);
-            *reinterpret_cast<uint2*>(out + (size_t)t * out_stride + h * D + d) = packed;
+            store_result4(out, (size_t)t * out_stride + h * D + d, total, extras);
         }
     }
     // nobody's shared memory goes away before it was read
@@ -338,7 +332,7 @@ template <int D, int NG>
 int launch(const void* q, int q_stride, void* out, int out_stride, const void* k_pool, const void* v_pool, long long page_stride,
            const int* token_item, const int* token_row, const int* positions, const int* block_table, int bt_stride,
            const int* q_start, const int* kv_len, int T, int n_heads, int n_kv_heads, int page_size, int window, float scale,
-           int splits, float softcap, const float* sink, const float* mix, cudaStream_t s) {
+           int splits, float softcap, const float* sink, const float* mix, int wide, cudaStream_t s) {
     auto kernel = attention_rows_kernel<D, NG>;
     static size_t raised[MAX_DEVICES] = {0};
     if (!ensure_dynamic_smem((const void*)kernel, Layout<D, NG>::BYTES, raised)) return PS_ERR_LAUNCH;
@@ -346,7 +340,7 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
                               (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pool,
                               (const __nv_bfloat16*)v_pool, page_stride, token_item, token_row, positions, block_table,
                               bt_stride, q_start, kv_len, n_heads, n_kv_heads, page_size, window,
-                              scale * 1.4426950408889634f, softmax_extras(scale, softcap, sink), mix);
+                              scale * 1.4426950408889634f, softmax_extras(scale, softcap, sink, wide), mix);
 }
 
 }  // namespace rows
@@ -356,12 +350,13 @@ int launch(const void* q, int q_stride, void* out, int out_stride, const void* k
 // in block-table row token_row[t] (null: token_item[t]); out likewise.  mix null: plain attention, groups of at most 16 heads.
 // mix float32 [n_heads][n_heads]: the heads' weights are mixed by it; at most 16 heads, and n_kv_heads rounded up to a power
 // of two times head_dim at most 256.  Head sizes: multiples of 16 up to 128.  splits: 1, 2, 4 or 8 CTAs share a token's keys.
-// q_start / kv_len (per item, both or neither): which keys are older than this step.  softcap, sink: see common.cuh.
+// q_start / kv_len (per item, both or neither): which keys are older than this step.  softcap, sink, wide (out is
+// float32): see common.cuh.
 PS_EXPORT int ps_attention_rows(const void* q, int q_stride, void* out, int out_stride, const void* k_pool, const void* v_pool,
                                 long long page_stride, const int* token_item, const int* token_row, const int* positions,
                                 const int* block_table, int bt_stride, const int* q_start, const int* kv_len, int T,
                                 int n_heads, int n_kv_heads, int head_dim, int page_size, int window, float scale, int splits,
-                                float softcap, const float* sink, const float* mix, void* stream) {
+                                float softcap, const float* sink, const float* mix, int wide, void* stream) {
     if (T <= 0) return PS_OK;
     if (!q || !out || !k_pool || !v_pool || !token_item || !positions || !block_table) return PS_ERR_BAD_ARGUMENT;
     if ((q_start == nullptr) != (kv_len == nullptr)) return PS_ERR_BAD_ARGUMENT;
@@ -371,14 +366,14 @@ PS_EXPORT int ps_attention_rows(const void* q, int q_stride, void* out, int out_
     if (page_size <= 0 || page_size > 64 || (page_size & (page_size - 1))) return PS_ERR_UNSUPPORTED;
     if ((mix ? n_heads : n_heads / n_kv_heads) > ps::rows::M) return PS_ERR_UNSUPPORTED;
     if (q_stride % 8 != 0 || out_stride % 4 != 0 || page_stride % 8 != 0) return PS_ERR_UNSUPPORTED;
-    if (((uintptr_t)q & 15) || ((uintptr_t)out & 7) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15))
+    if (((uintptr_t)q & 15) || ((uintptr_t)out & (wide ? 15 : 7)) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15))
         return PS_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const int ng = mix ? n_kv_heads : 1;
 #define PS_ROWS(D, NG)                                                                                                 \
     return ps::rows::launch<D, NG>(q, q_stride, out, out_stride, k_pool, v_pool, page_stride, token_item, token_row,    \
                                    positions, block_table, bt_stride, q_start, kv_len, T, n_heads, n_kv_heads, page_size, \
-                                   window, scale, splits, softcap, sink, mix, s)
+                                   window, scale, splits, softcap, sink, mix, wide, s)
 #define PS_ROWS_2(D)                \
     case D:                         \
         if (ng <= 1) PS_ROWS(D, 1); \

@@ -108,7 +108,7 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
                             const int* __restrict__ token_item, const int* __restrict__ positions,
                             const int* __restrict__ block_table, int bt_stride,
                             int n_heads, int n_kv_heads, int head_dim, int page_size, int window, float scale,
-                            float softcap, const float* __restrict__ sink, int all_values) {
+                            float softcap, const float* __restrict__ sink, int all_values, int wide_out) {
     extern __shared__ float smem[];
     float* q_s = smem;                                   // [head_dim]
     float* acc_s = smem + head_dim;                      // [ATT_WARPS][head_dim]
@@ -196,7 +196,9 @@ paged_attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < ATT_WARPS; ++w) o += acc_s[w * head_dim + d] * wgt[w];
-        out[(size_t)t * out_stride + column * head_dim + d] = from_float<T>(o * inv);
+        const size_t at = (size_t)t * out_stride + column * head_dim + d;
+        if (wide_out) reinterpret_cast<float*>(out)[at] = o * inv;
+        else out[at] = from_float<T>(o * inv);
     }
 }
 
@@ -227,12 +229,13 @@ PS_EXPORT int ps_kv_append(const void* k_src, const void* v_src, int src_stride,
     return PS_ERR_UNSUPPORTED;
 }
 
+// wide_out: out is float32.
 PS_EXPORT int ps_paged_attention_simt(const void* q, int q_stride, void* out, int out_stride,
                                       const void* k_pool, const void* v_pool, long long page_stride,
                                       const int* token_item, const int* positions, const int* block_table,
                                       int bt_stride, int T, int n_heads, int n_kv_heads, int head_dim,
                                       int page_size, int window, float scale, float softcap, const float* sink,
-                                      int all_values, int dtype, void* stream) {
+                                      int all_values, int wide_out, int dtype, void* stream) {
     if (T <= 0) return PS_OK;
     int rc = check_attention_sizes(n_heads, n_kv_heads, head_dim, page_size);
     if (rc) return rc;
@@ -248,7 +251,7 @@ PS_EXPORT int ps_paged_attention_simt(const void* q, int q_stride, void* out, in
         return ps::launch_pdl(kernel, grid, dim3(ps::ATT_WARPS * 32), smem, s,
                               (const float*)q, q_stride, (float*)out, out_stride, (const float*)k_pool,
                               (const float*)v_pool, page_stride, token_item, positions, block_table, bt_stride,
-                              n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap, sink, all_values);
+                              n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap, sink, all_values, wide_out);
     }
     if (dtype == PS_BF16) {
         auto kernel = wide ? ps::paged_attention_simt_kernel<__nv_bfloat16, ps::ATT_MAX_HD / 32>
@@ -257,7 +260,7 @@ PS_EXPORT int ps_paged_attention_simt(const void* q, int q_stride, void* out, in
                               (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride,
                               (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, page_stride, token_item,
                               positions, block_table, bt_stride, n_heads, n_kv_heads, head_dim, page_size, window,
-                              scale, softcap, sink, all_values);
+                              scale, softcap, sink, all_values, wide_out);
     }
     return PS_ERR_UNSUPPORTED;
 }

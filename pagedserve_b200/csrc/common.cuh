@@ -138,17 +138,41 @@ __device__ __forceinline__ unsigned long long pair_fma(unsigned long long a, uns
 //   sink:         one float per query head (natural units) whose exponential joins the denominator. A kernel
 //                 gives it to exactly one of the partial softmax states of a row as that state's start:
 //                 (max, sum) = (sink * log2 e, 1) instead of (-inf, 0), which is a key without a value.
+//   wide:         the result is stored as float32 (`out` is then an array of floats with the same strides in elements),
+//                 for layers that go on calculating with it.
 struct SoftmaxExtras {
     float cap_log2;
     float scale_over_cap;
     const float* sink;
+    int wide;
 };
-__host__ __device__ inline SoftmaxExtras softmax_extras(float scale, float softcap, const float* sink) {
+__host__ __device__ inline SoftmaxExtras softmax_extras(float scale, float softcap, const float* sink, int wide = 0) {
     SoftmaxExtras e;
+    e.wide = wide;
     e.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     e.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
     e.sink = sink;
     return e;
+}
+// one number of an attention result, and two or four neighbouring ones (aligned to their size)
+__device__ __forceinline__ void store_result(__nv_bfloat16* out, size_t at, float v, const SoftmaxExtras& x) {
+    if (x.wide) reinterpret_cast<float*>(out)[at] = v;
+    else out[at] = __float2bfloat16_rn(v);
+}
+__device__ __forceinline__ void store_result2(__nv_bfloat16* out, size_t at, float a, float b, const SoftmaxExtras& x) {
+    if (x.wide) *reinterpret_cast<float2*>(reinterpret_cast<float*>(out) + at) = make_float2(a, b);
+    else *reinterpret_cast<__nv_bfloat162*>(out + at) = __floats2bfloat162_rn(a, b);
+}
+__device__ __forceinline__ void store_result4(__nv_bfloat16* out, size_t at, const float4& v, const SoftmaxExtras& x) {
+    if (x.wide) {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + at) = v;
+    } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+        uint2 packed;
+        packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+        packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(out + at) = packed;
+    }
 }
 // tanh from one ex2 and one reciprocal: 1 - 2 / (1 + e^(2x)); absolute error about 1e-7, exact at both ends
 __device__ __forceinline__ float tanh_ex2(float x) {

@@ -139,9 +139,20 @@ diff_prepare_kernel(const T* __restrict__ row, long long row_stride, int k_offse
     }
 }
 
+// V neighbouring numbers of a map's result: of the output's type, or float32
 template <typename T, int V>
+__device__ __forceinline__ void diff_fetch(const T* p, float (&x)[V]) {
+    if constexpr (V == 8 && sizeof(T) == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+    } else {
+        diff_unpack(*reinterpret_cast<const typename DiffPack<T, V>::type*>(p), x);
+    }
+}
+
+template <typename TM, typename T, int V>
 __global__ void __launch_bounds__(DIFF_WARPS * 32)
-diff_combine_kernel(const T* __restrict__ maps, long long maps_stride, const T* __restrict__ gate, long long gate_stride,
+diff_combine_kernel(const TM* __restrict__ maps, long long maps_stride, const T* __restrict__ gate, long long gate_stride,
                     T* __restrict__ out, long long out_stride, float share, float eps, float scale, int rows, int n_heads,
                     int vdim, int slot, int lanes) {
     using P = typename DiffPack<T, V>::type;
@@ -157,14 +168,14 @@ diff_combine_kernel(const T* __restrict__ maps, long long maps_stride, const T* 
         const long long unit = base + group;
         const bool here = unit < total;
         const int t = here ? (int)(unit / n_heads) : 0, h = here ? (int)(unit - (long long)t * n_heads) : 0;
-        const T* a1 = maps + (size_t)t * maps_stride + (size_t)(2 * h) * slot;
-        const T* a2 = a1 + slot;
+        const TM* a1 = maps + (size_t)t * maps_stride + (size_t)(2 * h) * slot;
+        const TM* a2 = a1 + slot;
         float sq = 0.f, held[V];                             // the first V numbers of a lane stay in registers
         if (here) {
             for (int d = V * gl; d < vdim; d += V * lanes) {
                 float x[V], y[V];
-                diff_unpack(*reinterpret_cast<const P*>(a1 + d), x);
-                diff_unpack(*reinterpret_cast<const P*>(a2 + d), y);
+                diff_fetch(a1 + d, x);
+                diff_fetch(a2 + d, y);
 #pragma unroll
                 for (int e = 0; e < V; ++e) {
                     x[e] = fmaf(-share, y[e], x[e]);
@@ -185,8 +196,8 @@ diff_combine_kernel(const T* __restrict__ maps, long long maps_stride, const T* 
                 for (int e = 0; e < V; ++e) x[e] = held[e];
             } else {
                 float y[V];
-                diff_unpack(*reinterpret_cast<const P*>(a1 + d), x);
-                diff_unpack(*reinterpret_cast<const P*>(a2 + d), y);
+                diff_fetch(a1 + d, x);
+                diff_fetch(a2 + d, y);
 #pragma unroll
                 for (int e = 0; e < V; ++e) x[e] = fmaf(-share, y[e], x[e]);
             }
@@ -221,14 +232,14 @@ int launch_diff_prepare(const void* row, long long row_stride, int k_offset, int
                       vdim, slot, has_kv, lanes);
 }
 
-template <typename T, int V>
+template <typename TM, typename T, int V>
 int launch_diff_combine(const void* maps, long long maps_stride, const void* gate, long long gate_stride, void* out,
                         long long out_stride, float share, float eps, float scale, int rows, int n_heads, int vdim, int slot,
                         cudaStream_t s) {
     const int lanes = diff_lanes(vdim, V), per_cta = DIFF_WARPS * (32 / lanes);
     const long long ctas = ((long long)rows * n_heads + per_cta - 1) / per_cta;
-    return launch_pdl(diff_combine_kernel<T, V>, dim3((unsigned)(ctas < 148 * 16 ? ctas : 148 * 16)), dim3(DIFF_WARPS * 32), 0, s,
-                      (const T*)maps, maps_stride, (const T*)gate, gate_stride, (T*)out, out_stride, share, eps, scale, rows,
+    return launch_pdl(diff_combine_kernel<TM, T, V>, dim3((unsigned)(ctas < 148 * 16 ? ctas : 148 * 16)), dim3(DIFF_WARPS * 32), 0, s,
+                      (const TM*)maps, maps_stride, (const T*)gate, gate_stride, (T*)out, out_stride, share, eps, scale, rows,
                       n_heads, vdim, slot, lanes);
 }
 
@@ -268,26 +279,31 @@ PS_EXPORT int ps_diff_prepare(const void* row, long long row_stride, int k_offse
     return PS_ERR_UNSUPPORTED;
 }
 
-// maps [T][2 * n_heads * slot], gate [T][n_heads] or null, out [T][n_heads * vdim], all of `dtype`
+// maps [T][2 * n_heads * slot] of maps_dtype (`dtype` or float32), gate [T][n_heads] or null, out [T][n_heads * vdim] of `dtype`
 PS_EXPORT int ps_diff_combine(const void* maps, long long maps_stride, const void* gate, long long gate_stride, void* out,
                               long long out_stride, float share, float eps, float scale, int T, int n_heads, int vdim,
-                              int slot, int dtype, void* stream) {
+                              int slot, int maps_dtype, int dtype, void* stream) {
     if (T <= 0) return PS_OK;
     if (!maps || !out || n_heads <= 0 || vdim <= 0 || slot < vdim) return PS_ERR_BAD_ARGUMENT;
     cudaStream_t s = (cudaStream_t)stream;
     const int V = dtype == PS_F32 ? 4 : 8;
     const bool wide = vdim % V == 0 && slot % V == 0 && maps_stride % V == 0 && out_stride % V == 0 &&
                       !(((uintptr_t)maps | (uintptr_t)out) & 15);
-#define PS_DIFF_COMBINE(TYPE, V)                                                                                        \
-    return ps::launch_diff_combine<TYPE, V>(maps, maps_stride, gate, gate_stride, out, out_stride, share, eps, scale, T, \
-                                            n_heads, vdim, slot, s)
-    if (dtype == PS_F32) {
-        if (wide) PS_DIFF_COMBINE(float, 4);
-        PS_DIFF_COMBINE(float, 1);
+#define PS_DIFF_COMBINE(MAPS, TYPE, V)                                                                                  \
+    return ps::launch_diff_combine<MAPS, TYPE, V>(maps, maps_stride, gate, gate_stride, out, out_stride, share, eps, scale, T, \
+                                                  n_heads, vdim, slot, s)
+    using bf = __nv_bfloat16;
+    if (dtype == PS_F32 && maps_dtype == PS_F32) {
+        if (wide) PS_DIFF_COMBINE(float, float, 4);
+        PS_DIFF_COMBINE(float, float, 1);
     }
-    if (dtype == PS_BF16) {
-        if (wide) PS_DIFF_COMBINE(__nv_bfloat16, 8);
-        PS_DIFF_COMBINE(__nv_bfloat16, 1);
+    if (dtype == PS_BF16 && maps_dtype == PS_F32) {
+        if (wide) PS_DIFF_COMBINE(float, bf, 8);
+        PS_DIFF_COMBINE(float, bf, 1);
+    }
+    if (dtype == PS_BF16 && maps_dtype == PS_BF16) {
+        if (wide) PS_DIFF_COMBINE(bf, bf, 8);
+        PS_DIFF_COMBINE(bf, bf, 1);
     }
 #undef PS_DIFF_COMBINE
     return PS_ERR_UNSUPPORTED;

@@ -36,7 +36,7 @@ __global__ void embed_kernel(const int* __restrict__ ids, const int* __restrict_
 
 // h[t] = wte[id_t] + sinusoids of the position: number 2i is sin(p f_i), number 2i + 1 is cos(p f_i).  The angle is formed to
 // more than one float: f_i comes as (high, low) parts, the product's rounding error is recovered with an fma, and what the
-// float that sincosf takes cannot hold is applied to first order.
+// float that sincosf takes cannot hold is applied to second order.
 template <typename T>
 __global__ void embed_sinusoid_kernel(const int* __restrict__ ids, const int* __restrict__ pos, const T* __restrict__ wte,
                                       const float2* __restrict__ freq, float* __restrict__ out, int H, int V,
@@ -56,8 +56,9 @@ __global__ void embed_sinusoid_kernel(const int* __restrict__ ids, const int* __
         const float high = p * f.x, low = fmaf(p, f.x, -high) + p * f.y;
         float sn, cs;
         sincosf(high, &sn, &cs);
-        out[(size_t)t * H + c] = bad ? 0.f : a + fmaf(low, cs, sn);
-        if (c + 1 < H) out[(size_t)t * H + c + 1] = bad ? 0.f : b + fmaf(-low, sn, cs);
+        const float half = 0.5f * low * low;                 // sin(high + low), cos(high + low) to second order
+        out[(size_t)t * H + c] = bad ? 0.f : a + fmaf(low, cs, fmaf(-half, sn, sn));
+        if (c + 1 < H) out[(size_t)t * H + c + 1] = bad ? 0.f : b + fmaf(-low, sn, fmaf(-half, cs, cs));
     }
 }
 

@@ -79,7 +79,7 @@ _SIGNATURES = {
         "ps_gemm_simt": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "ps_kv_append": [_P, _P, _I, _P, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I, _P],
         "ps_paged_attention_simt": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P,
-                                    _I, _I, _P],
+                                    _I, _I, _I, _P],
         "ps_rotary_cache_write": [_P, _I, _P, _I, _P, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _I,
                                   _I, _P],
         "ps_token_shift_mix": [_P, _I, _P, _I, _P, _L, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P],
@@ -111,7 +111,7 @@ _SIGNATURES = {
                    _P],
         "ps_diff_prepare": [_P, _L, _I, _I, _P, _P, _F, _F, _I, _P, _P, _P, _I, _P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _I,
                             _I, _I, _I, _P],
-        "ps_diff_combine": [_P, _L, _P, _L, _P, _L, _F, _F, _F, _I, _I, _I, _I, _I, _P],
+        "ps_diff_combine": [_P, _L, _P, _L, _P, _L, _F, _F, _F, _I, _I, _I, _I, _I, _I, _P],
         "ps_head_mix": [_P, _L, _P, _P, _L, _I, _I, _I, _I, _I, _P],
         "ps_moe_plan": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P],
         "ps_moe_gather": [_P, _I, _P, _P, _I, _I, _I, _I, _P],
@@ -134,12 +134,12 @@ _SIGNATURES = {
         "ps_paged_attention_decode_checked": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
                                               _F, _I, _I, _P, _P, _P, _P, _P],
         "ps_paged_attention_decode_ex": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I,
-                                         _I, _I, _F, _I, _I, _I, _P, _P, _P, _P, _F, _P, _I, _P],
+                                         _I, _I, _F, _I, _I, _I, _P, _P, _P, _P, _F, _P, _I, _I, _P],
         "ps_shared_position_attention": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P],
         "ps_attention_rows": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P,
-                              _P, _P],
+                              _P, _I, _P],
         "ps_prefill_attention": [_P, _I, _P, _I, _P, _P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F,
-                                 _F, _P, _I, _P],
+                                 _F, _P, _I, _I, _P],
     },
     "tc": {
         "ps_gemm_tc": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
@@ -149,7 +149,7 @@ _SIGNATURES = {
         "ps_gemm_tc_experts": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P],
         "ps_gemm_tc_qkv": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "ps_prefill_attention_tc": [_P, _I, _I, _P, _I, _P, _L, _L, _L, _L, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I,
-                                    _I, _I, _F, _I, _P, _F, _P, _I, _P],
+                                    _I, _I, _F, _I, _P, _F, _P, _I, _I, _P],
     },
 }
 
@@ -663,6 +663,14 @@ class Ops:
                                       n_kv_heads, head_dim, page_size,
                                       self.code, _stream()), "kv_append")
 
+    @staticmethod
+    def _wide(out):
+        """Whether a bfloat16 attention kernel leaves its result as float32: where ``out`` is."""
+        _require(out, "out")
+        if out.dtype not in (torch.bfloat16, torch.float32):
+            raise KernelError("attention: out is bfloat16 or float32")
+        return 1 if out.dtype == torch.float32 else 0
+
     def paged_attention_simt(self, q, out, k_pool, v_pool, page_stride, token_item, positions, block_table,
                              n_heads, n_kv_heads, head_dim, page_size, window, scale, softcap=None, sink=None, all_values=False):
         """out[t, h] = softmax(q[t,h] . K[<=pos]) V over the request's pages; CUDA cores.  ``softcap``:
@@ -675,7 +683,7 @@ class Ops:
                 raise KernelError("attention: one sink per query head")
         T = q.shape[0]
         _require(q, "q", self.dtype)
-        _require(out, "out", self.dtype)
+        _require(out, "out", out.dtype if out.dtype == torch.float32 else self.dtype)
         if q.stride(1) != 1 or out.stride(1) != 1:
             raise KernelError("attention: innermost stride must be 1")
         self.launches += 1
@@ -683,8 +691,8 @@ class Ops:
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_pool), _ptr(v_pool),
             page_stride, _ptr(token_item), _ptr(positions), _ptr(block_table),
             block_table.stride(0), T, n_heads, n_kv_heads, head_dim,
-            page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), 1 if all_values else 0, self.code, _stream()),
-            "paged_attention_simt")
+            page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), 1 if all_values else 0,
+            1 if out.dtype == torch.float32 and self.dtype != torch.float32 else 0, self.code, _stream()), "paged_attention_simt")
         return out
 
     @staticmethod
@@ -736,7 +744,6 @@ class Ops:
         :meth:`paged_attention_simt`."""
         T = q.shape[0]
         _require(q, "q", torch.bfloat16)
-        _require(out, "out", torch.bfloat16)
         columns = n_heads * n_kv_heads if all_values else n_heads          # results per token
         plan = None
         if merge == "cluster":
@@ -763,7 +770,7 @@ class Ops:
             block_table.stride(0), _ptr(q_start), _ptr(kv_len), T, n_heads, n_kv_heads, head_dim,
             page_size, window or 0, scale, split_tiles, n_splits, cluster,
             _ptr(part_acc), _ptr(part_ml), _ptr(counters), _ptr(status), float(softcap or 0.0), _ptr(sink),
-            1 if all_values else 0, _stream()), "paged_attention_decode")
+            1 if all_values else 0, self._wide(out), _stream()), "paged_attention_decode")
         return out
 
     def prefill_attention(self, q, out, k_pool, v_pool, page_stride, q_start, kv_len, block_table, first_item,
@@ -774,7 +781,6 @@ class Ops:
         token arrays (row 0 = token 0).  ``item_row``: the block-table row of each item (a table kept by request
         slot); without it item i uses row i."""
         _require(q, "q", torch.bfloat16)
-        _require(out, "out", torch.bfloat16)
         if head_dim > 128:
             raise KernelError("prefill_attention: head sizes above 128 are not supported")
         self.launches += 1
@@ -783,7 +789,7 @@ class Ops:
             page_stride, _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), _ptr(item_row),
             first_item, n_items, max_blocks, n_heads, n_kv_heads,
             head_dim, page_size, window or 0, scale, float(softcap or 0.0), _ptr(sink), 1 if all_values else 0,
-            _stream()), "prefill_attention")
+            self._wide(out), _stream()), "prefill_attention")
         return out
 
     def shared_position_attention(self, q, out, k_pool, v_pool, page_stride, positions, block_table, token_row,
@@ -851,7 +857,6 @@ class Ops:
         heads' weights are mixed by it before they meet the values.  Otherwise as :meth:`paged_attention_decode`."""
         T = q.shape[0]
         _require(q, "q", torch.bfloat16)
-        _require(out, "out", torch.bfloat16)
         if q.shape[1] != n_heads * head_dim or out.shape != q.shape or q.stride(1) != 1 or out.stride(1) != 1:
             raise KernelError("attention_rows: q and out must be rows of n_heads * head_dim")
         for name, vector, count in (("sink", sink, n_heads), ("mix", mix, n_heads * n_heads)):
@@ -866,7 +871,7 @@ class Ops:
             _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_pool), _ptr(v_pool), page_stride, _ptr(token_item),
             _ptr(token_row), _ptr(positions), _ptr(block_table), block_table.stride(0), _ptr(q_start), _ptr(kv_len), T, n_heads,
             n_kv_heads, head_dim, page_size, window or 0, scale, splits, float(softcap or 0.0), _ptr(sink), _ptr(mix),
-            _stream()), "attention_rows")
+            self._wide(out), _stream()), "attention_rows")
         return out
 
     @staticmethod
@@ -882,7 +887,6 @@ class Ops:
         layer's index inside it; ``max_blocks`` >= the number of 128-query blocks of the items.
         ``row_threads``: 1 or 2 threads per query row (0: the kernel's launcher decides)."""
         _require(q, "q", torch.bfloat16)
-        _require(out, "out", torch.bfloat16)
         if self._tc is None:
             self._tc = _declare(_load_library("tc"), "tc")
         if status is None:
@@ -897,18 +901,20 @@ class Ops:
             (cache_layer_local * planes + planes - 1) * rows_per_tensor, page_rows,
             _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), _ptr(item_row), first_item,
             n_items, max_blocks, n_heads, n_kv_heads, head_dim, page_size, window or 0, scale, row_threads,
-            _ptr(status), float(softcap or 0.0), _ptr(sink), 1 if all_values else 0, _stream()),
-            "prefill_attention_tc")
+            _ptr(status), float(softcap or 0.0), _ptr(sink), 1 if all_values else 0, self._wide(out),
+            _stream()), "prefill_attention_tc")
         return out
 
     def attention(self, q, k, v, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, scale,
                   write_cache=True, softcap=None, sink=None, chunk=None, mix=None):
         """Write the step's keys and values into the pages, then attend from the pages.  ``softcap`` and ``sink`` as in
         :meth:`paged_attention_simt`; ``mix`` float32 [n_heads, n_heads]: the heads' weights are mixed by it before they
-        meet the values (:meth:`head_mix`).  Besides "no later key", a query sees the last ``window``
+        meet the values (:meth:`head_mix`).  ``out`` may be float32 in a bfloat16 engine (not with ``mix``).  Besides "no later key", a query sees the last ``window``
         keys, or (``chunk`` C instead of a window) the keys j of its own run of C positions,
         ``j // C == i // C``, runs counted from position 0 of the sequence; neither: every earlier key.  Below
         this method the two travel as one integer: the window, or minus the chunk."""
+        if mix is not None and out.dtype != self.dtype:
+            raise KernelError("attention: mixed heads leave rows of the compute type")
         if chunk:
             if window:
                 raise KernelError("attention: a window or a chunked mask, not both")
@@ -1463,10 +1469,11 @@ class Ops:
 
     def diff_combine(self, maps, gate, out, share, eps, scale, n_heads, vdim, slot):
         """Per head o = a1 - share * a2 of the two maps' results in ``maps`` [T, 2 * n_heads * slot]; ``out``
-        [T, n_heads * vdim] = o / sqrt(mean(o^2) + eps) * scale * sigmoid(gate), ``gate`` [T, n_heads] or None."""
+        [T, n_heads * vdim] = o / sqrt(mean(o^2) + eps) * scale * sigmoid(gate), ``gate`` [T, n_heads] or None.  ``maps`` of
+        the compute dtype or float32."""
         T = maps.shape[0]
-        for name, tensor in (("maps", maps), ("out", out)):
-            _require(tensor, name, self.dtype)
+        _require(maps, "maps", maps.dtype if maps.dtype in (self.dtype, torch.float32) else self.dtype)
+        _require(out, "out", self.dtype)
         if gate is not None:
             _require(gate, "gate", self.dtype)
             if gate.shape != (T, n_heads) or gate.stride(1) != 1:
@@ -1477,7 +1484,7 @@ class Ops:
         self.launches += 1
         _check(self.core.ps_diff_combine(_ptr(maps), maps.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0,
                                          _ptr(out), out.stride(0), float(share), float(eps), float(scale), T, n_heads, vdim,
-                                         slot, self.code, _stream()), "diff_combine")
+                                         slot, dtype_code(maps.dtype), self.code, _stream()), "diff_combine")
         return out
 
     # ------------------------------------------------------------------ minGRU

@@ -75,7 +75,8 @@ def attention(ops, q, out, ctx, layer, n_heads, n_kv_heads, head_dim, window, sc
             every = ops.empty((ctx.num_tokens, columns * head_dim), out.dtype, out.device)
     all_values = mix is not None
     if short_tokens >= SHARED_POSITION_FROM and n_kv_heads == 1 and n_heads >= 4 and head_dim <= 128 \
-            and softcap is None and sink is None and mix is None and q.is_contiguous() and out.is_contiguous():
+            and softcap is None and sink is None and mix is None and q.is_contiguous() and out.is_contiguous() \
+            and out.dtype == q.dtype:
         # Every query head reads the one key/value head: the heads of a token become the query rows of one
         # tile of the prompt kernel, all at the token's position, and the token's keys are fetched once instead
         # of once per head; with few tokens the key tiles of a token are shared out over up to 8 CTAs and merged

@@ -101,7 +101,8 @@ class DifferentialAttention(Mixer):
         queries = ops.empty((tokens, 2 * H * D), dtype, device)
         ops.diff_prepare(row, self.k_offset, self.v_offset, self.q_gain, self.k_gain, float(p["eps"]), self.q_temp, ctx, layer,
                          queries, H, G, p["head_dim"], p["v_dim"], D, has_kv=self.kv_source)
-        maps = ops.empty((tokens, 2 * H * D), dtype, device)
+        # (the two maps' results stay float32: their difference may be much smaller than they are)
+        maps = ops.empty((tokens, 2 * H * D), torch.float32, device)
         ops.attention(queries, None, None, maps, ctx, layer, 2 * H, G, D, None, float(p["scale"]), write_cache=False)
         context = ops.empty((tokens, H * p["v_dim"]), dtype, device)
         ops.diff_combine(maps, row[:, self.gate_offset:self.gate_offset + H], context, self.share, float(p["eps"]),
