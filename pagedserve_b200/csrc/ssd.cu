@@ -10,9 +10,15 @@
 //
 // ssd_step_kernel: steps in which every entry brings one token (decode).  One CTA per (entry, head); S goes through registers,
 //                  four columns an access, the first rows on their way before the wait for the kernel that makes the token's row.
-// ssd_scan_kernel: everything else, on CUDA cores, any size.  One CTA per (entry, head, 32 columns, run of tokens): a lane is a
-//                  column, a warp holds N / 8 rows of S in registers, two rows to a packed pair; tokens come in chunks of
-//                  SSD_CHUNK through shared memory, the sums over the warps are formed for a whole chunk at once.
+// ssd_scan_kernel: everything else, float32 arithmetic on CUDA cores, any size.  One CTA per (entry, head, tile of columns, run
+//                  of tokens): a lane holds one or two columns, a warp N / 8 rows of S in registers, two rows to a packed pair.
+//                  Tokens come in chunks of 16, the next chunk's rows on their way in registers while one is worked on.  With
+//                  S the state ahead of a chunk and L_t the sum of the chunk's -exp(A_h) d up to and including token t,
+//                      y_t = exp(L_t) C_t S + sum over s <= t of exp(L_t - L_s) d_s (C_t . B_s) x_s,
+//                      S  <- exp(L_end) S + sum over s of exp(L_end - L_s) d_s B_s x_s^T,
+//                  so that a state element takes one multiply-add per token for the result and one for the update.  (Exponents
+//                  are never positive: nothing overflows however fast a head forgets.)  The 16 x 16 products C_t . B_s come
+//                  from mma.sync where B and C are bfloat16 (exact products, float32 sums).
 // The recurrence is linear in S, so the entries from `first_cut` on (prompt portions) are cut into `segments` runs of tokens that
 // are worked on side by side: a first launch (STATE_ONLY) leaves every run's own contribution to S (started from zero) and the
 // product of its decays in scratch, ssd_fold_kernel folds them in order into the S that every run starts from, the second
@@ -32,34 +38,67 @@ struct SsdInputs {
 
 __device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
-constexpr int SSD_THREADS = 256, SSD_WARPS = 8, SSD_CHUNK = 16, SSD_COLS = 32;
+constexpr int SSD_THREADS = 256, SSD_WARPS = 8, SSD_CHUNK = 16;
 
 // how an entry of `count` tokens is cut into runs of whole chunks
 __host__ __device__ __forceinline__ int ssd_run_length(int count, int segments, int chunk) {
     return ((count + segments - 1) / segments + chunk - 1) / chunk * chunk;
 }
 
-// R: rows of S of a warp (N <= 8 R)
-template <typename T, typename TO, int R, bool STATE_ONLY>
-__global__ void __launch_bounds__(SSD_THREADS)
-ssd_scan_kernel(const T* __restrict__ conv, const T* __restrict__ raw, const SsdInputs in, float* __restrict__ state,
+// elements of one 16-byte access, as floats
+__device__ __forceinline__ void ssd_unpack(const uint4& raw, float (&x)[4]) {
+    x[0] = __uint_as_float(raw.x); x[1] = __uint_as_float(raw.y); x[2] = __uint_as_float(raw.z); x[3] = __uint_as_float(raw.w);
+}
+__device__ __forceinline__ void ssd_unpack(const uint4& raw, float (&x)[8]) {
+    const __nv_bfloat162* pair = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(pair[i]);
+        x[2 * i] = f.x;
+        x[2 * i + 1] = f.y;
+    }
+}
+
+// R: rows of S of a warp (N <= 8 R); CPL: columns of a lane
+template <typename T, int R, int CPL>
+struct SsdLayout {
+    static constexpr int CH = SSD_CHUNK, NP = SSD_WARPS * R, COLS = 32 * CPL, ROW = NP + 4;      // ROW: padded against bank conflicts
+    static constexpr int VEC = 16 / (int)sizeof(T);
+    static constexpr int up(int a, int b) { return (a + b - 1) / b; }
+    static constexpr int N_PIECES = up(CH * NP / VEC, SSD_THREADS), P_PIECES = up(CH * COLS / VEC, SSD_THREADS);
+    // floats: B, C (padded rows), x, z, the warps' sums, the chunk's weights W; then B and C as they came (bfloat16 only)
+    static constexpr int B = 0, C = CH * ROW, X = 2 * CH * ROW, Z = X + CH * COLS, Y = Z + CH * COLS, W = Y + SSD_WARPS * CH * COLS,
+                         TYPED = W + CH * (CH + 4);
+    static constexpr int TROW = NP + 8;                          // a row of the typed tiles, in elements
+    static constexpr size_t BYTES = (size_t)TYPED * 4 + (sizeof(T) == 2 ? (size_t)2 * CH * TROW * 2 : 0);
+};
+
+template <typename T, typename TO, int R, int CPL, bool STATE_ONLY>
+__global__ void __launch_bounds__(SSD_THREADS, R * CPL <= 32 ? 2 : 1)
+ssd_scan_kernel(const T* __restrict__ conv, const T* __restrict__ raw, const SsdInputs in, int wide, float* __restrict__ state,
                 long long state_stride, const int* __restrict__ q_start, const int* __restrict__ item_slot, int first_item,
-                int last_item, int first_cut, int segments, int chunk_unit, float* __restrict__ run_state,
-                float* __restrict__ run_decay, TO* __restrict__ out, long long out_stride) {
-    constexpr int NP = SSD_WARPS * R, CH = SSD_CHUNK;
+                int last_item, int first_cut, int segments, float* __restrict__ run_state, float* __restrict__ run_decay,
+                TO* __restrict__ out, long long out_stride) {
+    using L = SsdLayout<T, R, CPL>;
+    constexpr int CH = L::CH, NP = L::NP, COLS = L::COLS, ROW = L::ROW, VEC = L::VEC, TROW = L::TROW;
     extern __shared__ __align__(16) float ssd_smem[];
-    float* const s_b = ssd_smem;                                 // [CH][NP]
-    float* const s_c = s_b + CH * NP;                            // [CH][NP]
-    float* const s_x = s_c + CH * NP;                            // [CH][32]
-    float* const s_y = s_x + CH * SSD_COLS;                      // [WARPS][CH][32]
-    __shared__ float s_dt[CH], s_keep[CH];
+    float* const s_b = ssd_smem + L::B;
+    float* const s_c = ssd_smem + L::C;
+    float* const s_x = ssd_smem + L::X;
+    float* const s_z = ssd_smem + L::Z;
+    float* const s_y = ssd_smem + L::Y;
+    float* const s_w = ssd_smem + L::W;                          // [CH][CH + 4]
+    T* const t_b = reinterpret_cast<T*>(ssd_smem + L::TYPED);
+    T* const t_c = t_b + CH * TROW;
+    // of the chunk's tokens: step size, sum of the decays' logarithms so far, its exponential, weight in the update
+    __shared__ float s_dt[CH], s_log[CH], s_from[CH], s_to[CH];
     const int item = first_item + blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int col_tiles = (in.P + SSD_COLS - 1) / SSD_COLS;
-    const int p0 = (blockIdx.z % col_tiles) * SSD_COLS, segment = blockIdx.z / col_tiles, p = p0 + lane;
+    const int col_tiles = (in.P + COLS - 1) / COLS;
+    const int p0 = (blockIdx.z % col_tiles) * COLS, segment = blockIdx.z / col_tiles, p = p0 + CPL * lane;
     if (item >= last_item) return;
     const int begin = q_start[item], count = q_start[item + 1] - begin;
     const bool cut = segments > 1 && item >= first_cut;
-    const int per = cut ? ssd_run_length(count, segments, chunk_unit) : count;
+    const int per = cut ? ssd_run_length(count, segments, CH) : count;
     const int runs = cut && count > 0 ? (count + per - 1) / per : 1;
     if (count <= 0 || segment >= (STATE_ONLY ? runs - 1 : runs)) return;
     const int lo = begin + segment * per, hi = min(lo + per, begin + count);
@@ -68,115 +107,274 @@ ssd_scan_kernel(const T* __restrict__ conv, const T* __restrict__ raw, const Ssd
     const size_t block = (size_t)N * P;
     float* S = state + (size_t)item_slot[item] * state_stride + (size_t)h * block;
     const size_t cut_base = cut ? ((size_t)(item - first_cut) * in.heads + h) * segments : 0;
+
+    unsigned long long s[R / 2][CPL];                            // s[r][c]: rows n0 + 2r and + 1 of column p + c
+    auto load_state = [&](const float* from) {
+#pragma unroll
+        for (int r = 0; r < R / 2; ++r)
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) {
+                const int n = n0 + 2 * r;
+                const float a = (p + c < P && n < N) ? from[(size_t)n * P + p + c] : 0.f;
+                const float b = (p + c < P && n + 1 < N) ? from[(size_t)(n + 1) * P + p + c] : 0.f;
+                s[r][c] = pair_of(a, b);
+            }
+    };
+    auto store_state = [&](float* to) {
+#pragma unroll
+        for (int r = 0; r < R / 2; ++r)
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) {
+                const int n = n0 + 2 * r;
+                float a, b;
+                pair_split(s[r][c], a, b);
+                if (p + c < P && n < N) to[(size_t)n * P + p + c] = a;
+                if (p + c < P && n + 1 < N) to[(size_t)(n + 1) * P + p + c] = b;
+            }
+    };
+    // S of the slot: only this kernel of an earlier step wrote it, and that one is done
+    if (STATE_ONLY ? segment == 0 : runs == 1) load_state(S);
     pdl_prologue();
     conv = pdl_fresh(conv);
     raw = pdl_fresh(raw);
 
-    unsigned long long s[R / 2];
-    auto load_state = [&](const float* from) {
+    // ---- the rows of a chunk: 16-byte pieces on their way in registers (wide), or straight into shared memory
+    uint4 in_b[L::N_PIECES], in_c[L::N_PIECES], in_x[L::P_PIECES], in_z[L::P_PIECES];
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    float in_dt = 0.f;
+    auto fetch = [&](int t0) {
+        const int n = min(CH, hi - t0);
+        if (tid < n) in_dt = to_float(raw[(size_t)(t0 + tid) * in.ld_raw + in.dt + h]);
+        if (!wide) return;
 #pragma unroll
-        for (int r = 0; r < R / 2; ++r) {
-            const int n = n0 + 2 * r;
-            const float a = (p < P && n < N) ? from[(size_t)n * P + p] : 0.f;
-            const float b = (p < P && n + 1 < N) ? from[(size_t)(n + 1) * P + p] : 0.f;
-            s[r] = pair_of(a, b);
+        for (int q = 0; q < L::N_PIECES; ++q) {
+            const int e = tid + q * SSD_THREADS, tt = e / (NP / VEC), i = (e % (NP / VEC)) * VEC;
+            const bool here = tt < n && i < N;
+            const T* at = conv + (size_t)(t0 + tt) * in.ld_conv + (size_t)g * N + i;
+            in_b[q] = here ? *reinterpret_cast<const uint4*>(at + in.b) : zero;
+            if (!STATE_ONLY) in_c[q] = here ? *reinterpret_cast<const uint4*>(at + in.c) : zero;
+        }
+#pragma unroll
+        for (int q = 0; q < L::P_PIECES; ++q) {
+            const int e = tid + q * SSD_THREADS, tt = e / (COLS / VEC), j = (e % (COLS / VEC)) * VEC;
+            const bool here = tt < n && p0 + j < P;
+            in_x[q] = here ? *reinterpret_cast<const uint4*>(conv + (size_t)(t0 + tt) * in.ld_conv + in.x + (size_t)h * P + p0 + j) : zero;
+            if (!STATE_ONLY)
+                in_z[q] = here ? *reinterpret_cast<const uint4*>(raw + (size_t)(t0 + tt) * in.ld_raw + in.z + (size_t)h * P + p0 + j) : zero;
         }
     };
-    auto store_state = [&](float* to) {
+    auto place = [&](float* to, const uint4& piece) {
+        float x[VEC];
+        ssd_unpack(piece, x);
 #pragma unroll
-        for (int r = 0; r < R / 2; ++r) {
-            const int n = n0 + 2 * r;
-            float a, b;
-            pair_split(s[r], a, b);
-            if (p < P && n < N) to[(size_t)n * P + p] = a;
-            if (p < P && n + 1 < N) to[(size_t)(n + 1) * P + p] = b;
+        for (int w = 0; w < VEC; w += 4) *reinterpret_cast<float4*>(to + w) = make_float4(x[w], x[w + 1], x[w + 2], x[w + 3]);
+    };
+    auto settle = [&](int t0) {
+        const int n = min(CH, hi - t0);
+        if (wide) {
+#pragma unroll
+            for (int q = 0; q < L::N_PIECES; ++q) {
+                const int e = tid + q * SSD_THREADS, tt = e / (NP / VEC), i = (e % (NP / VEC)) * VEC;
+                if (tt < CH) {
+                    place(s_b + tt * ROW + i, in_b[q]);
+                    if (!STATE_ONLY) place(s_c + tt * ROW + i, in_c[q]);
+                    if constexpr (sizeof(T) == 2 && !STATE_ONLY) {
+                        *reinterpret_cast<uint4*>(t_b + tt * TROW + i) = in_b[q];
+                        *reinterpret_cast<uint4*>(t_c + tt * TROW + i) = in_c[q];
+                    }
+                }
+            }
+#pragma unroll
+            for (int q = 0; q < L::P_PIECES; ++q) {
+                const int e = tid + q * SSD_THREADS, tt = e / (COLS / VEC), j = (e % (COLS / VEC)) * VEC;
+                if (tt < CH) {
+                    place(s_x + tt * COLS + j, in_x[q]);
+                    if (!STATE_ONLY) place(s_z + tt * COLS + j, in_z[q]);
+                }
+            }
+        } else {
+            for (int e = tid; e < CH * NP; e += SSD_THREADS) {
+                const int tt = e / NP, i = e - tt * NP;
+                const bool here = tt < n && i < N;
+                const T* at = conv + (size_t)(t0 + tt) * in.ld_conv + (size_t)g * N + i;
+                const T b = here ? at[in.b] : from_float<T>(0.f), c = here ? at[in.c] : from_float<T>(0.f);
+                s_b[tt * ROW + i] = to_float(b);
+                s_c[tt * ROW + i] = to_float(c);
+                if constexpr (sizeof(T) == 2) {
+                    t_b[tt * TROW + i] = b;
+                    t_c[tt * TROW + i] = c;
+                }
+            }
+            for (int e = tid; e < CH * COLS; e += SSD_THREADS) {
+                const int tt = e / COLS, j = p0 + e % COLS;
+                const bool here = tt < n && j < P;
+                s_x[e] = here ? to_float(conv[(size_t)(t0 + tt) * in.ld_conv + in.x + (size_t)h * P + j]) : 0.f;
+                s_z[e] = here ? to_float(raw[(size_t)(t0 + tt) * in.ld_raw + in.z + (size_t)h * P + j]) : 0.f;
+            }
+        }
+        if (warp == 0) {                                         // (tokens behind the last: no step, nothing decays)
+            const float dt = lane < n ? softplus(in_dt + bias) : 0.f;
+            float sum = rate * dt;
+#pragma unroll
+            for (int o = 1; o < CH; o <<= 1) {
+                const float other = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += other;
+            }
+            const float end = __shfl_sync(0xffffffffu, sum, CH - 1);
+            if (lane < CH) {
+                s_dt[lane] = dt;
+                s_log[lane] = sum;
+                s_from[lane] = expf(sum);
+                s_to[lane] = expf(end - sum) * dt;
+            }
         }
     };
+    fetch(lo);
     if (STATE_ONLY) {
-        if (segment == 0) {                                      // the first run's start is the slot's state
-            load_state(S);
-            store_state(run_state + cut_base * block);
-        }
+        if (segment == 0) store_state(run_state + cut_base * block);         // the first run's start is the slot's state
 #pragma unroll
-        for (int r = 0; r < R / 2; ++r) s[r] = pair_of(0.f, 0.f);
+        for (int r = 0; r < R / 2; ++r)
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) s[r][c] = pair_of(0.f, 0.f);
     } else if (runs > 1) {
         load_state(pdl_fresh(run_state) + (cut_base + segment) * block);
-    } else {
-        load_state(S);
     }
     float exponent = 0.f;                                        // STATE_ONLY: the sum of the run's logarithms of decays
     for (int t0 = lo; t0 < hi; t0 += CH) {
         const int n = min(CH, hi - t0);
-        __syncthreads();                                         // the chunk before is done with shared memory
-        for (int e = tid; e < CH * NP; e += SSD_THREADS) {
-            const int tt = e / NP, i = e - tt * NP;
-            const bool here = tt < n && i < N;
-            const T* at = conv + (size_t)(t0 + tt) * in.ld_conv + (size_t)g * N + i;
-            s_b[e] = here ? to_float(at[in.b]) : 0.f;
-            if (!STATE_ONLY) s_c[e] = here ? to_float(at[in.c]) : 0.f;
-        }
-        for (int e = tid; e < CH * SSD_COLS; e += SSD_THREADS) {
-            const int tt = e / SSD_COLS, j = p0 + (e & (SSD_COLS - 1));
-            s_x[e] = tt < n && j < P ? to_float(conv[(size_t)(t0 + tt) * in.ld_conv + in.x + (size_t)h * P + j]) : 0.f;
-        }
-        if (tid < CH) {
-            const float dt = tid < n ? softplus(to_float(raw[(size_t)(t0 + tid) * in.ld_raw + in.dt + h]) + bias) : 0.f;
-            s_dt[tid] = dt;
-            s_keep[tid] = expf(rate * dt);                       // (1 behind the last token)
-        }
+        settle(t0);
         __syncthreads();
-        float y[CH];
-        auto token = [&](int tt) {
-            const float xd = s_x[tt * SSD_COLS + lane] * s_dt[tt], keep = s_keep[tt];
-            const unsigned long long x2 = pair_of(xd, xd), k2 = pair_of(keep, keep);
-            unsigned long long sum = pair_of(0.f, 0.f);
+        if (t0 + CH < hi) fetch(t0 + CH);
+        if constexpr (!STATE_ONLY) {
+            // ---- the weights W[t][s] of the chunk's own tokens
+            if constexpr (sizeof(T) == 2) {
+                if (warp < 2) {
+                    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+                    const uint32_t a_at = (uint32_t)__cvta_generic_to_shared(t_c + (lane & 15) * TROW + (lane >> 4) * 8);
+                    const uint32_t b_at = (uint32_t)__cvta_generic_to_shared(t_b + (8 * warp + (lane & 7)) * TROW + ((lane >> 3) & 1) * 8);
 #pragma unroll
-            for (int r = 0; r < R / 2; r += 2) {
-                const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(s_b + tt * NP + n0 + 2 * r);
-                s[r] = pair_fma(bb.x, x2, pair_mul(k2, s[r]));
-                s[r + 1] = pair_fma(bb.y, x2, pair_mul(k2, s[r + 1]));
-                if (!STATE_ONLY) {
-                    const ulonglong2 cc = *reinterpret_cast<const ulonglong2*>(s_c + tt * NP + n0 + 2 * r);
-                    sum = pair_fma(cc.x, s[r], sum);
-                    sum = pair_fma(cc.y, s[r + 1], sum);
+                    for (int k = 0; k < NP / 16; ++k) {
+                        uint32_t a[4], b[2];
+                        asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                                     : "=r"(a[0]), "=r"(a[1]), "=r"(a[2]), "=r"(a[3]) : "r"(a_at + 32 * k) : "memory");
+                        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
+                                     : "=r"(b[0]), "=r"(b[1]) : "r"(b_at + 32 * k) : "memory");
+                        asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                                     : "+f"(acc[0]), "+f"(acc[1]), "+f"(acc[2]), "+f"(acc[3])
+                                     : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+                    }
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int t = (lane >> 2) + 8 * (i >> 1), u = 8 * warp + 2 * (lane & 3) + (i & 1);
+                        s_w[t * (CH + 4) + u] = u <= t ? acc[i] * expf(s_log[t] - s_log[u]) * s_dt[u] : 0.f;
+                    }
                 }
+            } else {
+                const int t = tid >> 4, u = tid & 15;
+                float dot = 0.f;
+                if (u <= t) {
+                    for (int i = 0; i < NP; i += 4) {
+                        const float4 a = *reinterpret_cast<const float4*>(s_c + t * ROW + i);
+                        const float4 b = *reinterpret_cast<const float4*>(s_b + u * ROW + i);
+                        dot = fmaf(a.x, b.x, dot); dot = fmaf(a.y, b.y, dot);
+                        dot = fmaf(a.z, b.z, dot); dot = fmaf(a.w, b.w, dot);
+                    }
+                    dot *= expf(s_log[t] - s_log[u]) * s_dt[u];
+                }
+                s_w[t * (CH + 4) + u] = dot;
             }
-            float even, odd;
-            pair_split(sum, even, odd);
-            y[tt] = even + odd;
-        };
-        if (STATE_ONLY) {
-#pragma unroll 1
-            for (int tt = 0; tt < n; ++tt) {
-                const float xd = s_x[tt * SSD_COLS + lane] * s_dt[tt], keep = s_keep[tt];
-                exponent = fmaf(rate, s_dt[tt], exponent);
-                const unsigned long long x2 = pair_of(xd, xd), k2 = pair_of(keep, keep);
+            // ---- what the state ahead of the chunk gives to its tokens
+#pragma unroll
+            for (int tt = 0; tt < CH; ++tt) {
+                unsigned long long sum[CPL];
 #pragma unroll
                 for (int r = 0; r < R / 2; r += 2) {
-                    const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(s_b + tt * NP + n0 + 2 * r);
-                    s[r] = pair_fma(bb.x, x2, pair_mul(k2, s[r]));
-                    s[r + 1] = pair_fma(bb.y, x2, pair_mul(k2, s[r + 1]));
+                    const ulonglong2 cc = *reinterpret_cast<const ulonglong2*>(s_c + tt * ROW + n0 + 2 * r);
+#pragma unroll
+                    for (int c = 0; c < CPL; ++c) {
+                        sum[c] = r == 0 ? pair_mul(cc.x, s[r][c]) : pair_fma(cc.x, s[r][c], sum[c]);
+                        sum[c] = pair_fma(cc.y, s[r + 1][c], sum[c]);
+                    }
+                }
+                float y[CPL];
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) {
+                    float even, odd;
+                    pair_split(sum[c], even, odd);
+                    y[c] = even + odd;
+                }
+                float* to = s_y + (warp * CH + tt) * COLS + CPL * lane;
+                if constexpr (CPL == 2) *reinterpret_cast<float2*>(to) = make_float2(y[0], y[1]);
+                else *to = y[0];
+            }
+        }
+        // ---- the state behind the chunk
+        {
+            const float keep = s_from[CH - 1];
+            const unsigned long long k2 = pair_of(keep, keep);
+            if (STATE_ONLY) exponent += s_log[CH - 1];
+#pragma unroll
+            for (int r = 0; r < R / 2; ++r)
+#pragma unroll
+                for (int c = 0; c < CPL; ++c) s[r][c] = pair_mul(k2, s[r][c]);
+#pragma unroll 4
+            for (int tt = 0; tt < CH; ++tt) {
+                const float weight = s_to[tt];
+                unsigned long long x2[CPL];
+                if constexpr (CPL == 2) {
+                    const float2 x = *reinterpret_cast<const float2*>(s_x + tt * COLS + 2 * lane);
+                    x2[0] = pair_of(x.x * weight, x.x * weight);
+                    x2[1] = pair_of(x.y * weight, x.y * weight);
+                } else {
+                    const float x = s_x[tt * COLS + lane] * weight;
+                    x2[0] = pair_of(x, x);
+                }
+#pragma unroll
+                for (int r = 0; r < R / 2; r += 2) {
+                    const ulonglong2 bb = *reinterpret_cast<const ulonglong2*>(s_b + tt * ROW + n0 + 2 * r);
+#pragma unroll
+                    for (int c = 0; c < CPL; ++c) {
+                        s[r][c] = pair_fma(bb.x, x2[c], s[r][c]);
+                        s[r + 1][c] = pair_fma(bb.y, x2[c], s[r + 1][c]);
+                    }
                 }
             }
-            continue;
         }
-#pragma unroll
-        for (int tt = 0; tt < CH; ++tt) {
-            if (tt < n) token(tt);
-            else y[tt] = 0.f;
-        }
-#pragma unroll
-        for (int tt = 0; tt < CH; ++tt) s_y[(warp * CH + tt) * SSD_COLS + lane] = y[tt];
         __syncthreads();
-        for (int e = tid; e < n * SSD_COLS; e += SSD_THREADS) {
-            const int tt = e / SSD_COLS, col = e & (SSD_COLS - 1), j = p0 + col;
-            if (j >= P) continue;
-            float total = 0.f;
+        if constexpr (!STATE_ONLY) {
+            // ---- the sums over the warps, the chunk's own tokens, the skip and the gate: CPL neighbouring columns at a time
+            for (int e = tid; e < CH * 32; e += SSD_THREADS) {
+                const int tt = e >> 5, col = (e & 31) * CPL;
+                if (tt >= n || p0 + col >= P) continue;
+                float total[CPL], own[CPL];
 #pragma unroll
-            for (int w = 0; w < SSD_WARPS; ++w) total += s_y[(w * CH + tt) * SSD_COLS + col];
-            total = fmaf(skip, s_x[e], total);
-            const float z = to_float(raw[(size_t)(t0 + tt) * in.ld_raw + in.z + (size_t)h * P + j]);
-            out[(size_t)(t0 + tt) * out_stride + (size_t)h * P + j] = from_float<TO>(total * silu(z));
+                for (int c = 0; c < CPL; ++c) total[c] = own[c] = 0.f;
+                auto take = [&](const float* from, float weight, float (&to)[CPL]) {
+                    if constexpr (CPL == 2) {
+                        const float2 f = *reinterpret_cast<const float2*>(from);
+                        to[0] = fmaf(weight, f.x, to[0]);
+                        to[1] = fmaf(weight, f.y, to[1]);
+                    } else {
+                        to[0] = fmaf(weight, *from, to[0]);
+                    }
+                };
+#pragma unroll
+                for (int w = 0; w < SSD_WARPS; ++w) take(s_y + (w * CH + tt) * COLS + col, 1.f, total);
+#pragma unroll
+                for (int u = 0; u < CH; u += 4) {
+                    const float4 w = *reinterpret_cast<const float4*>(s_w + tt * (CH + 4) + u);
+                    take(s_x + u * COLS + col, w.x, own);
+                    take(s_x + (u + 1) * COLS + col, w.y, own);
+                    take(s_x + (u + 2) * COLS + col, w.z, own);
+                    take(s_x + (u + 3) * COLS + col, w.w, own);
+                }
+                take(s_x + tt * COLS + col, skip, own);
+                TO* to = out + (size_t)(t0 + tt) * out_stride + (size_t)h * P + p0 + col;
+#pragma unroll
+                for (int c = 0; c < CPL; ++c)
+                    if (p0 + col + c < P) to[c] = from_float<TO>(fmaf(s_from[tt], total[c], own[c]) * silu(s_z[tt * COLS + col + c]));
+            }
+            __syncthreads();                                     // before the next chunk's rows arrive
         }
     }
     if (STATE_ONLY) {
@@ -321,34 +519,47 @@ ssd_step_kernel(const T* __restrict__ conv, const T* __restrict__ raw, const Ssd
     }
 }
 
-template <typename T, typename TO, int R, bool STATE_ONLY>
+template <typename T, typename TO, int R, int CPL, bool STATE_ONLY>
 int launch_ssd_scan_rows(const T* conv, const T* raw, const SsdInputs& in, float* state, long long state_stride,
                          const int* q_start, const int* item_slot, int first_item, int last_item, int first_cut, int segments,
-                         int chunk_unit, int depth, float* run_state, float* run_decay, TO* out, long long out_stride,
-                         cudaStream_t s) {
-    auto kernel = ssd_scan_kernel<T, TO, R, STATE_ONLY>;
-    const int tiles = (in.P + SSD_COLS - 1) / SSD_COLS;
-    const size_t smem = (size_t)(2 * SSD_CHUNK * SSD_WARPS * R + SSD_CHUNK * SSD_COLS + SSD_WARPS * SSD_CHUNK * SSD_COLS) * sizeof(float);
+                         int depth, float* run_state, float* run_decay, TO* out, long long out_stride, cudaStream_t s) {
+    using L = SsdLayout<T, R, CPL>;
+    auto kernel = ssd_scan_kernel<T, TO, R, CPL, STATE_ONLY>;
+    const int tiles = (in.P + L::COLS - 1) / L::COLS;
     static size_t raised[MAX_DEVICES] = {0};
-    if (!ensure_dynamic_smem((const void*)kernel, smem, raised)) return PS_ERR_LAUNCH;
+    if (!ensure_dynamic_smem((const void*)kernel, L::BYTES, raised)) return PS_ERR_LAUNCH;
     if ((long long)tiles * depth > 65535) return PS_ERR_UNSUPPORTED;
-    return launch_pdl(kernel, dim3(last_item - first_item, in.heads, tiles * depth), dim3(SSD_THREADS), smem, s, conv, raw, in,
-                      state, state_stride, q_start, item_slot, first_item, last_item, first_cut, segments, chunk_unit, run_state,
+    constexpr int V = L::VEC;
+    const int wide = in.N % V == 0 && in.P % V == 0 && in.ld_conv % V == 0 && in.ld_raw % V == 0 && in.x % V == 0 && in.b % V == 0 &&
+                     in.c % V == 0 && in.z % V == 0 && !(((uintptr_t)conv | (uintptr_t)raw) & 15);
+    return launch_pdl(kernel, dim3(last_item - first_item, in.heads, tiles * depth), dim3(SSD_THREADS), L::BYTES, s, conv, raw, in,
+                      wide, state, state_stride, q_start, item_slot, first_item, last_item, first_cut, segments, run_state,
                       run_decay, out, out_stride);
 }
 
 template <typename T, typename TO, bool STATE_ONLY>
 int launch_ssd_scan(const T* conv, const T* raw, const SsdInputs& in, float* state, long long state_stride, const int* q_start,
-                    const int* item_slot, int first_item, int last_item, int first_cut, int segments, int chunk_unit, int depth,
+                    const int* item_slot, int first_item, int last_item, int first_cut, int segments, int depth,
                     float* run_state, float* run_decay, TO* out, long long out_stride, cudaStream_t s) {
-#define PS_SSD_ROWS(R)                                                                                                  \
-    return launch_ssd_scan_rows<T, TO, R, STATE_ONLY>(conv, raw, in, state, state_stride, q_start, item_slot, first_item, last_item, \
-                                                      first_cut, segments, chunk_unit, depth, run_state, run_decay, out, out_stride, s)
-    if (in.N <= 32) PS_SSD_ROWS(4);
-    if (in.N <= 64) PS_SSD_ROWS(8);
-    if (in.N <= 128) PS_SSD_ROWS(16);
-    if (in.N <= 256) PS_SSD_ROWS(32);
-    PS_SSD_ROWS(64);
+#define PS_SSD_ROWS(R, CPL)                                                                                             \
+    return launch_ssd_scan_rows<T, TO, R, CPL, STATE_ONLY>(conv, raw, in, state, state_stride, q_start, item_slot, first_item, \
+                                                           last_item, first_cut, segments, depth, run_state, run_decay, out, \
+                                                           out_stride, s)
+    const bool two = in.P > 32;                                  // columns of a lane
+    if (in.N <= 32) {
+        if (two) PS_SSD_ROWS(4, 2);
+        PS_SSD_ROWS(4, 1);
+    }
+    if (in.N <= 64) {
+        if (two) PS_SSD_ROWS(8, 2);
+        PS_SSD_ROWS(8, 1);
+    }
+    if (in.N <= 128) {
+        if (two) PS_SSD_ROWS(16, 2);
+        PS_SSD_ROWS(16, 1);
+    }
+    if (in.N <= 256) PS_SSD_ROWS(32, 1);
+    PS_SSD_ROWS(64, 1);
 #undef PS_SSD_ROWS
 }
 
@@ -379,7 +590,7 @@ int pick_ssd(const T* conv, const T* raw, const SsdInputs& in, int single, float
     }
     if (segments > 1) {
         int status = launch_ssd_scan<T, TO, true>(conv, raw, in, state, state_stride, q_start, item_slot, first_cut, n_items,
-                                                  first_cut, segments, SSD_CHUNK, segments - 1, run_state, run_decay, out,
+                                                  first_cut, segments, segments - 1, run_state, run_decay, out,
                                                   out_stride, s);
         if (status != PS_OK) return status;
         const int block = in.N * in.P;
@@ -392,7 +603,7 @@ int pick_ssd(const T* conv, const T* raw, const SsdInputs& in, int single, float
         if (status != PS_OK) return status;
     }
     return launch_ssd_scan<T, TO, false>(conv, raw, in, state, state_stride, q_start, item_slot, 0, n_items, first_cut, segments,
-                                         SSD_CHUNK, segments, run_state, run_decay, out, out_stride, s);
+                                         segments, run_state, run_decay, out, out_stride, s);
 }
 
 }  // namespace ps
