@@ -22,6 +22,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import statistics
 import subprocess
@@ -309,7 +310,8 @@ def _run_reference(args, ref):
 # results and end with an average over depth, a gated recurrence, latent attention without a window, attention with
 # short convolutions, routed experts) beside a Gozunex of equal width, depth, heads, latent and experts; Suvunex (norms
 # before and after each sublayer, attention beside gated linear attention, attention with mixed heads) beside a Tefopel in
-# which every other layer is recurrent.
+# which every other layer is recurrent; Vozirax (state-space layers, differential attention, mixer and feed-forward side by
+# side, experts without gates) beside a Suvunex of equal weights, whose kernels are the likes of most of its own.
 DESIGN_SIZES = {"w1024": "w1024", "w2048": "w2048"}      # named sizes of config/tefopel.py and config/gozunex.py
 DESIGN_CONTEXT = 2048
 
@@ -334,8 +336,24 @@ def design_arm(args):
     steps, warmup = min(args.steps, 64), max(args.warmup, 3)
 
     def configs(name):
-        from pagedserve_b200.config import gozunex, pagatar, suvunex, tefopel, zositar
+        from pagedserve_b200.config import gozunex, pagatar, suvunex, tefopel, vozirax, zositar
 
+        if args.design == "vozirax":
+            # Suvunex of equal size: same width, depth and vocabulary, as many attention heads of the cached heads' size on as
+            # many key heads, a recurrence in every other layer, and a dense feed-forward that makes the weights equal
+            from pagedserve_b200.models import init_plan
+            from pagedserve_b200.models.suvunex import build_suvunex_spec
+            from pagedserve_b200.models.vozirax import build_vozirax_spec
+
+            count = lambda spec: sum(math.prod(drawn[2] if len(drawn) > 2 else param.shape) for param, drawn in init_plan(spec))
+            size = vozirax.NAMED_CONFIGS["vozirax-" + name]
+            own = vozirax.named_config("vozirax-" + name)
+            like = lambda ff: suvunex.repeating_config(
+                width=size["width"], heads=size["heads"], head_dim=2 * size["head_dim"], kv_heads=size["kv_heads"],
+                layers=size["layers"], vocab=size["vocab"], ff=ff, right_heads=size["width"] // 64, right_dim=64)
+            spare = count(build_vozirax_spec(own)) - count(build_suvunex_spec(like(64)))
+            ff = 64 + spare // (3 * size["width"] * size["layers"]) // 64 * 64
+            return size, {"vozirax": own, "suvunex": like(ff)}
         if args.design == "suvunex":
             # Tefopel of equal size: same width, depth, heads and head size, a recurrent layer wherever the design has a
             # recurrence beside attention, windows that see every key, and a dense feed-forward that makes the weights equal
@@ -475,6 +493,54 @@ def design_arm(args):
             run = microbench.time_experts(2048, width, size["experts"], size["top"], size["ff"])
             kernels[f"experts_2048_tokens_{name}"] = {**run, "frac_tensor": run["tflops"] / tensor,
                                                       "dense_frac_tensor": run["dense_tflops"] / tensor}
+    elif args.dtype == "bfloat16" and not args.skip_points and args.design == "vozirax":
+        from pagedserve_b200.config import vozirax
+
+        hbm, tensor = peaks["hbm_gbs"], peaks["bf16_tflops"]
+        kernels = report["kernels"]
+
+        def of_hbm(run):
+            return {**run, "frac_hbm": run["gbs"] / hbm}
+
+        def of_tensor(run):
+            return {**run, "frac_tensor": run["tflops"] / tensor}
+
+        for name in (args.design_sizes.split(",") if args.design_sizes else DESIGN_SIZES):
+            size = vozirax.NAMED_CONFIGS["vozirax-" + name]
+            H, G, d, width = size["heads"], size["kv_heads"], size["head_dim"], size["width"]
+            slot, inner, channels = 2 * d, size["ssm_heads"] * size["ssm_dim"], size["ssm_heads"] * size["ssm_dim"] + 2 * size["ssm_state"]
+            for label, items, each in (("prefill_2x1024", 2, 1024), ("decode_b64", 64, 1), ("decode_b8", 8, 1)):
+                kernels[f"recurrence_{label}_{name}"] = {
+                    "suvunex": of_hbm(microbench.time_gla(items, each, width // 64, 64, 64)),
+                    "vozirax": of_hbm(microbench.time_ssd(items, each, size["ssm_heads"], 1, size["ssm_state"], size["ssm_dim"]))}
+            # attention with two maps per head: twice the query heads on the same cache, results left as float32
+            for batch in (8, 64):
+                kernels[f"decode_attention_b{batch}_{name}"] = {
+                    "suvunex": of_hbm(microbench.time_decode_attention(batch, 1024, H, G, slot, sink=True, as_rows=True)),
+                    "vozirax": of_hbm(microbench.time_decode_attention(batch, 1024, 2 * H, G, slot, as_rows=True, wide=True))}
+            kernels[f"prefill_attention_{name}"] = {
+                "suvunex": of_tensor(microbench.time_prefill_attention(2, 1024, H, G, slot, sink=True)),
+                "vozirax": of_tensor(microbench.time_prefill_attention(2, 1024, 2 * H, G, slot, wide=True))}
+            for label, tokens in (("prefill_2048", 2048), ("decode_b64", 64), ("decode_b8", 8)):
+                items = 2 if tokens > 64 else tokens
+                kernels[f"cache_write_{label}_{name}"] = {
+                    "suvunex": of_hbm(microbench.time_head_norm_cache_write(tokens, H, G, slot, rot_dims=slot)),
+                    "vozirax": of_hbm(microbench.time_diff_prepare(tokens, H, G, d, 2 * d)),
+                    "vozirax_combine": of_hbm(microbench.time_diff_combine(tokens, H, 2 * d, slot))}
+                kernels[f"norms_{label}_{name}"] = {
+                    "suvunex_close": of_hbm(microbench.time_sandwich_close(tokens, width)),
+                    "tefopel_norm": of_hbm(microbench.time_layernorm(tokens, width)),
+                    "vozirax_two_norms": of_hbm(microbench.time_norm_pair(tokens, width)),
+                    "vozirax_gated_norm": of_hbm(microbench.time_group_norm(tokens, inner, 1))}
+                kernels[f"convolution_{label}_{name}"] = {
+                    "pagatar": of_hbm(microbench.time_short_conv(tokens, items, H, H, slot, 3)),
+                    "suvunex": of_hbm(microbench.time_row_conv(tokens, items, width, 4)),
+                    "vozirax": of_hbm(microbench.time_gated_conv(tokens, items, channels, 4, beside=inner))}
+            like = microbench.time_experts(2048, width, size["experts"], size["top"], size["expert_ff"], score="sigmoid",
+                                           normalize=False)
+            own = microbench.time_experts(2048, width, size["experts"], size["top"], size["expert_ff"], score="sigmoid",
+                                          form="relu_squared")
+            kernels[f"experts_2048_tokens_{name}"] = {"pagatar": of_tensor(like), "vozirax": of_tensor(own)}
     elif args.dtype == "bfloat16" and not args.skip_points and args.design == "suvunex":
         from pagedserve_b200.config import suvunex
 
@@ -637,7 +703,7 @@ def main():
     parser.add_argument("--serving", type=int, default=0, metavar="REQUESTS",
                         help="instead of the decode measurement: this many requests (prompts U[64,1024), outputs "
                              "U[32,256]) through the scheduler, chunked prefill under a 2,048-token budget")
-    parser.add_argument("--design", default=None, choices=("tefopel", "gozunex", "zositar", "pagatar", "suvunex"),
+    parser.add_argument("--design", default=None, choices=("tefopel", "gozunex", "zositar", "pagatar", "suvunex", "vozirax"),
                         help="instead of the default workload: prefill and decode throughput of this design at a few "
                              "sizes beside GPT-2 of equal size, and its kernels alone against the measured peaks")
     parser.add_argument("--design-sizes", default=None, help="comma-separated names out of: " + ", ".join(DESIGN_SIZES))

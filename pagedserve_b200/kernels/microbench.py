@@ -102,7 +102,7 @@ def bench_attention(args):
     pool = torch.randn(B * pages_per + 1, layers, 2, H, page, D, device="cuda").to(torch.bfloat16)
     table = torch.randperm(B * pages_per, device="cuda").to(torch.int32).view(B, pages_per)
     q = torch.randn(B, H * D, device="cuda").to(torch.bfloat16)
-    out = torch.empty_like(q)
+    out = torch.empty_like(q, dtype=torch.float32 if wide else None)
     token_item = torch.arange(B, dtype=torch.int32, device="cuda")
     positions = torch.full((B,), ctx - 1, dtype=torch.int32, device="cuda")
     stride = layers * 2 * H * page * D
@@ -132,11 +132,12 @@ def _paged_inputs(items, context, kv_heads, head_dim, page, rotate_mb=200, plane
 
 
 def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, window=None, softcap=None,
-                          sink=False, iters=20, planes=2, chunk=None, mixed=False, as_rows=False, splits=None):
+                          sink=False, iters=20, planes=2, chunk=None, mixed=False, as_rows=False, splits=None, wide=False):
     """One decode token per request over ``context`` keys (bfloat16 split-key kernel); GB/s over the K and V
     bytes a token may see (with one plane: over the rows once).  ``mixed``: a layer whose heads' weights are mixed
     across heads (every query head meets all values, then the mixing kernel).  ``as_rows``: the kernel with the heads of a
-    group (mixed: all heads) as the rows of a tile, a token's keys shared out over ``splits`` CTAs (None: its own rule)."""
+    group (mixed: all heads) as the rows of a tile, a token's keys shared out over ``splits`` CTAs (None: its own rule).
+    ``wide``: the result is left as float32."""
     from pagedserve_b200.kernels.ops import Ops
 
     ops = Ops(torch.bfloat16)
@@ -176,16 +177,16 @@ def time_decode_attention(batch, context, heads, kv_heads, head_dim, page=16, wi
 
 
 def time_prefill_attention(prompts, prompt_len, heads, kv_heads, head_dim, page=16, window=None, softcap=None,
-                           sink=False, iters=10, planes=2, chunk=None, mixed=False):
+                           sink=False, iters=10, planes=2, chunk=None, mixed=False, wide=False):
     """Whole prompts through the tcgen05 prompt kernel (bfloat16, head size 64 or 128); TFLOP/s over the
-    products of the keys a query may see.  ``mixed`` as in :func:`time_decode_attention` (the same products counted)."""
+    products of the keys a query may see.  ``mixed`` and ``wide`` as in :func:`time_decode_attention` (the same products counted)."""
     from pagedserve_b200.kernels.ops import Ops
 
     ops = Ops(torch.bfloat16)
     pool, table, layers, _ = _paged_inputs(prompts, prompt_len, kv_heads, head_dim, page, rotate_mb=0, planes=planes)
     total = prompts * prompt_len
     q = torch.randn(total, heads * head_dim, device="cuda").to(torch.bfloat16)
-    out = torch.empty_like(q)
+    out = torch.empty_like(q, dtype=torch.float32 if wide else None)
     q_start = torch.arange(0, total + 1, prompt_len, dtype=torch.int32, device="cuda")
     kv_len = torch.full((prompts,), prompt_len, dtype=torch.int32, device="cuda")
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
@@ -465,6 +466,128 @@ def time_gla(items, tokens_each, heads, dk, dv, rank=16, dtype=torch.bfloat16, i
     return {"us": seconds * 1e6, "gbs": nbytes / seconds / 1e9, "tokens_per_s": total / seconds}
 
 
+def time_ssd(items, tokens_each, heads, groups, state, vdim, dtype=torch.bfloat16, iters=10, segments=None):
+    """The state-space recurrence alone (all its launches where entries are cut into runs) on ``items`` entries of
+    ``tokens_each`` tokens; GB/s over what it must move: x, B, C, z and dt in, one row out, every entry's state in and
+    out."""
+    from types import SimpleNamespace
+
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    total, inner, shared = items * tokens_each, heads * vdim, groups * state
+    columns, rows = inner + 2 * shared, 2 * inner + 2 * shared + heads
+    copies = min(64, max(1, int(200e6 // (total * (columns + rows) * 2)) + 1))            # rotate past the L2
+    conv = torch.randn(copies, total, columns, device="cuda").to(dtype)
+    raw = torch.randn(copies, total, rows + (-rows % 8), device="cuda").to(dtype)
+    vectors = [torch.randn(heads, device="cuda") for _ in range(3)]
+    states = max(1, min(16, int(200e6 // (items * heads * state * vdim * 4)) + 1))
+    kept = torch.zeros(states, items, heads * state * vdim, device="cuda")
+    out = torch.empty(total, inner, dtype=dtype, device="cuda")
+    ctx = SimpleNamespace(q_start=torch.arange(0, total + 1, tokens_each, dtype=torch.int32, device="cuda"),
+                          item_slot=torch.arange(items, dtype=torch.int32, device="cuda"), num_items=items,
+                          num_short_items=items if tokens_each < 16 else 0, max_q_len=tokens_each,
+                          single_tokens=tokens_each == 1)
+    offsets = (0, inner, inner + shared, 0, 2 * inner + 2 * shared)
+
+    def run(i):
+        ops.ssd(conv[i % copies], raw[i % copies], offsets, *vectors, kept[i % states], ctx, out, heads, groups, state, vdim,
+                segments=segments)
+
+    seconds = _time(run, iters, graph=True)
+    nbytes = total * (3 * inner + 2 * shared + heads) * out.element_size() + items * heads * state * vdim * 4 * 2
+    return {"us": seconds * 1e6, "gbs": nbytes / seconds / 1e9, "tokens_per_s": total / seconds}
+
+
+def time_gated_conv(tokens, items, channels, taps, beside=0, iters=20):
+    """The short convolution with bias and silu on ``channels`` of a projection's rows (``beside`` others stand beside them);
+    GB/s over rows of the compute type read and written and the kept rows."""
+    from types import SimpleNamespace
+
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = min(256, max(1, int(200e6 // (tokens * channels * 4)) + 1))            # rotate past the L2
+    u = torch.randn(copies, tokens, beside + channels, device="cuda").to(torch.bfloat16)
+    out = torch.empty(tokens, channels, dtype=torch.bfloat16, device="cuda")
+    weight, bias = torch.randn(channels, taps, device="cuda"), torch.randn(channels, device="cuda")
+    state = torch.zeros(items + 1, (taps - 1) * channels, device="cuda")
+    each = tokens // items
+    ctx = SimpleNamespace(q_start=torch.arange(0, tokens + 1, each, dtype=torch.int32, device="cuda"),
+                          item_slot=torch.arange(items, dtype=torch.int32, device="cuda"), num_items=items,
+                          token_item=(torch.arange(tokens, device="cuda") // each).to(torch.int32), single_tokens=each == 1)
+    seconds = _time(lambda i: ops.short_conv(u[i % copies][:, beside:], weight, taps, channels, state, ctx, out, bias=bias,
+                                             act="silu"), iters, graph=True)
+    return {"us": seconds * 1e6, "gbs": (tokens * channels * 4 + 2 * items * (taps - 1) * channels * 4) / seconds / 1e9}
+
+
+def time_diff_prepare(tokens, heads, kv_heads, dim, vdim, page=16, iters=20):
+    """Norms, temperature and cache write of attention with two maps per head; GB/s over the projected row read, the queries
+    and the pages written."""
+    from types import SimpleNamespace
+
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    slot = -(-max(2 * dim, vdim) // 16) * 16
+    pool, table, layers, stride = _paged_inputs(1, tokens, kv_heads, slot, page)
+    widths = (2 * heads * dim, 2 * kv_heads * dim, kv_heads * vdim)
+    copies = min(256, max(1, int(200e6 // (tokens * sum(widths) * 2)) + 1))         # rotate past the L2
+    row = torch.randn(copies, tokens, sum(widths), device="cuda").to(torch.bfloat16)
+    gain = torch.ones(dim, device="cuda")
+    out = torch.empty(tokens, 2 * heads * slot, dtype=torch.bfloat16, device="cuda")
+    ctx = SimpleNamespace(token_slot=torch.zeros(tokens, dtype=torch.int32, device="cuda"),
+                          positions=torch.arange(tokens, dtype=torch.int32, device="cuda"))
+
+    def run(i):
+        layer = SimpleNamespace(k_pool=pool[:, i % layers, 0], v_pool=pool[:, i % layers, 1], page_stride=stride, page_size=page,
+                                block_table=table)
+        ops.diff_prepare(row[i % copies], widths[0], widths[0] + widths[1], gain, gain, 1e-6, (0.1, 64), ctx, layer, out, heads,
+                         kv_heads, dim, vdim, slot)
+
+    seconds = _time(run, iters, graph=True)
+    return {"us": seconds * 1e6, "gbs": tokens * (sum(widths) + 2 * heads * slot + 2 * kv_heads * slot) * 2 / seconds / 1e9}
+
+
+def time_diff_combine(tokens, heads, vdim, slot, iters=20):
+    """Difference, norm and gate of two maps per head; GB/s over float32 maps read and rows written."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = min(64, max(1, int(200e6 // (tokens * 2 * heads * slot * 4)) + 1))     # rotate past the L2
+    maps = torch.randn(copies, tokens, 2 * heads * slot, device="cuda")
+    gate = torch.randn(tokens, heads, device="cuda").to(torch.bfloat16)
+    out = torch.empty(tokens, heads * vdim, dtype=torch.bfloat16, device="cuda")
+    seconds = _time(lambda i: ops.diff_combine(maps[i % copies], gate, out, 0.5, 1e-6, 0.6, heads, vdim, slot), iters, graph=True)
+    return {"us": seconds * 1e6, "gbs": tokens * heads * (2 * vdim * 4 + vdim * 2) / seconds / 1e9}
+
+
+def time_norm_pair(tokens, width, iters=20):
+    """Two norms of one row; GB/s over float32 rows read and two rounded rows written."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = min(256, max(1, int(200e6 // (tokens * width * 4)) + 1))               # rotate past the L2
+    x = torch.randn(copies, tokens, width, device="cuda")
+    gain = torch.ones(width, device="cuda")
+    outs = [torch.empty(tokens, width, dtype=torch.bfloat16, device="cuda") for _ in range(2)]
+    seconds = _time(lambda i: ops.rms_norm_pair(x[i % copies], gain, gain, 1e-6, *outs), iters, graph=True)
+    return {"us": seconds * 1e6, "gbs": tokens * width * 8 / seconds / 1e9}
+
+
+def time_group_norm(tokens, width, groups, iters=20):
+    """The norm in groups on rows of the compute type; GB/s over rows read and written."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(torch.bfloat16)
+    copies = min(256, max(1, int(200e6 // (tokens * width * 2)) + 1))               # rotate past the L2
+    x = torch.randn(copies, tokens, width, device="cuda").to(torch.bfloat16)
+    gain = torch.ones(width, device="cuda")
+    out = torch.empty(tokens, width, dtype=torch.bfloat16, device="cuda")
+    seconds = _time(lambda i: ops.group_rms_norm(x[i % copies], gain, 1e-6, groups, out), iters, graph=True)
+    return {"us": seconds * 1e6, "gbs": tokens * width * 4 / seconds / 1e9}
+
+
 def time_sandwich_close(tokens, width, rows_out=True, iters=20):
     """The kernel that closes a sublayer of a layer with norms before and after its sublayers; GB/s over the sublayer's
     row read and zeroed, the residual row read and written and (``rows_out``) the next sublayer's row written."""
@@ -524,14 +647,16 @@ def time_experts(tokens, width, experts, top, ff, iters=10, score="softmax", nor
     two tcgen05 products over expert tiles, gate, combine; beside the two plain tcgen05 products of a dense
     feed-forward with the same inner size per token (top * ff).  TFLOP/s over the useful products.  ``score``,
     ``normalize`` and ``form`` as the router and the inner activation take them (sigmoid scores that are the
-    weights; clamped experts)."""
+    weights; clamped experts; "relu_squared": experts without a gate, two products instead of three, whose activation is the
+    first product's epilogue)."""
     from pagedserve_b200.kernels.ops import Ops
 
     ops = Ops(torch.bfloat16)
     dev = "cuda"
     x = torch.randn(tokens, width, device=dev).to(torch.bfloat16)
     router = (torch.randn(experts, width, device=dev) * 0.05).to(torch.bfloat16)
-    w_gu = (torch.randn(experts * 2 * ff, width, device=dev) * width ** -0.5).to(torch.bfloat16)
+    gated = form != "relu_squared"
+    w_gu = (torch.randn(experts * (2 if gated else 1) * ff, width, device=dev) * width ** -0.5).to(torch.bfloat16)
     w_down = (torch.randn(width, experts * ff, device=dev) * ff ** -0.5).to(torch.bfloat16)
     dense = torch.empty(tokens, experts, device=dev)
     chosen = torch.empty(tokens, top, dtype=torch.int32, device=dev)
@@ -542,10 +667,11 @@ def time_experts(tokens, width, experts, top, ff, iters=10, score="softmax", nor
     row_weight = torch.empty(rows_cap, device=dev)
     tile_expert = torch.empty(rows_cap // ops.EXPERT_TILE, dtype=torch.int32, device=dev)
     rows = torch.empty(rows_cap, width, dtype=torch.bfloat16, device=dev)
-    gate_up = torch.empty(rows_cap, 2 * ff, dtype=torch.bfloat16, device=dev)
+    gate_up = torch.empty(rows_cap, (2 if gated else 1) * ff, dtype=torch.bfloat16, device=dev)
     inner = torch.empty(rows_cap, ff, dtype=torch.bfloat16, device=dev)
     down = torch.empty(rows_cap, width, device=dev)
     y = torch.zeros(tokens, width, device=dev)
+    ones = torch.ones(width, device=dev)
     status = ops.status_flag(dev)
     parts = {}
 
@@ -553,10 +679,13 @@ def time_experts(tokens, width, experts, top, ff, iters=10, score="softmax", nor
         ops.moe_route(x, router, None, dense, chosen, chosen_w, None, top, 0, 0, score=score, normalize=normalize)
         ops.moe_plan(chosen, chosen_w, experts, row_of, row_token, row_weight, tile_expert)
         ops.moe_gather(x, row_token, rows)
-        ops.linear_experts(rows, w_gu, gate_up, tile_expert, experts)
-        ops.moe_gate_mul_rows(gate_up, row_weight, inner, form=form)
+        if gated:
+            ops.linear_experts(rows, w_gu, gate_up, tile_expert, experts)
+            ops.moe_gate_mul_rows(gate_up, row_weight, inner, form=form)
+        else:
+            ops.linear_experts(rows, w_gu, inner, tile_expert, experts, act="relu_squared")
         ops.linear_experts(inner, w_down, down, tile_expert, experts, along_k=True)
-        ops.moe_combine(down, row_of, top, y)
+        ops.moe_combine(down, row_of, top, y, **({} if gated else dict(weights=chosen_w, factor=ones)))
 
     seconds = _time(routed, iters, graph=True)
     parts["route_us"] = _time(lambda i: ops.moe_route(x, router, None, dense, chosen, chosen_w, None, top, 0, 0, score=score, normalize=normalize), iters,
@@ -566,15 +695,16 @@ def time_experts(tokens, width, experts, top, ff, iters=10, score="softmax", nor
     parts["gather_us"] = _time(lambda i: ops.moe_gather(x, row_token, rows), iters, graph=True) * 1e6
     parts["gate_up_us"] = _time(lambda i: ops.linear_experts(rows, w_gu, gate_up, tile_expert, experts), iters,
                                 graph=True) * 1e6
-    parts["gate_mul_us"] = _time(lambda i: ops.moe_gate_mul_rows(gate_up, row_weight, inner, form=form), iters, graph=True) * 1e6
+    if gated:
+        parts["gate_mul_us"] = _time(lambda i: ops.moe_gate_mul_rows(gate_up, row_weight, inner, form=form), iters, graph=True) * 1e6
     parts["down_us"] = _time(lambda i: ops.linear_experts(inner, w_down, down, tile_expert, experts, along_k=True), iters,
                              graph=True) * 1e6
     parts["combine_us"] = _time(lambda i: ops.moe_combine(down, row_of, top, y), iters, graph=True) * 1e6
     # a dense feed-forward of the same inner size per token: up to 2 * top * ff columns, down from top * ff
     wide = top * ff
-    w_up_d = (torch.randn(2 * wide, width, device=dev) * width ** -0.5).to(torch.bfloat16)
+    w_up_d = (torch.randn((2 if gated else 1) * wide, width, device=dev) * width ** -0.5).to(torch.bfloat16)
     w_down_d = (torch.randn(width, wide, device=dev) * wide ** -0.5).to(torch.bfloat16)
-    up_d = torch.empty(tokens, 2 * wide, dtype=torch.bfloat16, device=dev)
+    up_d = torch.empty(tokens, (2 if gated else 1) * wide, dtype=torch.bfloat16, device=dev)
     inner_d = up_d[:, :wide]
 
     def plain(i):
@@ -582,7 +712,7 @@ def time_experts(tokens, width, experts, top, ff, iters=10, score="softmax", nor
         ops.linear_tc(inner_d, w_down_d, None, y, accumulate=True, status=status)
 
     plain_seconds = _time(plain, iters, graph=True)
-    flops = 2.0 * tokens * top * (3 * ff) * width
+    flops = 2.0 * tokens * top * ((3 if gated else 2) * ff) * width
     return {"us": seconds * 1e6, "tflops": flops / seconds / 1e12, "dense_us": plain_seconds * 1e6,
             "dense_tflops": flops / plain_seconds / 1e12, "status": int(status.item()), **parts}
 

@@ -1387,13 +1387,13 @@ class Ops:
     SSD_SCRATCH_BYTES = 256 << 20
 
     def ssd_segments(self, ctx, heads, N, P):
-        """Runs that a prompt portion is cut into: about as many CTAs as the device holds at once."""
+        """Runs that a prompt portion is cut into: about as many CTAs as two on every SM."""
         long_items = ctx.num_items - ctx.num_short_items
         longest = int(ctx.max_q_len)
         if long_items <= 0 or longest < 2 * self.SSD_RUN:
             return 1
-        tiles = -(-P // 32)
-        wanted = min(148 * 3 // (long_items * heads * tiles), longest // self.SSD_RUN,
+        tiles = -(-P // (64 if P > 32 and N <= 128 else 32))
+        wanted = min(148 * 2 // (long_items * heads * tiles), longest // self.SSD_RUN,
                      self.SSD_SCRATCH_BYTES // (4 * long_items * heads * N * P))
         return max(1, min(64, wanted))
 
