@@ -8,9 +8,14 @@
 //     S_t    = exp(-exp(A_h) d_t) S_(t-1) + d_t B_t x_t^T
 //     out_t  = (S_t^T C_t + D_h x_t) * silu(z_t)                    (rows of heads * P numbers; the norm behind is another kernel)
 //
-// ssd_step_kernel: steps in which every entry brings one token (decode).  One CTA per (entry, head); S goes through registers,
-//                  four columns an access, the first rows on their way before the wait for the kernel that makes the token's row.
-// ssd_scan_kernel: everything else, float32 arithmetic on CUDA cores, any size.  One CTA per (entry, head, tile of columns, run
+// ssd_step_kernel: entries of few tokens (decode).  One CTA per (entry, head); S goes through registers, four columns an
+//                  access, the first rows on their way before the wait for the kernel that makes the token's row.
+// ssd_prompt_kernel: prompt portions in bfloat16, on tensor cores to float32 accuracy.  One CTA per (entry, head, tile of
+//                  columns, run of tokens), chunks of 64 tokens (copied in by cp.async, the next chunk's on their way), S as
+//                  float32 mma accumulators that stay in registers.  The equations are those of the next kernel; every matrix
+//                  product has one operand that is bfloat16 as it comes (x, B, C) and one float32 operand, which is cut into
+//                  three bfloat16 pieces (together its 24 bits), so that the products are those of float32 numbers.
+// ssd_scan_kernel: all other portions, float32 arithmetic on CUDA cores, any size.  One CTA per (entry, head, tile of columns, run
 //                  of tokens): a lane holds one or two columns, a warp N / 8 rows of S in registers, two rows to a packed pair.
 //                  Tokens come in chunks of 16, the next chunk's rows on their way in registers while one is worked on.  With
 //                  S the state ahead of a chunk and L_t the sum of the chunk's -exp(A_h) d up to and including token t,
@@ -430,19 +435,19 @@ ssd_fold_kernel(float* __restrict__ run_state, const float* __restrict__ run_dec
     }
 }
 
-// One token per entry.  Thread (part, group) works on the columns [V group, V group + V) of the rows part, part + parts, ...;
+// Entries [0, gridDim.x) of few tokens, token by token.  Thread (part, group) works on the columns [V group, V group + V) of the rows part, part + parts, ...;
 // `lanes` (a power of two, at least P / V) threads share a row.
 constexpr int SSD_STEP_ROWS = 8;                                 // rows of a thread that are on their way together
 
 template <typename T, typename TO, int V>
-__global__ void __launch_bounds__(SSD_THREADS)
+__global__ void __launch_bounds__(SSD_THREADS, 4)
 ssd_step_kernel(const T* __restrict__ conv, const T* __restrict__ raw, const SsdInputs in, float* __restrict__ state,
                 long long state_stride, const int* __restrict__ q_start, const int* __restrict__ item_slot, int lanes,
                 TO* __restrict__ out, long long out_stride) {
     extern __shared__ __align__(16) float ssd_smem[];             // B [N], C [N], then the sums [warps or parts][P]
     const int item = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
-    const int t = q_start[item];
-    if (q_start[item + 1] <= t) return;
+    const int begin = q_start[item], end = q_start[item + 1];
+    if (end <= begin) return;
     const int N = in.N, P = in.P, g = h / (in.heads / in.groups);
     const int parts = SSD_THREADS / lanes, part = tid / lanes, col = (tid - part * lanes) * V;
     const bool mine = col < P;
@@ -469,53 +474,372 @@ ssd_step_kernel(const T* __restrict__ conv, const T* __restrict__ raw, const Ssd
     fetch(0);
     const float rate = -expf(in.a_log[h]), bias = in.dt_bias[h], skip = in.d[h];
     pdl_prologue();
-    conv = pdl_fresh(conv) + (size_t)t * in.ld_conv;
-    raw = pdl_fresh(raw) + (size_t)t * in.ld_raw;
-    for (int i = tid; i < N; i += SSD_THREADS) {
-        s_b[i] = to_float(conv[in.b + g * N + i]);
-        s_c[i] = to_float(conv[in.c + g * N + i]);
-    }
-    float x[V], y[V];
-    const float dt = softplus(to_float(raw[in.dt + h]) + bias), keep = expf(rate * dt);
+    conv = pdl_fresh(conv) + (size_t)begin * in.ld_conv;
+    raw = pdl_fresh(raw) + (size_t)begin * in.ld_raw;
+    for (int t = begin; t < end; ++t, conv += in.ld_conv, raw += in.ld_raw) {
+        if (t > begin) {                                             // (S: what this thread has just stored)
+            __syncthreads();
+            fetch(0);
+        }
+        for (int i = tid; i < N; i += SSD_THREADS) {
+            s_b[i] = to_float(conv[in.b + g * N + i]);
+            s_c[i] = to_float(conv[in.c + g * N + i]);
+        }
+        float x[V], y[V];
+        const float dt = softplus(to_float(raw[in.dt + h]) + bias), keep = expf(rate * dt);
 #pragma unroll
-    for (int v = 0; v < V; ++v) {
-        x[v] = mine && col + v < P ? to_float(conv[in.x + (size_t)h * P + col + v]) * dt : 0.f;
-        y[v] = 0.f;
-    }
-    __syncthreads();
-    for (int first = 0; first < N; first += SSD_STEP_ROWS * parts) {
-        if (first) fetch(first);
+        for (int v = 0; v < V; ++v) {
+            x[v] = mine && col + v < P ? to_float(conv[in.x + (size_t)h * P + col + v]) * dt : 0.f;
+            y[v] = 0.f;
+        }
+        __syncthreads();
+        for (int first = 0; first < N; first += SSD_STEP_ROWS * parts) {
+            if (first) fetch(first);
 #pragma unroll
-        for (int r = 0; r < SSD_STEP_ROWS; ++r) {
-            const int n = first + part + r * parts;
-            if (mine && n < N) {
-                const float b = s_b[n], c = s_c[n];
+            for (int r = 0; r < SSD_STEP_ROWS; ++r) {
+                const int n = first + part + r * parts;
+                if (mine && n < N) {
+                    const float b = s_b[n], c = s_c[n];
 #pragma unroll
-                for (int v = 0; v < V; ++v) {
-                    s[r][v] = fmaf(b, x[v], keep * s[r][v]);
-                    y[v] = fmaf(c, s[r][v], y[v]);
+                    for (int v = 0; v < V; ++v) {
+                        s[r][v] = fmaf(b, x[v], keep * s[r][v]);
+                        y[v] = fmaf(c, s[r][v], y[v]);
+                    }
+                    if constexpr (V == 4) *reinterpret_cast<float4*>(S + (size_t)n * P) = make_float4(s[r][0], s[r][1], s[r][2], s[r][3]);
+                    else S[(size_t)n * P] = s[r][0];
                 }
-                if constexpr (V == 4) *reinterpret_cast<float4*>(S + (size_t)n * P) = make_float4(s[r][0], s[r][1], s[r][2], s[r][3]);
-                else S[(size_t)n * P] = s[r][0];
+            }
+        }
+        // the sums over the parts: first inside a warp, then between its rows in shared memory
+        for (int o = lanes; o < 32; o <<= 1)
+#pragma unroll
+            for (int v = 0; v < V; ++v) y[v] += __shfl_xor_sync(0xffffffffu, y[v], o);
+        const int rows = lanes < 32 ? SSD_WARPS : parts, own = lanes < 32 ? tid >> 5 : part;
+        if (mine && (lanes >= 32 || (tid & 31) < lanes)) {
+#pragma unroll
+            for (int v = 0; v < V; ++v)
+                if (col + v < P) s_y[own * P + col + v] = y[v];
+        }
+        __syncthreads();
+        for (int j = tid; j < P; j += SSD_THREADS) {
+            float total = 0.f;
+            for (int w = 0; w < rows; ++w) total += s_y[w * P + j];
+            total = fmaf(skip, to_float(conv[in.x + (size_t)h * P + j]), total);
+            out[(size_t)t * out_stride + (size_t)h * P + j] = from_float<TO>(total * silu(to_float(raw[in.z + (size_t)h * P + j])));
+        }
+    }
+}
+
+// ---- prompt portions on tensor cores
+constexpr int SSD_PROMPT_CHUNK = 64, SSD_PIECES = 3;
+
+__device__ __forceinline__ void ssd_ldm(uint32_t (&r)[4], uint32_t at) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at) : "memory");
+}
+__device__ __forceinline__ void ssd_ldm_t(uint32_t (&r)[4], uint32_t at) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at) : "memory");
+}
+__device__ __forceinline__ void ssd_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// two float32 numbers as three pairs of bfloat16 numbers that add up to them
+__device__ __forceinline__ void ssd_split(float x, float y, uint32_t (&piece)[SSD_PIECES]) {
+#pragma unroll
+    for (int i = 0; i < SSD_PIECES; ++i) {
+        const __nv_bfloat162 rounded = __floats2bfloat162_rn(x, y);
+        piece[i] = *reinterpret_cast<const uint32_t*>(&rounded);
+        const float2 back = __bfloat1622float2(rounded);
+        x -= back.x;
+        y -= back.y;
+    }
+}
+
+// NT: rows of S, PT: columns of S of a CTA (both padded with zeros)
+template <int NT, int PT>
+struct SsdPromptLayout {
+    static constexpr int CH = SSD_PROMPT_CHUNK, TROW = NT + 8, PROW = PT + 8;           // padded rows, in elements
+    static constexpr int B = 0, C = CH * TROW, X = 2 * CH * TROW, Z = X + CH * PROW, STAGE = Z + CH * PROW;
+    static constexpr int WX = 2 * STAGE, S = WX + SSD_PIECES * CH * PROW, END = S + SSD_PIECES * NT * PROW;
+    static constexpr size_t BYTES = (size_t)END * 2;
+    // warps as tiles of 16 rows of S by groups of 8-column tiles (the update), and as tiles of 16 tokens by halves (the result)
+    static constexpr int NTILES = NT / 16, P_SPLITS = SSD_WARPS / NTILES, UPDATE = PT / 8 / P_SPLITS, RESULT = PT / 8 / 2;
+    static_assert(NTILES * P_SPLITS == SSD_WARPS && UPDATE >= 1 && RESULT >= 2, "layout");
+};
+
+template <typename TO, int NT, int PT, bool STATE_ONLY>
+__global__ void __launch_bounds__(SSD_THREADS, 1)
+ssd_prompt_kernel(const __nv_bfloat16* __restrict__ conv, const __nv_bfloat16* __restrict__ raw, const SsdInputs in,
+                  float* __restrict__ state, long long state_stride, const int* __restrict__ q_start,
+                  const int* __restrict__ item_slot, int first_item, int segments, float* __restrict__ run_state,
+                  float* __restrict__ run_decay, TO* __restrict__ out, long long out_stride) {
+    using L = SsdPromptLayout<NT, PT>;
+    constexpr int CH = L::CH, TROW = L::TROW, PROW = L::PROW;
+    extern __shared__ __align__(16) __nv_bfloat16 ssd_tiles[];
+    __shared__ float s_dt[CH], s_log[CH], s_from[CH], s_to[CH];
+    const int item = first_item + blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int col_tiles = (in.P + PT - 1) / PT, p0 = (blockIdx.z % col_tiles) * PT, segment = blockIdx.z / col_tiles;
+    const int begin = q_start[item], count = q_start[item + 1] - begin;
+    const int per = ssd_run_length(count, segments, CH), runs = count > 0 ? (count + per - 1) / per : 1;
+    if (count <= 0 || segment >= (STATE_ONLY ? runs - 1 : runs)) return;
+    const int lo = begin + segment * per, hi = min(lo + per, begin + count);
+    const int N = in.N, P = in.P, g = h / (in.heads / in.groups);
+    const float rate = -expf(in.a_log[h]), bias = in.dt_bias[h], skip = in.d[h];
+    const size_t block = (size_t)N * P;
+    float* S = state + (size_t)item_slot[item] * state_stride + (size_t)h * block;
+    const size_t cut_base = ((size_t)blockIdx.x * in.heads + h) * segments;
+
+    // ---- S as accumulators: rows n_row and n_row + 8, columns p0 + 8 (u_first + j) + 2 (lane & 3) and the next
+    const int n_tile = warp % L::NTILES, u_first = warp / L::NTILES * L::UPDATE;
+    const int n_row = 16 * n_tile + (lane >> 2), s_col = 8 * u_first + 2 * (lane & 3);
+    float s[L::UPDATE][4];
+    auto each_pair = [&](auto&& visit) {
+#pragma unroll
+        for (int j = 0; j < L::UPDATE; ++j)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int n = n_row + 8 * half, p = p0 + s_col + 8 * j;
+                visit(j, 2 * half, n < N && p < P, (size_t)n * P + p);
+            }
+    };
+    auto load_state = [&](const float* from) {
+        each_pair([&](int j, int i, bool here, size_t at) {
+            const float2 v = here ? *reinterpret_cast<const float2*>(from + at) : make_float2(0.f, 0.f);
+            s[j][i] = v.x;
+            s[j][i + 1] = v.y;
+        });
+    };
+    auto store_state = [&](float* to) {
+        each_pair([&](int j, int i, bool here, size_t at) {
+            if (here) *reinterpret_cast<float2*>(to + at) = make_float2(s[j][i], s[j][i + 1]);
+        });
+    };
+    // S of the slot: only these kernels of an earlier step wrote it, and they are done
+    if (STATE_ONLY ? segment == 0 : runs == 1) load_state(S);
+    pdl_prologue();
+    conv = pdl_fresh(conv);
+    raw = pdl_fresh(raw);
+
+    const uint32_t tiles = (uint32_t)__cvta_generic_to_shared(ssd_tiles);
+    auto copy = [&](int to, const __nv_bfloat16* from, bool here) {
+        const int bytes = here ? 16 : 0;                                       // 0: sixteen bytes of zeros
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(tiles + 2 * to), "l"(here ? from : conv), "r"(bytes) : "memory");
+    };
+    float dt_next[2] = {0.f, 0.f};                                             // warp 0: the tokens 2 lane and 2 lane + 1
+    auto fetch = [&](int t0, int stage) {
+        const int n = min(CH, hi - t0), base = stage * L::STAGE;
+        for (int e = tid; e < CH * (NT / 8); e += SSD_THREADS) {
+            const int tt = e / (NT / 8), i = (e % (NT / 8)) * 8;
+            const bool here = tt < n && i < N;
+            const __nv_bfloat16* at = conv + (size_t)(t0 + tt) * in.ld_conv + (size_t)g * N + i;
+            copy(base + L::B + tt * TROW + i, at + in.b, here);
+            if (!STATE_ONLY) copy(base + L::C + tt * TROW + i, at + in.c, here);
+        }
+        for (int e = tid; e < CH * (PT / 8); e += SSD_THREADS) {
+            const int tt = e / (PT / 8), j = (e % (PT / 8)) * 8;
+            const bool here = tt < n && p0 + j < P;
+            copy(base + L::X + tt * PROW + j, conv + (size_t)(t0 + tt) * in.ld_conv + in.x + (size_t)h * P + p0 + j, here);
+            if (!STATE_ONLY) copy(base + L::Z + tt * PROW + j, raw + (size_t)(t0 + tt) * in.ld_raw + in.z + (size_t)h * P + p0 + j, here);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (warp == 0) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                if (2 * lane + i < n) dt_next[i] = to_float(raw[(size_t)(t0 + 2 * lane + i) * in.ld_raw + in.dt + h]);
+        }
+    };
+    fetch(lo, 0);
+    if (STATE_ONLY) {
+        if (segment == 0) store_state(run_state + cut_base * block);           // the first run's start is the slot's state
+#pragma unroll
+        for (int j = 0; j < L::UPDATE; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+    } else if (runs > 1) {
+        load_state(pdl_fresh(run_state) + (cut_base + segment) * block);
+    }
+    // lane addresses (bytes) of the fragments: rows of a tile as they lie, and transposed
+    const uint32_t straight_row = (lane & 15), straight_col = (lane >> 4) * 8;            // A: [row][k]
+    const uint32_t pair_row = (lane & 7) + ((lane >> 4) & 1) * 8, pair_col = ((lane >> 3) & 1) * 8;    // B from [n][k]; A from [k][row]
+    const uint32_t trans_row = (lane & 7) + ((lane >> 3) & 1) * 8, trans_col = ((lane >> 4) & 1) * 8;  // B from [k][n]
+    float exponent = 0.f;                                                      // STATE_ONLY: the sum of the run's logarithms of decays
+    int stage = 0;
+    for (int t0 = lo; t0 < hi; t0 += CH, stage ^= 1) {
+        const int n = min(CH, hi - t0);
+        const uint32_t here = tiles + 2 * stage * L::STAGE;
+        const __nv_bfloat16* x_tile = ssd_tiles + stage * L::STAGE + L::X;
+        // ---- step sizes and decays; the state's pieces
+        if (warp == 0) {
+            float dt[2], v[2];
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                dt[i] = 2 * lane + i < n ? softplus(dt_next[i] + bias) : 0.f;
+                v[i] = rate * dt[i];
+            }
+            float sum = v[0] + v[1];
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float other = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += other;
+            }
+            const float end = __shfl_sync(0xffffffffu, sum, 31), mid = sum - v[1];
+            s_dt[2 * lane] = dt[0];             s_dt[2 * lane + 1] = dt[1];
+            s_log[2 * lane] = mid;              s_log[2 * lane + 1] = sum;
+            s_from[2 * lane] = expf(mid);       s_from[2 * lane + 1] = expf(sum);
+            s_to[2 * lane] = expf(end - mid) * dt[0];
+            s_to[2 * lane + 1] = expf(end - sum) * dt[1];
+        }
+        if (!STATE_ONLY) {
+#pragma unroll
+            for (int j = 0; j < L::UPDATE; ++j)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    uint32_t piece[SSD_PIECES];
+                    ssd_split(s[j][2 * half], s[j][2 * half + 1], piece);
+#pragma unroll
+                    for (int q = 0; q < SSD_PIECES; ++q)
+                        *reinterpret_cast<uint32_t*>(ssd_tiles + L::S + (q * NT + n_row + 8 * half) * PROW + s_col + 8 * j) = piece[q];
+                }
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (t0 + CH < hi) fetch(t0 + CH, stage ^ 1);
+        // ---- the pieces of the weighted x
+        for (int e = tid; e < CH * (PT / 2); e += SSD_THREADS) {
+            const int tt = e / (PT / 2), j = (e % (PT / 2)) * 2;
+            const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x_tile + tt * PROW + j));
+            const float weight = s_to[tt];
+            uint32_t piece[SSD_PIECES];
+            ssd_split(x.x * weight, x.y * weight, piece);
+#pragma unroll
+            for (int q = 0; q < SSD_PIECES; ++q)
+                *reinterpret_cast<uint32_t*>(ssd_tiles + L::WX + (q * CH + tt) * PROW + j) = piece[q];
+        }
+        if constexpr (!STATE_ONLY) {
+            const int m_tile = warp & 3, r_first = (warp >> 2) * L::RESULT;    // 16 tokens, half of the columns
+            const int row = 16 * m_tile + (lane >> 2);
+            float y[L::RESULT][4];
+#pragma unroll
+            for (int j = 0; j < L::RESULT; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+            uint32_t c_frag[NT / 16][4];
+#pragma unroll
+            for (int k = 0; k < NT / 16; ++k)
+                ssd_ldm(c_frag[k], here + 2 * (L::C + (16 * m_tile + straight_row) * TROW + 16 * k + straight_col));
+            // what the state ahead of the chunk gives
+#pragma unroll
+            for (int k = 0; k < NT / 16; ++k)
+#pragma unroll
+                for (int q = 0; q < SSD_PIECES; ++q)
+#pragma unroll
+                    for (int j = 0; j < L::RESULT; j += 2) {
+                        uint32_t b[4];
+                        ssd_ldm_t(b, tiles + 2 * (L::S + (q * NT + 16 * k + trans_row) * PROW + 8 * (r_first + j) + trans_col));
+                        ssd_mma(y[j], c_frag[k], b[0], b[1]);
+                        ssd_mma(y[j + 1], c_frag[k], b[2], b[3]);
+                    }
+            const float from[2] = {s_from[row], s_from[row + 8]};
+#pragma unroll
+            for (int j = 0; j < L::RESULT; ++j) {
+                y[j][0] *= from[0]; y[j][1] *= from[0];
+                y[j][2] *= from[1]; y[j][3] *= from[1];
+            }
+            // the chunk's own tokens, 16 at a time
+            const float log_row[2] = {s_log[row], s_log[row + 8]};
+#pragma unroll
+            for (int kk = 0; kk < CH / 16; ++kk) {
+                if (kk > m_tile) continue;
+                float w[2][4];
+#pragma unroll
+                for (int j = 0; j < 2; ++j) w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.f;
+#pragma unroll
+                for (int k = 0; k < NT / 16; ++k) {
+                    uint32_t b[4];
+                    ssd_ldm(b, here + 2 * (L::B + (16 * kk + pair_row) * TROW + 16 * k + pair_col));
+                    ssd_mma(w[0], c_frag[k], b[0], b[1]);
+                    ssd_mma(w[1], c_frag[k], b[2], b[3]);
+                }
+                uint32_t a[SSD_PIECES][4];
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    const int u = 16 * kk + 8 * j + 2 * (lane & 3);
+                    const float2 log_u = *reinterpret_cast<const float2*>(s_log + u), dt_u = *reinterpret_cast<const float2*>(s_dt + u);
+#pragma unroll
+                    for (int half = 0; half < 2; ++half) {
+                        const int t = row + 8 * half;
+                        const float v0 = u <= t ? w[j][2 * half] * expf(log_row[half] - log_u.x) * dt_u.x : 0.f;
+                        const float v1 = u + 1 <= t ? w[j][2 * half + 1] * expf(log_row[half] - log_u.y) * dt_u.y : 0.f;
+                        uint32_t piece[SSD_PIECES];
+                        ssd_split(v0, v1, piece);
+#pragma unroll
+                        for (int q = 0; q < SSD_PIECES; ++q) a[q][2 * j + half] = piece[q];
+                    }
+                }
+#pragma unroll
+                for (int j = 0; j < L::RESULT; j += 2) {
+                    uint32_t b[4];
+                    ssd_ldm_t(b, here + 2 * (L::X + (16 * kk + trans_row) * PROW + 8 * (r_first + j) + trans_col));
+#pragma unroll
+                    for (int q = 0; q < SSD_PIECES; ++q) {
+                        ssd_mma(y[j], a[q], b[0], b[1]);
+                        ssd_mma(y[j + 1], a[q], b[2], b[3]);
+                    }
+                }
+            }
+            // skip, gate, out
+            const __nv_bfloat16* z_tile = ssd_tiles + stage * L::STAGE + L::Z;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int tt = row + 8 * half;
+                if (tt >= n) continue;
+                TO* to = out + (size_t)(t0 + tt) * out_stride + (size_t)h * P + p0;
+#pragma unroll
+                for (int j = 0; j < L::RESULT; ++j) {
+                    const int col = 8 * (r_first + j) + 2 * (lane & 3);
+                    if (p0 + col >= P) continue;
+                    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x_tile + tt * PROW + col));
+                    const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(z_tile + tt * PROW + col));
+                    const float v0 = fmaf(skip, x.x, y[j][2 * half]) * silu(z.x), v1 = fmaf(skip, x.y, y[j][2 * half + 1]) * silu(z.y);
+                    if constexpr (sizeof(TO) == 4) *reinterpret_cast<float2*>(to + col) = make_float2(v0, v1);
+                    else *reinterpret_cast<__nv_bfloat162*>(to + col) = __floats2bfloat162_rn(v0, v1);
+                }
+            }
+        }
+        // (the decays are read ahead of the barrier: behind it the first warp may already form the next chunk's)
+        const float keep = s_from[CH - 1];
+        if (STATE_ONLY) exponent += s_log[CH - 1];
+        __syncthreads();
+        // ---- the state behind the chunk
+#pragma unroll
+        for (int j = 0; j < L::UPDATE; ++j) {
+            s[j][0] *= keep; s[j][1] *= keep; s[j][2] *= keep; s[j][3] *= keep;
+        }
+#pragma unroll
+        for (int k = 0; k < CH / 16; ++k) {
+            uint32_t a[4];
+            ssd_ldm_t(a, here + 2 * (L::B + (16 * k + pair_row) * TROW + 16 * n_tile + pair_col));
+#pragma unroll
+            for (int q = 0; q < SSD_PIECES; ++q) {
+                if constexpr (L::UPDATE == 1) {
+                    uint32_t b[4];                                             // (the neighbouring tile's fragments are not used)
+                    ssd_ldm_t(b, tiles + 2 * (L::WX + (q * CH + 16 * k + trans_row) * PROW + 8 * (u_first & ~1) + trans_col));
+                    if (u_first & 1) ssd_mma(s[0], a, b[2], b[3]);
+                    else ssd_mma(s[0], a, b[0], b[1]);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < L::UPDATE; j += 2) {
+                        uint32_t b[4];
+                        ssd_ldm_t(b, tiles + 2 * (L::WX + (q * CH + 16 * k + trans_row) * PROW + 8 * (u_first + j) + trans_col));
+                        ssd_mma(s[j], a, b[0], b[1]);
+                        ssd_mma(s[j + 1], a, b[2], b[3]);
+                    }
+                }
             }
         }
     }
-    // the sums over the parts: first inside a warp, then between its rows in shared memory
-    for (int o = lanes; o < 32; o <<= 1)
-#pragma unroll
-        for (int v = 0; v < V; ++v) y[v] += __shfl_xor_sync(0xffffffffu, y[v], o);
-    const int rows = lanes < 32 ? SSD_WARPS : parts, own = lanes < 32 ? tid >> 5 : part;
-    if (mine && (lanes >= 32 || (tid & 31) < lanes)) {
-#pragma unroll
-        for (int v = 0; v < V; ++v)
-            if (col + v < P) s_y[own * P + col + v] = y[v];
-    }
-    __syncthreads();
-    for (int j = tid; j < P; j += SSD_THREADS) {
-        float total = 0.f;
-        for (int w = 0; w < rows; ++w) total += s_y[w * P + j];
-        total = fmaf(skip, to_float(conv[in.x + (size_t)h * P + j]), total);
-        out[(size_t)t * out_stride + (size_t)h * P + j] = from_float<TO>(total * silu(to_float(raw[in.z + (size_t)h * P + j])));
+    if (STATE_ONLY) {
+        const size_t entry = cut_base + segment + 1;
+        store_state(run_state + entry * block);
+        if (tid == 0 && p0 == 0) run_decay[entry] = expf(exponent);
+    } else if (segment == runs - 1) {
+        store_state(S);
     }
 }
 
@@ -563,59 +887,100 @@ int launch_ssd_scan(const T* conv, const T* raw, const SsdInputs& in, float* sta
 #undef PS_SSD_ROWS
 }
 
+template <typename TO, int NT, int PT, bool STATE_ONLY>
+int launch_ssd_prompt(const __nv_bfloat16* conv, const __nv_bfloat16* raw, const SsdInputs& in, float* state,
+                      long long state_stride, const int* q_start, const int* item_slot, int n_items, int first_item,
+                      int segments, int depth, float* run_state, float* run_decay, TO* out, long long out_stride, cudaStream_t s) {
+    using L = SsdPromptLayout<NT, PT>;
+    auto kernel = ssd_prompt_kernel<TO, NT, PT, STATE_ONLY>;
+    static size_t raised[MAX_DEVICES] = {0};
+    if (!ensure_dynamic_smem((const void*)kernel, L::BYTES, raised)) return PS_ERR_LAUNCH;
+    const int tiles = (in.P + PT - 1) / PT;
+    if ((long long)tiles * depth > 65535) return PS_ERR_UNSUPPORTED;
+    return launch_pdl(kernel, dim3(n_items - first_item, in.heads, tiles * depth), dim3(SSD_THREADS), L::BYTES, s, conv, raw, in,
+                      state, state_stride, q_start, item_slot, first_item, segments, run_state, run_decay, out, out_stride);
+}
+
+template <typename TO, bool STATE_ONLY>
+int pick_ssd_prompt(const __nv_bfloat16* conv, const __nv_bfloat16* raw, const SsdInputs& in, float* state,
+                    long long state_stride, const int* q_start, const int* item_slot, int n_items, int first_item,
+                    int segments, int depth, float* run_state, float* run_decay, TO* out, long long out_stride, cudaStream_t s) {
+#define PS_SSD_PROMPT(NT, PT)                                                                                           \
+    return launch_ssd_prompt<TO, NT, PT, STATE_ONLY>(conv, raw, in, state, state_stride, q_start, item_slot, n_items, first_item, \
+                                                     segments, depth, run_state, run_decay, out, out_stride, s)
+    if (in.P <= 32) {
+        if (in.N <= 32) PS_SSD_PROMPT(32, 32);
+        if (in.N <= 64) PS_SSD_PROMPT(64, 32);
+        PS_SSD_PROMPT(128, 32);
+    }
+    if (in.N <= 32) PS_SSD_PROMPT(32, 64);
+    if (in.N <= 64) PS_SSD_PROMPT(64, 64);
+    PS_SSD_PROMPT(128, 64);
+#undef PS_SSD_PROMPT
+}
+
 template <typename T, typename TO>
-int pick_ssd(const T* conv, const T* raw, const SsdInputs& in, int single, float* state, long long state_stride,
-             const int* q_start, const int* item_slot, int n_items, int first_cut, int segments, float* run_state,
-             float* run_decay, TO* out, long long out_stride, cudaStream_t s) {
-    if (single) {
-        const bool by4 = in.P % 4 == 0 && state_stride % 4 == 0 && !((uintptr_t)state & 15);
-        const int V = by4 ? 4 : 1;
-        int lanes = 1;
-        while (lanes < SSD_THREADS && lanes * V < in.P) lanes <<= 1;
-        if (lanes * V < in.P) return PS_ERR_UNSUPPORTED;
+int pick_ssd(const T* conv, const T* raw, const SsdInputs& in, float* state, long long state_stride, const int* q_start,
+             const int* item_slot, int n_items, int first_cut, int segments, float* run_state, float* run_decay, TO* out,
+             long long out_stride, cudaStream_t s) {
+    int status = PS_OK, first = 0;                                // entries [0, first) are done
+    const bool by4 = in.P % 4 == 0 && state_stride % 4 == 0 && !((uintptr_t)state & 15);
+    const int V = by4 ? 4 : 1;
+    int lanes = 1;
+    while (lanes < SSD_THREADS && lanes * V < in.P) lanes <<= 1;
+    if (first_cut > 0 && lanes * V >= in.P) {
         const int parts = SSD_THREADS / lanes, rows = lanes < 32 ? SSD_WARPS : parts;
         const size_t smem = (size_t)(2 * in.N + rows * in.P) * sizeof(float);
-        if (by4) {
-            auto kernel = ssd_step_kernel<T, TO, 4>;
-            static size_t raised[MAX_DEVICES] = {0};
-            if (!ensure_dynamic_smem((const void*)kernel, smem, raised)) return PS_ERR_LAUNCH;
-            return launch_pdl(kernel, dim3(n_items, in.heads), dim3(SSD_THREADS), smem, s, conv, raw, in, state, state_stride,
-                              q_start, item_slot, lanes, out, out_stride);
-        }
-        auto kernel = ssd_step_kernel<T, TO, 1>;
-        static size_t raised[MAX_DEVICES] = {0};
-        if (!ensure_dynamic_smem((const void*)kernel, smem, raised)) return PS_ERR_LAUNCH;
-        return launch_pdl(kernel, dim3(n_items, in.heads), dim3(SSD_THREADS), smem, s, conv, raw, in, state, state_stride, q_start,
-                          item_slot, lanes, out, out_stride);
+        auto kernel = by4 ? ssd_step_kernel<T, TO, 4> : ssd_step_kernel<T, TO, 1>;
+        if (smem > 48 * 1024) return PS_ERR_UNSUPPORTED;
+        status = launch_pdl(kernel, dim3(first_cut, in.heads), dim3(SSD_THREADS), smem, s, conv, raw, in, state, state_stride,
+                            q_start, item_slot, lanes, out, out_stride);
+        if (status != PS_OK) return status;
+        first = first_cut;
     }
+    if (first == n_items) return PS_OK;
+    const bool prompt = sizeof(T) == 2 && first == first_cut && in.N <= 128 && in.N % 8 == 0 && in.P % 8 == 0 && in.ld_conv % 8 == 0 &&
+                        in.ld_raw % 8 == 0 && in.x % 8 == 0 && in.b % 8 == 0 && in.c % 8 == 0 && in.z % 8 == 0 &&
+                        !(((uintptr_t)conv | (uintptr_t)raw) & 15) && out_stride % 2 == 0 && !((uintptr_t)out & 7) &&
+                        state_stride % 2 == 0 && !((uintptr_t)state & 7) && !((uintptr_t)run_state & 7);
     if (segments > 1) {
-        int status = launch_ssd_scan<T, TO, true>(conv, raw, in, state, state_stride, q_start, item_slot, first_cut, n_items,
-                                                  first_cut, segments, segments - 1, run_state, run_decay, out,
-                                                  out_stride, s);
+        if constexpr (sizeof(T) == 2) {
+            if (prompt)
+                status = pick_ssd_prompt<TO, true>(conv, raw, in, state, state_stride, q_start, item_slot, n_items, first_cut,
+                                                   segments, segments - 1, run_state, run_decay, out, out_stride, s);
+        }
+        if (!prompt)
+            status = launch_ssd_scan<T, TO, true>(conv, raw, in, state, state_stride, q_start, item_slot, first_cut, n_items,
+                                                  first_cut, segments, segments - 1, run_state, run_decay, out, out_stride, s);
         if (status != PS_OK) return status;
         const int block = in.N * in.P;
-        const bool by4 = block % 4 == 0 && !((uintptr_t)run_state & 15);
-        const int units = by4 ? block / 4 : block;
-        status = launch_pdl(by4 ? ssd_fold_kernel<4> : ssd_fold_kernel<1>,
+        const bool quads = block % 4 == 0 && !((uintptr_t)run_state & 15);
+        const int units = quads ? block / 4 : block;
+        status = launch_pdl(quads ? ssd_fold_kernel<4> : ssd_fold_kernel<1>,
                             dim3((units + SSD_FOLD_THREADS - 1) / SSD_FOLD_THREADS, in.heads, n_items - first_cut),
                             dim3(SSD_FOLD_THREADS), 0, s, run_state, (const float*)run_decay, q_start, first_cut, segments,
-                            (int)SSD_CHUNK, in.heads, block);
+                            (int)(prompt ? SSD_PROMPT_CHUNK : SSD_CHUNK), in.heads, block);
         if (status != PS_OK) return status;
     }
-    return launch_ssd_scan<T, TO, false>(conv, raw, in, state, state_stride, q_start, item_slot, 0, n_items, first_cut, segments,
+    if constexpr (sizeof(T) == 2) {
+        if (prompt)
+            return pick_ssd_prompt<TO, false>(conv, raw, in, state, state_stride, q_start, item_slot, n_items, first_cut, segments,
+                                              segments, run_state, run_decay, out, out_stride, s);
+    }
+    return launch_ssd_scan<T, TO, false>(conv, raw, in, state, state_stride, q_start, item_slot, first, n_items, first_cut, segments,
                                          segments, run_state, run_decay, out, out_stride, s);
 }
 
 }  // namespace ps
 
 // conv, raw: rows of `dtype`, ld_conv / ld_raw elements apart; offsets: where x, B, C (in conv), z and dt (in raw) begin.
-// state: float32 [slots] rows of state_stride, of which the first heads * N * P numbers are S.  single: every entry brings
-// exactly one token.  Entries [first_cut, n_items) are cut into up to `segments` runs: run_state float32
+// state: float32 [slots] rows of state_stride, of which the first heads * N * P numbers are S.  Entries [0, first_cut) bring
+// few tokens and run token by token; entries [first_cut, n_items) are cut into up to `segments` runs: run_state float32
 // [(n_items - first_cut) * heads * segments][N * P] and run_decay [...] are scratch (null when segments is 1).  out: rows of
 // heads * P numbers of out_dtype (`dtype` or float32), out_stride apart.
 PS_EXPORT int ps_ssd(const void* conv, long long ld_conv, const void* raw, long long ld_raw, const int* offsets,
                      const float* a_log, const float* dt_bias, const float* d, float* state, long long state_stride,
-                     const int* q_start, const int* item_slot, int n_items, int T, int single, int first_cut, int segments,
+                     const int* q_start, const int* item_slot, int n_items, int T, int first_cut, int segments,
                      float* run_state, float* run_decay, void* out, long long out_stride, int heads, int groups, int N, int P,
                      int dtype, int out_dtype, void* stream) {
     if (n_items <= 0 || T <= 0) return PS_OK;
@@ -631,13 +996,13 @@ PS_EXPORT int ps_ssd(const void* conv, long long ld_conv, const void* raw, long 
     cudaStream_t s = (cudaStream_t)stream;
     using bf = __nv_bfloat16;
     if (dtype == PS_F32 && out_dtype == PS_F32)
-        return ps::pick_ssd<float, float>((const float*)conv, (const float*)raw, in, single, state, state_stride, q_start,
+        return ps::pick_ssd<float, float>((const float*)conv, (const float*)raw, in, state, state_stride, q_start,
                                           item_slot, n_items, first_cut, segments, run_state, run_decay, (float*)out, out_stride, s);
     if (dtype == PS_BF16 && out_dtype == PS_F32)
-        return ps::pick_ssd<bf, float>((const bf*)conv, (const bf*)raw, in, single, state, state_stride, q_start, item_slot,
+        return ps::pick_ssd<bf, float>((const bf*)conv, (const bf*)raw, in, state, state_stride, q_start, item_slot,
                                        n_items, first_cut, segments, run_state, run_decay, (float*)out, out_stride, s);
     if (dtype == PS_BF16 && out_dtype == PS_BF16)
-        return ps::pick_ssd<bf, bf>((const bf*)conv, (const bf*)raw, in, single, state, state_stride, q_start, item_slot, n_items,
+        return ps::pick_ssd<bf, bf>((const bf*)conv, (const bf*)raw, in, state, state_stride, q_start, item_slot, n_items,
                                     first_cut, segments, run_state, run_decay, (bf*)out, out_stride, s);
     return PS_ERR_UNSUPPORTED;
 }

@@ -107,7 +107,7 @@ _SIGNATURES = {
         "ps_sandwich_close_conv": [_P, _P, _I, _I, _P, _F, _F, _P, _I, _P, _L, _P, _P, _I, _P],
         "ps_gla_recurrence": [_P, _L, _P, _P, _P, _I, _F, _F, _P, _F, _F, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P,
                               _L, _I, _I, _I, _I, _P],
-        "ps_ssd": [_P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I,
+        "ps_ssd": [_P, _L, _P, _L, _P, _P, _P, _P, _P, _L, _P, _P, _I, _I, _I, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I,
                    _P],
         "ps_diff_prepare": [_P, _L, _I, _I, _P, _P, _F, _F, _I, _P, _P, _P, _I, _P, _P, _L, _I, _P, _L, _I, _I, _I, _I, _I,
                             _I, _I, _I, _P],
@@ -1387,13 +1387,15 @@ class Ops:
     SSD_SCRATCH_BYTES = 256 << 20
 
     def ssd_segments(self, ctx, heads, N, P):
-        """Runs that a prompt portion is cut into: about as many CTAs as two on every SM."""
+        """Runs that a prompt portion is cut into, so that about every SM has a CTA (in float32, and at sizes that the
+        tensor-core kernel does not take, two)."""
         long_items = ctx.num_items - ctx.num_short_items
         longest = int(ctx.max_q_len)
         if long_items <= 0 or longest < 2 * self.SSD_RUN:
             return 1
         tiles = -(-P // (64 if P > 32 and N <= 128 else 32))
-        wanted = min(148 * 2 // (long_items * heads * tiles), longest // self.SSD_RUN,
+        each = 1 if self.dtype == torch.bfloat16 and N <= 128 and N % 8 == 0 and P % 8 == 0 else 2
+        wanted = min(148 * each // (long_items * heads * tiles), longest // self.SSD_RUN,
                      self.SSD_SCRATCH_BYTES // (4 * long_items * heads * N * P))
         return max(1, min(64, wanted))
 
@@ -1419,8 +1421,8 @@ class Ops:
         single = bool(getattr(ctx, "single_tokens", False))
         if segments is None:
             segments = 1 if single else self.ssd_segments(ctx, heads, N, P)
-        first_cut = ctx.num_short_items
-        if single or first_cut >= ctx.num_items:
+        first_cut = ctx.num_items if single else ctx.num_short_items
+        if first_cut >= ctx.num_items:
             segments = 1
         run_state = run_decay = None
         if segments > 1:
@@ -1428,10 +1430,11 @@ class Ops:
             run_state = self.empty((runs, N * P), torch.float32, conv.device)
             run_decay = self.empty((runs,), torch.float32, conv.device)
         places = (ctypes.c_int * 5)(*[int(o) for o in offsets])
-        self.launches += 3 if segments > 1 else 1
+        long_items = first_cut < ctx.num_items
+        self.launches += (1 if first_cut else 0) + (0 if not long_items else 3 if segments > 1 else 1)
         _check(self.core.ps_ssd(_ptr(conv), conv.stride(0), _ptr(raw), raw.stride(0), ctypes.addressof(places), _ptr(a_log),
                                 _ptr(dt_bias), _ptr(d), _ptr(state), state.stride(0), _ptr(ctx.q_start), _ptr(ctx.item_slot),
-                                ctx.num_items, T, 1 if single else 0, first_cut, segments, _ptr(run_state), _ptr(run_decay),
+                                ctx.num_items, T, first_cut, segments, _ptr(run_state), _ptr(run_decay),
                                 _ptr(out), out.stride(0), heads, groups, N, P, self.code, dtype_code(out.dtype), _stream()),
                "ssd")
         return out
