@@ -62,63 +62,72 @@ __global__ void embed_sinusoid_kernel(const int* __restrict__ ids, const int* __
     }
 }
 
-// Two RMS norms of the same row with gains of their own, out_a = n(x) gain_a and out_b = n(x) gain_b: one warp per row held in
-// registers (H <= 128 * WMAX, a multiple of four, 16-byte addresses), or one CTA per row of any width (WMAX 0).
-template <typename TOut, int WMAX>
+// Two RMS norms of the same row with gains of their own, out_a = n(x) gain_a and out_b = n(x) gain_b, one CTA per row: the row
+// in registers, QUADS pieces of four numbers a thread, the gains fetched before the wait (QUADS 0: rows of any width and
+// alignment).
+template <typename TOut, int QUADS>
 __global__ void __launch_bounds__(256)
 rms_norm_pair_kernel(const float* __restrict__ x, const float* __restrict__ gain_a, const float* __restrict__ gain_b, float eps,
-                     TOut* __restrict__ out_a, TOut* __restrict__ out_b, int n_rows, int H) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+                     TOut* __restrict__ out_a, TOut* __restrict__ out_b, int H) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const float inv_h = 1.0f / (float)H;
-    if constexpr (WMAX > 0) {
+    __shared__ float red[8];
+    const size_t base = (size_t)blockIdx.x * H;
+    if constexpr (QUADS > 0) {
         const int quads = H >> 2;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        float4 ga[QUADS], gb[QUADS], v[QUADS];
+#pragma unroll
+        for (int i = 0; i < QUADS; ++i) {
+            const int c = threadIdx.x + i * blockDim.x;
+            ga[i] = c < quads ? reinterpret_cast<const float4*>(gain_a)[c] : zero;
+            gb[i] = c < quads ? reinterpret_cast<const float4*>(gain_b)[c] : zero;
+        }
         pdl_prologue();
         x = pdl_fresh(x);
-        const int r = blockIdx.x * (blockDim.x >> 5) + warp;
-        if (r >= n_rows) return;
-        const float4* xr = reinterpret_cast<const float4*>(x + (size_t)r * H);
-        float4 v[WMAX];
+        const float4* row = reinterpret_cast<const float4*>(x + base);
+#pragma unroll
+        for (int i = 0; i < QUADS; ++i) {
+            const int c = threadIdx.x + i * blockDim.x;
+            v[i] = c < quads ? row[c] : zero;
+        }
         float sq = 0.f;
 #pragma unroll
-        for (int i = 0; i < WMAX; ++i) {
-            const int c = lane + 32 * i;
-            v[i] = c < quads ? xr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
+        for (int i = 0; i < QUADS; ++i) sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+        sq = warp_sum(sq);
+        if (lane == 0) red[warp] = sq;
+        __syncthreads();
+        float total = 0.f;
+        for (int w = 0; w < warps; ++w) total += red[w];
+        const float inverse = 1.0f / sqrtf(total * inv_h + eps);
+        auto put = [&](TOut* out, const float4 (&g)[QUADS]) {
 #pragma unroll
-        for (int i = 0; i < WMAX; ++i) sq += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
-        const float inverse = 1.0f / sqrtf(warp_sum(sq) * inv_h + eps);
-        auto put = [&](TOut* out, const float* gain) {
-#pragma unroll
-            for (int i = 0; i < WMAX; ++i) {
-                const int c = lane + 32 * i;
-                if (c < quads) {
-                    const float4 g = reinterpret_cast<const float4*>(gain)[c];
-                    const float y0 = v[i].x * inverse * g.x, y1 = v[i].y * inverse * g.y;
-                    const float y2 = v[i].z * inverse * g.z, y3 = v[i].w * inverse * g.w;
-                    if constexpr (sizeof(TOut) == 2) {
-                        __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
-                        *reinterpret_cast<uint2*>(out + (size_t)r * H + 4 * c) =
-                            make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
-                    } else {
-                        *reinterpret_cast<float4*>(out + (size_t)r * H + 4 * c) = make_float4(y0, y1, y2, y3);
-                    }
+            for (int i = 0; i < QUADS; ++i) {
+                const int c = threadIdx.x + i * blockDim.x;
+                if (c >= quads) continue;
+                const float y0 = v[i].x * inverse * g[i].x, y1 = v[i].y * inverse * g[i].y;
+                const float y2 = v[i].z * inverse * g[i].z, y3 = v[i].w * inverse * g[i].w;
+                if constexpr (sizeof(TOut) == 2) {
+                    __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
+                    *reinterpret_cast<uint2*>(out + base + 4 * c) =
+                        make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+                } else {
+                    *reinterpret_cast<float4*>(out + base + 4 * c) = make_float4(y0, y1, y2, y3);
                 }
             }
         };
-        put(out_a, gain_a);
-        put(out_b, gain_b);
+        put(out_a, ga);
+        put(out_b, gb);
     } else {
-        __shared__ float red[8];
         pdl_prologue();
         x = pdl_fresh(x);
-        const size_t base = (size_t)blockIdx.x * H;
         float sq = 0.f;
         for (int c = threadIdx.x; c < H; c += blockDim.x) sq = fmaf(x[base + c], x[base + c], sq);
         sq = warp_sum(sq);
         if (lane == 0) red[warp] = sq;
         __syncthreads();
         float total = 0.f;
-        for (int w = 0; w < (int)(blockDim.x >> 5); ++w) total += red[w];
+        for (int w = 0; w < warps; ++w) total += red[w];
         const float inverse = 1.0f / sqrtf(total * inv_h + eps);
         for (int c = threadIdx.x; c < H; c += blockDim.x) {
             const float n = x[base + c] * inverse;
@@ -134,15 +143,14 @@ int launch_rms_norm_pair(const float* x, const float* gain_a, const float* gain_
     // (which form runs depends on the width and the alignment alone)
     const bool aligned = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)gain_a | (uintptr_t)gain_b | (uintptr_t)out_a |
                                          (uintptr_t)out_b) & 15) == 0;
-    if (aligned && H <= 2048) {
-        const int warps = n_rows <= 256 ? 2 : 8;
-        const dim3 grid((n_rows + warps - 1) / warps), block(32 * warps);
-        if (H <= 1024)
-            return launch_pdl(rms_norm_pair_kernel<TOut, 8>, grid, block, 0, s, x, gain_a, gain_b, eps, out_a, out_b, n_rows, H);
-        return launch_pdl(rms_norm_pair_kernel<TOut, 16>, grid, block, 0, s, x, gain_a, gain_b, eps, out_a, out_b, n_rows, H);
-    }
-    return launch_pdl(rms_norm_pair_kernel<TOut, 0>, dim3(n_rows), dim3(256), 0, s, x, gain_a, gain_b, eps, out_a, out_b,
-                      n_rows, H);
+    const int quads = H / 4;
+    if (!aligned || quads > 4 * 256)
+        return launch_pdl(rms_norm_pair_kernel<TOut, 0>, dim3(n_rows), dim3(256), 0, s, x, gain_a, gain_b, eps, out_a, out_b, H);
+    // half a thousand numbers a warp at most; two pieces a thread where a row has enough of them
+    const int each = quads <= 128 ? 1 : quads <= 512 ? 2 : 4;
+    const dim3 block((quads + each * 32 - 1) / (each * 32) * 32);
+    auto kernel = each == 1 ? rms_norm_pair_kernel<TOut, 1> : each == 2 ? rms_norm_pair_kernel<TOut, 2> : rms_norm_pair_kernel<TOut, 4>;
+    return launch_pdl(kernel, dim3(n_rows), block, 0, s, x, gain_a, gain_b, eps, out_a, out_b, H);
 }
 
 // One CTA per row. Row kept in registers when H <= NT*MAXV, else re-read.

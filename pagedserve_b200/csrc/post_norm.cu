@@ -60,6 +60,97 @@ group_rms_norm_kernel(const TIn* x, long long x_stride, const int* __restrict__ 
     for (int j = threadIdx.x; j < H; j += blockDim.x) target[j] = from_float<TOut>(staged[j] * inverse[j / run] * gain[j]);
 }
 
+// The same for rows in 16-byte pieces (V numbers of the input's type) and one group, or groups that are whole warps' passes
+// (run a multiple of 32 V): a row stays in registers, PASSES pieces a thread; the gains are fetched before the wait.
+template <typename T, int V> __device__ __forceinline__ void norm_piece(const T* p, float (&x)[V]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    if constexpr (V == 4) {
+        x[0] = __uint_as_float(raw.x); x[1] = __uint_as_float(raw.y); x[2] = __uint_as_float(raw.z); x[3] = __uint_as_float(raw.w);
+    } else {
+        const __nv_bfloat162* pair = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = __bfloat1622float2(pair[i]);
+            x[2 * i] = f.x;
+            x[2 * i + 1] = f.y;
+        }
+    }
+}
+template <int V> __device__ __forceinline__ void norm_store(float* p, const float (&x)[V]) {
+#pragma unroll
+    for (int i = 0; i < V; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+}
+template <int V> __device__ __forceinline__ void norm_store(__nv_bfloat16* p, const float (&x)[V]) {
+#pragma unroll
+    for (int i = 0; i < V; i += 4) {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(x[i], x[i + 1]), hi = __floats2bfloat162_rn(x[i + 2], x[i + 3]);
+        *reinterpret_cast<uint2*>(p + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+}
+
+template <typename TIn, typename TOut, int PASSES>
+__global__ void __launch_bounds__(GROUP_NORM_THREADS)
+group_rms_norm_pieces_kernel(const TIn* x, long long x_stride, const int* __restrict__ rows, int H, int groups,
+                             const float* __restrict__ gain, float eps, TOut* out, long long out_stride) {
+    constexpr int V = 16 / (int)sizeof(TIn);
+    __shared__ float partial[PASSES * GROUP_NORM_THREADS / 32];
+    __shared__ float inverse[GROUP_NORM_MAX_GROUPS];
+    const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, run = H / groups;
+    float g[PASSES][V];
+#pragma unroll
+    for (int p = 0; p < PASSES; ++p) {
+        const int j = V * (threadIdx.x + p * blockDim.x);
+#pragma unroll
+        for (int i = 0; i < V; i += 4) {
+            const float4 f = j < H ? *reinterpret_cast<const float4*>(gain + j + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            g[p][i] = f.x; g[p][i + 1] = f.y; g[p][i + 2] = f.z; g[p][i + 3] = f.w;
+        }
+    }
+    pdl_prologue();
+    x = pdl_fresh(x);
+    const int r = blockIdx.x;
+    const TIn* source = x + (size_t)(rows ? rows[r] : r) * x_stride;
+    float v[PASSES][V];
+#pragma unroll
+    for (int p = 0; p < PASSES; ++p) {
+        const int j = V * (threadIdx.x + p * blockDim.x);
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[p][i] = 0.f;
+        if (j < H) norm_piece<TIn, V>(source + j, v[p]);
+    }
+#pragma unroll
+    for (int p = 0; p < PASSES; ++p) {
+        float sq = 0.f;
+#pragma unroll
+        for (int i = 0; i < V; ++i) sq = fmaf(v[p][i], v[p][i], sq);
+        sq = warp_sum(sq);
+        if (lane == 0) partial[p * warps + warp] = sq;                   // the pieces p * warps + warp, in the row's order
+    }
+    __syncthreads();
+    float whole = 0.f;
+    if (groups == 1) {                                                   // at most 32 partial sums: every warp adds them itself
+        whole = 1.0f / sqrtf(warp_sum(lane < PASSES * warps ? partial[lane] : 0.f) / (float)run + eps);
+    } else {
+        const int each = run / (32 * V);                                 // partial sums of a group
+        for (int k = threadIdx.x; k < groups; k += blockDim.x) {
+            float total = 0.f;
+            for (int i = 0; i < each; ++i) total += partial[k * each + i];
+            inverse[k] = 1.0f / sqrtf(total / (float)run + eps);
+        }
+        __syncthreads();
+    }
+    TOut* target = out + (size_t)r * out_stride;
+#pragma unroll
+    for (int p = 0; p < PASSES; ++p) {
+        const int j = V * (threadIdx.x + p * blockDim.x);
+        if (j >= H) continue;
+        const float scale = groups == 1 ? whole : inverse[j / run];
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[p][i] = v[p][i] * scale * g[p][i];
+        norm_store<V>(target + j, v[p]);
+    }
+}
+
 // V numbers per access (4 where the width allows it).  The older entries of the history do not depend on the
 // sublayer's row: their weighted sum and the residual row are fetched in the first pass, beside the row itself, so
 // that their latency lies behind the row's statistics instead of behind them.
@@ -376,6 +467,18 @@ int launch_sandwich_rows(float* y, float* x, int T, int H, const float* gain, fl
 template <typename TIn, typename TOut>
 inline int launch_group_norm(const void* x, long long x_stride, const int* rows, int n_rows, int H, int groups,
                              const float* gain, float eps, void* out, long long out_stride, cudaStream_t s) {
+    constexpr int V = 16 / (int)sizeof(TIn), OUT = (int)sizeof(TOut);
+    if (H % V == 0 && x_stride % V == 0 && out_stride % (16 / OUT) == 0 && (groups == 1 || H / groups % (32 * V) == 0) &&
+        !(((uintptr_t)x | (uintptr_t)gain | (uintptr_t)out) & 15) && H / V <= 4 * GROUP_NORM_THREADS) {
+        const int pieces = H / V, threads = pieces < GROUP_NORM_THREADS ? (pieces + 31) / 32 * 32 : GROUP_NORM_THREADS;
+        const int passes = (pieces + threads - 1) / threads;
+        auto kernel = passes == 1 ? group_rms_norm_pieces_kernel<TIn, TOut, 1>
+                                  : passes == 2 ? group_rms_norm_pieces_kernel<TIn, TOut, 2> : group_rms_norm_pieces_kernel<TIn, TOut, 4>;
+        return launch_pdl(kernel, dim3(n_rows), dim3(threads), 0, s, (const TIn*)x, x_stride, rows, H, groups, gain, eps,
+                          (TOut*)out, out_stride);
+    }
+    static size_t raised[MAX_DEVICES] = {0};
+    if (!ensure_dynamic_smem((const void*)group_rms_norm_kernel<TIn, TOut>, (size_t)H * sizeof(float), raised)) return PS_ERR_LAUNCH;
     return launch_pdl(group_rms_norm_kernel<TIn, TOut>, dim3(n_rows), dim3(GROUP_NORM_THREADS), (size_t)H * sizeof(float),
                       s, (const TIn*)x, x_stride, rows, H, groups, gain, eps, (TOut*)out, out_stride);
 }
@@ -389,7 +492,7 @@ PS_EXPORT int ps_group_rms_norm(const void* x, long long x_stride, int in_dtype,
                                 int out_dtype, void* stream) {
     if (n_rows <= 0) return PS_OK;
     if (!x || !gain || !out || H <= 0 || groups <= 0 || H % groups) return PS_ERR_BAD_ARGUMENT;
-    if (groups > ps::GROUP_NORM_MAX_GROUPS || (size_t)H * sizeof(float) > 48 * 1024) return PS_ERR_UNSUPPORTED;
+    if (groups > ps::GROUP_NORM_MAX_GROUPS || (size_t)H * sizeof(float) > 200 * 1024) return PS_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
 #define PS_GROUP_NORM(TIN, TOUT) \
     return ps::launch_group_norm<TIN, TOUT>(x, x_stride, rows, n_rows, H, groups, gain, eps, out, out_stride, s)

@@ -207,8 +207,9 @@ short_conv_runs_kernel(const TI* __restrict__ u, long long u_stride, const float
         for (int k = TAPS - 2; k > 0; --k) held[k] = held[k - 1];
         if (TAPS > 1) held[0] = now;
         if constexpr (FORM == 2) {
-            y[0] = silu(y[0] + shift.x); y[1] = silu(y[1] + shift.y);
-            y[2] = silu(y[2] + shift.z); y[3] = silu(y[3] + shift.w);
+            auto gate = [](float v) { return sizeof(TC) == 2 ? silu_fast(v) : silu(v); };
+            y[0] = gate(y[0] + shift.x); y[1] = gate(y[1] + shift.y);
+            y[2] = gate(y[2] + shift.z); y[3] = gate(y[3] + shift.w);
         }
         if (common >= 0) {
             float* place = shared_values + (size_t)t * mix_heads * head_values + common;

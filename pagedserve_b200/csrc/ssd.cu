@@ -796,7 +796,7 @@ ssd_prompt_kernel(const __nv_bfloat16* __restrict__ conv, const __nv_bfloat16* _
                     if (p0 + col >= P) continue;
                     const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x_tile + tt * PROW + col));
                     const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(z_tile + tt * PROW + col));
-                    const float v0 = fmaf(skip, x.x, y[j][2 * half]) * silu(z.x), v1 = fmaf(skip, x.y, y[j][2 * half + 1]) * silu(z.y);
+                    const float v0 = fmaf(skip, x.x, y[j][2 * half]) * silu_fast(z.x), v1 = fmaf(skip, x.y, y[j][2 * half + 1]) * silu_fast(z.y);
                     if constexpr (sizeof(TO) == 4) *reinterpret_cast<float2*>(to + col) = make_float2(v0, v1);
                     else *reinterpret_cast<__nv_bfloat162*>(to + col) = __floats2bfloat162_rn(v0, v1);
                 }

@@ -492,7 +492,7 @@ def test_sines_of_far_positions(width, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("rows,width", [(1, 64), (37, 50), (300, 1024), (5, 2048), (3, 2052), (6, 37)])
+@pytest.mark.parametrize("rows,width", [(1, 64), (37, 50), (300, 1024), (5, 2048), (3, 2052), (6, 37), (2, 4096), (4, 5000), (3, 132)])
 def test_two_norms_of_one_row(rows, width, dtype):
     from pagedserve_b200.kernels.ops import Ops
 
@@ -504,6 +504,27 @@ def test_two_norms_of_one_row(rows, width, dtype):
     ops.rms_norm_pair(x.to(DEV), gains[0].to(DEV), gains[1].to(DEV), 1e-4, *outs)
     for out, gain in zip(outs, gains):
         assert rel_err(out, plain.unit_rms(x.double(), 1e-4) * gain.double()) < (2e-6 if dtype == torch.float32 else 5e-3)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("width,groups", [(64, 1), (512, 2), (4096, 1), (4096, 8), (1536, 3), (768, 6), (2048, 64), (8192, 4), (13000, 1), (200, 5)])
+def test_norm_in_groups_of_wide_rows(width, groups, dtype):
+    """Rows of the compute type whose groups differ a hundredfold in size, in 16-byte pieces where groups are whole passes of
+    a warp, and otherwise."""
+    from pagedserve_b200.kernels.ops import Ops
+
+    ops = Ops(dtype)
+    g = torch.Generator().manual_seed(width + groups)
+    rows = torch.randn(9, groups, width // groups, generator=g) * (10.0 ** (torch.arange(groups) % 3))[None, :, None]
+    rows = rows.reshape(9, width).to(dtype)
+    gain = 1.0 + 0.2 * torch.randn(width, generator=g)
+    out = torch.full((9, width + 8), 5.0, dtype=dtype, device=DEV)
+    ops.group_rms_norm(rows.to(DEV), gain.to(DEV), 1e-4, groups, out[:, :width])
+    want = plain.unit_rms_in_parts(rows.double(), groups, 1e-4) * gain.double()
+    assert rel_err(out[:, :width], want) < (2e-6 if dtype == torch.float32 else 5e-3) and bool((out[:, width:] == 5.0).all())
+    picks = torch.tensor([4, 4, 0], dtype=torch.int32)
+    ops.group_rms_norm(rows.to(DEV), gain.to(DEV), 1e-4, groups, out[:3, :width], rows=picks.to(DEV))
+    assert rel_err(out[:3, :width], want[picks.long()]) < (2e-6 if dtype == torch.float32 else 5e-3)
 
 
 # ------------------------------------------------------------------ products with a factor per column
