@@ -164,7 +164,7 @@ short_conv_runs_kernel(const TI* __restrict__ u, long long u_stride, const float
         return v;
     };
     if (c >= channels) return;
-    constexpr int AHEAD = 4;                                      // tokens whose rows are fetched together
+    constexpr int AHEAD = sizeof(TI) == 2 ? 8 : 4;                // tokens whose rows are fetched together
     if (!convolved) {
         for (int t = t0; t < t1; t += AHEAD) {
             float4 rows[AHEAD];
@@ -311,7 +311,9 @@ PS_EXPORT int ps_short_conv(const void* u, int u_dtype, long long u_stride, cons
         // runs of 16 tokens re-read (taps - 1) / 16 of the rows; shorter runs where the step has too few for the SMs
         const int columns = (channels / 4 + ps::SHORT_CONV_THREADS - 1) / ps::SHORT_CONV_THREADS;
         int run = 16;
-        while (run > 1 && (long long)columns * ((T + run - 1) / run) < 1200) run >>= 1;
+        // (rows of two bytes a number: as many bytes on their way as with four take twice the tokens a thread)
+        const long long enough = in_elem == 2 ? 1000 : 1200;
+        while (run > 1 && (long long)columns * ((T + run - 1) / run) < enough) run >>= 1;
         const dim3 grid(columns, (T + run - 1) / run), block(ps::SHORT_CONV_THREADS);
 #define PS_CONV_RUNS(TI, TC, TAPS, FORM)                                                                              \
     return ps::launch_pdl(ps::short_conv_runs_kernel<TI, TC, TAPS, FORM>, grid, block, 0, s, (const TI*)u, u_stride,    \
