@@ -120,6 +120,8 @@ class VoziraxConfig(ModelConfig):
         else:
             temp = _object(mixer["q_temp"], f"{where}: mixer.q_temp")
             temp["coef"] = _any_number(temp.get("coef"), f"{where}: mixer.q_temp.coef")
+            if isinstance(temp.get("every"), float) and temp["every"].is_integer():
+                temp["every"] = int(temp["every"])
             _positive_int(temp.get("every"), f"{where}: mixer.q_temp.every")
         if mixer.get("kv_from") is None:
             mixer.pop("kv_from", None)
